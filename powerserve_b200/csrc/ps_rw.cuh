@@ -181,8 +181,8 @@ PS_D float ps_rw_row_result(const PsRwAcc &acc) {
 // ---------------------------------------------------------------------------------------------------- the kernel
 // quantise one 256-block held as e[8] per lane (see ps_quant_block_q8k_regs) into the shared-memory image the block
 // math reads: qa[i][j2][q] = {sub-block 2*j2 words 2q, 2q+1 ; sub-block 2*j2+1 words 2q, 2q+1}, meta[i][q] = {d, bsums pair q}
-// (the eight elements travel BY VALUE: a pointer to the caller's register array would force it through local memory - two
-// STL.128 + two LDL.128 per call, L2 round trips when the 24 KB of L1 left beside the shared-memory carve-out miss)
+// (the eight elements travel BY VALUE: a pointer to the caller's register array would force it through local memory and
+// the 24 KB of L1 left beside the shared-memory carve-out)
 __device__ __noinline__ void ps_rw_quant_store_v(float4 ea, float4 eb, int lane, uint32_t *qw, uint2 *meta) {
     uint32_t words[2], bsp4;
     float yd;
