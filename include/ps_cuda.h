@@ -210,12 +210,14 @@ int ps_cuda_tp_import(ps_cuda_ctx *ctx, const void *handles, int n);
 /* ---------------------------------------------------------------------------------------------- layer-list models
  * Models that a configuration file describes layer by layer (config.json + model.safetensors, weights in bfloat16)
  * instead of the fixed llama / qwen2 stack above.  A layer is a token mixer plus an optional feed-forward.
- *   block_kind PS_BLOCK_PARALLEL: both read ONE norm's output, x <- x + (mixer(N(x)) + ff(N(x)));
+ *   block_kind PS_BLOCK_PARALLEL: both read ONE norm's output, x <- x + residual_scale * (mixer(N(x)) + ff(N(x)));
  *   block_kind PS_BLOCK_SEQUENTIAL: x <- x + P1(mixer(N1(x))), then x <- x + P2(ff(N2(x))); P1 / P2 are norms of the
  *   sublayer's OUTPUT when post_norm = 1, the identity otherwise.
  * Every mechanism is a parameter set of its own, so that another design can combine them differently:
  *   attention  - grouped-query, separate query/key and value head sizes, projection biases, no rotation;
  *                qk_norm = 1: every head's q and k are divided by their root mean square (no weight, eps = norm_eps);
+ *                qk_norm = PS_QKNORM_HEAD_W: the same, times the weights q_norm / k_norm [qk_dim] that all heads share;
+ *                q_temp_coef != 0: q at position p is multiplied by 1 + q_temp_coef ln(floor((p + 1) / q_temp_every) + 1);
  *                score = q.k * score_scale [* head_temp[h]] [+ rel[bucket(i - j)][h]] [- r1[h] ln(1 + r2[h] (i - j))]
  *                [mixed over heads by head_mix]; window > 0: query i sees the keys i - window < j <= i only;
  *                soft-max with an optional sink (one more term in the denominator that carries no value: exp(0) for
@@ -228,7 +230,7 @@ int ps_cuda_tp_import(ps_cuda_ctx *ctx, const void *handles, int n);
  *                rot_dim dims of ONE rotated key part shared by all heads; per head k = W_uk c, v = W_uv c;
  *                score = (q_plain . k + q_rot . k_rot) * score_scale, causal or windowed, sink as above.  The cache
  *                holds c and the rotated key part only: the executor folds W_uk into the query and applies W_uv to
- *                the weighted sum of latents.
+ *                the weighted sum of latents.  q_rank = 0: the queries are projected from the input itself (tensor q, no dq / uq).
  *   rotation   - the first rope_dims dims of a rotated vector, pairs (i, i + rope_dims / 2), angle pos * f_i with
  *                f_i = rope_base^(-2 i / rope_dims); rope_factor > 0 adds YaRN: f_i <- f_i / factor * ramp_i +
  *                f_i (1 - ramp_i) with the ramp between the dims whose wavelength fits rope_original positions
@@ -246,6 +248,10 @@ int ps_cuda_tp_import(ps_cuda_ctx *ctx, const void *handles, int n);
  *                S_t = exp(-exp(A_log[h]) dt) S_(t-1) + dt B_t x_t^T, y_t = S_t^T C_t + D[h] x_t; y silu(z) is RMS-normed in
  *                gate_norm_groups equal parts times mix_norm, then the output projection.  State: S per head, ssm_state x v_dim, fp32,
  *                and the last conv_taps - 1 inputs of the convolution.
+ *   rg-lru     - PS_MIXER_RGLRU: two branches of rec_width channels, y = gelu_tanh(W_y h + b_y) and u = conv(W_x h + b_x) (causal
+ *                convolution of conv_taps taps with bias); u in rec_blocks equal parts, in part b r = sigmoid(R_b u_b + ..),
+ *                i = sigmoid(I_b u_b + ..); log a = -rec_rate r softplus(lam), S_t = a S_(t-1) + sqrt(1 - a^2) i u (zero before the
+ *                start), then the output projection of S y.  State: S (fp32) and the convolution's last inputs (a ring of conv_taps rows).
  *   recurrent state lives where a cache set keeps an attention layer's K rows (first buffer) and V^T rows (second buffer);
  *                a sequence at position 0 starts from zero state whatever the buffers hold; ps_cuda_kv_rollback to a
  *                position other than 0 is refused for models with such layers.
@@ -256,6 +262,7 @@ int ps_cuda_tp_import(ps_cuda_ctx *ctx, const void *handles, int n);
  *                the experts form that many equal groups of neighbours, a group is worth its best score and only the
  *                route_keep best groups can be chosen from.  Expert: g = min(Wg z, act_limit), u = clamp(Wu z, +-act_limit),
  *                y = g * sigmoid(act_alpha * g) * (u + up_shift), out = Wd y; act_kind PS_ACT_GELU_TANH: y = gelu_tanh(Wg z) * (Wu z).
+ *                router_bias = 1: a bias on the logits; router_act 3 = the top_k largest LOGITS choose, weights = soft-max over those alone;
  *                shared_ff > 0: one more expert of that many rows runs for every token and is added, times
  *                sigmoid(shared_sg . z) when shared_gate = 1.
  *   raw_input  - sequential blocks: the sublayers read the residual stream itself (no norm on the way in).
@@ -268,18 +275,24 @@ int ps_cuda_tp_import(ps_cuda_ctx *ctx, const void *handles, int n);
  *                carries no distance term.  The cache set keeps the means behind the layer's K rows and V^T rows.
  *   linear distance bias - lin_bias = 1: score -= lin[h] * (i - j).
  *   output gate - out_gate = 1: the concatenated heads are multiplied by sigmoid(W_g h) (tensor g, [H * v_dim][dim]) before the
- *                output projection; W_g reads the mixer's input.
+ *                output projection; W_g reads the mixer's input.  out_gate = PS_GATE_HEAD: W_g has one row per head, a head's whole
+ *                output is multiplied by its number.
  *   side mixer - side_kind = PS_MIXER_MINGRU: a gated recurrence beside the attention, reading the same input: z = sigmoid(W_z h + b_z),
  *                u = W_x h + b_x, candidate c = u + 1/2 (u >= 0) or sigmoid(u) (u < 0), S_t = (1 - z) S_(t-1) + z c element by
  *                element over side_width channels (fp32, zero at position 0), output W_so (S_t silu(W_sg h)).  The layer's mixer
  *                output is mix_scale * attention + side_scale * side (one product over the concatenated inputs).
  *   interleaved rotation - rope_interleaved = 1: the rotation pairs dims (2i, 2i + 1) instead of (i, i + rope_dims / 2).
- *   ungated ff - mlp_ungated = 1 (PS_MLP_DENSE): out = W_down act(W_up h), act the one-argument form of act_kind; PS_ACT_XIELU with the
+ *   ungated ff - mlp_ungated = 1: out = W_down act(W_up h), act the one-argument form of act_kind, for the dense feed-forward, the
+ *                experts and the shared expert; PS_ACT_RELU2: max(z, 0)^2; PS_ACT_XIELU (dense only) with the
  *                two numbers p, q of tensor act: z > 0: softplus(p) z^2 + z / 2; z <= 0: (1/2 + softplus(q)) (exp(z) - 1 - z) + z / 2.
  *   layer runs - the descriptor's layer list is the list of layer RUNS: share_weights = j + 1 makes a run use the weights of run j
  *                (same sizes; its own cache and state), so a group of layers can be passed through several times.  pass_embed = 1
  *                adds the embedding output (the residual stream as it was before the first run) to the stream before the run,
- *                pass_step = r + 1 adds row r of the model's pass_steps table [n_pass_steps][dim].
+ *                pass_step = r + 1 adds row r of the model's pass_steps table [n_pass_steps][dim]; pass_in = 1 replaces the stream x by
+ *                W_in [x; x0] (tensor pass_in [dim][2 dim], x0 the embedding output) before the run.
+ *   general parallel blocks - a parallel block with any of: a layer norm, latent attention or an rg-lru as its mixer, an ungated dense or
+ *                routed feed-forward (also with a shared expert), PS_QKNORM_HEAD_W, a query temperature, a gate per head, proj_bias = 2,
+ *                a residual scale, a pass_in.  Its feed-forward has no gate (or there is none).
  *   norm       - RMS norm with eps inside the root; norm_kind = PS_NORM_LAYER: the mean is taken off first and the divisor is
  *                sqrt(variance + eps) (a weight, no bias); norm_unit_offset = 1: the stored weight is around zero (1 + w);
  *                norm_groups > 1: the vector is cut into that many equal parts, each divided by its own root mean square;
@@ -292,21 +305,22 @@ int ps_cuda_tp_import(ps_cuda_ctx *ctx, const void *handles, int n);
  * compute = PS_COMPUTE_BF16: matrix products take bfloat16 operands and accumulate in fp32; the residual stream, norms,
  * attention scores / weights, routers and the cache stay fp32.  PS_COMPUTE_F32: every product in true fp32 (FMA). */
 enum ps_cuda_compute { PS_COMPUTE_BF16 = 0, PS_COMPUTE_F32 = 1 };
-enum ps_cuda_mixer_kind { PS_MIXER_ATTENTION = 1, PS_MIXER_LATENT = 2, PS_MIXER_RETENTION = 3, PS_MIXER_MAMBA2 = 4, PS_MIXER_MINGRU = 5 /* side mixer only */ };
+enum ps_cuda_mixer_kind { PS_MIXER_ATTENTION = 1, PS_MIXER_LATENT = 2, PS_MIXER_RETENTION = 3, PS_MIXER_MAMBA2 = 4, PS_MIXER_MINGRU = 5 /* side mixer only */, PS_MIXER_RGLRU = 6 };
 enum ps_cuda_mlp_kind { PS_MLP_NONE = 0, PS_MLP_ROUTED = 1, PS_MLP_DENSE = 2 };
 enum ps_cuda_block_kind { PS_BLOCK_PARALLEL = 0, PS_BLOCK_SEQUENTIAL = 1 };
 enum ps_cuda_sink_kind { PS_SINK_NONE = 0, PS_SINK_ZERO = 1, PS_SINK_LEARNED = 2 };
 enum ps_cuda_vmix_kind { PS_VMIX_NONE = 0, PS_VMIX_SOURCE = 1, PS_VMIX_BLEND = 2 };
-enum ps_cuda_qknorm_kind { PS_QKNORM_NONE = 0, PS_QKNORM_HEAD = 1, PS_QKNORM_WHOLE = 2 };
-enum ps_cuda_act_kind { PS_ACT_SWISH = 0, PS_ACT_GELU_TANH = 1, PS_ACT_XIELU = 2 };
+enum ps_cuda_qknorm_kind { PS_QKNORM_NONE = 0, PS_QKNORM_HEAD = 1, PS_QKNORM_WHOLE = 2, PS_QKNORM_HEAD_W = 3 };
+enum ps_cuda_gate_kind { PS_GATE_NONE = 0, PS_GATE_ELEMENT = 1, PS_GATE_HEAD = 2 };
+enum ps_cuda_act_kind { PS_ACT_SWISH = 0, PS_ACT_GELU_TANH = 1, PS_ACT_XIELU = 2, PS_ACT_RELU2 = 3 /* one-argument only */ };
 enum ps_cuda_norm_kind { PS_NORM_RMS = 0, PS_NORM_LAYER = 1 };
-enum ps_cuda_router_act { PS_ROUTER_SIGMOID = 1, PS_ROUTER_SOFTMAX = 2 };
+enum ps_cuda_router_act { PS_ROUTER_SIGMOID = 1, PS_ROUTER_SOFTMAX = 2, PS_ROUTER_TOPK_SOFTMAX = 3 };
 
 typedef struct {
     int32_t mixer_kind;
     int32_t n_heads, n_kv_heads, qk_dim, v_dim;
     float   score_scale;
-    int32_t proj_bias;                  /* q, k, v and output projections carry biases */
+    int32_t proj_bias;                  /* 1: q, k, v and output projections carry biases; 2: q, k and v do */
     int32_t head_temp;                  /* per-head score multiplier */
     int32_t rel_buckets; float rel_max_dist; /* rows of the distance-bias table (0 = none) and the distance of its last bucket */
     int32_t head_mix;                   /* [H][H] mixing of the heads' scores before the soft-max */
@@ -337,13 +351,18 @@ typedef struct {
     int32_t v_is_k;                     /* the value rows are the projected key rows (no W_v) */
     int32_t pool;                       /* > 0: mean key / value per block of this many positions wholly before the window */
     int32_t lin_bias;                   /* score -= lin[h] * distance */
-    int32_t out_gate;                   /* heads' outputs times sigmoid(W_g h) before the output projection */
+    int32_t out_gate;                   /* enum ps_cuda_gate_kind: heads' outputs times sigmoid(W_g h) before the output projection */
     int32_t side_kind, side_width;      /* a second mixer beside the attention (0 = none, PS_MIXER_MINGRU) and its channels */
     float   mix_scale, side_scale;      /* mixer output = mix_scale * attention + side_scale * side (used when side_kind != 0) */
     int32_t rope_interleaved;           /* rotation pairs (2i, 2i + 1) */
-    int32_t mlp_ungated;                /* dense feed-forward without a gate: down(act(up h)) */
+    int32_t mlp_ungated;                /* feed-forward (experts, shared expert) without a gate: down(act(up h)) */
+    float   q_temp_coef, q_temp_every;  /* query temperature (coef 0 = none) */
+    int32_t rec_width, rec_blocks;      /* rg-lru: channels, equal parts of the gates' matrices */
+    float   rec_rate;                   /* rg-lru: factor of the decay's logarithm */
+    int32_t router_bias;                /* the router's logits carry a bias */
     int32_t share_weights;              /* j + 1: this run uses the weights of run j */
     int32_t pass_embed, pass_step;      /* before the run: add the embedding output; add row pass_step - 1 of pass_steps */
+    int32_t pass_in;                    /* before the run: x <- W_in [x; embedding output] */
 } ps_cuda_layer_desc;
 
 typedef struct {
@@ -357,6 +376,7 @@ typedef struct {
     int32_t norm_scalar;                /* the norms' weights are single numbers */
     int32_t norm_kind;                  /* enum ps_cuda_norm_kind: the block norms and the final norm */
     int32_t n_pass_steps;               /* rows of the pass_steps table */
+    float   residual_scale;             /* factor on what a block adds to the residual stream (0: 1) */
 } ps_cuda_arch_desc;
 
 /* matrices [out][in] in bfloat16; vectors and the small tables in bfloat16 or fp32 */
@@ -373,12 +393,16 @@ typedef struct {
     ps_cuda_tensor shared_gate, shared_up, shared_down, shared_sg; /* shared expert */
     ps_cuda_tensor lin, act;            /* linear distance-bias slopes [H]; the activation's numbers [2] */
     ps_cuda_tensor side_z, side_z_bias, side_x, side_x_bias, side_g, side_o; /* side mixer: [W][dim], [W], [W][dim], [W], [W][dim], [dim][W] */
+    ps_cuda_tensor router_bias;         /* [n_experts] */
+    ps_cuda_tensor rec_y, rec_y_bias, rec_x, rec_x_bias;   /* rg-lru: [W][dim], [W] twice (conv_w [W][taps] and conv_b [W] above) */
+    ps_cuda_tensor rec_r, rec_r_bias, rec_i, rec_i_bias, rec_lam; /* [blocks][W / blocks][W / blocks], [W] twice; [W] */
 } ps_cuda_arch_layer_weights;
 
 typedef struct {
     ps_cuda_tensor embed, final_norm, head;
     const ps_cuda_arch_layer_weights *layers; /* one entry per run; the entries of runs that share another run's weights are not read */
     ps_cuda_tensor pass_steps;          /* [n_pass_steps][dim] */
+    ps_cuda_tensor pass_in;             /* [dim][2 dim] */
 } ps_cuda_arch_weights;
 
 int ps_cuda_create_arch(ps_cuda_ctx **out, int device, const ps_cuda_arch_desc *desc);

@@ -41,7 +41,7 @@ class LayerListModel(capi.CudaModel):
         self._layer_descs = (LayerDesc * len(layers))(*layers)
         self.desc = ArchDesc(top["dim"], top["vocab_size"], len(layers), int(n_ctx), int(max_batch), top["norm_eps"], top["embed_scale"],
                              top["norm_unit_offset"], compute, self._layer_descs, int(top.get("norm_groups", 1)), int(top.get("norm_scalar", 0)),
-                             int(top.get("norm_kind", 0)), int(top.get("n_pass_steps", 0)))
+                             int(top.get("norm_kind", 0)), int(top.get("n_pass_steps", 0)), float(top.get("residual_scale", 1.0)))
         self.vocab = self.desc.vocab_size
         self.be = capi.CudaBackend(self.desc, device)
 
@@ -70,7 +70,7 @@ class LayerListModel(capi.CudaModel):
                     self._keep.append(arr)
                     setattr(lw, f, arr)
             self._lw[i] = lw
-        self._w = ArchWeights(T(names["embed"]), T(names["final_norm"]), T(names["head"]), self._lw, T(names.get("pass_steps")))
+        self._w = ArchWeights(T(names["embed"]), T(names["final_norm"]), T(names["head"]), self._lw, T(names.get("pass_steps")), T(names.get("pass_in")))
         self.be._ck(self.be.L.ps_cuda_bind_arch(self.be.h, C.byref(self._w)))
 
     def layer_tap(self, layer: int, bs: int):
@@ -314,13 +314,13 @@ def _dozotar_tensor_names(cfg: dict) -> dict:
 #   "latent_attention"  queries through a normed latent, keys / values from a shared normed latent plus one rotated key part common to
 #                       all heads; rotation in neighbouring pairs (2i, 2i + 1); a window.
 # Feed-forward: down(xIELU(up h)) with the activation's two numbers per layer.  Embedding scaled; final layer norm; untied head.
-def _pidenex_runs(cfg: dict) -> List[Tuple[int, Optional[int]]]:
-    """(layer, number of the pass that this run opens or None) in execution order"""
+def _layer_runs(cfg: dict) -> List[Tuple[int, Optional[int]]]:
+    """(layer, number of the pass that this run opens or None) in execution order, by config "loop" = {start, stop, times}"""
     n = len(cfg["layers"])
     lp = cfg.get("loop") or {}
     a, b, times = int(lp.get("start", 0)), int(lp.get("stop", 0)), int(lp.get("times", 1))
     if not (0 <= a <= b <= n) or times < 1:
-        raise capi.PsCudaError(f"Pidenex: loop {lp!r} does not fit {n} layers")
+        raise capi.PsCudaError(f"loop {lp!r} does not fit {n} layers")
     runs: List[Tuple[int, Optional[int]]] = [(i, None) for i in range(a)]
     if b > a:
         for t in range(times):
@@ -340,7 +340,7 @@ def _pidenex_attention(d: LayerDesc, m: dict) -> None:
 def _pidenex_describe(cfg: dict, tensors) -> Tuple[List[LayerDesc], dict]:
     layers = []
     first_run: Dict[int, int] = {}
-    for r, (i, t) in enumerate(_pidenex_runs(cfg)):
+    for r, (i, t) in enumerate(_layer_runs(cfg)):
         l = cfg["layers"][i]
         m = l["mixer"]
         d = LayerDesc()
@@ -390,7 +390,7 @@ def _pidenex_tensor_names(cfg: dict) -> dict:
     if int(lp.get("stop", 0)) > int(lp.get("start", 0)):
         out["pass_steps"] = "loop.step"
     seen = set()
-    for i, _ in _pidenex_runs(cfg):
+    for i, _ in _layer_runs(cfg):
         if i in seen:                 # a repeated run: the weights of its first run
             out["layers"].append({})
             continue
@@ -415,8 +415,110 @@ def _pidenex_tensor_names(cfg: dict) -> dict:
     return out
 
 
+# ------------------------------------------------------------------------------------------------------------ Momedra
+# Decoder-only; every layer is a parallel block behind one layer norm (weight, no bias), x <- x + residual_mult (mixer(h) + ff(h)).
+# config "loop" as in Pidenex; before the first layer of every pass - the first pass too - x <- W_in [x; x0], x0 the embedding output.
+# Three mixers, chosen by "type":
+#   "attention"         grouped-query, no rotation; q / k / v biases; q and k of every head RMS-normed with a weight the heads share; q at
+#                       position p times 1 + coef ln(floor((p + 1) / every) + 1); every head's output times sigmoid((W_g h)_head).
+#   "latent_attention"  queries straight from h; keys / values from a normed latent plus one rotated key part common to all heads,
+#                       rotation in neighbouring pairs; a learned sink per head.
+#   "rglru"             gelu branch times a real-gated linear recurrence over a short convolution's output, block-diagonal gates.
+# Feed-forwards have no gate, down(max(up h, 0)^2): one, or `top` of `experts` small ones by their (biased) router logits, weights the
+# soft-max over the chosen, plus a shared one for every token.
+_MOMEDRA_RG_RATE = 8.0
+
+
+def _momedra_describe(cfg: dict, tensors) -> Tuple[List[LayerDesc], dict]:
+    layers = []
+    first_run: Dict[int, int] = {}
+    for r, (i, t) in enumerate(_layer_runs(cfg)):
+        l = cfg["layers"][i]
+        m = l["mixer"]
+        d = LayerDesc()
+        d.block_kind = capi.BLOCK_PARALLEL
+        if l["type"] == "attention":
+            d.mixer_kind = capi.MIXER_ATTENTION
+            d.n_heads, d.n_kv_heads, d.qk_dim, d.v_dim = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+            d.score_scale = m["scale"]
+            d.proj_bias, d.qk_norm, d.out_gate = 2, capi.QKNORM_HEAD_W, capi.GATE_HEAD
+            qt = m.get("q_temp")
+            if qt:
+                d.q_temp_coef, d.q_temp_every = float(qt["coef"]), float(qt["every"])
+        elif l["type"] == "latent_attention":
+            d.mixer_kind = capi.MIXER_LATENT
+            d.n_heads, d.n_kv_heads, d.qk_dim, d.v_dim = m["heads"], 1, m["dim"], m["vdim"]
+            d.score_scale = m["scale"]
+            d.q_rank, d.kv_rank, d.rot_dim = 0, m["kv_rank"], m["rot_dim"]
+            d.rope_dims, d.rope_base, d.rope_interleaved = int(m["rot"].get("dims", d.rot_dim)), float(m["rot"]["base"]), 1
+            d.sink = capi.SINK_LEARNED
+        elif l["type"] == "rglru":
+            d.mixer_kind = capi.MIXER_RGLRU
+            d.rec_width, d.rec_blocks, d.conv_taps, d.rec_rate = m["width"], m["blocks"], m["conv"], _MOMEDRA_RG_RATE
+        else:
+            raise capi.PsCudaError(f"Momedra layer {i}: unknown mixer type {l['type']!r}")
+        mlp = l.get("mlp")
+        if mlp is None:
+            d.mlp_kind = capi.MLP_NONE
+        else:
+            d.mlp_ungated, d.act_kind = 1, capi.ACT_RELU2
+            if mlp.get("kind") == "dense":
+                d.mlp_kind, d.expert_ff = capi.MLP_DENSE, mlp["ff"]
+            elif mlp.get("kind") == "moe":
+                d.mlp_kind = capi.MLP_ROUTED
+                d.n_experts, d.top_k, d.expert_ff = mlp["router"]["experts"], mlp["router"]["top"], mlp["expert"]["ff"]
+                d.router_act, d.router_bias = capi.ROUTER_TOPK_SOFTMAX, 1
+                if mlp.get("shared"):
+                    d.shared_ff = mlp["shared"]["ff"]
+            else:
+                raise capi.PsCudaError(f"Momedra layer {i}: unknown feed-forward kind {mlp.get('kind')!r}")
+        if i in first_run:
+            d.share_weights = first_run[i] + 1
+        else:
+            first_run[i] = r
+        d.pass_in = int(t is not None)
+        layers.append(d)
+    top = {"dim": cfg["width"], "vocab_size": cfg["vocab"], "norm_eps": cfg["norm"]["eps"], "embed_scale": 1.0, "norm_unit_offset": 0,
+           "norm_kind": capi.NORM_LAYER, "residual_scale": float(cfg["residual_mult"])}
+    return layers, top
+
+
+def _momedra_tensor_names(cfg: dict) -> dict:
+    out = {"embed": "embed", "final_norm": "final.norm", "head": "head", "layers": []}
+    seen = set()
+    for i, t in _layer_runs(cfg):
+        if t is not None:
+            out["pass_in"] = "loop.in"
+        if i in seen:                 # a repeated run: the weights of its first run
+            out["layers"].append({})
+            continue
+        seen.add(i)
+        l = cfg["layers"][i]
+        p, a = f"l{i}.", f"l{i}.mix."
+        n = {"norm": p + "norm1", "o": a + "o"}
+        if l["type"] == "attention":
+            n.update({"q": a + "q", "q_bias": a + "q.b", "k": a + "k", "k_bias": a + "k.b", "v": a + "v", "v_bias": a + "v.b", "q_norm": a + "q.norm", "k_norm": a + "k.norm",
+                      "g": a + "g"})
+        elif l["type"] == "latent_attention":
+            n.update({"q": a + "q", "dkv": a + "dkv", "dkv_norm": a + "dkv.norm", "uk": a + "uk", "uv": a + "uv", "sink": a + "sink"})
+        else:
+            n.update({"rec_y": a + "y", "rec_y_bias": a + "y.b", "rec_x": a + "x", "rec_x_bias": a + "x.b", "conv_w": a + "conv", "conv_b": a + "conv.b", "rec_r": a + "ra",
+                      "rec_r_bias": a + "ra.b", "rec_i": a + "ri", "rec_i_bias": a + "ri.b", "rec_lam": a + "lam"})
+        mlp = l.get("mlp")
+        if mlp is not None and mlp.get("kind") == "moe":
+            E = mlp["router"]["experts"]
+            n.update({"router": p + "mlp.router", "router_bias": p + "mlp.router.b", "up": [f"{p}mlp.e{e}.up" for e in range(E)], "down": [f"{p}mlp.e{e}.down" for e in range(E)]})
+            if mlp.get("shared"):
+                n.update({"shared_up": p + "mlp.shared.up", "shared_down": p + "mlp.shared.down"})
+        elif mlp is not None:
+            n.update({"up": [p + "mlp.up"], "down": [p + "mlp.down"]})
+        out["layers"].append(n)
+    return out
+
+
 ARCHITECTURES: Dict[str, Tuple[Callable, Callable]] = {
     "Dozotar": (_dozotar_describe, _dozotar_tensor_names),
+    "Momedra": (_momedra_describe, _momedra_tensor_names),
     "Pidenex": (_pidenex_describe, _pidenex_tensor_names),
     "Nufusun": (_nufusun_describe, _nufusun_tensor_names),
     "Vanapel": (_vanapel_describe, _vanapel_tensor_names),

@@ -297,7 +297,7 @@ def run_size_pidenex(name, prompt_len, steps, warmup, seed, chunk):
     m = _load_synth(cfg, arch_synth.pidenex_weights(cfg, seed=seed, fast=True), chunk, n_ctx)
     t_pre, t_dec, launches, e2e = _measure(m, prompt, chunk, steps, warmup)
     m.close()
-    runs = "".join(kinds[i] for i, _ in arch._pidenex_runs(cfg))
+    runs = "".join(kinds[i] for i, _ in arch._layer_runs(cfg))
     na, npar, nlat = runs.count("a"), runs.count("p"), runs.count("l")
     p_att = (H + G) * hs * W + H * hs * W
     p_par = (H + G) * hs * W + 2 * H * hs * W + 4 * R * W

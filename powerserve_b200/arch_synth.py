@@ -330,3 +330,102 @@ def pidenex_weights(cfg: dict, seed: int = 0, fast: bool = False) -> Dict[str, n
             t[p + "norm2"], t[p + "norm2b"] = vec(W, 1.0), vec(W, 0.5)
             t[p + "mlp.up"], t[p + "mlp.down"], t[p + "mlp.act"] = mat(ff, W, 1.5), mat(W, ff), rnd(rng.standard_normal(2).astype(np.float32))
     return t
+
+
+# ------------------------------------------------------------------------------------------------------------ Momedra
+def _momedra_mlp(ff: int = 0, experts: int = 0, top: int = 1, shared_ff: int = 0) -> Optional[dict]:
+    """ff == 0: no feed-forward; experts == 0: dense of ff rows; else routed experts of ff rows (+ a shared expert of shared_ff rows)"""
+    if not ff:
+        return None
+    if not experts:
+        return {"kind": "dense", "ff": ff}
+    mlp = {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": experts, "top": top}}
+    if shared_ff:
+        mlp["shared"] = {"ff": shared_ff}
+    return mlp
+
+
+def momedra_attention_layer(heads: int, kv_heads: int, dim: int, vdim: int, *, scale: Optional[float] = None, q_temp: Optional[tuple] = (0.4, 100), **mlp) -> dict:
+    """q_temp = (coef, every) or None"""
+    mixer = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": float(scale if scale is not None else dim ** -0.5)}
+    if q_temp:
+        mixer["q_temp"] = {"coef": q_temp[0], "every": q_temp[1]}
+    return {"type": "attention", "mixer": mixer, "mlp": _momedra_mlp(**mlp)}
+
+
+def momedra_latent_layer(heads: int, dim: int, rot_dim: int, vdim: int, kv_rank: int, *, scale: Optional[float] = None, rope_base: float = 10000.0, **mlp) -> dict:
+    mixer = {"heads": heads, "dim": dim, "rot_dim": rot_dim, "vdim": vdim, "kv_rank": kv_rank, "rot": {"base": rope_base, "dims": rot_dim},
+             "scale": float(scale if scale is not None else (dim + rot_dim) ** -0.5)}
+    return {"type": "latent_attention", "mixer": mixer, "mlp": _momedra_mlp(**mlp)}
+
+
+def momedra_rglru_layer(width: int, blocks: int, *, conv: int = 3, **mlp) -> dict:
+    return {"type": "rglru", "mixer": {"width": width, "blocks": blocks, "conv": conv}, "mlp": _momedra_mlp(**mlp)}
+
+
+def momedra_config(width: int, vocab: int, layers: List[dict], *, loop: Optional[tuple] = None, eps: float = 1e-5, residual_mult: float = 0.6) -> dict:
+    """loop = (start, stop, times): the layers start .. stop - 1 run `times` times with the same weights"""
+    a, b, n = loop if loop else (0, 0, 1)
+    return {"architecture": "Momedra", "layers": layers, "loop": {"start": a, "stop": b, "times": n}, "norm": {"eps": eps}, "residual_mult": residual_mult,
+            "vocab": vocab, "width": width}
+
+
+def momedra_weights(cfg: dict, seed: int = 0, fast: bool = False) -> Dict[str, np.ndarray]:
+    """float32 arrays of bfloat16-representable values keyed by tensor name (fast = True: big matrices as random bfloat16 bit patterns)"""
+    rng = np.random.default_rng(seed)
+    W, V = cfg["width"], cfg["vocab"]
+
+    def rnd(a):
+        return (safetensors.float32_to_bf16_bits(np.asarray(a, np.float32)).astype(np.uint32) << 16).view(np.float32)
+
+    def mat(out_dim, in_dim, gain=1.0):
+        if fast:
+            e = int(np.floor(np.log2(gain / np.sqrt(in_dim)))) + 127
+            bits = rng.integers(0, 1 << 7, size=(out_dim, in_dim), dtype=np.uint16) | np.uint16(e << 7)
+            return bits | (rng.integers(0, 2, size=(out_dim, in_dim), dtype=np.uint16) << 15).astype(np.uint16)
+        return rnd(rng.standard_normal((out_dim, in_dim), dtype=np.float32) * np.float32(gain / np.sqrt(in_dim)))
+
+    def vec(n, mean=0.0, dev=0.1):
+        return rnd(mean + rng.standard_normal(n).astype(np.float32) * dev)
+
+    t: Dict[str, np.ndarray] = {"embed": mat(V, W, np.sqrt(W)), "final.norm": vec(W, 1.0), "head": mat(V, W)}
+    lp = cfg.get("loop") or {}
+    if lp.get("stop", 0) > lp.get("start", 0):
+        t["loop.in"] = mat(W, 2 * W)
+    for i, l in enumerate(cfg["layers"]):
+        p, a, m = f"l{i}.", f"l{i}.mix.", l["mixer"]
+        t[p + "norm1"] = vec(W, 1.0)
+        if l["type"] == "attention":
+            H, G, dq, dv = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+            t[a + "q"], t[a + "k"], t[a + "v"] = mat(H * dq, W), mat(G * dq, W), mat(G * dv, W)
+            t[a + "q.b"], t[a + "k.b"], t[a + "v.b"] = vec(H * dq, 0.0, 0.3), vec(G * dq, 0.0, 0.3), vec(G * dv, 0.0, 0.3)
+            t[a + "q.norm"], t[a + "k.norm"] = vec(dq, 1.4, 0.3), vec(dq, 1.4, 0.3)
+            t[a + "g"], t[a + "o"] = mat(H, W, 2.0), mat(W, H * dv)
+        elif l["type"] == "latent_attention":
+            H, dn, dr, dv, rk = m["heads"], m["dim"], m["rot_dim"], m["vdim"], m["kv_rank"]
+            t[a + "q"], t[a + "dkv"], t[a + "dkv.norm"] = mat(H * (dn + dr), W, 2.0), mat(rk + dr, W), vec(rk, 1.0)
+            t[a + "uk"], t[a + "uv"], t[a + "o"] = mat(H * dn, rk, 1.5), mat(H * dv, rk), mat(W, H * dv)
+            t[a + "sink"] = vec(H, 0.5, 1.0)
+        else:
+            R, nb, taps = m["width"], m["blocks"], m["conv"]
+            s = R // nb
+            t[a + "y"], t[a + "y.b"], t[a + "x"], t[a + "x.b"] = mat(R, W), vec(R, 0.0, 0.3), mat(R, W), vec(R, 0.0, 0.3)
+            t[a + "conv"] = rnd(rng.standard_normal((R, taps)) * 0.4 + np.eye(taps)[taps - 1])
+            t[a + "conv.b"] = vec(R, 0.0, 0.2)
+            t[a + "ra"], t[a + "ri"] = mat(nb * s, s, 1.5).reshape(nb, s, s), mat(nb * s, s, 1.5).reshape(nb, s, s)
+            t[a + "ra.b"], t[a + "ri.b"] = vec(R, 0.0, 0.3).reshape(nb, s), vec(R, 0.0, 0.3).reshape(nb, s)
+            t[a + "lam"] = rnd(rng.uniform(-7.0, -2.0, R))
+            t[a + "o"] = mat(W, R)
+        f = l.get("mlp")
+        if f is None:
+            continue
+        if f["kind"] == "dense":
+            t[p + "mlp.up"], t[p + "mlp.down"] = mat(f["ff"], W), mat(W, f["ff"])
+        else:
+            E = f["router"]["experts"]
+            t[p + "mlp.router"], t[p + "mlp.router.b"] = mat(E, W, 2.0), vec(E, 0.0, 0.5)
+            for e in range(E):
+                t[p + f"mlp.e{e}.up"], t[p + f"mlp.e{e}.down"] = mat(f["expert"]["ff"], W), mat(W, f["expert"]["ff"])
+            if f.get("shared"):
+                t[p + "mlp.shared.up"], t[p + "mlp.shared.down"] = mat(f["shared"]["ff"], W), mat(W, f["shared"]["ff"])
+    return t

@@ -61,6 +61,14 @@ struct PsArchLayer {
     float act_a = 0.f, act_b = 0.f;       // xIELU: softplus(p), 1/2 + softplus(q)
     int n_pool = 0;                       // pooled blocks of a cache set, padded to a multiple of 4
     int64_t state_off = 0;                // the side mixer's state in the K buffer (floats from its start)
+    // general parallel blocks: ONE product reads the normed input - rows [mixer's projections (pw) | up rows of the feed-forward or the
+    // shared expert (upn)] - and one writes the residual: [W_o | W_down] over [mixer's heads | activated up rows].  A projected row keeps
+    // the mixer's columns first, then from o_off on the heads' outputs (od columns) right before the up columns
+    bool gpar = false;
+    int upn = 0, o_off = 0, ldp = 0;
+    float *router_b = nullptr;
+    bf16 *wri = nullptr;                  // rg-lru: [block][r rows | i rows][W / blocks]
+    float *rec_rb = nullptr, *rec_ib = nullptr, *rec_sp = nullptr; // gate biases; rec_rate * softplus(lam)
 };
 
 static inline PaAct pa_act_of(const ps_cuda_layer_desc &l) { return PaAct{l.act_limit, l.act_alpha, l.up_shift, l.act_kind}; }
@@ -113,8 +121,16 @@ struct PsArch {
     int opt_prefetch = 1; // 1: a mat-vec CTA requests its first row group into L2 before the dependency wait; 2: every next group too
     int opt_pdl = 1;    // single-token kernels on the main stream are launched with programmatic stream serialisation
     int opt_scan_nc = 0; // value columns per lane of the recurrence scan (0: chosen by the grid's size)
-    bool has_seq = false, has_par = false; // some layer is a sequential / a parallel block
+    bool has_seq = false, has_par = false; // some block's output waits for the next seam (sequential, general parallel) / joins the stream itself
     bool keep_embed = false;               // some run adds the embedding output back
+    float res_scale = 1.0f;                // factor on what a block adds to the residual stream
+    bool has_pass_in = false;              // some run opens with x <- W_in [x; embedding output]
+    bf16 *pass_in = nullptr;
+    uint8_t *t_pass_in = nullptr;
+    float *xcat = nullptr;                 // [max_batch][2 dim]: stream | embedding output
+    float *gts = nullptr;                  // rg-lru: gate logits of a batch
+    float *hn = nullptr;                   // single-token step: the normed input, for the experts
+    int max_rec = 0;
 };
 
 namespace {
@@ -272,31 +288,121 @@ extern "C" float ps_cuda_host_rope_freq(int dims, float base, float factor, int 
     return (float)m;
 }
 
+// a parallel block that needs more than Nufusun's: its output waits for the next seam like a sequential block's
+static bool pa_general_parallel(const ps_cuda_arch_desc &d, const ps_cuda_layer_desc &l) {
+    if (l.block_kind != PS_BLOCK_PARALLEL) return false;
+    return d.norm_kind == PS_NORM_LAYER || (d.residual_scale != 0.f && d.residual_scale != 1.0f) || l.pass_in || l.mixer_kind == PS_MIXER_LATENT || l.mixer_kind == PS_MIXER_RGLRU ||
+           l.mlp_ungated || l.mlp_kind == PS_MLP_DENSE || l.qk_norm || l.q_temp_coef != 0.f || l.out_gate || l.proj_bias == 2;
+}
+
+// sizes, limits and workspace needs of one general parallel block
+static int par_layer_sizes(PsArch *a, int i, std::string &err) {
+    const ps_cuda_arch_desc &d = a->d;
+    PsArchLayer &w = a->L[(size_t)i];
+    const ps_cuda_layer_desc &l = w.d;
+    const bool latent = l.mixer_kind == PS_MIXER_LATENT, rec = l.mixer_kind == PS_MIXER_RGLRU, routed = l.mlp_kind == PS_MLP_ROUTED;
+#define PA_BAD(...) return afail(err, PS_CUDA_ERR_UNSUPPORTED, __VA_ARGS__)
+    if (l.raw_input || l.post_norm || l.v_mix || l.v_is_k || l.pool || l.side_kind || l.head_mix || l.head_temp || d.norm_groups > 1 || d.norm_unit_offset || d.norm_scalar || (l.conv_taps > 0 && !rec))
+        PA_BAD("layer %d: raw inputs, output norms, value blending, values from keys, pooled windows, side mixers, head mixing / temperatures and group, offset or scalar norms are not combined with a general parallel block", i);
+    if (l.mixer_kind != PS_MIXER_ATTENTION && !latent && !rec) PA_BAD("layer %d: mixer kind %d in a general parallel block", i, l.mixer_kind);
+    if (l.mlp_kind != PS_MLP_NONE && !routed && l.mlp_kind != PS_MLP_DENSE) PA_BAD("layer %d: unknown feed-forward kind %d", i, l.mlp_kind);
+    if (l.mlp_kind != PS_MLP_NONE && (!l.mlp_ungated || l.expert_ff <= 0 || l.act_kind < PS_ACT_SWISH || l.act_kind > PS_ACT_RELU2 || l.act_kind == PS_ACT_XIELU))
+        PA_BAD("layer %d: a general parallel block's feed-forward has no gate (%d rows, activation %d)", i, l.expert_ff, l.act_kind);
+    if (routed && (l.n_experts <= 0 || l.n_experts > PA_MAX_EXPERTS || l.top_k <= 0 || l.top_k > l.n_experts || l.shared_ff < 0 || l.shared_gate || l.route_on_input ||
+                   l.router_act != PS_ROUTER_TOPK_SOFTMAX || l.route_groups > 1))
+        PA_BAD("layer %d: unsupported routed feed-forward (%d experts, top %d, router activation %d, shared expert of %d rows)", i, l.n_experts, l.top_k, l.router_act, l.shared_ff);
+    if ((size_t)d.dim * (l.pass_in ? 8 : 4) > 160 * 1024) PA_BAD("layer %d: width %d exceeds the single-token kernels' shared memory", i, d.dim);
+    if (rec) {
+        if (l.rec_width <= 0 || l.rec_blocks <= 0 || l.rec_width % l.rec_blocks || l.conv_taps < 1 || l.conv_taps > 64 || l.rec_width / l.rec_blocks > 8192)
+            PA_BAD("layer %d: rg-lru of %d channels in %d blocks, %d taps", i, l.rec_width, l.rec_blocks, l.conv_taps);
+        w.pw = 2 * l.rec_width; // y | x
+        w.od = l.rec_width;
+        w.conv_c = l.rec_width;
+        w.k_floats = l.rec_width;
+        w.v_floats = (int64_t)l.conv_taps * l.rec_width;
+        a->has_state = true;
+        a->max_cv = std::max(a->max_cv, l.rec_width);
+        a->max_rec = std::max(a->max_rec, l.rec_width);
+    } else {
+        const int dq = latent ? l.kv_rank + l.rot_dim : l.qk_dim, dv = latent ? l.kv_rank : l.v_dim;
+        if (l.n_heads <= 0 || l.n_heads > PA_MAX_HEADS || l.n_kv_heads <= 0 || l.n_heads % l.n_kv_heads || l.qk_dim <= 0 || l.v_dim <= 0 || l.window < 0 || l.chunk < 0)
+            PA_BAD("layer %d: unsupported head geometry (%d / %d heads, sizes %d / %d; at most %d heads)", i, l.n_heads, l.n_kv_heads, l.qk_dim, l.v_dim, PA_MAX_HEADS);
+        if (l.sink < PS_SINK_NONE || l.sink > PS_SINK_LEARNED || l.rel_buckets || l.log_bias || l.lin_bias || (l.proj_bias != 0 && l.proj_bias != 2) || (l.out_gate != PS_GATE_NONE && l.out_gate != PS_GATE_HEAD) ||
+            l.qk_norm == PS_QKNORM_WHOLE || l.qk_norm > PS_QKNORM_HEAD_W || (l.q_temp_coef != 0.f && (!(l.q_temp_every > 0.f) || l.qk_norm == PS_QKNORM_NONE)))
+            PA_BAD("layer %d: sink %d, biases %d, gate %d, q / k norm %d, query temperature %g / %g", i, l.sink, l.proj_bias, l.out_gate, l.qk_norm, (double)l.q_temp_coef, (double)l.q_temp_every);
+        if (latent && (l.q_rank != 0 || l.kv_rank <= 0 || l.rot_dim < 0 || l.rope_dims < 0 || l.rope_dims > l.rot_dim || (l.rope_dims & 1) || (l.rope_dims > 0 && !(l.rope_base > 0.f)) || l.n_kv_heads != 1 ||
+                       l.proj_bias || l.out_gate || l.qk_norm))
+            PA_BAD("layer %d: unsupported latent attention (ranks %d / %d, %d rotated dims of which %d rotate)", i, l.q_rank, l.kv_rank, l.rot_dim, l.rope_dims);
+        if (pa_dec_scores_smem(l.n_heads, l.n_kv_heads, dq) > 160 * 1024) PA_BAD("layer %d: %d heads of size %d exceed the single-token kernels' shared memory", i, l.n_heads, dq);
+        w.qd = l.n_heads * dq; w.kd = l.n_kv_heads * dq; w.vd = l.n_kv_heads * dv; w.od = l.n_heads * l.v_dim;
+        w.v_off = w.qd + w.kd;
+        if (latent) {
+            w.pw = l.n_heads * (l.qk_dim + l.rot_dim) + l.kv_rank + l.rot_dim; // q | kv latent | rotated key part
+            a->max_qa = std::max(a->max_qa, w.qd);
+        } else {
+            w.pw = w.qd + w.kd + w.vd;
+            if (l.out_gate) { w.g_off = w.pw; w.pw += l.n_heads; }
+        }
+        a->max_h = std::max(a->max_h, l.n_heads);
+        a->max_dv = std::max(a->max_dv, dv);
+        w.aw = l.n_heads * dv;
+        a->max_od = std::max(a->max_od, w.aw);
+    }
+    w.ho = w.od;
+    w.upn = l.mlp_kind == PS_MLP_DENSE ? l.expert_ff : routed ? l.shared_ff : 0;
+    w.o_off = (w.pw + 7) & ~7;
+    w.ldp = (w.o_off + w.od + w.upn + 7) & ~7;
+    a->max_qkv = std::max(a->max_qkv, w.ldp);
+    a->max_k = std::max(a->max_k, std::max(l.pass_in ? 2 * d.dim : d.dim, w.od + w.upn));
+    if (routed) {
+        a->max_top = std::max(a->max_top, l.top_k);
+        a->max_ff = std::max(a->max_ff, l.expert_ff);
+        a->max_e = std::max(a->max_e, l.n_experts);
+        a->max_k = std::max(a->max_k, l.expert_ff);
+    }
+#undef PA_BAD
+    return 0;
+}
+
 int ps_arch_create(PsArch **out, const ps_cuda_arch_desc *desc, std::string &err) {
     *out = nullptr;
     const ps_cuda_arch_desc &d = *desc;
     if (d.dim <= 0 || d.vocab_size <= 0 || d.n_layers <= 0 || d.n_ctx <= 0 || d.max_batch <= 0 || !d.layers)
         return afail(err, PS_CUDA_ERR_INVALID, "layer-list descriptor has non-positive fields");
     if (d.compute != PS_COMPUTE_BF16 && d.compute != PS_COMPUTE_F32) return afail(err, PS_CUDA_ERR_INVALID, "unknown compute mode %d", d.compute);
+    if (d.norm_kind != PS_NORM_RMS && d.norm_kind != PS_NORM_LAYER) return afail(err, PS_CUDA_ERR_INVALID, "unknown norm kind %d", d.norm_kind);
     if (d.norm_groups < 0 || (d.norm_groups > 1 && d.dim % d.norm_groups)) return afail(err, PS_CUDA_ERR_INVALID, "width %d does not split into %d norm groups", d.dim, d.norm_groups);
     PsArch *a = new PsArch();
     a->d = d;
     a->round = d.compute == PS_COMPUTE_BF16;
+    a->res_scale = d.residual_scale != 0.f ? d.residual_scale : 1.0f;
     a->L.resize((size_t)d.n_layers);
     auto bail = [&](int rc) { ps_arch_destroy(a); return rc; };
     for (int i = 0; i < d.n_layers; i++) {
         const ps_cuda_layer_desc &l = d.layers[i];
         PsArchLayer &w = a->L[(size_t)i];
         w.d = l;
-        (l.block_kind == PS_BLOCK_SEQUENTIAL ? a->has_seq : a->has_par) = true;
+        w.gpar = pa_general_parallel(d, l);
+        (l.block_kind == PS_BLOCK_SEQUENTIAL || w.gpar ? a->has_seq : a->has_par) = true;
         if (l.pass_embed) a->keep_embed = true;
+        if (l.pass_in) a->has_pass_in = true;
+        if ((l.pass_embed && a->has_pass_in) || (l.pass_in && a->keep_embed)) return bail(afail(err, PS_CUDA_ERR_UNSUPPORTED, "layer %d: passes either add the embedding output or project it in", i));
+        if (l.pass_in && !w.gpar) return bail(afail(err, PS_CUDA_ERR_UNSUPPORTED, "layer %d: a pass that projects the embedding output in opens at a general parallel block", i));
         if ((l.pass_embed || l.pass_step) && l.block_kind != PS_BLOCK_SEQUENTIAL) return bail(afail(err, PS_CUDA_ERR_UNSUPPORTED, "layer %d: passes open at sequential blocks", i));
         if (l.share_weights < 0 || l.share_weights > i || l.pass_embed < 0 || l.pass_step < 0 || l.pass_step > d.n_pass_steps)
             return bail(afail(err, PS_CUDA_ERR_INVALID, "layer %d: shares the weights of run %d, pass step %d of %d", i, l.share_weights - 1, l.pass_step, d.n_pass_steps));
         if (l.share_weights > 0 && memcmp(&d.layers[l.share_weights - 1], &l, offsetof(ps_cuda_layer_desc, share_weights)) != 0)
             return bail(afail(err, PS_CUDA_ERR_INVALID, "layer %d: a run that shares weights must have the sizes of run %d", i, l.share_weights - 1));
-        if (l.mixer_kind < PS_MIXER_ATTENTION || l.mixer_kind > PS_MIXER_MAMBA2) return bail(afail(err, PS_CUDA_ERR_UNSUPPORTED, "layer %d: unknown mixer kind %d", i, l.mixer_kind));
+        if (l.mixer_kind < PS_MIXER_ATTENTION || l.mixer_kind > PS_MIXER_RGLRU || l.mixer_kind == PS_MIXER_MINGRU) return bail(afail(err, PS_CUDA_ERR_UNSUPPORTED, "layer %d: unknown mixer kind %d", i, l.mixer_kind));
+        if (w.gpar) {
+            const int rc = par_layer_sizes(a, i, err);
+            if (rc) return bail(rc);
+            continue;
+        }
         const bool latent = l.mixer_kind == PS_MIXER_LATENT, recur = pa_recurrent(l);
+        if (l.mixer_kind == PS_MIXER_RGLRU || l.act_kind == PS_ACT_RELU2 || l.qk_norm == PS_QKNORM_HEAD_W || l.out_gate == PS_GATE_HEAD || l.q_temp_coef != 0.f || l.proj_bias == 2 || l.router_bias ||
+            l.router_act == PS_ROUTER_TOPK_SOFTMAX)
+            return bail(afail(err, PS_CUDA_ERR_UNSUPPORTED, "layer %d: rg-lru, squared relu, weighted head norms, gates per head, query temperatures, q / k / v-only and router biases need a general parallel block", i));
         const bool newer = l.v_is_k || l.pool > 0 || l.lin_bias || l.out_gate || l.side_kind; // mechanisms of the general sequential layer only
         w.gen2 = l.block_kind == PS_BLOCK_SEQUENTIAL && !latent &&
                  (l.raw_input || recur || l.conv_taps > 0 || l.qk_norm == PS_QKNORM_WHOLE || l.chunk > 0 || l.mlp_kind == PS_MLP_ROUTED || l.rel_buckets > 0 ||
@@ -317,7 +423,7 @@ int ps_arch_create(PsArch **out, const ps_cuda_arch_desc *desc, std::string &err
             return bail(afail(err, PS_CUDA_ERR_UNSUPPORTED, "layer %d: latent attention, value blending, per-head unit norms, projection biases and head mixing are not combined with this layer's other mechanisms", i));
         if (w.gen2 && l.mlp_kind == PS_MLP_ROUTED && !l.raw_input && d.norm_groups > 1)
             return bail(afail(err, PS_CUDA_ERR_UNSUPPORTED, "layer %d: routed experts behind a group norm", i));
-        if (l.chunk < 0 || l.conv_taps < 0 || l.conv_taps > 64 || l.act_kind < PS_ACT_SWISH || l.act_kind > PS_ACT_XIELU || l.shared_ff < 0)
+        if (l.chunk < 0 || l.conv_taps < 0 || l.conv_taps > 64 || l.act_kind < PS_ACT_SWISH || l.act_kind > PS_ACT_RELU2 || l.shared_ff < 0)
             return bail(afail(err, PS_CUDA_ERR_UNSUPPORTED, "layer %d: chunk %d, %d convolution taps, activation %d, shared expert of %d rows", i, l.chunk, l.conv_taps, l.act_kind, l.shared_ff));
         if (l.mixer_kind == PS_MIXER_RETENTION && (l.rope_dims < 0 || l.rope_dims > l.qk_dim || (l.rope_dims & 1) || (l.rope_dims > 0 && !(l.rope_base > 0.f)) || l.qk_dim > 256 || l.rope_factor != 0.f))
             return bail(afail(err, PS_CUDA_ERR_UNSUPPORTED, "layer %d: retention with heads of %d of which %d rotate (at most 256)", i, l.qk_dim, l.rope_dims));
@@ -418,7 +524,6 @@ int ps_arch_create(PsArch **out, const ps_cuda_arch_desc *desc, std::string &err
     }
     a->d.layers = nullptr; // the caller's array need not outlive this call: the copies live in L
     const int64_t B = d.max_batch, dim = d.dim;
-    if (d.norm_kind != PS_NORM_RMS && d.norm_kind != PS_NORM_LAYER) return bail(afail(err, PS_CUDA_ERR_INVALID, "unknown norm kind %d", d.norm_kind));
     a->pool_off = (d.n_ctx + 3) & ~3;
     a->ldS = (int64_t)a->pool_off + a->max_pool; // a score row: the tokens, then the pooled blocks
     int rc = 0;
@@ -461,6 +566,10 @@ int ps_arch_create(PsArch **out, const ps_cuda_arch_desc *desc, std::string &err
         AL(a->qa, 4 * (size_t)a->max_qa * B);
         AL(a->att2, 4 * (size_t)a->max_att2 * B);
     }
+    if (a->max_qa && !a->qa) AL(a->qa, 4 * (size_t)a->max_qa * B);
+    if (a->has_pass_in) AL(a->xcat, 8 * dim * B);
+    if (a->max_rec) AL(a->gts, 8 * (size_t)a->max_rec * B);
+    AL(a->hn, 4 * dim);
     if (a->vsrc_w) AL(a->vsrc, 4 * (size_t)a->vsrc_w * B);
     if (rc) return bail(rc);
     int dev = 0;
@@ -532,6 +641,108 @@ int ps_arch_set_option(PsArch *a, const char *name, int value) {
     return 0;
 }
 
+// latent attention: W_uk [H * dn][rk] -> per head transposed [H][rk][dn], q_h . (W_uk,h c) = (W_uk,h^T q_h) . c; the rotation's frequencies
+static int latent_bind(PsArch *a, PsArchLayer &w, const ps_cuda_arch_layer_weights &s, std::string &err) {
+    const ps_cuda_layer_desc &l = w.d;
+    const size_t H = (size_t)l.n_heads, rk = (size_t)l.kv_rank, dn = (size_t)l.qk_dim;
+    int rc;
+    if (!s.uk.host || s.uk.type != PS_TYPE_BF16) return afail(err, PS_CUDA_ERR_INVALID, "bind: matrix uk is missing or not bfloat16");
+    std::vector<uint16_t> tr(H * rk * dn);
+    const uint16_t *src = static_cast<const uint16_t *>(s.uk.host);
+    for (size_t hh = 0; hh < H; hh++)
+        for (size_t r = 0; r < dn; r++)
+            for (size_t c = 0; c < rk; c++) tr[(hh * rk + c) * dn + r] = src[(hh * dn + r) * rk + c];
+    if ((rc = aalloc(a, (void **)&w.wukt, 2 * tr.size(), err))) return rc;
+    PA_CK(cudaMemcpy(w.wukt, tr.data(), 2 * tr.size(), cudaMemcpyHostToDevice));
+    if (l.rope_dims > 0) {
+        std::vector<double> fd((size_t)l.rope_dims / 2);
+        w.rope_mscale = (float)rope_freq_host(l.rope_dims, l.rope_base, l.rope_factor, l.rope_original, l.rope_fast, l.rope_slow, fd.data());
+        if ((rc = aalloc(a, (void **)&w.rope_freq, fd.size() * 8, err))) return rc;
+        PA_CK(cudaMemcpy(w.rope_freq, fd.data(), fd.size() * 8, cudaMemcpyHostToDevice));
+    }
+    return 0;
+}
+
+// weights of one general parallel block (its norm is bound already)
+static int par_layer_bind(PsArch *a, PsArchLayer &w, const ps_cuda_arch_layer_weights &s, int i, std::string &err) {
+    const ps_cuda_layer_desc &l = w.d;
+    const size_t dim = (size_t)a->d.dim, up = (size_t)w.upn, od = (size_t)w.od, H = (size_t)l.n_heads;
+    const bool routed = l.mlp_kind == PS_MLP_ROUTED;
+    int rc;
+    std::vector<float> tmp, bias((size_t)w.pw + up, 0.f);
+    bool biased = false;
+    auto vec = [&](float **dst, const ps_cuda_tensor &t, size_t n, const char *what) -> int {
+        int r = small_to_f32(t, n, tmp, what, err);
+        return r ? r : upload_f32(a, dst, tmp, err);
+    };
+    auto add_bias = [&](const ps_cuda_tensor &t, size_t at, size_t n, const char *what) -> int {
+        int r = small_to_f32(t, n, tmp, what, err);
+        if (!r) std::copy(tmp.begin(), tmp.end(), bias.begin() + (ptrdiff_t)at);
+        biased = true;
+        return r;
+    };
+    if ((rc = aalloc(a, (void **)&w.wqkv, 2 * ((size_t)w.pw + up) * dim, err))) return rc;
+    auto rows = [&](size_t at, const ps_cuda_tensor &t, size_t n, const char *what) { return upload_mat(w.wqkv + at * dim, t, n * dim, what, err); };
+    if (l.mixer_kind == PS_MIXER_LATENT) {
+        const size_t rk = (size_t)l.kv_rank, dr = (size_t)l.rot_dim, lq = H * ((size_t)l.qk_dim + dr);
+        if ((rc = rows(0, s.q, lq, "q")) || (rc = rows(lq, s.dkv, rk + dr, "dkv")) || (rc = vec(&w.dkv_norm, s.dkv_norm, rk, "dkv norm"))) return rc;
+        if ((rc = aalloc(a, (void **)&w.wuv, 2 * od * rk, err)) || (rc = upload_mat(w.wuv, s.uv, od * rk, "uv", err)) || (rc = latent_bind(a, w, s, err))) return rc;
+    } else if (l.mixer_kind == PS_MIXER_RGLRU) {
+        const size_t W = (size_t)l.rec_width, nb = (size_t)l.rec_blocks, bs = W / nb;
+        if ((rc = rows(0, s.rec_y, W, "rec y")) || (rc = rows(W, s.rec_x, W, "rec x")) || (rc = add_bias(s.rec_y_bias, 0, W, "rec y bias")) || (rc = add_bias(s.rec_x_bias, W, W, "rec x bias"))) return rc;
+        if ((rc = vec(&w.conv_w, s.conv_w, W * l.conv_taps, "convolution")) || (rc = vec(&w.conv_b, s.conv_b, W, "convolution bias")) || (rc = vec(&w.rec_rb, s.rec_r_bias, W, "rec r bias")) ||
+            (rc = vec(&w.rec_ib, s.rec_i_bias, W, "rec i bias")))
+            return rc;
+        if (!s.rec_r.host || !s.rec_i.host || s.rec_r.type != PS_TYPE_BF16 || s.rec_i.type != PS_TYPE_BF16) return afail(err, PS_CUDA_ERR_INVALID, "bind: layer %d: the recurrence's gate matrices are missing or not bfloat16", i);
+        std::vector<uint16_t> ri(2 * W * bs);
+        for (size_t b = 0; b < nb; b++) {
+            memcpy(&ri[2 * b * bs * bs], static_cast<const uint16_t *>(s.rec_r.host) + b * bs * bs, 2 * bs * bs);
+            memcpy(&ri[(2 * b + 1) * bs * bs], static_cast<const uint16_t *>(s.rec_i.host) + b * bs * bs, 2 * bs * bs);
+        }
+        if ((rc = aalloc(a, (void **)&w.wri, 2 * ri.size(), err))) return rc;
+        PA_CK(cudaMemcpy(w.wri, ri.data(), 2 * ri.size(), cudaMemcpyHostToDevice));
+        if ((rc = small_to_f32(s.rec_lam, W, tmp, "rec lam", err))) return rc;
+        for (float &v : tmp) v = (float)((double)l.rec_rate * (std::log1p(std::exp(-std::fabs((double)v))) + std::max((double)v, 0.0)));
+        if ((rc = upload_f32(a, &w.rec_sp, tmp, err))) return rc;
+    } else {
+        const size_t nq = (size_t)w.qd, nk = (size_t)w.kd, nv = (size_t)w.vd;
+        if ((rc = rows(0, s.q, nq, "q")) || (rc = rows(nq, s.k, nk, "k")) || (rc = rows(nq + nk, s.v, nv, "v"))) return rc;
+        if (l.out_gate && (rc = rows((size_t)w.g_off, s.g, H, "head gate"))) return rc;
+        if (l.proj_bias && ((rc = add_bias(s.q_bias, 0, nq, "q bias")) || (rc = add_bias(s.k_bias, nq, nk, "k bias")) || (rc = add_bias(s.v_bias, nq + nk, nv, "v bias")))) return rc;
+        if (l.qk_norm == PS_QKNORM_HEAD_W && ((rc = vec(&w.q_norm, s.q_norm, (size_t)l.qk_dim, "q norm")) || (rc = vec(&w.k_norm, s.k_norm, (size_t)l.qk_dim, "k norm")))) return rc;
+    }
+    if (l.sink == PS_SINK_LEARNED && (rc = vec(&w.sink_v, s.sink, H, "sink logits"))) return rc;
+    // [W_o | W_down]: every output row reads the heads' outputs, then the activated up rows
+    const ps_cuda_tensor *dn = nullptr;
+    if (l.mlp_kind == PS_MLP_DENSE) {
+        if (!s.up || !s.down) return afail(err, PS_CUDA_ERR_INVALID, "bind: layer %d has no feed-forward tensors", i);
+        if ((rc = rows((size_t)w.pw, s.up[0], up, "up"))) return rc;
+        dn = &s.down[0];
+    } else if (up > 0) {
+        if ((rc = rows((size_t)w.pw, s.shared_up, up, "shared up rows"))) return rc;
+        dn = &s.shared_down;
+    }
+    if (!s.o.host || s.o.type != PS_TYPE_BF16 || (dn && (!dn->host || dn->type != PS_TYPE_BF16))) return afail(err, PS_CUDA_ERR_INVALID, "bind: layer %d: matrix o or down is missing or not bfloat16", i);
+    std::vector<uint16_t> cat(dim * (od + up));
+    for (size_t r = 0; r < dim; r++) {
+        memcpy(&cat[r * (od + up)], static_cast<const uint16_t *>(s.o.host) + r * od, 2 * od);
+        if (dn) memcpy(&cat[r * (od + up) + od], static_cast<const uint16_t *>(dn->host) + r * up, 2 * up);
+    }
+    if ((rc = aalloc(a, (void **)&w.wo, 2 * cat.size(), err))) return rc;
+    PA_CK(cudaMemcpy(w.wo, cat.data(), 2 * cat.size(), cudaMemcpyHostToDevice));
+    if (biased && (rc = upload_f32(a, &w.bqkv, bias, err))) return rc;
+    if (routed) {
+        const size_t E = (size_t)l.n_experts, ff = (size_t)l.expert_ff;
+        if (!s.up || !s.down) return afail(err, PS_CUDA_ERR_INVALID, "bind: layer %d has no expert tensors", i);
+        if ((rc = aalloc(a, (void **)&w.router, 2 * E * dim, err)) || (rc = upload_mat(w.router, s.router, E * dim, "router", err))) return rc;
+        if (l.router_bias && (rc = vec(&w.router_b, s.router_bias, E, "router bias"))) return rc;
+        if ((rc = aalloc(a, (void **)&w.wup, 2 * E * ff * dim, err)) || (rc = aalloc(a, (void **)&w.wdown, 2 * E * ff * dim, err))) return rc;
+        for (size_t e = 0; e < E; e++)
+            if ((rc = upload_mat(w.wup + e * ff * dim, s.up[e], ff * dim, "expert up", err)) || (rc = upload_mat(w.wdown + e * ff * dim, s.down[e], ff * dim, "expert down", err))) return rc;
+    }
+    return 0;
+}
+
 int ps_arch_bind(PsArch *a, const ps_cuda_arch_weights *wt, cudaStream_t stream, std::string &err) {
     (void)stream;
     if (a->bound) return afail(err, PS_CUDA_ERR_INVALID, "bind: a model is already bound");
@@ -560,6 +771,7 @@ int ps_arch_bind(PsArch *a, const ps_cuda_arch_weights *wt, cudaStream_t stream,
         int r = aalloc(a, (void **)dst, 2 * n, err);
         return r ? r : upload_mat(*dst, t, n, what, err);
     };
+    if (a->has_pass_in && (rc = mat(&a->pass_in, wt->pass_in, 2 * dim * dim, "pass input"))) return rc;
     if (d.n_pass_steps > 0 && (rc = vec(&a->pass_steps, wt->pass_steps, (size_t)d.n_pass_steps * dim, "pass steps", false))) return rc;
     a->taps.assign((size_t)d.n_layers, nullptr);
     for (int i = 0; i < d.n_layers; i++) {
@@ -571,27 +783,17 @@ int ps_arch_bind(PsArch *a, const ps_cuda_arch_weights *wt, cudaStream_t stream,
         snprintf(nm, sizeof nm, "layer %d", i);
         if (!l.raw_input && (rc = normvec(&w.norm, s.norm, nm))) return rc;
         const size_t nq = (size_t)w.qd, nk = (size_t)w.kd, nv = (size_t)w.vd;
+        if (w.gpar) {
+            if ((rc = par_layer_bind(a, w, s, i, err))) return rc;
+            continue;
+        }
         if ((rc = aalloc(a, (void **)&w.wqkv, 2 * (size_t)w.pw * dim, err))) return rc;
         if (l.mixer_kind == PS_MIXER_LATENT) {
             const size_t H = (size_t)l.n_heads, rq = (size_t)l.q_rank, rk = (size_t)l.kv_rank, dr = (size_t)l.rot_dim, dn = (size_t)l.qk_dim, dv = (size_t)l.v_dim;
             if ((rc = upload_mat(w.wqkv, s.dq, rq * dim, "dq", err)) || (rc = upload_mat(w.wqkv + rq * dim, s.dkv, (rk + dr) * dim, "dkv", err))) return rc;
             if ((rc = mat(&w.wuq, s.uq, H * (dn + dr) * rq, "uq")) || (rc = mat(&w.wuv, s.uv, H * dv * rk, "uv"))) return rc;
             if ((rc = vec(&w.dq_norm, s.dq_norm, rq, "dq norm", false)) || (rc = vec(&w.dkv_norm, s.dkv_norm, rk, "dkv norm", false))) return rc;
-            // W_uk [H * dn][rk] -> per head transposed [H][rk][dn]: q_h . (W_uk,h c) = (W_uk,h^T q_h) . c
-            if (!s.uk.host || s.uk.type != PS_TYPE_BF16) return afail(err, PS_CUDA_ERR_INVALID, "bind: matrix uk is missing or not bfloat16");
-            std::vector<uint16_t> tr(H * rk * dn);
-            const uint16_t *src = static_cast<const uint16_t *>(s.uk.host);
-            for (size_t hh = 0; hh < H; hh++)
-                for (size_t r = 0; r < dn; r++)
-                    for (size_t c = 0; c < rk; c++) tr[(hh * rk + c) * dn + r] = src[(hh * dn + r) * rk + c];
-            if ((rc = aalloc(a, (void **)&w.wukt, 2 * tr.size(), err))) return rc;
-            PA_CK(cudaMemcpy(w.wukt, tr.data(), 2 * tr.size(), cudaMemcpyHostToDevice));
-            if (l.rope_dims > 0) {
-                std::vector<double> fd((size_t)l.rope_dims / 2);
-                w.rope_mscale = (float)rope_freq_host(l.rope_dims, l.rope_base, l.rope_factor, l.rope_original, l.rope_fast, l.rope_slow, fd.data());
-                if ((rc = aalloc(a, (void **)&w.rope_freq, fd.size() * 8, err))) return rc;
-                PA_CK(cudaMemcpy(w.rope_freq, fd.data(), fd.size() * 8, cudaMemcpyHostToDevice));
-            }
+            if ((rc = latent_bind(a, w, s, err))) return rc;
         } else if (l.mixer_kind == PS_MIXER_MAMBA2) {
             const size_t H = (size_t)l.n_heads;
             if ((rc = upload_mat(w.wqkv, s.w_in, (size_t)w.pw * dim, "in", err))) return rc;
@@ -719,9 +921,16 @@ int ps_arch_bind(PsArch *a, const ps_cuda_arch_weights *wt, cudaStream_t stream,
             return 0;
         };
         if ((rc = tile(&a->t_head, a->head, 1, d.vocab_size, d.dim))) return rc;
+        if (a->pass_in && (rc = tile(&a->t_pass_in, a->pass_in, 1, d.dim, 2 * d.dim))) return rc;
         for (int i = 0; i < d.n_layers; i++) {
             PsArchLayer &w = a->L[(size_t)i];
             if (w.d.share_weights > 0) continue;
+            if (w.gpar) {
+                if ((rc = tile(&w.t_qkv, w.wqkv, 1, w.pw + w.upn, d.dim)) || (rc = tile(&w.t_o, w.wo, 1, d.dim, w.od + w.upn)) ||
+                    (w.d.mlp_kind == PS_MLP_ROUTED && ((rc = tile(&w.t_up, w.wup, w.d.n_experts, w.d.expert_ff, d.dim)) || (rc = tile(&w.t_down, w.wdown, w.d.n_experts, d.dim, w.d.expert_ff)))))
+                    return rc;
+                continue;
+            }
             if ((rc = tile(&w.t_qkv, w.wqkv, 1, w.pw, d.dim)) || (rc = tile(&w.t_o, w.wo, 1, d.dim, w.od))) return rc;
             if (w.wuq && (rc = tile(&w.t_uq, w.wuq, 1, w.d.n_heads * (w.d.qk_dim + w.d.rot_dim), w.d.q_rank))) return rc;
             if (w.d.mlp_kind == PS_MLP_DENSE &&
@@ -775,13 +984,14 @@ static int forward_t(PsArch *a, const PsArchIO &io, int bs, int pos0, int lm_hea
     };
     const bool tc = ROUND && a->opt_tc && !single && !a->opt_simple;
     // C[m][n] = sum_k X[m][k] W[n][k] + bias[n] on the tensor cores: round + tile the activations, then the GEMM
-    auto tc_dense = [&](const float *X, int ldx, int M, int K, const uint8_t *wt, int N, const float *bias, float *C, int ldc, const PaAct *act1 = nullptr) -> int {
+    auto tc_dense = [&](const float *X, int ldx, int M, int K, const uint8_t *wt, int N, const float *bias, float *C, int ldc, const PaAct *act1 = nullptr, int act_from = 0,
+                        int gap = 0) -> int {
         const int nkb = (K + PT_KB - 1) / PT_KB, n_ct = (M + PT_N - 1) / PT_N, n_rt = (N + PT_M - 1) / PT_M;
         pa_k_tc_prep_x<<<dim3((unsigned)nkb, (unsigned)n_ct), 256, 0, st>>>(a->tcx, X, ldx, M, K, nkb, nullptr, nullptr, nullptr, nullptr, nullptr);
         PA_LAUNCH();
         PtArgs g{};
         g.a0 = wt; g.b = a->tcx; g.nkb = nkb; g.n_rt = n_rt; g.n_ct = n_ct; g.M = M; g.N = N; g.mode = PT_MODE_DENSE; g.C = C; g.ldc = ldc; g.bias = bias; g.err = io.err_dev;
-        if (act1) { g.act = *act1; g.act1 = 1; }
+        if (act1) { g.act = *act1; g.act1 = 1; g.act_from = act_from; g.gap = gap; }
         pa_k_tc_gemm<1><<<std::min(a->n_sm, n_ct * n_rt), PT_THREADS, PT_SMEM, st>>>(g);
         PA_LAUNCH();
         return 0;
@@ -801,7 +1011,7 @@ static int forward_t(PsArch *a, const PsArchIO &io, int bs, int pos0, int lm_hea
         return 0;
     };
     // scores -> soft-max -> P.V of a batch against the cache rows 0 .. n_kv - 1 (keys before the first query's window are skipped)
-    auto attend = [&](const PaAttn &at, const float *q, int ldq, int kd, int li, int aw) -> int {
+    auto attend = [&](const PaAttn &at, const float *q, int ldq, int kd, int li, float *out, int aw) -> int {
         int lo0 = at.window > 0 ? std::max(0, pos0 - at.window + 1) : 0; // the first key the first query sees
         if (at.chunk > 0) lo0 = std::max(lo0, pos0 - pos0 % at.chunk);
         const int tile0 = lo0 / PA_TN, tok_tiles = (int)cdiv(n_kv, PA_TN) - tile0;
@@ -811,7 +1021,7 @@ static int forward_t(PsArch *a, const PsArchIO &io, int bs, int pos0, int lm_hea
         PA_LAUNCH();
         pa_k_mix_softmax<<<bs, 256, 4 * (size_t)at.H * at.H, st>>>(at, a->S, io.pos_dev, bs);
         PA_LAUNCH();
-        pa_k_pv<<<dim3(cdiv(at.dv, PA_TN), cdiv(bs, PA_TM), at.H), blk, 0, st>>>(at, a->S, io.vct[li], a->att, aw, io.pos_dev, bs);
+        pa_k_pv<<<dim3(cdiv(at.dv, PA_TN), cdiv(bs, PA_TM), at.H), blk, 0, st>>>(at, a->S, io.vct[li], out, aw, io.pos_dev, bs);
         PA_LAUNCH();
         return 0;
     };
@@ -819,9 +1029,9 @@ static int forward_t(PsArch *a, const PsArchIO &io, int bs, int pos0, int lm_hea
     const float *pend_y = nullptr, *pend_w = nullptr;
     // ... and what a new pass of a looped model adds before its first layer (the embedding output, a row of the pass steps)
     const float *add_tok = nullptr, *add_vec = nullptr;
-    auto seam = [&](float *h_out, const float *w_in) -> int {
+    auto seam = [&](float *h_out, const float *w_in, int ldh = 0) -> int {
         if (!pend_y && !h_out && !add_tok && !add_vec) return 0;
-        pa_k_seam_norm<<<bs, 256, 0, st>>>(a->x, pend_y, pend_w, h_out, w_in, dim, groups, d.norm_eps, center, add_tok, add_vec);
+        pa_k_seam_norm<<<bs, 256, 0, st>>>(a->x, pend_y, pend_w, h_out, w_in, dim, groups, d.norm_eps, center, add_tok, add_vec, a->res_scale, ldh > 0 ? ldh : dim);
         PA_LAUNCH();
         pend_y = pend_w = add_tok = add_vec = nullptr;
         return 0;
@@ -831,7 +1041,7 @@ static int forward_t(PsArch *a, const PsArchIO &io, int bs, int pos0, int lm_hea
     float *xc = a->x, *xo = a->x2;
     auto seam_mv = [&](PaMv &mv, const float *norm_w) {
         mv.x = xc; mv.groups = groups; mv.eps = d.norm_eps; mv.norm_w = norm_w; mv.seam_y = pend_y; mv.seam_w = pend_w;
-        mv.center = center; mv.add_tok = add_tok; mv.add_vec = add_vec;
+        mv.center = center; mv.y_scale = a->res_scale; mv.add_tok = add_tok; mv.add_vec = add_vec;
         if (pend_y || add_tok || add_vec) { mv.x_out = xo; std::swap(xc, xo); }
         pend_y = pend_w = add_tok = add_vec = nullptr;
     };
@@ -842,7 +1052,7 @@ static int forward_t(PsArch *a, const PsArchIO &io, int bs, int pos0, int lm_hea
         return 0;
     };
     // scores and P.V of one query against the cache; the grids do not depend on the position (a window bounds the blocks of keys)
-    auto attend_single = [&](const PaAttn &at, const float *q, int li, bool pool_here = false) -> int {
+    auto attend_single = [&](const PaAttn &at, const float *q, int li, float *out, bool pool_here = false) -> int {
         unsigned blocks = cdiv(n_kv_cap, PA_DS_KEYS);
         if (at.window > 0) blocks = std::min(blocks, cdiv(at.window, PA_DS_KEYS) + 1);
         if (at.chunk > 0) blocks = std::min(blocks, cdiv(at.chunk, PA_DS_KEYS) + 1);
@@ -850,7 +1060,7 @@ static int forward_t(PsArch *a, const PsArchIO &io, int bs, int pos0, int lm_hea
         pa_launch_dep(pdl, pa_k_dec_scores, dim3(blocks + pooled), dim3(256), pa_dec_scores_smem(at.H, at.G, at.dq), st, at, q, (const float *)io.kc[li], io.pos_dev, a->S, io.err_dev, (int)blocks,
                       pool_here && pooled ? io.vct[li] : (float *)nullptr);
         PA_LAUNCH();
-        pa_launch_dep(pdl, pa_k_dec_pv, dim3(cdiv(at.dv, PA_DP_DIMS), at.G, pa_dec_pv_split(at.H, at.G)), dim3(256), pa_dec_pv_smem(at.H, at.G), st, at, (const float *)a->S, (const float *)io.vct[li], io.pos_dev, a->att,
+        pa_launch_dep(pdl, pa_k_dec_pv, dim3(cdiv(at.dv, PA_DP_DIMS), at.G, pa_dec_pv_split(at.H, at.G)), dim3(256), pa_dec_pv_smem(at.H, at.G), st, at, (const float *)a->S, (const float *)io.vct[li], io.pos_dev, out,
                       pa_dec_pv_chunk(at.H, at.G), io.err_dev);
         PA_LAUNCH();
         return 0;
@@ -870,7 +1080,12 @@ static int forward_t(PsArch *a, const PsArchIO &io, int bs, int pos0, int lm_hea
             g.a0 = w.t_gate; g.a1 = w.t_up; g.b = a->tcx; g.nkb = nkb1; g.n_rt = (ff + PT_M - 1) / PT_M; g.n_ct = max_tiles; g.n_ct_dev = a->n_tiles;
             g.tile_e = a->tile_e; g.tile_row0 = a->tile_row0; g.tile_end = a->tile_end; g.M = n; g.N = ff; g.mode = PT_MODE_EXPERT_UP; g.C = a->y; g.ldc = ff;
             g.act = pa_act_of(l); g.err = io.err_dev;
-            pa_k_tc_gemm<2><<<std::min(a->n_sm, max_tiles * g.n_rt), PT_THREADS, PT_SMEM, st>>>(g);
+            if (w.t_gate) {
+                pa_k_tc_gemm<2><<<std::min(a->n_sm, max_tiles * g.n_rt), PT_THREADS, PT_SMEM, st>>>(g);
+            } else { // no gate
+                g.a0 = w.t_up; g.a1 = nullptr;
+                pa_k_tc_gemm<1><<<std::min(a->n_sm, max_tiles * g.n_rt), PT_THREADS, PT_SMEM, st>>>(g);
+            }
             PA_LAUNCH();
             pa_k_tc_prep_x<<<dim3((unsigned)nkb2, (unsigned)max_tiles), 256, 0, st>>>(a->tcx, a->y, ff, n, ff, nkb2, a->n_tiles, a->tile_row0, a->tile_end, nullptr, nullptr);
             PA_LAUNCH();
@@ -884,8 +1099,9 @@ static int forward_t(PsArch *a, const PsArchIO &io, int bs, int pos0, int lm_hea
             const int max_tiles = n / PA_TM + E + 1;
             pa_k_dispatch<<<1, 256, 0, st>>>(a->sel_e, a->sel_w, n, top, E, PA_TM, a->row_token, a->row_slot, a->row_w, a->tile_e, a->tile_row0, a->tile_end, a->n_tiles);
             PA_LAUNCH();
-            pa_k_expert_up<ROUND><<<dim3(cdiv(ff, PA_TN), max_tiles), blk, 0, st>>>(X, dim, a->row_token, a->row_w, a->tile_e, a->tile_row0, a->tile_end, a->n_tiles,
-                                                                                    w.wgate, w.wup, a->y, ff, dim, l.route_on_input, pa_act_of(l));
+            auto *up_kern = w.wgate ? pa_k_expert_up<ROUND, 2> : pa_k_expert_up<ROUND, 1>;
+            up_kern<<<dim3(cdiv(ff, PA_TN), max_tiles), blk, 0, st>>>(X, dim, a->row_token, a->row_w, a->tile_e, a->tile_row0, a->tile_end, a->n_tiles, w.wgate, w.wup, a->y, ff, dim,
+                                                                      l.route_on_input, pa_act_of(l));
             PA_LAUNCH();
             pa_k_expert_down<ROUND><<<dim3(cdiv(dim, PA_TN), max_tiles), blk, 0, st>>>(a->y, ff, a->row_token, a->row_slot, a->row_w, a->tile_e, a->tile_row0, a->tile_end,
                                                                                       a->n_tiles, w.wdown, a->slot, top, dim, ff, l.route_on_input);
@@ -925,7 +1141,7 @@ static int forward_t(PsArch *a, const PsArchIO &io, int bs, int pos0, int lm_hea
         const int ff = w.d.expert_ff;
         const unsigned rows_cta = w.wgate ? PA_DV_ROWS / 2 : PA_DV_ROWS;
         pa_launch_dep(pdl, pa_k_dec_dense_up<ROUND>, dim3(std::min(cdiv(ff, rows_cta), (unsigned)(4 * a->n_sm))), dim3(PA_DV_THREADS), 4 * (size_t)dim, st, (const float *)xc, pend_y, pend_w, w_in,
-                      xo, groups, d.norm_eps, (const bf16 *)w.wgate, (const bf16 *)w.wup, a->y, ff, dim, pa_act_of(w), (const bf16 *)nullptr, 0, (float *)nullptr, center);
+                      xo, groups, d.norm_eps, (const bf16 *)w.wgate, (const bf16 *)w.wup, a->y, ff, dim, pa_act_of(w), (const bf16 *)nullptr, 0, (float *)nullptr, center, a->res_scale);
         PA_LAUNCH();
         std::swap(xc, xo);
         PaMv mv{};
@@ -969,21 +1185,22 @@ static int forward_t(PsArch *a, const PsArchIO &io, int bs, int pos0, int lm_hea
                 if ((rc = linear_heads(a->lq, lqw, dn + dr, dn, w.wukt, rk, a->qa, w.qd, rk + dr, H))) return rc; // W_uk folded into the query
             }
             if (dr > 0) {
-                pa_k_rope_q<<<bs, 256, 0, st>>>(a->lq, a->qa, H, dn, dr, rk, rope, io.pos_dev);
+                pa_k_rope_q<<<bs, 256, 0, st>>>(a->lq, lqw, a->qa, H, dn, dr, rk, rope, io.pos_dev);
                 PA_LAUNCH();
             }
             at.dq = rk + dr; at.dv = rk; q = a->qa; ldq = w.qd;
         } else {
             at.dq = l.qk_dim; at.dv = l.v_dim;
             if (l.qk_norm || l.v_mix)
-                pa_k_qkv_post<<<bs, 256, 0, st>>>(a->qkv, w.pw, H, G, l.qk_dim, l.v_dim, l.qk_norm, d.norm_eps, l.v_mix, w.vmix, a->vsrc, a->vsrc_w, io.kc[li], io.vct[li], d.n_ctx, io.pos_dev);
+                pa_k_qkv_post<<<bs, 256, 0, st>>>(a->qkv, w.pw, H, G, l.qk_dim, l.v_dim, l.qk_norm, d.norm_eps, l.v_mix, w.vmix, a->vsrc, a->vsrc_w, io.kc[li], io.vct[li], d.n_ctx, io.pos_dev,
+                                                   nullptr, nullptr, 0.f, 1.f);
             else
                 pa_k_kv_store<<<dim3(cdiv(w.kd + w.vd, 256), bs), 256, 0, st>>>(a->qkv, w.pw, w.qd, w.kd, w.vd, io.kc[li], io.vct[li], d.n_ctx, io.pos_dev, w.qd + w.kd);
             PA_LAUNCH();
         }
         if (single) {
-            if ((rc = attend_single(at, q, li))) return rc;
-        } else if ((rc = attend(at, q, ldq, w.kd, li, w.aw))) {
+            if ((rc = attend_single(at, q, li, a->att))) return rc;
+        } else if ((rc = attend(at, q, ldq, w.kd, li, a->att, w.aw))) {
             return rc;
         }
         const float *ain = a->att;
@@ -1072,7 +1289,7 @@ static int forward_t(PsArch *a, const PsArchIO &io, int bs, int pos0, int lm_hea
                 if (bs == 1) {
                     pa_k_conv_step<<<cdiv(w.pw, 256), 256, 0, st>>>(a->qkv, w.conv_w, nullptr, w.pw, l.conv_taps, tail, 0, a->cv, io.pos_dev);
                 } else {
-                    pa_k_short_conv<<<dim3(cdiv(w.pw, 256), bs), 256, 0, st>>>(a->qkv, w.pw, w.conv_w, nullptr, w.pw, l.conv_taps, tail, 0, a->cv, w.pw, io.pos_dev);
+                    pa_k_short_conv<<<dim3(cdiv(w.pw, 256), bs), 256, 0, st>>>(a->qkv, w.pw, w.conv_w, nullptr, w.pw, l.conv_taps, tail, 0, a->cv, w.pw, io.pos_dev, 0);
                     if (l.conv_taps > 1) {
                         PA_LAUNCH();
                         pa_k_conv_tail<<<cdiv(w.pw, 256), 256, 0, st>>>(a->qkv, w.pw, w.pw, l.conv_taps, tail, io.pos_dev, bs);
@@ -1097,8 +1314,8 @@ static int forward_t(PsArch *a, const PsArchIO &io, int bs, int pos0, int lm_hea
             at.sink = l.sink != PS_SINK_NONE; at.sink_v = w.sink_v; at.r1 = w.r1; at.r2 = w.r2; at.window = l.window; at.chunk = l.chunk;
             at.n_ctx = d.n_ctx; at.ldS = a->ldS; at.B = B; at.pm = a->pm; at.pl = a->pl; at.ldP = a->ldP;
             at.lin = w.lin; at.pool = l.pool; at.n_pool = w.n_pool; at.pool_off = a->pool_off; at.stat_off = a->stat_off;
-            if (single) rc = attend_single(at, q, li, true);
-            else rc = attend(at, q, w.pw, w.kd, li, w.aw);
+            if (single) rc = attend_single(at, q, li, a->att, true);
+            else rc = attend(at, q, w.pw, w.kd, li, a->att, w.aw);
             if (rc) return rc;
             if (l.out_gate || l.side_kind) { // the heads' outputs through their gate; the side mixer's recurrence fills the columns behind them
                 const unsigned gate_ctas = cdiv(w.ho, PA_GG_THREADS), side_ctas = l.side_kind ? cdiv(l.side_width, 32) : 0;
@@ -1125,7 +1342,7 @@ static int forward_t(PsArch *a, const PsArchIO &io, int bs, int pos0, int lm_hea
                 pa_k_conv_step<<<cdiv(w.conv_c, 256), 256, 0, st>>>(a->qkv + inner, w.conv_w, w.conv_b, w.conv_c, T, tail, 1, a->cv, io.pos_dev);
                 PA_LAUNCH();
             } else {
-                pa_k_short_conv<<<dim3(cdiv(w.conv_c, 256), bs), 256, 0, st>>>(a->qkv + inner, w.pw, w.conv_w, w.conv_b, w.conv_c, T, tail, 1, a->cv, w.conv_c, io.pos_dev);
+                pa_k_short_conv<<<dim3(cdiv(w.conv_c, 256), bs), 256, 0, st>>>(a->qkv + inner, w.pw, w.conv_w, w.conv_b, w.conv_c, T, tail, 1, a->cv, w.conv_c, io.pos_dev, 0);
                 PA_LAUNCH();
                 if (T > 1) {
                     pa_k_conv_tail<<<cdiv(w.conv_c, 256), 256, 0, st>>>(a->qkv + inner, w.pw, w.conv_c, T, tail, io.pos_dev, bs);
@@ -1170,7 +1387,7 @@ static int forward_t(PsArch *a, const PsArchIO &io, int bs, int pos0, int lm_hea
             const int n_rt = E + (rt.shared_gate ? 1 : 0); // the router's rows (+ the shared gate's): logits from the unrounded input
             if (sff > 0) { // the shared expert's gate | up launch carries the seam and the router's rows
                 pa_launch_dep(pdl, pa_k_dec_dense_up<ROUND>, dim3(std::min(cdiv(sff + n_rt, PA_DV_ROWS / 2), up_cap)), dim3(PA_DV_THREADS), 4 * (size_t)dim, st, (const float *)xc, pend_y, pend_w, w_in,
-                              xo, groups, d.norm_eps, (const bf16 *)w.wsg, (const bf16 *)w.wsu, a->y, sff, dim, act, (const bf16 *)w.router, n_rt, a->z, 0);
+                              xo, groups, d.norm_eps, (const bf16 *)w.wsg, (const bf16 *)w.wsu, a->y, sff, dim, act, (const bf16 *)w.router, n_rt, a->z, 0, a->res_scale);
                 PA_LAUNCH();
                 std::swap(xc, xo);
                 pend_y = pend_w = nullptr;
@@ -1194,7 +1411,7 @@ static int forward_t(PsArch *a, const PsArchIO &io, int bs, int pos0, int lm_hea
             if ((rc = seam(raw ? nullptr : a->h, w_in))) return rc;
             const float *X = raw ? a->x : a->h;
             if (sff > 0 && (rc = dense_batch(X, w.wsg, w.wsu, w.wsd, w.t_sg, w.t_su, w.t_sd, sff, act, a->sh))) return rc;
-            pa_k_router<<<bs, 256, 0, st>>>(X, w.router, dim, rt, a->sel_e, a->sel_w, a->sgate);
+            pa_k_router<<<bs, 256, 0, st>>>(X, w.router, dim, rt, a->sel_e, a->sel_w, a->sgate, nullptr);
             PA_LAUNCH();
             if ((rc = routed_batch(X, w))) return rc;
             pa_k_moe_sum<<<dim3(cdiv(dim, 256), bs), 256, 0, st>>>(a->ffo, a->slot, top, sff > 0 ? a->sh : nullptr, rt.shared_gate ? a->sgate : nullptr, dim);
@@ -1204,15 +1421,160 @@ static int forward_t(PsArch *a, const PsArchIO &io, int bs, int pos0, int lm_hea
         return 0;
     };
 
-    pa_k_embed<<<bs, 128, 0, st>>>(a->x, a->embed, io.tokens_dev, dim, d.embed_scale, a->keep_embed ? a->xe : nullptr);
+    // A general parallel block.  One product reads the normed stream (mixer's projections, up rows through the activation), the mixer
+    // leaves its heads right before the up columns of the same rows, one product over both is what the next seam adds to the stream.
+    auto par_layer = [&](int li) -> int {
+        const PsArchLayer &w = a->L[(size_t)li];
+        const ps_cuda_layer_desc &l = w.d;
+        const int H = l.n_heads, n1 = w.pw + w.upn, k2 = w.od + w.upn, gap = w.o_off + w.od - w.pw;
+        const bool latent = l.mixer_kind == PS_MIXER_LATENT, rec = l.mixer_kind == PS_MIXER_RGLRU, routed = l.mlp_kind == PS_MLP_ROUTED;
+        const PaAct act = pa_act_of(l);
+        float *out = a->qkv + w.o_off; // the mixer's heads: rows of stride ldp
+        const int lq = l.qk_dim + l.rot_dim;
+        int rc;
+        if (l.pass_in) { // a new pass: x <- W_in [x; embedding output]
+            if (single) {
+                PaMv mv{};
+                seam_mv(mv, nullptr);
+                mv.x_out = nullptr; // (the sum itself is not kept: the product replaces the stream)
+                mv.W = a->pass_in; mv.N = dim; mv.K = 2 * dim; mv.cat = a->xcat + dim; mv.seam_dim = dim;
+                // seam_mv has swapped the buffers when something was pending; the other CTAs still read the one the seam came from
+                if (mv.x == xc) std::swap(xc, xo);
+                mv.y = xc;
+                if ((rc = dec_mv(mv, 8 * (size_t)dim))) return rc;
+            } else {
+                if ((rc = seam(a->xcat, nullptr, 2 * dim))) return rc;
+                if ((rc = linear(a->xcat, 2 * dim, 2 * dim, a->pass_in, a->t_pass_in, dim, a->x, dim))) return rc;
+            }
+        }
+        if (single) {
+            PaMv mv{};
+            seam_mv(mv, w.norm);
+            mv.W = w.wqkv; mv.bias = w.bqkv; mv.N = n1; mv.K = dim; mv.y = a->qkv;
+            if (w.upn > 0) { mv.act_from = w.pw; mv.gap = gap; mv.act = act; }
+            if (routed) { mv.Wr = w.router; mv.E = l.n_experts; mv.z = a->z; mv.zbias = w.router_b; mv.h_out = a->hn; }
+            if (!latent && !rec) { // value rows go straight into the cache; so do key rows that are not normed
+                const bool raw_k = l.qk_norm != PS_QKNORM_NONE;
+                mv.qd = raw_k ? w.qd + w.kd : w.qd; mv.kd = raw_k ? 0 : w.kd; mv.vd = w.vd;
+                mv.kc = io.kc[li]; mv.vct = io.vct[li]; mv.n_ctx = d.n_ctx; mv.pos = io.pos_dev;
+            }
+            if ((rc = dec_mv(mv, 4 * (size_t)dim))) return rc;
+            if (routed) { // the chosen experts' up rows beside the mixer (a fork in the captured graph); joined before `down`
+                cudaStream_t se = a->opt_fork ? a->side : st;
+                if (a->opt_fork) { PA_CK(cudaEventRecord(a->ev_fork, st)); PA_CK(cudaStreamWaitEvent(se, a->ev_fork, 0)); }
+                pa_k_dec_expert_up<ROUND><<<dim3(std::min(cdiv(l.expert_ff, PA_DV_ROWS), (unsigned)std::max(1, 4 * a->n_sm / l.top_k)), l.top_k), PA_DV_THREADS, 4 * (size_t)dim, se>>>(
+                    a->hn, nullptr, d.norm_eps, a->z, pa_route_of(l), nullptr, w.wup, a->y, l.expert_ff, dim, 0, act, a->sel_e, a->sel_w);
+                PA_LAUNCH();
+                if (a->opt_fork) PA_CK(cudaEventRecord(a->ev_join, se));
+            }
+        } else {
+            if ((rc = seam(a->h, w.norm))) return rc;
+            if (tc) {
+                if ((rc = tc_dense(a->h, dim, bs, dim, w.t_qkv, n1, w.bqkv, a->qkv, w.ldp, w.upn > 0 ? &act : nullptr, w.pw, gap))) return rc;
+            } else {
+                pa_k_linear<ROUND><<<dim3(cdiv(n1, PA_TN), cdiv(bs, PA_TM)), blk, 0, st>>>(a->h, dim, w.wqkv, w.bqkv, a->qkv, w.ldp, bs, n1, dim, 0, 0, w.pw, gap, act);
+                PA_LAUNCH();
+            }
+        }
+        if (rec) {
+            PaRglru g{};
+            g.y = a->qkv; g.x = a->qkv + l.rec_width; g.ld = w.ldp; g.u = a->cv; g.g = a->gts; g.rb = w.rec_rb; g.ib = w.rec_ib; g.sp = w.rec_sp;
+            g.W = l.rec_width; g.bsz = l.rec_width / l.rec_blocks; g.taps = l.conv_taps; g.conv_w = w.conv_w; g.conv_b = w.conv_b; g.wri = w.wri;
+            g.S = io.kc[li]; g.ring = io.vct[li]; g.o = out; g.ldo = w.ldp; g.pos = io.pos_dev; g.bs = bs;
+            if (single) {
+                pa_launch_dep(pdl, pa_k_dec_rglru, dim3(cdiv(g.bsz, 8), (unsigned)l.rec_blocks), dim3(256), 4 * (size_t)g.bsz, st, g);
+                PA_LAUNCH();
+            } else {
+                pa_k_short_conv<<<dim3(cdiv(g.W, 256), bs), 256, 0, st>>>(g.x, w.ldp, w.conv_w, w.conv_b, g.W, g.taps, g.ring, 0, a->cv, g.W, io.pos_dev, 1);
+                PA_LAUNCH();
+                pa_k_linear<false><<<dim3(cdiv(2 * g.bsz, PA_TN), cdiv(bs, PA_TM), (unsigned)l.rec_blocks), blk, 0, st>>>(a->cv, g.W, w.wri, nullptr, a->gts, 2 * g.W, bs, 2 * g.bsz, g.bsz, g.bsz, 2 * g.bsz);
+                PA_LAUNCH();
+                pa_k_rglru_scan<<<cdiv(g.W, 32), PA_GG_THREADS, 0, st>>>(g);
+                PA_LAUNCH();
+            }
+        } else {
+            PaAttn at{};
+            at.H = H; at.G = l.n_kv_heads; at.scale = l.score_scale; at.sink = l.sink != PS_SINK_NONE; at.sink_v = w.sink_v; at.window = l.window; at.chunk = l.chunk;
+            at.n_ctx = d.n_ctx; at.ldS = a->ldS; at.B = B; at.pm = a->pm; at.pl = a->pl; at.ldP = a->ldP;
+            at.dq = l.qk_dim; at.dv = l.v_dim;
+            if (l.out_gate) { at.gate = a->qkv + w.g_off; at.ld_gate = w.ldp; }
+            const float *q = a->qkv;
+            int ldq = w.ldp, ldo = w.ldp;
+            float *ho = out;
+            if (latent) {
+                const int rk = l.kv_rank, dr = l.rot_dim, dn = l.qk_dim;
+                const PaRope rope{w.rope_freq, l.rope_dims, w.rope_mscale, l.rope_interleaved};
+                at.dq = rk + dr; at.dv = rk; q = a->qa; ldq = w.qd; ho = a->att; ldo = w.aw;
+                if (single) {
+                    int lg = 0;
+                    while (lg < 5 && (8 << lg) < dn) lg++;
+                    pa_launch_dep(pdl, pa_k_dec_latent_q<ROUND>, dim3(std::min(cdiv((int64_t)H * rk, 8 * (32 >> lg)), (unsigned)(2 * a->n_sm)) + 1), dim3(256), 0, st, (const float *)a->qkv, H, dn, dr, rk,
+                                  (const bf16 *)w.wukt, a->qa, lg, (const float *)w.dkv_norm, d.norm_eps, rope, io.kc[li], io.vct[li], d.n_ctx, io.pos_dev);
+                    PA_LAUNCH();
+                } else {
+                    pa_k_latent_post<<<bs, 256, 0, st>>>(a->qkv + H * lq, w.ldp, 0, rk, dr, nullptr, w.dkv_norm, d.norm_eps, rope, nullptr, io.kc[li], io.vct[li], d.n_ctx, io.pos_dev);
+                    PA_LAUNCH();
+                    if ((rc = linear_heads(a->qkv, w.ldp, lq, dn, w.wukt, rk, a->qa, w.qd, rk + dr, H))) return rc; // W_uk folded into the query
+                    if (dr > 0) {
+                        pa_k_rope_q<<<bs, 256, 0, st>>>(a->qkv, w.ldp, a->qa, H, dn, dr, rk, rope, io.pos_dev);
+                        PA_LAUNCH();
+                    }
+                }
+            } else if (single) {
+                if (l.qk_norm != PS_QKNORM_NONE) { // the scores kernel norms q and the token's key
+                    at.qn = w.q_norm; at.kn = w.k_norm; at.eps = d.norm_eps; at.qt_coef = l.q_temp_coef; at.qt_every = l.q_temp_every; at.k_raw = a->qkv + w.qd; at.kc_out = io.kc[li];
+                }
+            } else {
+                pa_k_qkv_post<<<bs, 256, 0, st>>>(a->qkv, w.ldp, H, l.n_kv_heads, l.qk_dim, l.v_dim, l.qk_norm, d.norm_eps, 0, nullptr, nullptr, 0, io.kc[li], io.vct[li], d.n_ctx, io.pos_dev, w.q_norm,
+                                                  w.k_norm, l.q_temp_coef, l.q_temp_every);
+                PA_LAUNCH();
+            }
+            rc = single ? attend_single(at, q, li, ho) : attend(at, q, ldq, w.kd, li, ho, ldo);
+            if (rc) return rc;
+            if (latent) { // W_uv on every head's weighted sum of latents
+                if (single) {
+                    PaMv mv{};
+                    mv.x = a->att; mv.W = w.wuv; mv.N = w.od; mv.K = l.kv_rank; mv.y = out; mv.grp_rows = l.v_dim; mv.x_gs = l.kv_rank; mv.y_gs = l.v_dim;
+                    if ((rc = dec_mv(mv, 0))) return rc;
+                } else if ((rc = linear_heads(a->att, w.aw, l.kv_rank, l.kv_rank, w.wuv, l.v_dim, out, w.ldp, l.v_dim, H))) {
+                    return rc;
+                }
+            }
+        }
+        if (single) {
+            PaMv mv{};
+            mv.x = out; mv.W = w.wo; mv.N = dim; mv.K = k2; mv.y = a->ao;
+            if ((rc = dec_mv(mv, 0))) return rc;
+        } else if ((rc = linear(out, w.ldp, k2, w.wo, w.t_o, dim, a->ao, dim))) {
+            return rc;
+        }
+        pend_y = a->ao; pend_w = nullptr;
+        if (!routed) return 0;
+        if (single) {
+            if (a->opt_fork) PA_CK(cudaStreamWaitEvent(st, a->ev_join, 0));
+            const int ksd = pick_ksplit(dim, l.expert_ff);
+            pa_k_dec_expert_down<ROUND><<<cdiv(dim, PA_DV_ROWS / ksd), PA_DV_THREADS, 0, st>>>(a->y, a->sel_e, a->sel_w, l.top_k, w.wdown, nullptr, nullptr, dim, l.expert_ff, 0, ksd, a->ffo, a->ao, nullptr);
+            PA_LAUNCH();
+        } else {
+            pa_k_router<<<bs, 256, 0, st>>>(a->h, w.router, dim, pa_route_of(l), a->sel_e, a->sel_w, a->sgate, w.router_b);
+            PA_LAUNCH();
+            if ((rc = routed_batch(a->h, w))) return rc;
+            pa_k_moe_sum<<<dim3(cdiv(dim, 256), bs), 256, 0, st>>>(a->ffo, a->slot, l.top_k, a->ao, nullptr, dim);
+            PA_LAUNCH();
+        }
+        pend_y = a->ffo;
+        return 0;
+    };
+
+    pa_k_embed<<<bs, 128, 0, st>>>(a->x, a->embed, io.tokens_dev, dim, d.embed_scale, a->has_pass_in ? a->xcat + dim : a->keep_embed ? a->xe : nullptr, a->has_pass_in ? 2 * dim : dim);
     PA_LAUNCH();
     for (int li = 0; li < d.n_layers; li++) {
         const PsArchLayer &w = a->L[(size_t)li];
         const ps_cuda_layer_desc &l = w.d;
         if (l.pass_embed) add_tok = a->xe;   // a new pass: the run's first seam adds these to the stream
         if (l.pass_step) add_vec = a->pass_steps + (int64_t)(l.pass_step - 1) * dim;
-        if (l.block_kind == PS_BLOCK_SEQUENTIAL) {
-            int rc = w.gen2 ? gen_layer(li) : seq_layer(li);
+        if (l.block_kind == PS_BLOCK_SEQUENTIAL || w.gpar) {
+            int rc = w.gpar ? par_layer(li) : w.gen2 ? gen_layer(li) : seq_layer(li);
             if (rc) return rc;
             if (a->taps_on) {
                 if ((rc = seam(nullptr, nullptr))) return rc; // the tap shows the layer's whole effect
@@ -1295,7 +1657,7 @@ static int forward_t(PsArch *a, const PsArchIO &io, int bs, int pos0, int lm_hea
             const int ff = l.expert_ff;
             int rc = 0;
             if (!single) {
-                pa_k_router<<<bs, 256, 0, st>>>(a->h, w.router, dim, pa_route_of(l), a->sel_e, a->sel_w, a->sgate);
+                pa_k_router<<<bs, 256, 0, st>>>(a->h, w.router, dim, pa_route_of(l), a->sel_e, a->sel_w, a->sgate, nullptr);
                 PA_LAUNCH();
             }
             if (single) {

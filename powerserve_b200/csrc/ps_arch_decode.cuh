@@ -91,12 +91,12 @@ __device__ __forceinline__ void pa_norm_to_smem(float *hs, const float *__restri
     __syncthreads();
 }
 
-// block-wide seam of a sequential block (256 threads): hs = G(x + P(y) + add_tok + add_vec; w_in) with P(y) = G(y; w_out) (w_out
+// block-wide seam between two blocks (256 threads): hs = G(x + y_scale P(y) + add_tok + add_vec; w_in) with P(y) = G(y; w_out) (w_out
 // null: y itself; y / add_tok / add_vec null: nothing joins), G over `groups` equal parts, the part's mean taken off first when
 // `center`.  CTA 0 also stores the updated residual to x_out - a buffer other than x, which the other CTAs are still reading.
 __device__ __forceinline__ void pa_seam_to_smem(float *hs, const float *__restrict__ x, const float *__restrict__ y, const float *__restrict__ w_out,
                                                 const float *__restrict__ w_in, float *__restrict__ x_out, int dim, int groups, float eps, int center = 0,
-                                                const float *__restrict__ add_tok = nullptr, const float *__restrict__ add_vec = nullptr) {
+                                                const float *__restrict__ add_tok = nullptr, const float *__restrict__ add_vec = nullptr, float y_scale = 1.0f) {
     __shared__ float red[8];
     const int gs = dim / groups;
     for (int g = 0; g < groups; g++) {
@@ -105,7 +105,7 @@ __device__ __forceinline__ void pa_seam_to_smem(float *hs, const float *__restri
         if (y && w_out) inv = pa_block_stats(y + c0, gs, center, eps, red, mu);
         for (int c = threadIdx.x; c < gs; c += 256) {
             float v = x[c0 + c];
-            if (y) v += w_out ? (y[c0 + c] - mu) * inv * w_out[c0 + c] : y[c0 + c];
+            if (y) v += y_scale * (w_out ? (y[c0 + c] - mu) * inv * w_out[c0 + c] : y[c0 + c]);
             if (add_tok || add_vec) v += (add_tok ? add_tok[c0 + c] : 0.f) + (add_vec ? add_vec[c0 + c] : 0.f);
             hs[c0 + c] = v;
             if (x_out && blockIdx.x == 0 && blockIdx.y == 0) x_out[c0 + c] = v;
@@ -128,6 +128,10 @@ struct PaMv {
     const float *seam_y, *seam_w;
     float *x_out;
     int center;            // the norms take the mean off first
+    float y_scale;         // factor on seam_y's part
+    float *h_out;          // non-null: CTA 0 stores the seam's result (the normed input) there as well
+    const float *cat;      // non-null: the seam covers the first seam_dim inputs only, these K - seam_dim values follow
+    int seam_dim;
     const float *add_tok, *add_vec; // what a new pass of a looped model adds to the stream at this seam (null: nothing)
     // per-head products (grp_rows > 0): rows [g * grp_rows, (g + 1) * grp_rows) read x + g * x_gs and write y + g * y_gs
     int grp_rows, x_gs, y_gs;
@@ -136,7 +140,7 @@ struct PaMv {
     int N, K;
     float *y;              // [N] (rows routed to the cache below are not stored here)
     float *residual;       // non-null: residual[n] += result instead of y[n] = result
-    // q | k | v routing of the rows: [0, qd) -> y, [qd, qd + kd) -> K cache row `pos`, then vd rows -> V^T column `pos` (kd = 0: none)
+    // q | k | v routing of the rows: [0, qd) -> y, [qd, qd + kd) -> K cache row `pos`, then vd rows -> V^T column `pos` (kd = vd = 0: none)
     int qd, kd, vd;
     float *kc, *vct;
     int n_ctx;
@@ -146,6 +150,10 @@ struct PaMv {
     const bf16 *Wr;
     int E;
     float *z;
+    const float *zbias;    // [E] or null
+    // rows n >= act_from (> 0) leave through the one-argument activation, `gap` entries further on
+    int act_from, gap;
+    PaAct act;
     int ksplit;            // warps of a CTA that share a row pair, each taking K / ksplit of the columns (1, 2, 4 or 8)
     int prefetch;          // 1: request the first row group into L2 before the dependency wait; 2: also every next group one ahead
 };
@@ -171,7 +179,14 @@ __global__ void __launch_bounds__(PA_DV_THREADS) pa_k_dec_mv(const PaMv a) {
     ps_grid_dep_wait();
     const float *xin = a.x;
     if (a.groups > 0) {
-        pa_seam_to_smem(pa_hs, a.x, a.seam_y, a.seam_w, a.norm_w, a.x_out, a.K, a.groups, a.eps, a.center, a.add_tok, a.add_vec);
+        const int sd = a.cat ? a.seam_dim : a.K;
+        pa_seam_to_smem(pa_hs, a.x, a.seam_y, a.seam_w, a.norm_w, a.x_out, sd, a.groups, a.eps, a.center, a.add_tok, a.add_vec, a.y_scale);
+        if (a.cat) {
+            for (int c = threadIdx.x; c < a.K - sd; c += PA_DV_THREADS) pa_hs[sd + c] = a.cat[c];
+            __syncthreads();
+        }
+        if (a.h_out && blockIdx.x == 0)
+            for (int c = threadIdx.x; c < sd; c += PA_DV_THREADS) a.h_out[c] = pa_hs[c];
         xin = pa_hs;
     } else if (a.norm_w) {
         pa_norm_to_smem(pa_hs, a.x, a.norm_w, a.K, a.eps);
@@ -184,7 +199,9 @@ __global__ void __launch_bounds__(PA_DV_THREADS) pa_k_dec_mv(const PaMv a) {
         float s0 = 0.f, s1 = 0.f;
         if (live) {
             const bf16 *w0 = row(n0), *w1 = row(n1);
-            if (a.grp_rows > 0) { // every row reads its own head's slice of x
+            if (a.grp_rows > 0 && n0 / a.grp_rows == n1 / a.grp_rows) {
+                pa_dot2<ROUND>(w0, w1, xin + (n0 / a.grp_rows) * a.x_gs, a.K, 1.0f, lane, s0, s1, k_begin, k_end);
+            } else if (a.grp_rows > 0) { // every row reads its own head's slice of x
                 float t;
                 pa_dot2<ROUND>(w0, w0, xin + (n0 / a.grp_rows) * a.x_gs, a.K, 1.0f, lane, s0, t, k_begin, k_end);
                 pa_dot2<ROUND>(w1, w1, xin + (n1 / a.grp_rows) * a.x_gs, a.K, 1.0f, lane, s1, t, k_begin, k_end);
@@ -210,10 +227,10 @@ __global__ void __launch_bounds__(PA_DV_THREADS) pa_k_dec_mv(const PaMv a) {
             const int n = lane ? n1 : n0;
             float v = lane ? s1 : s0;
             if (n >= a.N) {
-                a.z[n - a.N] = v;
+                a.z[n - a.N] = a.zbias ? v + a.zbias[n - a.N] : v;
             } else {
                 if (a.bias) v += a.bias[n];
-                if (a.kd && n >= a.qd && n < a.qd + a.kd + a.vd) {
+                if (n >= a.qd && n < a.qd + a.kd + a.vd) {
                     const int p = a.pos[0];
                     if (n < a.qd + a.kd) {
                         a.kc[(int64_t)p * a.kd + (n - a.qd)] = v;
@@ -221,6 +238,8 @@ __global__ void __launch_bounds__(PA_DV_THREADS) pa_k_dec_mv(const PaMv a) {
                     } else {
                         a.vct[(int64_t)(n - a.qd - a.kd) * a.n_ctx + p] = v;
                     }
+                } else if (a.act_from > 0 && n >= a.act_from) {
+                    a.y[n + a.gap] = pa_act1(v, a.act);
                 } else if (a.residual) {
                     a.residual[n] += v;
                 } else if (a.grp_rows > 0) {
@@ -271,16 +290,38 @@ __global__ void __launch_bounds__(256) pa_k_dec_scores(PaAttn at, const float *_
     }
     if (nj <= 0) return;
     const bool bulk = (kd & 3) == 0;
+    const bool own = at.k_raw && !pooled && j0 + nj == pos + 1; // the token's own key: raw in k_raw, not in the cache yet
+    const int nc = own ? nj - 1 : nj;                           // rows that come from the cache
     if (bulk && tid == 0) {
         ps_mbar_init(&bar, 1);
         ps_fence_barrier_init();
         asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
-        ps_mbar_expect_tx(&bar, (uint32_t)(nj * kd * 4));
-        for (int jj = 0; jj < nj; jj++) ps_bulk_g2s(ks + jj * kds, kc + (int64_t)(j0 + jj) * kd, (uint32_t)(kd * 4), &bar);
+        ps_mbar_expect_tx(&bar, (uint32_t)(nc * kd * 4));
+        for (int jj = 0; jj < nc; jj++) ps_bulk_g2s(ks + jj * kds, kc + (int64_t)(j0 + jj) * kd, (uint32_t)(kd * 4), &bar);
     }
-    if (!bulk) for (int t = tid; t < nj * kd; t += 256) ks[(t / kd) * kds + t % kd] = kc[(int64_t)j0 * kd + t];
+    if (!bulk) for (int t = tid; t < nc * kd; t += 256) ks[(t / kd) * kds + t % kd] = kc[(int64_t)j0 * kd + t];
     for (int t = tid; t < H * dq; t += 256) qs[t] = q[t];
+    if (own) for (int t = tid; t < kd; t += 256) ks[nc * kds + t] = at.k_raw[t];
     __syncthreads();
+    if (at.k_raw) { // a warp per head: norm of q (times the position's temperature), and of the token's key on its way into the cache
+        const float qt = pa_q_temp(at.qt_coef, at.qt_every, pos);
+        for (int hh = tid >> 5; hh < H + (own ? G : 0); hh += 8) {
+            const int lane = tid & 31;
+            float *v = hh < H ? qs + hh * dq : ks + nc * kds + (hh - H) * dq;
+            const float inv = pa_warp_inv_rms(v, dq, at.eps, lane);
+            __syncwarp();
+            for (int c = lane; c < dq; c += 32) {
+                if (hh < H) {
+                    v[c] *= inv * (at.qn ? at.qn[c] : 1.0f) * qt;
+                } else {
+                    const float kv = v[c] * inv * (at.kn ? at.kn[c] : 1.0f);
+                    v[c] = kv;
+                    at.kc_out[(int64_t)pos * kd + (hh - H) * dq + c] = kv;
+                }
+            }
+        }
+        __syncthreads();
+    }
     if (bulk && !ps_tc_wait(&bar, 0)) { if (tid == 0) err[0] = 5; return; }
     for (int t = tid; t < PA_DS_KEYS * H; t += 256) {
         const int jj = t % PA_DS_KEYS, h = t / PA_DS_KEYS;
@@ -432,7 +473,69 @@ __global__ void __launch_bounds__(256) pa_k_dec_pv(PaAttn at, const float *__res
         if (c0 + cc >= dv) continue;
         float s = 0.f;
         for (int pp = 0; pp < n_part; pp++) s += acc[(pp * PA_DP_DIMS + cc) * rep + r];
-        att[(h0 + r) * dv + c0 + cc] = s * inv[r];
+        s *= inv[r];
+        att[(h0 + r) * dv + c0 + cc] = at.gate ? s * pa_sigmoid(at.gate[h0 + r]) : s;
+    }
+}
+
+// ---------------------------------------------------------------------------------------------------- latent attention
+// What lies between the first projection of a latent attention whose queries come straight from the input and its scores, in one
+// launch.  row = [q: H heads of dn + dr | kv latent (rk) | rotated key part (dr)].
+//   CTAs below gridDim.x - 1: W_uk folded into the query, qa[h][c] = sum_d wukt[h][c][d] round(q_h[d]); 2^lg lanes share an output row
+//     (a lane takes eight columns at a time), so short rows keep every lane busy
+//   the last CTA: the normed latent and the rotated key part into the cache, the rotated query parts into qa
+template <bool ROUND>
+__global__ void __launch_bounds__(256) pa_k_dec_latent_q(const float *__restrict__ row, int H, int dn, int dr, int rk, const bf16 *__restrict__ wukt, float *__restrict__ qa, int lg,
+                                                         const float *__restrict__ wk, float eps, PaRope rope, float *__restrict__ kc, float *__restrict__ vct, int n_ctx,
+                                                         const int32_t *__restrict__ pos) {
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, lqw = H * (dn + dr);
+    if (blockIdx.x + 1 == gridDim.x) {
+        __shared__ float red[8];
+        ps_grid_dep_launch();
+        ps_grid_dep_wait();
+        const int p = pos[0];
+        const float *c = row + lqw;
+        float s = 0.f;
+        for (int i = tid; i < rk; i += 256) s = fmaf(c[i], c[i], s);
+        const float inv = 1.0f / sqrtf(pa_block_sum(s, red) / (float)rk + eps);
+        float *krow = kc + (int64_t)p * (rk + dr);
+        for (int i = tid; i < rk; i += 256) {
+            const float v = c[i] * inv * wk[i];
+            krow[i] = v;
+            vct[(int64_t)i * n_ctx + p] = v;
+        }
+        for (int i = tid; i < dr; i += 256) pa_rope_store(rope, c + rk, krow + rk, dr, p, i);
+        for (int e = tid; e < H * dr; e += 256) pa_rope_store(rope, row + (e / dr) * (dn + dr) + dn, qa + (e / dr) * (rk + dr) + rk, dr, p, e % dr);
+        return;
+    }
+    const int lpr = 1 << lg, sub = lane & (lpr - 1), per_warp = 32 >> lg, rows = H * rk;
+    const int stride = ((int)gridDim.x - 1) * 8 * per_warp;
+    int n = (blockIdx.x * 8 + warp) * per_warp + (lane >> lg);
+    if (n < rows && sub * 64 < dn) asm volatile("prefetch.global.L2 [%0];" ::"l"(wukt + (int64_t)n * dn + sub * 64));
+    ps_grid_dep_launch();
+    ps_grid_dep_wait();
+    for (; __any_sync(0xffffffffu, n < rows); n += stride) {
+        const int nn = min(n, rows - 1), h = nn / rk;
+        const bf16 *w = wukt + (int64_t)nn * dn;
+        const float *x = row + h * (dn + dr);
+        float s = 0.f;
+        if ((dn & 7) == 0 && ((dn + dr) & 3) == 0) {
+            for (int k = sub * 8; k < dn; k += lpr * 8) {
+                const uint4 a = __ldg(reinterpret_cast<const uint4 *>(w + k));
+                const float4 x0 = *reinterpret_cast<const float4 *>(x + k), x1 = *reinterpret_cast<const float4 *>(x + k + 4);
+                const float xv[8] = {x0.x, x0.y, x0.z, x0.w, x1.x, x1.y, x1.z, x1.w};
+                const uint32_t au[4] = {a.x, a.y, a.z, a.w};
+#pragma unroll
+                for (int t = 0; t < 4; t++) {
+                    s = fmaf(__uint_as_float(au[t] << 16), pa_rnd<ROUND>(xv[2 * t]), s);
+                    s = fmaf(__uint_as_float(au[t] & 0xffff0000u), pa_rnd<ROUND>(xv[2 * t + 1]), s);
+                }
+            }
+        } else {
+            for (int k = sub; k < dn; k += lpr) s = fmaf(__bfloat162float(w[k]), pa_rnd<ROUND>(x[k]), s);
+        }
+        for (int o = lpr >> 1; o; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
+        if (sub == 0 && n < rows) qa[h * (rk + dr) + nn % rk] = s;
     }
 }
 
@@ -447,7 +550,14 @@ __global__ void __launch_bounds__(PA_DV_THREADS) pa_k_dec_expert_up(const float 
     __shared__ float sc[PA_MAX_EXPERTS];
     __shared__ int se[PA_MAX_EXPERTS];
     __shared__ float sw[PA_MAX_EXPERTS];
-    if (threadIdx.x == 0) {
+    if (rt.act == PS_ROUTER_TOPK_SOFTMAX) {
+        if (threadIdx.x < 32) {
+            pa_route_topk_warp(z, rt.E, rt.top, se, sw, threadIdx.x);
+            __syncwarp();
+            if (blockIdx.x == 0 && blockIdx.y == 0)
+                for (int r = threadIdx.x; r < rt.top; r += 32) { sel_e[r] = se[r]; sel_w[r] = sw[r]; }
+        }
+    } else if (threadIdx.x == 0) {
         pa_route_serial(z, rt, sc, se, sw);
         if (blockIdx.x == 0 && blockIdx.y == 0)
             for (int r = 0; r < rt.top; r++) { sel_e[r] = se[r]; sel_w[r] = sw[r]; }
@@ -462,6 +572,16 @@ __global__ void __launch_bounds__(PA_DV_THREADS) pa_k_dec_expert_up(const float 
     const float w = on_input ? sw[r] : 1.0f;
     // a warp owns one ff row at a time: its gate row and its up row are the pair; the CTAs walk the row groups with the grid's stride
     const int rows = PA_DV_ROWS / 2;
+    if (!Wg) { // no gate: the pair is two neighbouring up rows
+        for (int n0 = (blockIdx.x * rows + warp) * 2; n0 < ff; n0 += gridDim.x * rows * 2) {
+            const int n1 = min(n0 + 1, ff - 1);
+            float s0, s1;
+            pa_dot2<ROUND>(Wu + ((int64_t)e * ff + n0) * dim, Wu + ((int64_t)e * ff + n1) * dim, pa_hs, dim, w, lane, s0, s1);
+            if (lane == 0) y[(int64_t)r * ff + n0] = pa_act1(s0, act);
+            if (lane == 1 && n1 != n0) y[(int64_t)r * ff + n1] = pa_act1(s1, act);
+        }
+        return;
+    }
     for (int n = blockIdx.x * rows + warp; n < ff; n += gridDim.x * rows) {
         const bf16 *wg = Wg + ((int64_t)e * ff + n) * dim, *wu = Wu + ((int64_t)e * ff + n) * dim;
         float gsum, usum;
@@ -477,7 +597,7 @@ template <bool ROUND>
 __global__ void __launch_bounds__(PA_DV_THREADS) pa_k_dec_dense_up(const float *__restrict__ x, const float *__restrict__ seam_y, const float *__restrict__ seam_w,
                                                                    const float *__restrict__ norm_w, float *__restrict__ x_out, int groups, float eps, const bf16 *__restrict__ Wg,
                                                                    const bf16 *__restrict__ Wu, float *__restrict__ y, int ff, int dim, PaAct act,
-                                                                   const bf16 *__restrict__ Wr = nullptr, int E = 0, float *__restrict__ z = nullptr, int center = 0) {
+                                                                   const bf16 *__restrict__ Wr = nullptr, int E = 0, float *__restrict__ z = nullptr, int center = 0, float y_scale = 1.0f) {
     extern __shared__ __align__(16) float pa_hs[];
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, rows = PA_DV_ROWS / 2;
     if (!Wg) { // no gate: a warp's pair is two neighbouring up rows, y[n] = act(up[n] . h)
@@ -485,7 +605,7 @@ __global__ void __launch_bounds__(PA_DV_THREADS) pa_k_dec_dense_up(const float *
         if (n < ff) pa_prefetch2(Wu + (int64_t)n * dim, Wu + (int64_t)min(n + 1, ff - 1) * dim, 0, dim, lane);
         ps_grid_dep_launch();
         ps_grid_dep_wait();
-        pa_seam_to_smem(pa_hs, x, seam_y, seam_w, norm_w, x_out, dim, groups, eps, center);
+        pa_seam_to_smem(pa_hs, x, seam_y, seam_w, norm_w, x_out, dim, groups, eps, center, nullptr, nullptr, y_scale);
         for (int n0 = (blockIdx.x * rows + warp) * 2; n0 < ff; n0 += gridDim.x * rows * 2) {
             const int n1 = min(n0 + 1, ff - 1);
             float s0, s1;
@@ -501,7 +621,7 @@ __global__ void __launch_bounds__(PA_DV_THREADS) pa_k_dec_dense_up(const float *
     }
     ps_grid_dep_launch();
     ps_grid_dep_wait();
-    pa_seam_to_smem(pa_hs, x, seam_y, seam_w, norm_w, x_out, dim, groups, eps, center);
+    pa_seam_to_smem(pa_hs, x, seam_y, seam_w, norm_w, x_out, dim, groups, eps, center, nullptr, nullptr, y_scale);
     // E more rows behind the ff rows: a router's logits z[e] = Wr[e] . h from the UNROUNDED input (a shared expert's launch carries them)
     for (int n = blockIdx.x * rows + warp; n < ff + E; n += gridDim.x * rows) {
         float gsum, usum;

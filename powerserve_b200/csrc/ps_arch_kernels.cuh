@@ -21,6 +21,7 @@
 //                             PS_ACT_GELU_TANH  the tanh form of gelu on g, times u
 //                             PS_ACT_XIELU      one argument only: alpha z^2 + z / 2 above zero, shift (exp(z) - 1 - z) + z / 2 below
 //                                               (alpha = softplus(p), shift = 1/2 + softplus(q) of the layer's two numbers)
+//                             PS_ACT_RELU2      one argument only: max(z, 0)^2
 struct PaAct {
     float limit, alpha, shift;
     int kind;
@@ -47,6 +48,15 @@ struct PaAttn {
     int n_ctx;
     int64_t ldS;            // row stride of the score rows
     int B;                  // rows per head in the score buffer (max_batch)
+    // q / k of every head divided by their root mean square times qn / kn (shared by the heads), q at position p also times
+    // 1 + qt_coef ln(floor((p + 1) / qt_every) + 1): the batch kernels apply both before the scores, the single-token scores kernel in its
+    // prologue - it takes the token's raw key row from k_raw and stores the normed one to the cache row kc_out + pos * G * dq
+    const float *qn, *kn;
+    float eps, qt_coef, qt_every;
+    const float *k_raw;
+    float *kc_out;
+    const float *gate;      // one logit per query row and head (row stride ld_gate) or null: the head's output times sigmoid(logit)
+    int ld_gate;
     float *pm, *pl;         // single-token step: per head and block of keys, max and sum of exponentials of the mixed scores
     int ldP;                // blocks per head in pm / pl
 };
@@ -62,6 +72,25 @@ __device__ __forceinline__ float pa_ld(const float *p) { return *p; }
 template <bool ROUND>
 __device__ __forceinline__ void pa_dot2(const bf16 *__restrict__ w0, const bf16 *__restrict__ w1, const float *x, int K, float xscale, int lane, float &s0, float &s1,
                                         int k_begin = 0, int k_end = -1);
+
+// ---------------------------------------------------------------------------------------------------------------- activations
+__device__ __forceinline__ float pa_sigmoid(float v) { return 1.0f / (1.0f + expf(-v)); }
+__device__ __forceinline__ float pa_expert_act(float g, float u, PaAct act) {
+    if (act.kind == PS_ACT_GELU_TANH) // 0.5 g (1 + tanh(sqrt(2 / pi) (g + 0.044715 g^3))) * u
+        return 0.5f * g * (1.0f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g))) * u;
+    g = fminf(g, act.limit);
+    u = fminf(fmaxf(u, -act.limit), act.limit);
+    return g * (1.0f / (1.0f + expf(-act.alpha * g))) * (u + act.shift);
+}
+
+// the one-argument forms (a feed-forward without a gate)
+__device__ __forceinline__ float pa_act1(float z, PaAct act) {
+    if (act.kind == PS_ACT_RELU2) return z > 0.f ? z * z : 0.f;
+    if (act.kind == PS_ACT_XIELU) return z > 0.f ? fmaf(act.alpha * z, z, 0.5f * z) : fmaf(act.shift, expm1f(z) - z, 0.5f * z);
+    if (act.kind == PS_ACT_GELU_TANH) return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
+    z = fminf(z, act.limit);
+    return z * (1.0f / (1.0f + expf(-act.alpha * z)));
+}
 
 // ---------------------------------------------------------------------------------------------------------------- tile core
 // acc[i][j] += sum_k A(ty * 4 + i, k) * B(tx * 4 + j, k) for the CTA's 64 x 64 tile.  Every thread stages 4 k-values of ONE A
@@ -103,13 +132,13 @@ __device__ __forceinline__ void pa_tile_mm(float (&acc)[NB][4][4], const float *
     __shared__ __align__(16) float Bs[NB][PA_TK][PA_LD]
 
 // ---------------------------------------------------------------------------------------------------------------- small ops
-// keep (null or [tokens][dim]) receives the same rows once more: the embedding output that later passes of a looped model add back
+// keep (null or [tokens] rows of stride ld_keep) receives the same rows once more: the embedding output that later passes of a looped model add back
 __global__ void __launch_bounds__(128) pa_k_embed(float *__restrict__ x, const bf16 *__restrict__ table, const int32_t *__restrict__ tokens, int dim, float scale,
-                                                  float *__restrict__ keep) {
+                                                  float *__restrict__ keep, int ld_keep) {
     const int t = blockIdx.x;
     const bf16 *row = table + (int64_t)tokens[t] * dim;
     float *out = x + (int64_t)t * dim;
-    float *out2 = keep ? keep + (int64_t)t * dim : nullptr;
+    float *out2 = keep ? keep + (int64_t)t * ld_keep : nullptr;
     if ((dim & 7) == 0) { // 16-byte loads: the whole row is in flight at once
         for (int c = threadIdx.x * 8; c < dim; c += blockDim.x * 8) {
             const uint4 v = __ldg(reinterpret_cast<const uint4 *>(row + c));
@@ -223,14 +252,14 @@ __device__ __forceinline__ float pa_block_stats(const float *v, int n, int cente
 }
 
 // The seam between two sublayers of a sequential block, one CTA per token:
-//   y given:  x <- x + G(y; w_out)   (w_out null: x <- x + y)      the sublayer's output, normed, joins the residual stream
+//   y given:  x <- x + y_scale G(y; w_out)   (w_out null: y itself)  the sublayer's output, normed, joins the residual stream
 //   add_tok / add_vec given:  x <- x + add_tok[token] + add_vec     what a new pass of a looped model adds before its first layer
-//   h given:  h  = G(x; w_in)                                       the next sublayer's input
+//   h given:  h  = G(x; w_in)  (w_in null: x itself; rows of stride ldh)  the next sublayer's input
 // G cuts the vector into `groups` equal parts and divides each by its own sqrt(mean(part^2) + eps) before the weight; with
 // `center` the part's mean is taken off first (a layer norm without bias).
 __global__ void __launch_bounds__(256) pa_k_seam_norm(float *__restrict__ x, const float *__restrict__ y, const float *__restrict__ w_out, float *__restrict__ h,
                                                       const float *__restrict__ w_in, int dim, int groups, float eps, int center, const float *__restrict__ add_tok,
-                                                      const float *__restrict__ add_vec) {
+                                                      const float *__restrict__ add_vec, float y_scale, int ldh) {
     __shared__ float red[8];
     const int64_t base = (int64_t)blockIdx.x * dim;
     const int gs = dim / groups;
@@ -239,14 +268,16 @@ __global__ void __launch_bounds__(256) pa_k_seam_norm(float *__restrict__ x, con
         if (y) {
             float inv = 1.0f, mu = 0.f;
             if (w_out) inv = pa_block_stats(y + base + c0, gs, center, eps, red, mu);
-            for (int c = threadIdx.x; c < gs; c += 256) x[base + c0 + c] += w_out ? (y[base + c0 + c] - mu) * inv * w_out[c0 + c] : y[base + c0 + c];
+            for (int c = threadIdx.x; c < gs; c += 256) x[base + c0 + c] += y_scale * (w_out ? (y[base + c0 + c] - mu) * inv * w_out[c0 + c] : y[base + c0 + c]);
         }
         if (add_tok || add_vec)
             for (int c = threadIdx.x; c < gs; c += 256) x[base + c0 + c] += (add_tok ? add_tok[base + c0 + c] : 0.f) + (add_vec ? add_vec[c0 + c] : 0.f);
-        if (h) {
+        if (h && !w_in) {
+            for (int c = threadIdx.x; c < gs; c += 256) h[(int64_t)blockIdx.x * ldh + c0 + c] = x[base + c0 + c];
+        } else if (h) {
             float mu;
             const float inv = pa_block_stats(x + base + c0, gs, center, eps, red, mu); // (a thread reads back its own writes)
-            for (int c = threadIdx.x; c < gs; c += 256) h[base + c0 + c] = (x[base + c0 + c] - mu) * inv * w_in[c0 + c];
+            for (int c = threadIdx.x; c < gs; c += 256) h[(int64_t)blockIdx.x * ldh + c0 + c] = (x[base + c0 + c] - mu) * inv * w_in[c0 + c];
         }
     }
 }
@@ -260,22 +291,29 @@ __device__ __forceinline__ float pa_warp_inv_rms(const float *v, int n, float ep
     return 1.0f / sqrtf(s / (float)n + eps);
 }
 
-// After the q|k|v projection of a batch, one CTA per token: unit-RMS q heads (in place) and k heads (qk_norm), the value rows
-// blended with the source layer's (v_mix), K row -> kc[pos][:], V row transposed -> vct[:][pos].
+// factor on the query at position p (coef 0: 1); the quotient in double, so that the floor is right at every multiple
+__device__ __forceinline__ float pa_q_temp(float coef, float every, int p) {
+    return coef != 0.f ? 1.0f + coef * logf((float)floor((double)(p + 1) / (double)every) + 1.0f) : 1.0f;
+}
+
+// After the q|k|v projection of a batch, one CTA per token: unit-RMS q heads (in place) and k heads (qk_norm; times the weights qn / kn
+// and, for q, the position's temperature), the value rows blended with the source layer's (v_mix), K row -> kc[pos][:], V row transposed -> vct[:][pos].
 __global__ void __launch_bounds__(256) pa_k_qkv_post(float *__restrict__ qkv, int ld, int H, int G, int dq, int dv, int qk_norm, float eps, int v_mix,
                                                      const float *__restrict__ lambda, float *__restrict__ v_src, int ld_src, float *__restrict__ kc,
-                                                     float *__restrict__ vct, int n_ctx, const int32_t *__restrict__ pos) {
+                                                     float *__restrict__ vct, int n_ctx, const int32_t *__restrict__ pos, const float *__restrict__ qn, const float *__restrict__ kn,
+                                                     float qt_coef, float qt_every) {
     const int t = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, p = pos[t];
     float *row = qkv + (int64_t)t * ld;
+    const float qt = pa_q_temp(qt_coef, qt_every, p);
     const int qd = H * dq, kd = G * dq, vd = G * dv;
     for (int hh = warp; hh < H + G; hh += 8) { // q heads, then k heads
         float *v = row + hh * dq;
         const float inv = qk_norm ? pa_warp_inv_rms(v, dq, eps, lane) : 1.0f;
         if (hh < H) {
-            if (qk_norm) for (int c = lane; c < dq; c += 32) v[c] *= inv;
+            if (qk_norm) for (int c = lane; c < dq; c += 32) v[c] *= inv * (qn ? qn[c] : 1.0f) * qt;
         } else {
             float *dst = kc + (int64_t)p * kd + (hh - H) * dq;
-            for (int c = lane; c < dq; c += 32) dst[c] = v[c] * inv;
+            for (int c = lane; c < dq; c += 32) dst[c] = v[c] * inv * (kn ? kn[c] : 1.0f);
         }
     }
     const float lam = v_mix == PS_VMIX_BLEND ? lambda[0] : 0.f;
@@ -307,7 +345,7 @@ __device__ __forceinline__ void pa_rope_store(const PaRope &r, const float *src,
     else dst[c] = c < half ? src[c] * cs - src[c + half] * sn : src[c] * cs + src[c - half] * sn;
 }
 
-// After the down-projections W_dq | W_dkv of a latent attention, one CTA per token.  Row t = [q latent (rq) | kv latent (rk) |
+// After the down-projections W_dq | W_dkv of a latent attention, one CTA per token.  Row t = [q latent (rq, 0: none) | kv latent (rk) |
 // rotated key part (dr)]: cq = N(q latent; wq) -> cq[t];  c = N(kv latent; wk) -> kc[pos][0 .. rk) and vct[.][pos];
 // rot(key part, pos) -> kc[pos][rk .. rk + dr).
 __global__ void __launch_bounds__(256) pa_k_latent_post(const float *__restrict__ t_in, int ld, int rq, int rk, int dr, const float *__restrict__ wq, const float *__restrict__ wk,
@@ -317,10 +355,12 @@ __global__ void __launch_bounds__(256) pa_k_latent_post(const float *__restrict_
     const int t = blockIdx.x, p = pos[t];
     const float *row = t_in + (int64_t)t * ld;
     float s = 0.f;
-    for (int c = threadIdx.x; c < rq; c += 256) s = fmaf(row[c], row[c], s);
-    const float iq = 1.0f / sqrtf(pa_block_sum(s, red) / (float)rq + eps);
-    for (int c = threadIdx.x; c < rq; c += 256) cq[(int64_t)t * rq + c] = row[c] * iq * wq[c];
-    s = 0.f;
+    if (rq > 0) {
+        for (int c = threadIdx.x; c < rq; c += 256) s = fmaf(row[c], row[c], s);
+        const float iq = 1.0f / sqrtf(pa_block_sum(s, red) / (float)rq + eps);
+        for (int c = threadIdx.x; c < rq; c += 256) cq[(int64_t)t * rq + c] = row[c] * iq * wq[c];
+        s = 0.f;
+    }
     for (int c = threadIdx.x; c < rk; c += 256) s = fmaf(row[rq + c], row[rq + c], s);
     const float ik = 1.0f / sqrtf(pa_block_sum(s, red) / (float)rk + eps);
     float *krow = kc + (int64_t)p * (rk + dr);
@@ -332,21 +372,22 @@ __global__ void __launch_bounds__(256) pa_k_latent_post(const float *__restrict_
     for (int c = threadIdx.x; c < dr; c += 256) pa_rope_store(rope, row + rq + rk, krow + rk, dr, p, c);
 }
 
-// the rotated part of every query head: q[t][h * (dn + dr) + dn ..] -> qa[t][h * (rk + dr) + rk ..], rotated by the token's position
-__global__ void __launch_bounds__(256) pa_k_rope_q(const float *__restrict__ q, float *__restrict__ qa, int H, int dn, int dr, int rk, PaRope rope, const int32_t *__restrict__ pos) {
+// the rotated part of every query head: q[t * ldq + h * (dn + dr) + dn ..] -> qa[t][h * (rk + dr) + rk ..], rotated by the token's position
+__global__ void __launch_bounds__(256) pa_k_rope_q(const float *__restrict__ q, int ldq, float *__restrict__ qa, int H, int dn, int dr, int rk, PaRope rope, const int32_t *__restrict__ pos) {
     const int t = blockIdx.x, p = pos[t];
     for (int e = threadIdx.x; e < H * dr; e += 256) {
         const int hh = e / dr, c = e % dr;
-        pa_rope_store(rope, q + ((int64_t)t * H + hh) * (dn + dr) + dn, qa + ((int64_t)t * H + hh) * (rk + dr) + rk, dr, p, c);
+        pa_rope_store(rope, q + (int64_t)t * ldq + hh * (dn + dr) + dn, qa + ((int64_t)t * H + hh) * (rk + dr) + rk, dr, p, c);
     }
 }
 
 // ---------------------------------------------------------------------------------------------------------------- dense
 // C[m][n] = sum_k A[m][k] W[n][k] + bias[n].  blockIdx.z walks groups (per-head products): group z reads the columns of A from
-// z * a_gs on, the matrix z of N x K weights, and writes the columns of C from z * c_gs on.
+// z * a_gs on, the matrix z of N x K weights, and writes the columns of C from z * c_gs on.  Rows n >= act_from leave through the
+// one-argument activation, `gap` columns further on.
 template <bool ROUND>
 __global__ void __launch_bounds__(256) pa_k_linear(const float *__restrict__ A, int lda, const bf16 *__restrict__ W, const float *__restrict__ bias, float *__restrict__ C, int ldc,
-                                                   int M, int N, int K, int a_gs = 0, int c_gs = 0) {
+                                                   int M, int N, int K, int a_gs = 0, int c_gs = 0, int act_from = 1 << 30, int gap = 0, PaAct act = PaAct{}) {
     PA_TILE_SMEM(1);
     const int tid = threadIdx.x, lr = tid >> 2, tx = tid & 15, ty = tid >> 4;
     const int m0 = blockIdx.y * PA_TM, n0 = blockIdx.x * PA_TN;
@@ -364,7 +405,10 @@ __global__ void __launch_bounds__(256) pa_k_linear(const float *__restrict__ A, 
 #pragma unroll
         for (int j = 0; j < 4; j++) {
             const int n = n0 + tx * 4 + j;
-            if (n < N) C[(int64_t)m * ldc + n] = acc[0][i][j] + (bias ? bias[n] : 0.f);
+            if (n >= N) continue;
+            const float v = acc[0][i][j] + (bias ? bias[n] : 0.f);
+            if (n < act_from) C[(int64_t)m * ldc + n] = v;
+            else C[(int64_t)m * ldc + n + gap] = pa_act1(v, act);
         }
     }
 }
@@ -373,7 +417,8 @@ __global__ void __launch_bounds__(256) pa_k_linear(const float *__restrict__ A, 
 // how a router turns its logits into chosen experts and weights
 struct PaRoute {
     int E, top;
-    int act;           // PS_ROUTER_SIGMOID: every logit through a sigmoid; PS_ROUTER_SOFTMAX: soft-max over all experts
+    int act;           // PS_ROUTER_SIGMOID: every logit through a sigmoid; PS_ROUTER_SOFTMAX: soft-max over all experts;
+                       // PS_ROUTER_TOPK_SOFTMAX: the largest logits, soft-max over those alone (pa_route_topk_warp)
     int groups, keep;  // groups > 1: equal groups of neighbouring experts, a group is worth its best score, the `keep` best groups stay
     int renorm;        // the chosen scores are divided by their sum + eps
     float eps;
@@ -425,10 +470,38 @@ __device__ __forceinline__ void pa_route_serial(const float *__restrict__ z, con
         for (int n = 0; n < r.top; n++) sw[n] /= sum + r.eps;
 }
 
-// router logits W_r h in fp32 (h unrounded), then pa_route_serial -> sel_e / sel_w [token][top]; with a shared gate the matrix's
+// one warp: the `top` largest of E logits (ties: the lower expert), weights = soft-max over the chosen; se / sw are in shared memory
+__device__ __forceinline__ void pa_route_topk_warp(const float *__restrict__ z, int E, int top, int *se, float *sw, int lane) {
+    float v[PA_MAX_EXPERTS / 32], z0 = 0.f, sum = 0.f;
+    unsigned taken = 0;
+#pragma unroll
+    for (int i = 0; i < PA_MAX_EXPERTS / 32; i++) v[i] = lane + 32 * i < E ? z[lane + 32 * i] : 0.f;
+    for (int n = 0; n < top; n++) {
+        int be = -1;
+        float bv = 0.f;
+#pragma unroll
+        for (int i = 0; i < PA_MAX_EXPERTS / 32; i++)
+            if (lane + 32 * i < E && !((taken >> i) & 1) && (be < 0 || v[i] > bv)) { be = lane + 32 * i; bv = v[i]; }
+#pragma unroll
+        for (int o = 16; o; o >>= 1) {
+            const int oe = __shfl_xor_sync(0xffffffffu, be, o);
+            const float ov = __shfl_xor_sync(0xffffffffu, bv, o);
+            if (oe >= 0 && (be < 0 || ov > bv || (ov == bv && oe < be))) { be = oe; bv = ov; }
+        }
+        if ((be & 31) == lane) taken |= 1u << (be >> 5);
+        if (n == 0) z0 = bv;
+        const float e = expf(bv - z0);
+        sum += e;
+        if (lane == 0) { se[n] = be; sw[n] = e; }
+    }
+    __syncwarp();
+    for (int n = lane; n < top; n += 32) sw[n] /= sum;
+}
+
+// router logits W_r h (+ bias) in fp32 (h unrounded), then pa_route_serial -> sel_e / sel_w [token][top]; with a shared gate the matrix's
 // last row gives sgate[token] = sigmoid(w_sg . h)
 __global__ void __launch_bounds__(256) pa_k_router(const float *__restrict__ h, const bf16 *__restrict__ Wr, int dim, PaRoute r, int *__restrict__ sel_e,
-                                                   float *__restrict__ sel_w, float *__restrict__ sgate) {
+                                                   float *__restrict__ sel_w, float *__restrict__ sgate, const float *__restrict__ bias) {
     __shared__ float zs[PA_MAX_EXPERTS + 1], sc[PA_MAX_EXPERTS], sw[PA_MAX_EXPERTS];
     __shared__ int se[PA_MAX_EXPERTS];
     const int t = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
@@ -438,9 +511,18 @@ __global__ void __launch_bounds__(256) pa_k_router(const float *__restrict__ h, 
         const int e1 = min(e + 1, n_rows - 1);
         float s0, s1;
         pa_dot2<false>(Wr + (int64_t)e * dim, Wr + (int64_t)e1 * dim, hr, dim, 1.0f, lane, s0, s1);
-        if (lane == 0) { zs[e] = s0; zs[e1] = s1; }
+        if (lane == 0) { zs[e] = s0 + (bias && e < r.E ? bias[e] : 0.f); zs[e1] = s1 + (bias && e1 < r.E ? bias[e1] : 0.f); }
     }
     __syncthreads();
+    if (r.act == PS_ROUTER_TOPK_SOFTMAX) {
+        if (warp == 0) {
+            pa_route_topk_warp(zs, r.E, r.top, se, sw, lane);
+            __syncwarp();
+            for (int n = lane; n < r.top; n += 32) { sel_e[t * r.top + n] = se[n]; sel_w[t * r.top + n] = sw[n]; }
+            if (lane == 0 && r.shared_gate) sgate[t] = 1.0f / (1.0f + expf(-zs[r.E]));
+        }
+        return;
+    }
     if (threadIdx.x == 0) {
         pa_route_serial(zs, r, sc, se, sw);
         for (int n = 0; n < r.top; n++) { sel_e[t * r.top + n] = se[n]; sel_w[t * r.top + n] = sw[n]; }
@@ -476,39 +558,23 @@ __global__ void __launch_bounds__(256) pa_k_dispatch(const int *__restrict__ sel
     }
 }
 
-__device__ __forceinline__ float pa_expert_act(float g, float u, PaAct act) {
-    if (act.kind == PS_ACT_GELU_TANH) // 0.5 g (1 + tanh(sqrt(2 / pi) (g + 0.044715 g^3))) * u
-        return 0.5f * g * (1.0f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g))) * u;
-    g = fminf(g, act.limit);
-    u = fminf(fmaxf(u, -act.limit), act.limit);
-    return g * (1.0f / (1.0f + expf(-act.alpha * g))) * (u + act.shift);
-}
-
-// the one-argument forms (a feed-forward without a gate)
-__device__ __forceinline__ float pa_act1(float z, PaAct act) {
-    if (act.kind == PS_ACT_XIELU) return z > 0.f ? fmaf(act.alpha * z, z, 0.5f * z) : fmaf(act.shift, expm1f(z) - z, 0.5f * z);
-    if (act.kind == PS_ACT_GELU_TANH) return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
-    z = fminf(z, act.limit);
-    return z * (1.0f / (1.0f + expf(-act.alpha * z)));
-}
-
-// y[r][n] = act(gate_e . z_r, up_e . z_r), z_r = w_r * h[token_r] (route_on_input) or h[token_r]
-template <bool ROUND>
+// y[r][n] = act(gate_e . z_r, up_e . z_r), z_r = w_r * h[token_r] (route_on_input) or h[token_r]; NB = 1: no gate, act(up_e . z_r)
+template <bool ROUND, int NB>
 __global__ void __launch_bounds__(256) pa_k_expert_up(const float *__restrict__ h, int ldh, const int *__restrict__ row_token, const float *__restrict__ row_w,
                                                       const int *__restrict__ tile_e, const int *__restrict__ tile_row0, const int *__restrict__ tile_end,
                                                       const int *__restrict__ n_tiles, const bf16 *__restrict__ Wg, const bf16 *__restrict__ Wu, float *__restrict__ y, int ff,
                                                       int dim, int on_input, PaAct act) {
-    PA_TILE_SMEM(2);
+    PA_TILE_SMEM(NB);
     if ((int)blockIdx.y >= *n_tiles) return;
     const int tid = threadIdx.x, lr = tid >> 2, tx = tid & 15, ty = tid >> 4;
     const int e = tile_e[blockIdx.y], r0 = tile_row0[blockIdx.y], rend = tile_end[blockIdx.y], n0 = blockIdx.x * PA_TN;
-    float acc[2][4][4] = {};
+    float acc[NB][4][4] = {};
     const bool rin = r0 + lr < rend;
     const float *arow = rin ? h + (int64_t)row_token[r0 + lr] * ldh : nullptr;
     const float ascale = (rin && on_input) ? row_w[r0 + lr] : 1.0f;
     const int64_t wofs = ((int64_t)e * ff + n0 + lr) * dim;
     const bool nin = n0 + lr < ff;
-    pa_tile_mm<ROUND, bf16, 2>(acc, arow, ascale, nin ? Wg + wofs : nullptr, nin ? Wu + wofs : nullptr, dim, As, Bs);
+    pa_tile_mm<ROUND, bf16, NB>(acc, arow, ascale, nin ? (NB == 2 ? Wg : Wu) + wofs : nullptr, nin ? Wu + wofs : nullptr, dim, As, Bs);
 #pragma unroll
     for (int i = 0; i < 4; i++) {
         const int r = r0 + ty * 4 + i;
@@ -516,7 +582,7 @@ __global__ void __launch_bounds__(256) pa_k_expert_up(const float *__restrict__ 
 #pragma unroll
         for (int j = 0; j < 4; j++) {
             const int n = n0 + tx * 4 + j;
-            if (n < ff) y[(int64_t)r * ff + n] = pa_expert_act(acc[0][i][j], acc[1][i][j], act);
+            if (n < ff) y[(int64_t)r * ff + n] = NB == 2 ? pa_expert_act(acc[0][i][j], acc[NB - 1][i][j], act) : pa_act1(acc[0][i][j], act);
         }
     }
 }
@@ -752,7 +818,7 @@ __global__ void __launch_bounds__(256) pa_k_pv(PaAttn at, const float *__restric
 #pragma unroll
         for (int j = 0; j < 4; j++) {
             const int n = n0 + tx * 4 + j;
-            if (n < at.dv) att[(int64_t)m * od + h * at.dv + n] = acc[0][i][j];
+            if (n < at.dv) att[(int64_t)m * od + h * at.dv + n] = at.gate ? acc[0][i][j] * pa_sigmoid(at.gate[(int64_t)m * at.ld_gate + h]) : acc[0][i][j];
         }
     }
 }

@@ -5,7 +5,8 @@
 // whatever the state buffers hold (a cache set that is used again needs no clearing).
 //
 //   pa_k_short_conv      causal convolution over time on every channel, taps newest last, inputs before the batch from the `tail`
-//                        (the last taps - 1 inputs of the sequence), zeros before position 0; optional bias and silu
+//                        (the last taps - 1 inputs of the sequence; as a ring of `taps` rows, position p in row p mod taps, for the rg-lru),
+//                        zeros before position 0; optional bias and silu
 //   pa_k_conv_tail       the tail after the batch
 //   pa_k_conv_step       both for a single token
 //   pa_k_qkv_whole_norm  q (all heads) and k RMS-normed as one vector each with weights; K row and V^T column into the cache
@@ -16,6 +17,9 @@
 //                        depend on how a prompt was cut)
 //   pa_k_gate_gru        after an attention: the heads' outputs times their sigmoid gate, and the minGRU beside the attention
 //                        (S_t = (1 - z) S_(t-1) + z cand per channel, rounds of 32 tokens, gates formed ahead of the dependent steps)
+//   pa_k_rglru_scan      real-gated linear recurrence of a batch: S_t = a_t S_(t-1) + sqrt(1 - a_t^2) i_t u_t with log a_t = -rate r_t
+//                        softplus(lam), times gelu(y); rounds of 32 tokens like the minGRU; leaves the convolution's ring for the next batch
+//   pa_k_dec_rglru       convolution, both gates' block rows, recurrence and output product of a single token in one launch
 //   pa_k_gate_norm       RMS norm in equal parts around a silu gate: (y silu(g)) normed times w, or normed y times silu(g)
 //   pa_k_moe_sum         sum of a token's expert slots (fixed order) plus the gated shared expert
 #pragma once
@@ -25,7 +29,7 @@ __device__ __forceinline__ float pa_softplus(float v) { return v > 20.f ? v : lo
 
 // grid (channels / 256, tokens)
 __global__ void __launch_bounds__(256) pa_k_short_conv(const float *__restrict__ u, int ldu, const float *__restrict__ w, const float *__restrict__ b, int C, int T,
-                                                       const float *__restrict__ tail, int act_silu, float *__restrict__ y, int ldy, const int32_t *__restrict__ pos) {
+                                                       const float *__restrict__ tail, int act_silu, float *__restrict__ y, int ldy, const int32_t *__restrict__ pos, int ring) {
     const int t = blockIdx.y, c = blockIdx.x * 256 + threadIdx.x;
     if (c >= C) return;
     const int p0 = pos[0];
@@ -34,7 +38,7 @@ __global__ void __launch_bounds__(256) pa_k_short_conv(const float *__restrict__
         const int s = t - (T - 1) + j; // token of the batch this tap meets (negative: before the batch)
         float v = 0.f;
         if (s >= 0) v = u[(int64_t)s * ldu + c];
-        else if (p0 + s >= 0) v = tail[(int64_t)(T - 1 + s) * C + c];
+        else if (p0 + s >= 0) v = tail[(int64_t)(ring ? (p0 + s) % T : T - 1 + s) * C + c];
         acc = fmaf(w[(int64_t)c * T + j], v, acc);
     }
     y[(int64_t)t * ldy + c] = act_silu ? pa_silu(acc) : acc;
@@ -167,6 +171,105 @@ __global__ void __launch_bounds__(PA_GG_THREADS) pa_k_gate_gru(float *__restrict
         __syncthreads();
     }
     if (warp == 0 && live) state[c] = S;
+}
+
+struct PaRglru {
+    const float *y, *x;        // rows of the first projection: the gelu branch and the convolution's input, W channels each (row stride ld)
+    int ld;
+    const float *u, *g;        // batch: convolved inputs [t][W]; gate logits [t][block][r part | i part] without their biases
+    const float *rb, *ib, *sp; // [W]: gate biases, rate * softplus(lam)
+    int W, bsz, taps;          // channels, channels per block of the gates' matrices
+    const float *conv_w, *conv_b; // [W][taps], [W]
+    const bf16 *wri;           // [block][r rows | i rows][bsz]
+    float *S, *ring;           // [W]; [taps][W], the convolution's input of position p in row p mod taps
+    float *o;                  // S gelu(y), row stride ldo
+    int ldo;
+    const int32_t *pos;
+    int bs;
+};
+// one step's coefficients from the gate logits: a = exp(-sp r), b = sqrt(1 - a^2) i u (1 - a^2 without cancellation)
+__device__ __forceinline__ void pa_rglru_coef(float gr, float gi, float sp, float u, float &a, float &b) {
+    const float la = -sp * pa_sigmoid(gr);
+    a = expf(la);
+    b = sqrtf(-expm1f(2.0f * la)) * pa_sigmoid(gi) * u;
+}
+__device__ __forceinline__ float pa_gelu_tanh(float z) { return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z))); }
+
+// 32 channels per CTA, rounds of 32 tokens: the four warps form the coefficients of eight tokens each (nothing there depends on S), warp
+// 0 walks the 32 steps in order, a lane per channel - the same operations per step whatever the round and the cut of the prompt
+__global__ void __launch_bounds__(PA_GG_THREADS) pa_k_rglru_scan(const PaRglru a) {
+    __shared__ float aa[PA_GG_TOK][32], ba[PA_GG_TOK][32], ya[PA_GG_TOK][32];
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, c = blockIdx.x * 32 + lane, W = a.W;
+    const bool live = c < W;
+    const int cc = live ? c : W - 1, blk = cc / a.bsz, gc = blk * 2 * a.bsz + cc % a.bsz;
+    const int p0 = a.pos[0];
+    float S = p0 > 0 ? a.S[cc] : 0.f;
+    const float rb = a.rb[cc], ib = a.ib[cc], sp = a.sp[cc];
+    constexpr int PER = PA_GG_TOK / (PA_GG_THREADS / 32);
+    for (int t0 = 0; t0 < a.bs; t0 += PA_GG_TOK) {
+        float gr[PER], gi[PER], ur[PER], yr[PER];
+#pragma unroll
+        for (int i = 0; i < PER; i++) {
+            const int64_t t = min(t0 + warp * PER + i, a.bs - 1);
+            gr[i] = a.g[t * 2 * W + gc]; gi[i] = a.g[t * 2 * W + gc + a.bsz]; ur[i] = a.u[t * W + cc]; yr[i] = a.y[t * a.ld + cc];
+        }
+#pragma unroll
+        for (int i = 0; i < PER; i++) {
+            const int s = warp * PER + i;
+            pa_rglru_coef(gr[i] + rb, gi[i] + ib, sp, ur[i], aa[s][lane], ba[s][lane]);
+            ya[s][lane] = pa_gelu_tanh(yr[i]);
+        }
+        __syncthreads();
+        if (warp == 0 && live) {
+            const int n = min(PA_GG_TOK, a.bs - t0);
+#pragma unroll 8
+            for (int i = 0; i < n; i++) {
+                S = fmaf(aa[i][lane], S, ba[i][lane]);
+                a.o[(int64_t)(t0 + i) * a.ldo + c] = S * ya[i][lane];
+            }
+        }
+        __syncthreads();
+    }
+    if (warp == 0 && live) a.S[c] = S;
+    // the last taps - 1 inputs of the sequence (older ones than this batch's are in the ring already)
+    if (warp == 1 && live)
+        for (int t = max(0, a.bs - (a.taps - 1)); t < a.bs; t++) a.ring[(int64_t)((p0 + t) % a.taps) * W + c] = a.x[(int64_t)t * a.ld + c];
+}
+
+// grid (channels per block / 8, blocks): a CTA convolves the block's inputs into shared memory, then a warp takes one channel - its r and i
+// rows are the pair of dot products (fp32 inputs, never rounded).  The ring has `taps` rows, so the row this token writes (by the channel's
+// own CTA) is none of those that the other CTAs read.
+__global__ void __launch_bounds__(256) pa_k_dec_rglru(const PaRglru a) {
+    extern __shared__ __align__(16) float pa_us[]; // [bsz]
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, bsz = a.bsz, blk = blockIdx.y, n = blockIdx.x * 8 + warp;
+    const bf16 *wr = a.wri + ((int64_t)blk * 2 * bsz + min(n, bsz - 1)) * bsz, *wi = wr + (int64_t)bsz * bsz;
+    pa_prefetch2(wr, wi, 0, bsz, lane);
+    ps_grid_dep_launch();
+    ps_grid_dep_wait();
+    const int p = a.pos[0], T = a.taps;
+    for (int c = threadIdx.x; c < bsz; c += 256) {
+        const int ch = blk * bsz + c;
+        const float cur = a.x[ch];
+        float acc = a.conv_b[ch];
+        for (int j = 0; j < T - 1; j++) {
+            const int q = p - (T - 1) + j;
+            acc = fmaf(a.conv_w[(int64_t)ch * T + j], q >= 0 ? a.ring[(int64_t)(q % T) * a.W + ch] : 0.f, acc);
+        }
+        pa_us[c] = fmaf(a.conv_w[(int64_t)ch * T + T - 1], cur, acc);
+        if (c >= blockIdx.x * 8 && c < blockIdx.x * 8 + 8) a.ring[(int64_t)(p % T) * a.W + ch] = cur;
+    }
+    __syncthreads();
+    if (n >= bsz) return;
+    float gr, gi;
+    pa_dot2<false>(wr, wi, pa_us, bsz, 1.0f, lane, gr, gi);
+    if (lane == 0) {
+        const int ch = blk * bsz + n;
+        float ca, cb;
+        pa_rglru_coef(gr + a.rb[ch], gi + a.ib[ch], a.sp[ch], pa_us[n], ca, cb);
+        const float S = fmaf(ca, p > 0 ? a.S[ch] : 0.f, cb);
+        a.S[ch] = S;
+        a.o[ch] = S * pa_gelu_tanh(a.y[ch]);
+    }
 }
 
 #define PA_SC_TOK 32    // tokens staged per round (half as many for the widest states)

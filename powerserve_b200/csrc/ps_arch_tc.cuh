@@ -81,7 +81,8 @@ struct PtArgs {
     const float *row_w;
     int top, on_input;
     PaAct act;
-    int act1;               // PT_MODE_DENSE: the one-argument activation on every output (a feed-forward without a gate)
+    int act1;               // dense / expert up: the one-argument activation on the outputs n >= act_from (a feed-forward without a gate),
+    int act_from, gap;      // which are stored `gap` columns further on
     int *err;
 };
 
@@ -193,9 +194,10 @@ __global__ void __launch_bounds__(PT_THREADS, 1) pa_k_tc_gemm(const PtArgs a) {
                         if (r >= rend) break;
                         const float acc = __uint_as_float(v[c]);
                         if (a.mode == PT_MODE_DENSE) {
-                            a.C[(int64_t)r * a.ldc + n] = a.act1 ? pa_act1(acc + bias, a.act) : acc + bias;
+                            if (a.act1 && n >= a.act_from) a.C[(int64_t)r * a.ldc + n + a.gap] = pa_act1(acc + bias, a.act);
+                            else a.C[(int64_t)r * a.ldc + n] = acc + bias;
                         } else if (a.mode == PT_MODE_EXPERT_UP) {
-                            a.C[(int64_t)r * a.ldc + n] = pa_expert_act(acc, NA == 2 ? __uint_as_float(w2[c]) : 0.f, a.act);
+                            a.C[(int64_t)r * a.ldc + n] = NA == 2 ? pa_expert_act(acc, __uint_as_float(w2[c]), a.act) : pa_act1(acc, a.act);
                         } else {
                             a.C[((int64_t)a.row_token[r] * a.top + a.row_slot[r]) * a.ldc + n] = a.on_input ? acc : acc * a.row_w[r];
                         }

@@ -41,7 +41,7 @@ def test_registry_reads_every_size_from_the_configuration():
                                        (None, [0, 1, 2]), ((1, 1, 5), [0, 1, 2])])
 def test_runs_follow_the_loop(loop, want):
     cfg = arch_synth.pidenex_config(16, 8, [AT(1, 1, 4, window=3), AT(1, 1, 4, window=3), AT(1, 1, 4, window=3)], loop=loop)
-    runs = arch._pidenex_runs(cfg)
+    runs = arch._layer_runs(cfg)
     assert [i for i, _ in runs] == want == [i for i, _ in R.layer_runs(cfg)]
     assert runs == R.layer_runs(cfg)
     if loop and loop[1] > loop[0]:
@@ -58,7 +58,7 @@ def test_runs_follow_the_loop(loop, want):
 def test_bad_loops_and_types_are_refused():
     for loop in ((2, 1, 2), (0, 4, 2), (0, 1, 0), (-1, 1, 1)):
         with pytest.raises(capi.PsCudaError):
-            arch._pidenex_runs(arch_synth.pidenex_config(16, 8, [AT(1, 1, 4, window=3)] * 3, loop=loop))
+            arch._layer_runs(arch_synth.pidenex_config(16, 8, [AT(1, 1, 4, window=3)] * 3, loop=loop))
     cfg = arch_synth.pidenex_config(16, 8, [AT(1, 1, 4, window=3)])
     cfg["layers"][0]["type"] = "retention"
     with pytest.raises(capi.PsCudaError):
