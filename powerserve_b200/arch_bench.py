@@ -1,4 +1,4 @@
-"""bench.py --arch nufusun | vanapel | dozotar | pidenex: prefill and decode throughput of a layer-list design at layer sizes that resemble real
+"""bench.py --arch nufusun | vanapel | dozotar | pidenex | momedra: prefill and decode throughput of a layer-list design at layer sizes that resemble real
 models (random weights), beside the closest existing model of the framework.
 
 --arch vanapel: the Vanapel design (windowed attention layers and one latent-attention layer, dense gated feed-forward) beside
@@ -13,6 +13,11 @@ attention with rotation in neighbouring pairs, feed-forwards without a gate; the
 sizes s and m) beside Vanapel - the closest existing model: sequential blocks normed on both sides, windowed and latent attention,
 dense feed-forward - with as many layer runs, equal width, head geometry, windows, vocabulary and feed-forward bytes (a gated unit of
 ff rows against an ungated one of 3 ff / 2).
+
+--arch momedra: the Momedra design (parallel blocks: full attention with routed experts beside a shared one, latent attention and an
+RG-LRU with dense feed-forwards; the first two layers run twice at sizes s and m) beside Pidenex - the closest existing model: layer
+norms, layer runs, latent attention with neighbouring pairs, a gated recurrence, feed-forwards without a gate - with as many layer
+runs, equal width, head geometry, keys in sight, vocabulary and ACTIVE feed-forward rows per token.
 
 --arch nufusun: prefill and decode throughput of the Nufusun design at layer sizes that resemble real models
 (random weights), beside the closest existing model of the framework - a llama stack (Q4_K) with the same width, head
@@ -338,6 +343,80 @@ def run_size_pidenex(name, prompt_len, steps, warmup, seed, chunk):
     return out
 
 
+# name: (width, heads, kv heads, head size, active ff rows, latent (heads, plain dims, rotated dims, value dims, kv rank, Pidenex' q rank), rg-lru blocks, layer types, loop, vocab)
+MOMEDRA_SIZES = {
+    "s": (1024, 16, 4, 64, 3072, (16, 64, 32, 64, 256, 384), 16, "alr", (0, 2, 2), 32000),
+    "m": (2048, 16, 4, 128, 8448, (16, 128, 64, 128, 512, 768), 16, "alr", (0, 2, 2), 32000),
+    "l": (4096, 32, 8, 128, 21504, (32, 128, 64, 128, 512, 1536), 16, "alr", None, 32000),
+}
+
+
+def _momedra_model(name, seed, chunk, n_ctx):
+    W, H, G, hs, ff, (LH, dn, dr, dv, rk, _), nb, kinds, loop, V = MOMEDRA_SIZES[name]
+    layers = []
+    for k in kinds:
+        if k == "a":    # 2 of 8 experts of ff / 4 rows beside a shared one of ff / 2: ff active rows
+            layers.append(arch_synth.momedra_attention_layer(H, G, hs, hs, q_temp=(0.2, 512), ff=ff // 4, experts=8, top=2, shared_ff=ff // 2))
+        elif k == "l":
+            layers.append(arch_synth.momedra_latent_layer(LH, dn, dr, dv, rk, rope_base=5e5, ff=ff))
+        else:
+            layers.append(arch_synth.momedra_rglru_layer(W, nb, conv=4, ff=ff))
+    cfg = arch_synth.momedra_config(W, V, layers, loop=loop)
+    return cfg, _load_synth(cfg, arch_synth.momedra_weights(cfg, seed=seed, fast=True), chunk, n_ctx)
+
+
+def _momedra_comparator(name, seed, chunk, n_ctx):
+    """Pidenex with the same runs: a window that nothing leaves for the attention, the attention beside a minGRU in the RG-LRU's place"""
+    W, H, G, hs, ff, (LH, dn, dr, dv, rk, rq), _, kinds, loop, V = MOMEDRA_SIZES[name]
+    layers = []
+    for k in kinds:
+        if k == "a":
+            layers.append(arch_synth.pidenex_attention_layer(H, G, hs, window=n_ctx, ff=ff))
+        elif k == "l":
+            layers.append(arch_synth.pidenex_latent_layer(LH, dn, dr, dv, rq, rk, rope_base=5e5, ff=ff))
+        else:
+            layers.append(arch_synth.pidenex_parallel_layer(H, G, hs, window=n_ctx, gru_width=W // 2, ff=ff))
+    cfg = arch_synth.pidenex_config(W, V, layers, loop=loop)
+    return cfg, _load_synth(cfg, arch_synth.pidenex_weights(cfg, seed=seed, fast=True), chunk, n_ctx)
+
+
+def run_size_momedra(name, prompt_len, steps, warmup, seed, chunk):
+    W, H, G, hs, ff, (LH, dn, dr, dv, rk, rq), nb, kinds, loop, V = MOMEDRA_SIZES[name]
+    hbm, tflops, src = _peaks()
+    n_ctx = -(-(prompt_len + steps + warmup + 24) // 256) * 256
+    prompt = [int(v) for v in np.random.default_rng(1234).integers(0, V, prompt_len)]
+    out = {"size": name, "width": W, "heads": [H, G], "head_size": hs, "active_ff": ff, "latent": [LH, dn, dr, dv, rk], "rglru_blocks": nb, "layers": kinds, "loop": loop, "vocab": V,
+           "context": prompt_len}
+
+    def report(m, params, cache_bytes, mix_flops):
+        t_pre, t_dec, launches, e2e = _measure(m, prompt, chunk, steps, warmup)
+        m.close()
+        flops = (2 * params + mix_flops) * prompt_len / t_pre / 1e12
+        by = 2 * params + cache_bytes
+        return {"prefill_tok_s": prompt_len / t_pre, "prefill_chunk": chunk, "prefill_tflops": flops, "prefill_frac_of_bf16_peak": flops / tflops,
+                "decode_tok_s": 1 / t_dec, "decode_ms": t_dec * 1e3, "decode_launches_per_step": launches, "decode_bytes_per_token": by,
+                "decode_frac_of_hbm_peak": by / t_dec / 1e9 / hbm, "e2e_decode_tok_s": e2e}
+
+    cfg, m = _momedra_model(name, seed, chunk, n_ctx)
+    runs = "".join(kinds[i] for i, _ in arch._layer_runs(cfg))
+    na, nl, nr, n_pass = runs.count("a"), runs.count("l"), runs.count("r"), (loop[2] if loop else 0)
+    p_att = (H + 2 * G) * hs * W + H * W + H * hs * W + 8 * W
+    p_lat = LH * (dn + dr) * W + (rk + dr) * W + LH * dn * rk + LH * dv * rk + LH * dv * W
+    p_rec = 3 * W * W + 2 * W * W // nb
+    params = na * p_att + nl * p_lat + nr * p_rec + len(runs) * 2 * ff * W + n_pass * 2 * W * W + V * W
+    kv_a, fl_a = 2 * G * hs * 4 * prompt_len, 2 * 2 * H * hs * prompt_len / 2
+    kv_l, fl_l = (2 * rk + dr) * 4 * prompt_len, 2 * LH * (2 * rk + dr) * prompt_len / 2
+    out["momedra"] = dict(report(m, params, na * kv_a + nl * kv_l + nr * 2 * W * 4, na * fl_a + nl * fl_l), runs=runs)
+    cfg, m = _momedra_comparator(name, seed, chunk, n_ctx)
+    q_att = (2 * H + G) * hs * W
+    q_par = q_att + H * hs * W + 4 * (W // 2) * W
+    q_lat = (rq + rk + dr) * W + LH * (dn + dr) * rq + LH * dn * rk + LH * dv * rk + LH * dv * W
+    params = na * q_att + nl * q_lat + nr * q_par + len(runs) * 2 * ff * W + V * W
+    out["pidenex"] = dict(report(m, params, (na + nr) * kv_a + nl * kv_l + nr * W * 4, (na + nr) * fl_a + nl * fl_l), runs=runs.replace("r", "p"))
+    out["peaks"] = {"hbm_gbs": hbm, "bf16_tflops": tflops, "source": src}
+    return out
+
+
 def main(args) -> int:
     if capi.load_library().ps_cuda_device_count() == 0:
         print(json.dumps({"arch": args.arch, "unavailable": "no CUDA device: there is no CPU fallback"}))
@@ -351,6 +430,11 @@ def main(args) -> int:
     if args.arch == "pidenex":
         res = [run_size_pidenex(s, args.arch_prompt, max(args.steps, 8), max(args.warmup, 3), args.seed, args.arch_chunk) for s in sizes]
         print(json.dumps({"arch": "pidenex", "dtype": "bf16", "data": "synthetic", "timing": "CUDA events around every call, warm-up first; weights exceed L2",
+                          "sizes": res}))
+        return 0
+    if args.arch == "momedra":
+        res = [run_size_momedra(s, args.arch_prompt, max(args.steps, 8), max(args.warmup, 3), args.seed, args.arch_chunk) for s in sizes]
+        print(json.dumps({"arch": "momedra", "dtype": "bf16", "data": "synthetic", "timing": "CUDA events around every call, warm-up first; weights exceed L2",
                           "sizes": res}))
         return 0
     if args.arch == "vanapel":

@@ -300,28 +300,33 @@ __global__ void __launch_bounds__(256) pa_k_dec_scores(PaAttn at, const float *_
         for (int jj = 0; jj < nc; jj++) ps_bulk_g2s(ks + jj * kds, kc + (int64_t)(j0 + jj) * kd, (uint32_t)(kd * 4), &bar);
     }
     if (!bulk) for (int t = tid; t < nc * kd; t += 256) ks[(t / kd) * kds + t % kd] = kc[(int64_t)j0 * kd + t];
-    for (int t = tid; t < H * dq; t += 256) qs[t] = q[t];
-    if (own) for (int t = tid; t < kd; t += 256) ks[nc * kds + t] = at.k_raw[t];
-    __syncthreads();
     if (at.k_raw) { // a warp per head: norm of q (times the position's temperature), and of the token's key on its way into the cache
+        const int lane = tid & 31;
         const float qt = pa_q_temp(at.qt_coef, at.qt_every, pos);
         for (int hh = tid >> 5; hh < H + (own ? G : 0); hh += 8) {
-            const int lane = tid & 31;
-            float *v = hh < H ? qs + hh * dq : ks + nc * kds + (hh - H) * dq;
-            const float inv = pa_warp_inv_rms(v, dq, at.eps, lane);
-            __syncwarp();
+            const bool is_q = hh < H;
+            const float *src = is_q ? q + hh * dq : at.k_raw + (hh - H) * dq, *w = is_q ? at.qn : at.kn;
+            float *dst = is_q ? qs + hh * dq : ks + nc * kds + (hh - H) * dq;
+            float s = 0.f;
+#pragma unroll 4
             for (int c = lane; c < dq; c += 32) {
-                if (hh < H) {
-                    v[c] *= inv * (at.qn ? at.qn[c] : 1.0f) * qt;
-                } else {
-                    const float kv = v[c] * inv * (at.kn ? at.kn[c] : 1.0f);
-                    v[c] = kv;
-                    at.kc_out[(int64_t)pos * kd + (hh - H) * dq + c] = kv;
-                }
+                const float v = src[c];
+                dst[c] = w ? v * w[c] : v;
+                s = fmaf(v, v, s);
+            }
+#pragma unroll
+            for (int o = 16; o; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
+            const float inv = 1.0f / sqrtf(s / (float)dq + at.eps) * (is_q ? qt : 1.0f);
+            for (int c = lane; c < dq; c += 32) { // (a lane's own entries)
+                const float v = dst[c] * inv;
+                dst[c] = v;
+                if (!is_q) at.kc_out[(int64_t)pos * kd + (hh - H) * dq + c] = v;
             }
         }
-        __syncthreads();
+    } else {
+        for (int t = tid; t < H * dq; t += 256) qs[t] = q[t];
     }
+    __syncthreads();
     if (bulk && !ps_tc_wait(&bar, 0)) { if (tid == 0) err[0] = 5; return; }
     for (int t = tid; t < PA_DS_KEYS * H; t += 256) {
         const int jj = t % PA_DS_KEYS, h = t / PA_DS_KEYS;

@@ -291,9 +291,14 @@ __device__ __forceinline__ float pa_warp_inv_rms(const float *v, int n, float ep
     return 1.0f / sqrtf(s / (float)n + eps);
 }
 
-// factor on the query at position p (coef 0: 1); the quotient in double, so that the floor is right at every multiple
+// factor on the query at position p (coef 0: 1); the quotient's floor is corrected by the sign of an fma, which is exact
 __device__ __forceinline__ float pa_q_temp(float coef, float every, int p) {
-    return coef != 0.f ? 1.0f + coef * logf((float)floor((double)(p + 1) / (double)every) + 1.0f) : 1.0f;
+    if (coef == 0.f) return 1.0f;
+    const float x = (float)(p + 1);
+    float n = floorf(x / every);
+    if (fmaf(n, every, -x) > 0.f) n -= 1.0f;
+    else if (fmaf(n + 1.0f, every, -x) <= 0.f) n += 1.0f;
+    return 1.0f + coef * logf(n + 1.0f);
 }
 
 // After the q|k|v projection of a batch, one CTA per token: unit-RMS q heads (in place) and k heads (qk_norm; times the weights qn / kn
