@@ -119,7 +119,7 @@ def test_rglru_layer_alone(tmp_path, width, blocks, conv):
 
 @pytest.mark.parametrize("lam", [-20.0, -9.0, 0.0, 4.0])
 def test_decays_from_nearly_one_to_nearly_zero(tmp_path, lam):
-    """1 - a^2 must not cancel when a is close to one: there the oracle in float64 is the judge"""
+    """1 - a^2 must not cancel when a is close to one: the float64 oracle shows it"""
     def edit(t):
         t["l0.mix.lam"] = np.full_like(t["l0.mix.lam"], lam)
         t["l0.mix.o"] = t["l0.mix.o"] * np.float32({-20.0: 512.0, -9.0: 16.0}.get(lam, 1.0))
