@@ -218,13 +218,16 @@ int ps_cuda_tp_import(ps_cuda_ctx *ctx, const void *handles, int n);
  *                qk_norm = 1: every head's q and k are divided by their root mean square (no weight, eps = norm_eps);
  *                qk_norm = PS_QKNORM_HEAD_W: the same, times the weights q_norm / k_norm [qk_dim] that all heads share;
  *                q_temp_coef != 0: q at position p is multiplied by 1 + q_temp_coef ln(floor((p + 1) / q_temp_every) + 1);
+ *                rope_dims > 0: q and k of every head are rotated (rotation below) after their norm;
  *                score = q.k * score_scale [* head_temp[h]] [+ rel[bucket(i - j)][h]] [- r1[h] ln(1 + r2[h] (i - j))]
- *                [mixed over heads by head_mix]; window > 0: query i sees the keys i - window < j <= i only;
+ *                [mixed over heads by head_mix]; score_softcap > 0: score <- cap tanh(score / cap) (not with head_mix); window > 0: query i sees the keys i - window < j <= i only;
  *                soft-max with an optional sink (one more term in the denominator that carries no value: exp(0) for
  *                sink = PS_SINK_ZERO, exp(sink[h]) for PS_SINK_LEARNED);
  *                bucket(n) = n below rel_buckets / 2, then logarithmic up to rel_max_dist (last bucket beyond);
  *                v_mix: PS_VMIX_SOURCE keeps the layer's value rows of the tokens in flight, PS_VMIX_BLEND replaces
  *                v by (1 - vmix) v + vmix v_source before it is cached (same value width in both layers).
+ *                v_rope = 1: the value of position j is rotated by j over all v_dim dims (halves, pair m by j rope_base^(-2 m / v_dim), no
+ *                scaling) before it is cached, and every head's output at position i is turned back by i before any gate.
  *   latent attention - queries through a normed latent (c_q = N(W_dq h; dq_norm), q = W_uq c_q, per head qk_dim plain
  *                + rot_dim rotated dims); W_dkv h gives kv_rank latent dims (normed with dkv_norm: the latent c) and
  *                rot_dim dims of ONE rotated key part shared by all heads; per head k = W_uk c, v = W_uv c;
@@ -252,6 +255,10 @@ int ps_cuda_tp_import(ps_cuda_ctx *ctx, const void *handles, int n);
  *                convolution of conv_taps taps with bias); u in rec_blocks equal parts, in part b r = sigmoid(R_b u_b + ..),
  *                i = sigmoid(I_b u_b + ..); log a = -rec_rate r softplus(lam), S_t = a S_(t-1) + sqrt(1 - a^2) i u (zero before the
  *                start), then the output projection of S y.  State: S (fp32) and the convolution's last inputs (a ring of conv_taps rows).
+ *   gla        - PS_MIXER_GLA: gated linear attention; q = W_q h qk_dim^(-1/2), k = W_k h, v = W_v h; a decay per key channel
+ *                alpha = sigmoid(W_a2 W_a1 h + b)^(1 / decay_tau) with W_a1 of decay_rank rows; per head S_t = diag(alpha_t) S_(t-1) + k_t v_t^T,
+ *                o_t = S_t^T q_t; every head's o RMS-normed with the weight mix_norm [v_dim] that the heads share, the concatenation times
+ *                silu(W_g h), then the output projection.  State: S per head, qk_dim x v_dim, fp32.
  *   recurrent state lives where a cache set keeps an attention layer's K rows (first buffer) and V^T rows (second buffer);
  *                a sequence at position 0 starts from zero state whatever the buffers hold; ps_cuda_kv_rollback to a
  *                position other than 0 is refused for models with such layers.
@@ -265,6 +272,12 @@ int ps_cuda_tp_import(ps_cuda_ctx *ctx, const void *handles, int n);
  *                router_bias = 1: a bias on the logits; router_act 3 = the top_k largest LOGITS choose, weights = soft-max over those alone;
  *                shared_ff > 0: one more expert of that many rows runs for every token and is added, times
  *                sigmoid(shared_sg . z) when shared_gate = 1.
+ *                router_act 2 without groups: route_correction = 1: the experts are chosen by score + correction[e], weighted by the score alone;
+ *                route_identity = n: the router has n more outputs behind the experts', for experts whose output is the input itself.
+ *                act_kind PS_ACT_RELU: y = max(Wg z, 0) * (Wu z).
+ *   layer scale - layer_scale = 1 (with post_norm): a sublayer's normed output is multiplied element by element by scale_mix / scale_ff [dim].
+ *   per-layer token input - token_slot = s + 1: after the feed-forward e = the part [s token_dim, (s + 1) token_dim) of the token's row in
+ *                the model's token_embed table, y = W_proj (gelu_tanh(W_gate x) * e), x <- x + N(y; token_norm), N an RMS norm with a plain weight.
  *   raw_input  - sequential blocks: the sublayers read the residual stream itself (no norm on the way in).
  *   values from keys - v_is_k = 1: there is no W_v; a position's value row is its projected key row as it leaves the projection
  *                (before any q / k norm); v_dim = qk_dim.
@@ -281,6 +294,11 @@ int ps_cuda_tp_import(ps_cuda_ctx *ctx, const void *handles, int n);
  *                u = W_x h + b_x, candidate c = u + 1/2 (u >= 0) or sigmoid(u) (u < 0), S_t = (1 - z) S_(t-1) + z c element by
  *                element over side_width channels (fp32, zero at position 0), output W_so (S_t silu(W_sg h)).  The layer's mixer
  *                output is mix_scale * attention + side_scale * side (one product over the concatenated inputs).
+ *                side_kind = PS_MIXER_RWKV: a time mixing of side_heads heads of side_width / side_heads channels.  With h' the input of the
+ *                token before (zeros for the first), r, k, v, gate and decay each read h + (h' - h) mu_s; gate = silu(W_g ..), decay
+ *                w = exp(-exp(W_w2 tanh(W_w1 ..) + w0)) per head and key channel (W_w1 of decay_rank rows); per head
+ *                o_t = (S_(t-1) + diag(u) k_t v_t^T)^T r_t, then S_t = diag(w_t) S_(t-1) + k_t v_t^T; every head's o divided by its root mean
+ *                square, the concatenation times side_norm and the gate, then W_so.  State: S (fp32) and the last token's input.
  *   interleaved rotation - rope_interleaved = 1: the rotation pairs dims (2i, 2i + 1) instead of (i, i + rope_dims / 2).
  *   ungated ff - mlp_ungated = 1: out = W_down act(W_up h), act the one-argument form of act_kind, for the dense feed-forward, the
  *                experts and the shared expert; PS_ACT_RELU2: max(z, 0)^2; PS_ACT_XIELU (dense only) with the
@@ -305,14 +323,14 @@ int ps_cuda_tp_import(ps_cuda_ctx *ctx, const void *handles, int n);
  * compute = PS_COMPUTE_BF16: matrix products take bfloat16 operands and accumulate in fp32; the residual stream, norms,
  * attention scores / weights, routers and the cache stay fp32.  PS_COMPUTE_F32: every product in true fp32 (FMA). */
 enum ps_cuda_compute { PS_COMPUTE_BF16 = 0, PS_COMPUTE_F32 = 1 };
-enum ps_cuda_mixer_kind { PS_MIXER_ATTENTION = 1, PS_MIXER_LATENT = 2, PS_MIXER_RETENTION = 3, PS_MIXER_MAMBA2 = 4, PS_MIXER_MINGRU = 5 /* side mixer only */, PS_MIXER_RGLRU = 6 };
+enum ps_cuda_mixer_kind { PS_MIXER_ATTENTION = 1, PS_MIXER_LATENT = 2, PS_MIXER_RETENTION = 3, PS_MIXER_MAMBA2 = 4, PS_MIXER_MINGRU = 5 /* side mixer only */, PS_MIXER_RGLRU = 6, PS_MIXER_GLA = 7, PS_MIXER_RWKV = 8 /* side mixer only */ };
 enum ps_cuda_mlp_kind { PS_MLP_NONE = 0, PS_MLP_ROUTED = 1, PS_MLP_DENSE = 2 };
 enum ps_cuda_block_kind { PS_BLOCK_PARALLEL = 0, PS_BLOCK_SEQUENTIAL = 1 };
 enum ps_cuda_sink_kind { PS_SINK_NONE = 0, PS_SINK_ZERO = 1, PS_SINK_LEARNED = 2 };
 enum ps_cuda_vmix_kind { PS_VMIX_NONE = 0, PS_VMIX_SOURCE = 1, PS_VMIX_BLEND = 2 };
 enum ps_cuda_qknorm_kind { PS_QKNORM_NONE = 0, PS_QKNORM_HEAD = 1, PS_QKNORM_WHOLE = 2, PS_QKNORM_HEAD_W = 3 };
 enum ps_cuda_gate_kind { PS_GATE_NONE = 0, PS_GATE_ELEMENT = 1, PS_GATE_HEAD = 2 };
-enum ps_cuda_act_kind { PS_ACT_SWISH = 0, PS_ACT_GELU_TANH = 1, PS_ACT_XIELU = 2, PS_ACT_RELU2 = 3 /* one-argument only */ };
+enum ps_cuda_act_kind { PS_ACT_SWISH = 0, PS_ACT_GELU_TANH = 1, PS_ACT_XIELU = 2, PS_ACT_RELU2 = 3 /* one-argument only */, PS_ACT_RELU = 4 };
 enum ps_cuda_norm_kind { PS_NORM_RMS = 0, PS_NORM_LAYER = 1 };
 enum ps_cuda_router_act { PS_ROUTER_SIGMOID = 1, PS_ROUTER_SOFTMAX = 2, PS_ROUTER_TOPK_SOFTMAX = 3 };
 
@@ -352,7 +370,7 @@ typedef struct {
     int32_t pool;                       /* > 0: mean key / value per block of this many positions wholly before the window */
     int32_t lin_bias;                   /* score -= lin[h] * distance */
     int32_t out_gate;                   /* enum ps_cuda_gate_kind: heads' outputs times sigmoid(W_g h) before the output projection */
-    int32_t side_kind, side_width;      /* a second mixer beside the attention (0 = none, PS_MIXER_MINGRU) and its channels */
+    int32_t side_kind, side_width;      /* a second mixer beside the attention (0 = none, PS_MIXER_MINGRU, PS_MIXER_RWKV) and its channels */
     float   mix_scale, side_scale;      /* mixer output = mix_scale * attention + side_scale * side (used when side_kind != 0) */
     int32_t rope_interleaved;           /* rotation pairs (2i, 2i + 1) */
     int32_t mlp_ungated;                /* feed-forward (experts, shared expert) without a gate: down(act(up h)) */
@@ -360,9 +378,16 @@ typedef struct {
     int32_t rec_width, rec_blocks;      /* rg-lru: channels, equal parts of the gates' matrices */
     float   rec_rate;                   /* rg-lru: factor of the decay's logarithm */
     int32_t router_bias;                /* the router's logits carry a bias */
+    float   score_softcap;              /* > 0: score <- cap tanh(score / cap) */
+    int32_t v_rope;                     /* values rotated by their position, outputs turned back by the query's */
+    int32_t decay_rank; float decay_tau; /* gla, rwkv: rows of the decay's first matrix; gla: root of the decay */
+    int32_t side_heads;                 /* rwkv: heads of side_width / side_heads channels */
+    int32_t route_identity, route_correction; /* router outputs that stand for the input itself; corrections on the choice */
+    int32_t layer_scale;                /* sublayers' normed outputs times a vector */
     int32_t share_weights;              /* j + 1: this run uses the weights of run j */
     int32_t pass_embed, pass_step;      /* before the run: add the embedding output; add row pass_step - 1 of pass_steps */
     int32_t pass_in;                    /* before the run: x <- W_in [x; embedding output] */
+    int32_t token_slot;                 /* s + 1: the run takes part s of the token's row in token_embed (0 = no per-layer token input) */
 } ps_cuda_layer_desc;
 
 typedef struct {
@@ -377,6 +402,7 @@ typedef struct {
     int32_t norm_kind;                  /* enum ps_cuda_norm_kind: the block norms and the final norm */
     int32_t n_pass_steps;               /* rows of the pass_steps table */
     float   residual_scale;             /* factor on what a block adds to the residual stream (0: 1) */
+    int32_t token_dim, token_slots;     /* per-layer token input: size of a part, parts in a row of token_embed */
 } ps_cuda_arch_desc;
 
 /* matrices [out][in] in bfloat16; vectors and the small tables in bfloat16 or fp32 */
@@ -396,6 +422,12 @@ typedef struct {
     ps_cuda_tensor router_bias;         /* [n_experts] */
     ps_cuda_tensor rec_y, rec_y_bias, rec_x, rec_x_bias;   /* rg-lru: [W][dim], [W] twice (conv_w [W][taps] and conv_b [W] above) */
     ps_cuda_tensor rec_r, rec_r_bias, rec_i, rec_i_bias, rec_lam; /* [blocks][W / blocks][W / blocks], [W] twice; [W] */
+    ps_cuda_tensor a1, a2, a2_bias;     /* gla: decay [rank][dim], [H * qk_dim][rank], [H * qk_dim] */
+    ps_cuda_tensor side_mu_r, side_mu_k, side_mu_v, side_mu_g, side_mu_w; /* rwkv: [dim] each */
+    ps_cuda_tensor side_r, side_k, side_v, side_w1, side_w2, side_w0, side_u, side_norm; /* [W][dim] three times; [rank][dim], [W][rank], [W]; [W]; [W] (side_g, side_o above) */
+    ps_cuda_tensor correction;          /* [n_experts + route_identity] */
+    ps_cuda_tensor scale_mix, scale_ff; /* layer scale [dim] */
+    ps_cuda_tensor token_gate, token_proj, token_norm; /* per-layer token input: [token_dim][dim], [dim][token_dim], [dim] */
 } ps_cuda_arch_layer_weights;
 
 typedef struct {
@@ -403,6 +435,7 @@ typedef struct {
     const ps_cuda_arch_layer_weights *layers; /* one entry per run; the entries of runs that share another run's weights are not read */
     ps_cuda_tensor pass_steps;          /* [n_pass_steps][dim] */
     ps_cuda_tensor pass_in;             /* [dim][2 dim] */
+    ps_cuda_tensor token_embed;         /* [vocab][token_slots * token_dim] */
 } ps_cuda_arch_weights;
 
 int ps_cuda_create_arch(ps_cuda_ctx **out, int device, const ps_cuda_arch_desc *desc);

@@ -41,7 +41,8 @@ class LayerListModel(capi.CudaModel):
         self._layer_descs = (LayerDesc * len(layers))(*layers)
         self.desc = ArchDesc(top["dim"], top["vocab_size"], len(layers), int(n_ctx), int(max_batch), top["norm_eps"], top["embed_scale"],
                              top["norm_unit_offset"], compute, self._layer_descs, int(top.get("norm_groups", 1)), int(top.get("norm_scalar", 0)),
-                             int(top.get("norm_kind", 0)), int(top.get("n_pass_steps", 0)), float(top.get("residual_scale", 1.0)))
+                             int(top.get("norm_kind", 0)), int(top.get("n_pass_steps", 0)), float(top.get("residual_scale", 1.0)),
+                             int(top.get("token_dim", 0)), int(top.get("token_slots", 0)))
         self.vocab = self.desc.vocab_size
         self.be = capi.CudaBackend(self.desc, device)
 
@@ -70,7 +71,8 @@ class LayerListModel(capi.CudaModel):
                     self._keep.append(arr)
                     setattr(lw, f, arr)
             self._lw[i] = lw
-        self._w = ArchWeights(T(names["embed"]), T(names["final_norm"]), T(names["head"]), self._lw, T(names.get("pass_steps")), T(names.get("pass_in")))
+        self._w = ArchWeights(T(names["embed"]), T(names["final_norm"]), T(names["head"]), self._lw, T(names.get("pass_steps")), T(names.get("pass_in")),
+                              T(names.get("token_embed")))
         self.be._ck(self.be.L.ps_cuda_bind_arch(self.be.h, C.byref(self._w)))
 
     def layer_tap(self, layer: int, bs: int):
@@ -516,11 +518,98 @@ def _momedra_tensor_names(cfg: dict) -> dict:
     return out
 
 
+# ------------------------------------------------------------------------------------------------------------ Tegolix
+# Decoder-only; every layer is a sequential block whose sublayers are normed on the way in AND out (RMS norms, weights around zero) and scaled
+# element by element, x <- x + s1 N1b(mixer(N1(x))), x <- x + s2 N2b(ff(N2(x))), followed by a per-layer input from the token's own row,
+#   x <- x + N(W_proj (gelu(W_gate x) * e_token)).  Two mixers, chosen by "type":
+#   "gla"       gated linear attention with a decay per key channel, sigmoid(low-rank + bias)^(1 / tau).
+#   "parallel"  two mixers on the same input, summed with left_scale / right_scale: "left" a windowed soft-capped attention, q / k normed per
+#               head and rotated (rotate-half pairs, YaRN), values rotated by their position and turned back at the query's, one gate number
+#               a head; "right" a time mixing in the manner of RWKV.
+# Feed-forward: dense with relu, or soft-max-routed silu experts (choice by corrected scores, weights as they are, some router outputs stand
+# for the input itself) beside a shared expert behind a sigmoid gate.
+def _tegolix_describe(cfg: dict, tensors) -> Tuple[List[LayerDesc], dict]:
+    layers = []
+    for i, l in enumerate(cfg["layers"]):
+        m = l["mixer"]
+        d = LayerDesc()
+        d.block_kind, d.post_norm, d.layer_scale = capi.BLOCK_SEQUENTIAL, 1, 1
+        if l["type"] == "gla":
+            d.mixer_kind = capi.MIXER_GLA
+            d.n_heads, d.n_kv_heads, d.qk_dim, d.v_dim = m["heads"], m["heads"], m["dim"], m["vdim"]
+            d.decay_tau, d.decay_rank = float(m["tau"]), int(tensors[f"l{i}.mix.a1"].shape[0])          # the rows the stored matrix has
+        elif l["type"] == "parallel":
+            a, b, rot = m["left"], m["right"], m["left"]["rot"]
+            d.mixer_kind = capi.MIXER_ATTENTION
+            d.n_heads, d.n_kv_heads, d.qk_dim, d.v_dim = a["heads"], a["kv_heads"], a["dim"], a["vdim"]
+            d.score_scale, d.score_softcap = a["scale"], float(a.get("softcap") or 0.0)
+            d.window = int((a.get("mask") or {}).get("size", 0))
+            d.qk_norm, d.out_gate, d.v_rope = capi.QKNORM_HEAD_W, capi.GATE_HEAD, 1
+            d.rope_dims, d.rope_base = int(rot["dims"]), float(rot["base"])
+            sc = rot.get("scaling")
+            if sc:
+                d.rope_factor, d.rope_original, d.rope_fast, d.rope_slow = float(sc["factor"]), int(sc["original"]), float(sc["fast"]), float(sc["slow"])
+            d.side_kind, d.side_heads, d.side_width = capi.MIXER_RWKV, b["heads"], b["heads"] * b["dim"]
+            d.decay_rank = int(tensors[f"l{i}.mix.right.w1"].shape[0])
+            d.mix_scale, d.side_scale = float(m["left_scale"]), float(m["right_scale"])
+        else:
+            raise capi.PsCudaError(f"Tegolix layer {i}: unknown mixer type {l['type']!r}")
+        mlp = l.get("mlp")
+        d.act_limit, d.act_alpha, d.up_shift = float("inf"), 1.0, 0.0   # silu(gate) * up where the activation is the swish kind
+        if mlp is None:
+            d.mlp_kind = capi.MLP_NONE
+        elif mlp.get("kind") == "dense":
+            d.mlp_kind, d.expert_ff, d.act_kind = capi.MLP_DENSE, mlp["ff"], capi.ACT_RELU
+        elif mlp.get("kind") == "moe":
+            r = mlp["router"]
+            d.mlp_kind, d.act_kind = capi.MLP_ROUTED, capi.ACT_SWISH
+            d.n_experts, d.top_k, d.expert_ff, d.route_identity = r["experts"], r["top"], mlp["expert"]["ff"], int(r.get("identity", 0))
+            d.router_act, d.route_correction = capi.ROUTER_SOFTMAX, 1
+            if mlp.get("shared"):
+                d.shared_ff, d.shared_gate = mlp["shared"]["ff"], 1
+        else:
+            raise capi.PsCudaError(f"Tegolix layer {i}: unknown feed-forward kind {mlp.get('kind')!r}")
+        d.token_slot = i + 1
+        layers.append(d)
+    top = {"dim": cfg["width"], "vocab_size": cfg["vocab"], "norm_eps": cfg["norm"]["eps"], "embed_scale": 1.0, "norm_unit_offset": 1,
+           "token_dim": int(cfg["token_side"]["dim"]), "token_slots": len(cfg["layers"])}
+    return layers, top
+
+
+def _tegolix_tensor_names(cfg: dict) -> dict:
+    out = {"embed": "embed", "final_norm": "final.norm", "head": "head", "token_embed": "side.embed", "layers": []}
+    for i, l in enumerate(cfg["layers"]):
+        p, a = f"l{i}.", f"l{i}.mix."
+        n = {"norm": p + "norm1", "norm_mix_out": p + "norm1b", "scale_mix": p + "ls1", "token_gate": p + "side.gate", "token_proj": p + "side.proj", "token_norm": p + "side.norm"}
+        if l["type"] == "gla":
+            n.update({"q": a + "q", "k": a + "k", "v": a + "v", "g": a + "g", "o": a + "o", "mix_norm": a + "norm", "a1": a + "a1", "a2": a + "a2", "a2_bias": a + "a2.b"})
+        else:
+            b = a + "right."
+            n.update({k: a + "left." + t for k, t in (("q", "q"), ("k", "k"), ("v", "v"), ("q_norm", "q.norm"), ("k_norm", "k.norm"), ("g", "g"), ("o", "o"))})
+            n.update({"side_mu_" + s: b + "mu." + s for s in "rkvgw"})
+            n.update({"side_" + s: b + s for s in ("r", "k", "v", "g", "w1", "w2", "w0", "u", "norm", "o")})
+        mlp = l.get("mlp")
+        if mlp is not None:
+            n.update({"norm_ff": p + "norm2", "norm_ff_out": p + "norm2b", "scale_ff": p + "ls2"})
+            if mlp.get("kind") == "moe":
+                n.update({"router": p + "mlp.router", "correction": p + "mlp.correction"})
+                for f in ("gate", "up", "down"):
+                    n[f] = [f"{p}mlp.e{e}.{f}" for e in range(mlp["router"]["experts"])]
+                if mlp.get("shared"):
+                    n.update({"shared_gate": p + "mlp.shared.gate", "shared_up": p + "mlp.shared.up", "shared_down": p + "mlp.shared.down", "shared_sg": p + "mlp.shared.sg"})
+            else:
+                for f in ("gate", "up", "down"):
+                    n[f] = [f"{p}mlp.{f}"]
+        out["layers"].append(n)
+    return out
+
+
 ARCHITECTURES: Dict[str, Tuple[Callable, Callable]] = {
     "Dozotar": (_dozotar_describe, _dozotar_tensor_names),
     "Momedra": (_momedra_describe, _momedra_tensor_names),
     "Pidenex": (_pidenex_describe, _pidenex_tensor_names),
     "Nufusun": (_nufusun_describe, _nufusun_tensor_names),
+    "Tegolix": (_tegolix_describe, _tegolix_tensor_names),
     "Vanapel": (_vanapel_describe, _vanapel_tensor_names),
 }
 

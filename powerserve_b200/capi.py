@@ -59,22 +59,25 @@ class LayerDesc(C.Structure):
                 ("v_is_k", C.c_int32), ("pool", C.c_int32), ("lin_bias", C.c_int32), ("out_gate", C.c_int32), ("side_kind", C.c_int32),
                 ("side_width", C.c_int32), ("mix_scale", C.c_float), ("side_scale", C.c_float), ("rope_interleaved", C.c_int32),
                 ("mlp_ungated", C.c_int32), ("q_temp_coef", C.c_float), ("q_temp_every", C.c_float), ("rec_width", C.c_int32), ("rec_blocks", C.c_int32),
-                ("rec_rate", C.c_float), ("router_bias", C.c_int32), ("share_weights", C.c_int32), ("pass_embed", C.c_int32), ("pass_step", C.c_int32),
-                ("pass_in", C.c_int32)]
+                ("rec_rate", C.c_float), ("router_bias", C.c_int32), ("score_softcap", C.c_float), ("v_rope", C.c_int32), ("decay_rank", C.c_int32),
+                ("decay_tau", C.c_float), ("side_heads", C.c_int32), ("route_identity", C.c_int32), ("route_correction", C.c_int32), ("layer_scale", C.c_int32),
+                ("share_weights", C.c_int32), ("pass_embed", C.c_int32), ("pass_step", C.c_int32), ("pass_in", C.c_int32), ("token_slot", C.c_int32)]
 
 
 class ArchDesc(C.Structure):
     _fields_ = [("dim", C.c_int32), ("vocab_size", C.c_int32), ("n_layers", C.c_int32), ("n_ctx", C.c_int32), ("max_batch", C.c_int32),
                 ("norm_eps", C.c_float), ("embed_scale", C.c_float), ("norm_unit_offset", C.c_int32), ("compute", C.c_int32),
                 ("layers", C.POINTER(LayerDesc)), ("norm_groups", C.c_int32), ("norm_scalar", C.c_int32), ("norm_kind", C.c_int32),
-                ("n_pass_steps", C.c_int32), ("residual_scale", C.c_float)]
+                ("n_pass_steps", C.c_int32), ("residual_scale", C.c_float), ("token_dim", C.c_int32), ("token_slots", C.c_int32)]
 
 
 # the layer tensors after the expert lists, in the order of ps_cuda_arch_layer_weights
 ARCH_LAYER_VECTORS_2 = ("norm_mix_out", "norm_ff", "norm_ff_out", "r1", "r2", "sink", "vmix", "dq", "dq_norm", "uq", "dkv", "dkv_norm", "uk", "uv",
                         "q_norm", "k_norm", "q_conv", "k_conv", "v_conv", "g", "decay", "w_in", "conv_w", "conv_b", "dt_bias", "a_log", "d_skip", "mix_norm",
                         "shared_gate", "shared_up", "shared_down", "shared_sg", "lin", "act", "side_z", "side_z_bias", "side_x", "side_x_bias", "side_g",
-                        "side_o", "router_bias", "rec_y", "rec_y_bias", "rec_x", "rec_x_bias", "rec_r", "rec_r_bias", "rec_i", "rec_i_bias", "rec_lam")
+                        "side_o", "router_bias", "rec_y", "rec_y_bias", "rec_x", "rec_x_bias", "rec_r", "rec_r_bias", "rec_i", "rec_i_bias", "rec_lam",
+                        "a1", "a2", "a2_bias", "side_mu_r", "side_mu_k", "side_mu_v", "side_mu_g", "side_mu_w", "side_r", "side_k", "side_v", "side_w1", "side_w2",
+                        "side_w0", "side_u", "side_norm", "correction", "scale_mix", "scale_ff", "token_gate", "token_proj", "token_norm")
 
 
 class ArchLayerWeights(C.Structure):
@@ -84,7 +87,8 @@ class ArchLayerWeights(C.Structure):
 
 
 class ArchWeights(C.Structure):
-    _fields_ = [("embed", Tensor), ("final_norm", Tensor), ("head", Tensor), ("layers", C.POINTER(ArchLayerWeights)), ("pass_steps", Tensor), ("pass_in", Tensor)]
+    _fields_ = [("embed", Tensor), ("final_norm", Tensor), ("head", Tensor), ("layers", C.POINTER(ArchLayerWeights)), ("pass_steps", Tensor), ("pass_in", Tensor),
+                ("token_embed", Tensor)]
 
 
 COMPUTE_BF16, COMPUTE_F32 = 0, 1
@@ -96,8 +100,8 @@ VMIX_NONE, VMIX_SOURCE, VMIX_BLEND = 0, 1, 2
 MIXER_RETENTION, MIXER_MAMBA2 = 3, 4
 QKNORM_NONE, QKNORM_HEAD, QKNORM_WHOLE, QKNORM_HEAD_W = 0, 1, 2, 3
 GATE_NONE, GATE_ELEMENT, GATE_HEAD = 0, 1, 2
-ACT_SWISH, ACT_GELU_TANH, ACT_XIELU, ACT_RELU2 = 0, 1, 2, 3
-MIXER_MINGRU, MIXER_RGLRU = 5, 6
+ACT_SWISH, ACT_GELU_TANH, ACT_XIELU, ACT_RELU2, ACT_RELU = 0, 1, 2, 3, 4
+MIXER_MINGRU, MIXER_RGLRU, MIXER_GLA, MIXER_RWKV = 5, 6, 7, 8
 NORM_RMS, NORM_LAYER = 0, 1
 ROUTER_SIGMOID, ROUTER_SOFTMAX, ROUTER_TOPK_SOFTMAX = 1, 2, 3
 

@@ -7,6 +7,7 @@
 // bfloat16 already) and accumulates in fp32; PS_COMPUTE_F32 feeds the fp32 activations unrounded and uses FMA chains only.
 #include "ps_arch.h"
 
+#include <cooperative_groups.h>
 #include <cuda_bf16.h>
 
 #include <algorithm>
@@ -18,6 +19,7 @@
 #include <vector>
 
 typedef __nv_bfloat16 bf16;
+namespace cg = cooperative_groups;
 
 #include "ps_arch_kernels.cuh"
 #include "ps_arch_decode.cuh"
@@ -69,6 +71,18 @@ struct PsArchLayer {
     float *router_b = nullptr;
     bf16 *wri = nullptr;                  // rg-lru: [block][r rows | i rows][W / blocks]
     float *rec_rb = nullptr, *rec_ib = nullptr, *rec_sp = nullptr; // gate biases; rec_rate * softplus(lam)
+    // recurrences with a decay per key channel (gla as the mixer, time mixing beside an attention): first-projection rows
+    // q | k | v | gate | a1, or .. | r | k | v | gate | w1 behind the attention's (z_off); the decay's second matrix and bias, the bonus
+    bf16 *wa2 = nullptr;
+    float *a2b = nullptr, *bonus = nullptr, *mu = nullptr; // mu: [5][dim]
+    PtSegs seg{};                         // time mixing: which operand set the first projection's rows read
+    int64_t ring_off = 0;                 // the last token's input in the K buffer (two rows; floats from its start)
+    double *vrope_freq = nullptr;         // rotation of the values
+    float *corr = nullptr;                // corrections on the router's choice
+    // per-layer token input
+    bf16 *wtg = nullptr, *wtp = nullptr;
+    uint8_t *t_tg = nullptr, *t_tp = nullptr;
+    float *tok_norm = nullptr;
 };
 
 static inline PaAct pa_act_of(const ps_cuda_layer_desc &l) { return PaAct{l.act_limit, l.act_alpha, l.up_shift, l.act_kind}; }
@@ -76,9 +90,9 @@ static inline PaAct pa_act_of(const PsArchLayer &w) {
     return w.d.act_kind == PS_ACT_XIELU ? PaAct{0.f, w.act_a, w.act_b, PS_ACT_XIELU} : pa_act_of(w.d);
 }
 static inline PaRoute pa_route_of(const ps_cuda_layer_desc &l) {
-    return PaRoute{l.n_experts, l.top_k, l.router_act, l.route_groups, l.route_keep, l.route_renorm, l.route_renorm_eps, l.shared_ff > 0 && l.shared_gate};
+    return PaRoute{l.n_experts + l.route_identity, l.top_k, l.router_act, l.route_groups, l.route_keep, l.route_renorm, l.route_renorm_eps, nullptr, l.route_identity, l.shared_ff > 0 && l.shared_gate};
 }
-static inline bool pa_recurrent(const ps_cuda_layer_desc &l) { return l.mixer_kind == PS_MIXER_RETENTION || l.mixer_kind == PS_MIXER_MAMBA2; }
+static inline bool pa_recurrent(const ps_cuda_layer_desc &l) { return l.mixer_kind == PS_MIXER_RETENTION || l.mixer_kind == PS_MIXER_MAMBA2 || l.mixer_kind == PS_MIXER_GLA; }
 
 struct PsArch {
     ps_cuda_arch_desc d{};
@@ -130,6 +144,11 @@ struct PsArch {
     float *xcat = nullptr;                 // [max_batch][2 dim]: stream | embedding output
     float *gts = nullptr;                  // rg-lru: gate logits of a batch
     float *hn = nullptr;                   // single-token step: the normed input, for the experts
+    float *dcy = nullptr, *mixb = nullptr; // decays of a batch [max_batch][H * dk]; the five mixtures a time mixing reads [5][max_batch][dim]
+    int max_dcy = 0, max_seg_rt = 0;
+    bf16 *tok_embed = nullptr;             // per-layer token input: [vocab][token_slots * token_dim]
+    float *tg = nullptr, *ty = nullptr;    // its gated part [max_batch][token_dim] and its output [max_batch][dim]
+    bool has_shift = false;
     int max_rec = 0;
 };
 
@@ -223,7 +242,9 @@ void build_bucket_table(int rows, float dmax, int n, std::vector<uint16_t> &t) {
 }
 
 // shared memory of the single-token kernels
-size_t pa_dec_scores_smem(int H, int G, int dq) { return 4 * ((size_t)PA_DS_KEYS * (((G * dq + 3) & ~3) + 4) + (size_t)H * dq + (size_t)(PA_DS_KEYS + 1) * H + (size_t)H * H); }
+size_t pa_dec_scores_smem(int H, int G, int dq, int rope_dims = 0) {
+    return 4 * ((size_t)PA_DS_KEYS * (((G * dq + 3) & ~3) + 4) + (size_t)H * dq + (size_t)(PA_DS_KEYS + 1) * H + (size_t)std::max(H * H, rope_dims + 2));
+}
 // the P.V kernel splits more than 4 query heads per kv head over blockIdx.z, 4 (or fewer) to a CTA
 int pa_dec_pv_split(int H, int G) { return (H / G + 3) / 4; }
 int pa_dec_pv_rep(int H, int G) { const int z = pa_dec_pv_split(H, G); return (H / G + z - 1) / z; }
@@ -233,8 +254,47 @@ size_t pa_dec_pv_smem(int H, int G) {
     return 4 * ((size_t)(PA_DP_DIMS + rep) * pa_dec_pv_chunk(H, G) + (size_t)(2 + 8) * rep);
 }
 
+typedef void (*PaScanKernel)(PaScan);
+template <int IL> PaScanKernel pa_scan_pick(int nc, int mode) {
+    if (nc == 2) return mode == 0 ? pa_k_scan<IL, 2, 0> : mode == 1 ? pa_k_scan<IL, 2, 1> : pa_k_scan<IL, 2, 2>;
+    return mode == 0 ? pa_k_scan<IL, 1, 0> : mode == 1 ? pa_k_scan<IL, 1, 1> : pa_k_scan<IL, 1, 2>;
+}
+PaScanKernel pa_scan_kernel(int il, int nc, int mode) {
+    switch (il) {
+    case 1: return pa_scan_pick<1>(nc, mode);
+    case 2: return pa_scan_pick<2>(nc, mode);
+    case 4: return pa_scan_pick<4>(nc, mode);
+    case 8: return pa_scan_pick<8>(nc, mode);
+    default: return pa_scan_pick<16>(nc, mode);
+    }
+}
+
+// CTAs (a cluster) that share one head of the single-token recurrence: up to eight, while each keeps eight value columns
+int pa_rec_cluster(int dv) {
+    int n = 1;
+    while (n < 8 && dv / (2 * n) >= 8) n *= 2;
+    return n;
+}
+
 // a launch that may overlap the end of the kernel before it in the stream (the kernel calls griddepcontrol.wait before it reads
 // anything that kernel wrote)
+template <typename... KArgs, typename... Args>
+cudaError_t pa_launch_cluster(bool pdl, int n_cl, void (*kern)(KArgs...), dim3 grid, dim3 block, size_t smem, cudaStream_t st, Args... args) {
+    cudaLaunchConfig_t cfg{};
+    cfg.gridDim = grid;
+    cfg.blockDim = block;
+    cfg.dynamicSmemBytes = smem;
+    cfg.stream = st;
+    cudaLaunchAttribute at[2];
+    at[0].id = cudaLaunchAttributeClusterDimension;
+    at[0].val.clusterDim.x = (unsigned)n_cl;
+    at[0].val.clusterDim.y = at[0].val.clusterDim.z = 1;
+    at[1].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    at[1].val.programmaticStreamSerializationAllowed = 1;
+    cfg.attrs = at;
+    cfg.numAttrs = pdl ? 2 : 1;
+    return cudaLaunchKernelEx(&cfg, kern, KArgs(args)...);
+}
 template <typename... KArgs, typename... Args>
 cudaError_t pa_launch_dep(bool pdl, void (*kern)(KArgs...), dim3 grid, dim3 block, size_t smem, cudaStream_t st, Args... args) {
     cudaLaunchConfig_t cfg{};
@@ -302,6 +362,8 @@ static int par_layer_sizes(PsArch *a, int i, std::string &err) {
     const ps_cuda_layer_desc &l = w.d;
     const bool latent = l.mixer_kind == PS_MIXER_LATENT, rec = l.mixer_kind == PS_MIXER_RGLRU, routed = l.mlp_kind == PS_MLP_ROUTED;
 #define PA_BAD(...) return afail(err, PS_CUDA_ERR_UNSUPPORTED, __VA_ARGS__)
+    if (l.score_softcap != 0.f || l.v_rope || l.layer_scale || l.token_slot || l.route_identity || l.route_correction || l.act_kind == PS_ACT_RELU || (l.rope_dims > 0 && !latent))
+        PA_BAD("layer %d: soft-capped scores, rotated values or attention heads, layer scales, token inputs, identity experts, corrected choices and relu go with sequential blocks", i);
     if (l.raw_input || l.post_norm || l.v_mix || l.v_is_k || l.pool || l.side_kind || l.head_mix || l.head_temp || d.norm_groups > 1 || d.norm_unit_offset || d.norm_scalar || (l.conv_taps > 0 && !rec))
         PA_BAD("layer %d: raw inputs, output norms, value blending, values from keys, pooled windows, side mixers, head mixing / temperatures and group, offset or scalar norms are not combined with a general parallel block", i);
     if (l.mixer_kind != PS_MIXER_ATTENTION && !latent && !rec) PA_BAD("layer %d: mixer kind %d in a general parallel block", i, l.mixer_kind);
@@ -393,37 +455,52 @@ int ps_arch_create(PsArch **out, const ps_cuda_arch_desc *desc, std::string &err
             return bail(afail(err, PS_CUDA_ERR_INVALID, "layer %d: shares the weights of run %d, pass step %d of %d", i, l.share_weights - 1, l.pass_step, d.n_pass_steps));
         if (l.share_weights > 0 && memcmp(&d.layers[l.share_weights - 1], &l, offsetof(ps_cuda_layer_desc, share_weights)) != 0)
             return bail(afail(err, PS_CUDA_ERR_INVALID, "layer %d: a run that shares weights must have the sizes of run %d", i, l.share_weights - 1));
-        if (l.mixer_kind < PS_MIXER_ATTENTION || l.mixer_kind > PS_MIXER_RGLRU || l.mixer_kind == PS_MIXER_MINGRU) return bail(afail(err, PS_CUDA_ERR_UNSUPPORTED, "layer %d: unknown mixer kind %d", i, l.mixer_kind));
+        if (l.mixer_kind < PS_MIXER_ATTENTION || l.mixer_kind > PS_MIXER_GLA || l.mixer_kind == PS_MIXER_MINGRU) return bail(afail(err, PS_CUDA_ERR_UNSUPPORTED, "layer %d: unknown mixer kind %d", i, l.mixer_kind));
         if (w.gpar) {
             const int rc = par_layer_sizes(a, i, err);
             if (rc) return bail(rc);
             continue;
         }
         const bool latent = l.mixer_kind == PS_MIXER_LATENT, recur = pa_recurrent(l);
-        if (l.mixer_kind == PS_MIXER_RGLRU || l.act_kind == PS_ACT_RELU2 || l.qk_norm == PS_QKNORM_HEAD_W || l.out_gate == PS_GATE_HEAD || l.q_temp_coef != 0.f || l.proj_bias == 2 || l.router_bias ||
-            l.router_act == PS_ROUTER_TOPK_SOFTMAX)
-            return bail(afail(err, PS_CUDA_ERR_UNSUPPORTED, "layer %d: rg-lru, squared relu, weighted head norms, gates per head, query temperatures, q / k / v-only and router biases need a general parallel block", i));
-        const bool newer = l.v_is_k || l.pool > 0 || l.lin_bias || l.out_gate || l.side_kind; // mechanisms of the general sequential layer only
+        if (l.mixer_kind == PS_MIXER_RGLRU || l.act_kind == PS_ACT_RELU2 || l.q_temp_coef != 0.f || l.proj_bias == 2 || l.router_bias || l.router_act == PS_ROUTER_TOPK_SOFTMAX)
+            return bail(afail(err, PS_CUDA_ERR_UNSUPPORTED, "layer %d: rg-lru, squared relu, query temperatures, q / k / v-only and router biases need a general parallel block", i));
+        const bool turned = l.mixer_kind == PS_MIXER_ATTENTION && (l.rope_dims > 0 || l.v_rope); // rotated heads
+        // mechanisms of the general sequential layer's attention only
+        const bool newer = l.v_is_k || l.pool > 0 || l.lin_bias || l.out_gate || l.side_kind || l.qk_norm == PS_QKNORM_HEAD_W || turned || l.score_softcap != 0.f;
         w.gen2 = l.block_kind == PS_BLOCK_SEQUENTIAL && !latent &&
                  (l.raw_input || recur || l.conv_taps > 0 || l.qk_norm == PS_QKNORM_WHOLE || l.chunk > 0 || l.mlp_kind == PS_MLP_ROUTED || l.rel_buckets > 0 ||
-                  l.act_kind == PS_ACT_GELU_TANH || l.shared_ff > 0 || newer);
+                  l.act_kind == PS_ACT_GELU_TANH || l.act_kind == PS_ACT_RELU || l.shared_ff > 0 || newer);
         if (newer && (!w.gen2 || l.mixer_kind != PS_MIXER_ATTENTION))
-            return bail(afail(err, PS_CUDA_ERR_UNSUPPORTED, "layer %d: values from keys, pooled windows, linear distance biases, output gates and side mixers need an attention in a sequential block", i));
+            return bail(afail(err, PS_CUDA_ERR_UNSUPPORTED, "layer %d: values from keys, pooled windows, linear distance biases, soft-capped scores, weighted head norms, rotated heads, output gates and side mixers need an attention in a sequential block", i));
+        if (turned && (l.rope_dims < 0 || l.rope_dims > l.qk_dim || (l.rope_dims & 1) || !(l.rope_base > 0.f) || l.rope_interleaved || (l.v_rope && (l.v_dim & 1)) || l.qk_norm == PS_QKNORM_WHOLE || l.v_is_k ||
+                       l.pool > 0 || l.conv_taps > 0))
+            return bail(afail(err, PS_CUDA_ERR_UNSUPPORTED, "layer %d: rotated heads of %d (%d rotated) / %d entries go with no whole-projection norm, value sharing, pooling or convolution", i, l.qk_dim, l.rope_dims, l.v_dim));
+        if (l.score_softcap < 0.f || (l.qk_norm == PS_QKNORM_HEAD_W && (l.v_is_k || l.pool > 0 || l.conv_taps > 0)))
+            return bail(afail(err, PS_CUDA_ERR_UNSUPPORTED, "layer %d: score cap %g; weighted head norms go with no value sharing, pooling or convolution", i, (double)l.score_softcap));
+        if (l.mixer_kind == PS_MIXER_GLA && (l.block_kind != PS_BLOCK_SEQUENTIAL || l.qk_dim > 256 || l.decay_rank <= 0 || !(l.decay_tau > 0.f) || l.rope_dims || l.window || l.conv_taps || l.qk_norm))
+            return bail(afail(err, PS_CUDA_ERR_UNSUPPORTED, "layer %d: gated linear attention with heads of %d (at most 256), decay rank %d, root %g", i, l.qk_dim, l.decay_rank, (double)l.decay_tau));
+        if ((l.route_identity || l.route_correction) && (!w.gen2 || l.mlp_kind != PS_MLP_ROUTED || l.route_identity < 0 || l.router_act != PS_ROUTER_SOFTMAX || l.route_groups > 1 || l.route_on_input))
+            return bail(afail(err, PS_CUDA_ERR_UNSUPPORTED, "layer %d: identity experts (%d) and corrected choices need a soft-max router without groups in a sequential block", i, l.route_identity));
+        if ((l.layer_scale && (!l.post_norm || l.block_kind != PS_BLOCK_SEQUENTIAL)) || l.token_slot < 0 || l.token_slot > d.token_slots ||
+            (l.token_slot > 0 && (d.token_dim <= 0 || l.block_kind != PS_BLOCK_SEQUENTIAL || d.norm_kind != PS_NORM_RMS || d.norm_groups > 1 || l.pass_in)))
+            return bail(afail(err, PS_CUDA_ERR_UNSUPPORTED, "layer %d: layer scales need output norms in a sequential block; a token input (part %d of %d) a sequential block with plain RMS norms", i, l.token_slot, d.token_slots));
+
         if (l.v_is_k && l.v_dim != l.qk_dim) return bail(afail(err, PS_CUDA_ERR_UNSUPPORTED, "layer %d: values from keys of size %d cannot have size %d", i, l.qk_dim, l.v_dim));
         if (l.pool < 0 || (l.pool > 0 && (l.window <= 0 || l.chunk > 0 || l.conv_taps > 0 || l.rel_buckets > 0 || l.log_bias || l.lin_bias || l.head_mix)))
             return bail(afail(err, PS_CUDA_ERR_UNSUPPORTED, "layer %d: pooled blocks of %d need a window and go with no distance term, chunk, convolution or head mixing", i, l.pool));
-        if ((l.side_kind != 0 && (l.side_kind != PS_MIXER_MINGRU || l.side_width <= 0 || l.conv_taps > 0)) || (l.rope_interleaved && !latent))
+        if ((l.side_kind != 0 && ((l.side_kind != PS_MIXER_MINGRU && l.side_kind != PS_MIXER_RWKV) || l.side_width <= 0 || l.conv_taps > 0)) ||
+            (l.side_kind == PS_MIXER_RWKV && (l.side_heads <= 0 || l.side_width % std::max(l.side_heads, 1) || l.side_width / std::max(l.side_heads, 1) > 256 || l.decay_rank <= 0 || l.raw_input || (size_t)d.dim * 24 > 160 * 1024)) || (l.rope_interleaved && !latent))
             return bail(afail(err, PS_CUDA_ERR_UNSUPPORTED, "layer %d: side mixer %d of %d channels; interleaved rotation %d", i, l.side_kind, l.side_width, l.rope_interleaved));
         if ((l.mlp_ungated && l.mlp_kind != PS_MLP_DENSE) || (l.act_kind == PS_ACT_XIELU && !l.mlp_ungated) || (d.norm_kind == PS_NORM_LAYER && (l.block_kind != PS_BLOCK_SEQUENTIAL || l.mlp_kind == PS_MLP_ROUTED)))
             return bail(afail(err, PS_CUDA_ERR_UNSUPPORTED, "layer %d: a feed-forward without a gate is dense (xIELU has no gated form); layer norms go with sequential blocks and dense feed-forwards", i));
-        if (!w.gen2 && (l.raw_input || recur || l.conv_taps > 0 || l.qk_norm == PS_QKNORM_WHOLE || l.chunk > 0 || l.act_kind == PS_ACT_GELU_TANH || l.shared_ff > 0 ||
+        if (!w.gen2 && (l.raw_input || recur || l.conv_taps > 0 || l.qk_norm == PS_QKNORM_WHOLE || l.chunk > 0 || l.act_kind == PS_ACT_GELU_TANH || l.act_kind == PS_ACT_RELU || l.shared_ff > 0 ||
                         l.router_act == PS_ROUTER_SOFTMAX || l.route_groups > 1))
             return bail(afail(err, PS_CUDA_ERR_UNSUPPORTED, "layer %d: raw sublayer inputs, recurrent mixers, convolutions, whole-projection norms, chunked masks, gelu, soft-max / grouped routers and shared experts need a sequential block", i));
         if (w.gen2 && (latent || l.v_mix || l.qk_norm == PS_QKNORM_HEAD || l.proj_bias || l.head_mix || l.head_temp))
             return bail(afail(err, PS_CUDA_ERR_UNSUPPORTED, "layer %d: latent attention, value blending, per-head unit norms, projection biases and head mixing are not combined with this layer's other mechanisms", i));
         if (w.gen2 && l.mlp_kind == PS_MLP_ROUTED && !l.raw_input && d.norm_groups > 1)
             return bail(afail(err, PS_CUDA_ERR_UNSUPPORTED, "layer %d: routed experts behind a group norm", i));
-        if (l.chunk < 0 || l.conv_taps < 0 || l.conv_taps > 64 || l.act_kind < PS_ACT_SWISH || l.act_kind > PS_ACT_RELU2 || l.shared_ff < 0)
+        if (l.chunk < 0 || l.conv_taps < 0 || l.conv_taps > 64 || l.act_kind < PS_ACT_SWISH || l.act_kind > PS_ACT_RELU || l.shared_ff < 0)
             return bail(afail(err, PS_CUDA_ERR_UNSUPPORTED, "layer %d: chunk %d, %d convolution taps, activation %d, shared expert of %d rows", i, l.chunk, l.conv_taps, l.act_kind, l.shared_ff));
         if (l.mixer_kind == PS_MIXER_RETENTION && (l.rope_dims < 0 || l.rope_dims > l.qk_dim || (l.rope_dims & 1) || (l.rope_dims > 0 && !(l.rope_base > 0.f)) || l.qk_dim > 256 || l.rope_factor != 0.f))
             return bail(afail(err, PS_CUDA_ERR_UNSUPPORTED, "layer %d: retention with heads of %d of which %d rotate (at most 256)", i, l.qk_dim, l.rope_dims));
@@ -447,7 +524,7 @@ int ps_arch_create(PsArch **out, const ps_cuda_arch_desc *desc, std::string &err
         if (l.rel_buckets < 0 || l.rel_buckets > 65535 || (l.rel_buckets > 0 && (l.rel_buckets < 2 || !(l.rel_max_dist > (float)(l.rel_buckets / 2)))))
             return bail(afail(err, PS_CUDA_ERR_UNSUPPORTED, "layer %d: distance-bias table of %d rows up to distance %g", i, l.rel_buckets, (double)l.rel_max_dist));
         if (l.mlp_kind != PS_MLP_NONE && l.mlp_kind != PS_MLP_ROUTED && l.mlp_kind != PS_MLP_DENSE) return bail(afail(err, PS_CUDA_ERR_UNSUPPORTED, "layer %d: unknown feed-forward kind %d", i, l.mlp_kind));
-        if (l.mlp_kind == PS_MLP_ROUTED && (l.n_experts <= 0 || l.n_experts > PA_MAX_EXPERTS || l.top_k <= 0 || l.top_k > l.n_experts || l.expert_ff <= 0 ||
+        if (l.mlp_kind == PS_MLP_ROUTED && (l.n_experts <= 0 || l.n_experts + l.route_identity > PA_MAX_EXPERTS || l.top_k <= 0 || l.top_k > l.n_experts + l.route_identity || l.expert_ff <= 0 ||
                                          (l.router_act != PS_ROUTER_SIGMOID && l.router_act != PS_ROUTER_SOFTMAX) ||
                                          (l.route_groups > 1 && (l.n_experts % l.route_groups || l.route_keep <= 0 || l.route_keep > l.route_groups || l.top_k > l.route_keep * (l.n_experts / l.route_groups)))))
             return bail(afail(err, PS_CUDA_ERR_UNSUPPORTED, "layer %d: unsupported routed feed-forward (%d experts, top %d, ff %d, router activation %d)", i, l.n_experts,
@@ -455,7 +532,7 @@ int ps_arch_create(PsArch **out, const ps_cuda_arch_desc *desc, std::string &err
         if (l.mlp_kind == PS_MLP_DENSE && l.expert_ff <= 0) return bail(afail(err, PS_CUDA_ERR_UNSUPPORTED, "layer %d: dense feed-forward of %d rows", i, l.expert_ff));
         // the attention kernels see a latent layer as one shared key head of kv_rank + rot_dim dims whose values are the latents
         const int a_dq = latent ? l.kv_rank + l.rot_dim : l.qk_dim, a_dv = latent ? l.kv_rank : l.v_dim;
-        if ((!recur && pa_dec_scores_smem(l.n_heads, l.n_kv_heads, a_dq) > 160 * 1024) || (size_t)d.dim * 4 > 160 * 1024)
+        if ((!recur && pa_dec_scores_smem(l.n_heads, l.n_kv_heads, a_dq, l.rope_dims) > 160 * 1024) || (size_t)d.dim * 4 > 160 * 1024)
             return bail(afail(err, PS_CUDA_ERR_UNSUPPORTED, "layer %d: %d heads of size %d (or width %d) exceed the single-token kernels' shared memory", i, l.n_heads, a_dq, d.dim));
         w.qd = l.n_heads * a_dq; w.kd = l.n_kv_heads * a_dq; w.vd = l.n_kv_heads * a_dv; w.od = l.n_heads * l.v_dim;
         w.pw = latent ? l.q_rank + l.kv_rank + l.rot_dim : w.qd + w.kd + w.vd;
@@ -465,8 +542,9 @@ int ps_arch_create(PsArch **out, const ps_cuda_arch_desc *desc, std::string &err
         if (newer) { // q | k | [v] | [gate] | [z | u | side gate]
             w.v_off = l.v_is_k ? w.qd : w.qd + w.kd;
             w.pw = w.qd + w.kd + (l.v_is_k ? 0 : w.vd);
-            if (l.out_gate) { w.g_off = w.pw; w.pw += w.ho; }
-            if (l.side_kind) { w.z_off = w.pw; w.pw += 3 * l.side_width; w.od += l.side_width; w.aw = w.od; }
+            const bool rwkv = l.side_kind == PS_MIXER_RWKV;
+            if (l.out_gate) { w.g_off = w.pw; w.pw += l.out_gate == PS_GATE_HEAD ? l.n_heads : w.ho; }
+            if (l.side_kind) { w.z_off = w.pw; w.pw += rwkv ? 4 * l.side_width + l.decay_rank : 3 * l.side_width; w.od += l.side_width; w.aw = w.od; }
             int64_t kf = (int64_t)w.kd * d.n_ctx, vf = (int64_t)w.vd * d.n_ctx;
             if (l.pool > 0) {
                 w.n_pool = (d.n_ctx / l.pool + 3) & ~3;
@@ -474,10 +552,28 @@ int ps_arch_create(PsArch **out, const ps_cuda_arch_desc *desc, std::string &err
                 vf += (int64_t)w.n_pool * w.vd;
                 a->max_pool = std::max(a->max_pool, w.n_pool);
             }
-            if (l.side_kind) { w.state_off = kf; kf += l.side_width; }
+            if (rwkv) { // S [heads][channels][channels padded], then the last token's input (two rows)
+                const int sd = l.side_width / l.side_heads;
+                w.state_off = (kf + 3) & ~(int64_t)3;
+                w.ring_off = w.state_off + (int64_t)l.side_width * pa_scan_dkp(sd);
+                kf = w.ring_off + 2 * (int64_t)d.dim;
+                a->max_dcy = std::max(a->max_dcy, l.side_width);
+                a->has_shift = true;
+                // the first projection's rows by the mixture they read: the attention's (h), r, k, v, gate, w1
+                w.seg.n = PT_MAX_SEG;
+                w.seg.row[1] = w.z_off;
+                for (int k = 2; k < PT_MAX_SEG; k++) w.seg.row[k] = w.seg.row[k - 1] + l.side_width;
+                w.seg.row[PT_MAX_SEG] = w.pw;
+                for (int k = 0; k < PT_MAX_SEG; k++) w.seg.rt[k + 1] = w.seg.rt[k] + (w.seg.row[k + 1] - w.seg.row[k] + PT_M - 1) / PT_M;
+            } else if (l.side_kind) { w.state_off = kf; kf += l.side_width; }
             w.k_floats = kf; w.v_floats = vf;
         }
-        if (l.mixer_kind == PS_MIXER_RETENTION) { // q | k | v | gate; the state S [H][v_dim][qk_dim padded] takes the place of the K rows
+        if (l.mixer_kind == PS_MIXER_GLA) { // q | k | v | gate | a1
+            w.qd = w.kd = l.n_heads * l.qk_dim; w.vd = w.od = w.aw = l.n_heads * l.v_dim;
+            w.pw = 2 * w.qd + 2 * w.od + l.decay_rank;
+            w.k_floats = (int64_t)l.n_heads * pa_scan_dkp(l.qk_dim) * l.v_dim; w.v_floats = 4;
+            a->max_dcy = std::max(a->max_dcy, w.qd);
+        } else if (l.mixer_kind == PS_MIXER_RETENTION) { // q | k | v | gate; the state S [H][v_dim][qk_dim padded] takes the place of the K rows
             w.qd = w.kd = l.n_heads * l.qk_dim; w.vd = w.od = w.aw = l.n_heads * l.v_dim;
             w.pw = 2 * w.qd + 2 * w.od;
             w.k_floats = (int64_t)l.n_heads * pa_scan_dkp(l.qk_dim) * l.v_dim; w.v_floats = 4;
@@ -518,9 +614,10 @@ int ps_arch_create(PsArch **out, const ps_cuda_arch_desc *desc, std::string &err
         if (l.mlp_kind == PS_MLP_ROUTED) {
             a->max_top = std::max(a->max_top, l.top_k);
             a->max_ff = std::max(a->max_ff, l.expert_ff);
-            a->max_e = std::max(a->max_e, l.n_experts);
+            a->max_e = std::max(a->max_e, l.n_experts + l.route_identity);
             a->max_k = std::max(a->max_k, l.expert_ff);
         }
+        if (l.token_slot) a->max_k = std::max(a->max_k, d.token_dim);
     }
     a->d.layers = nullptr; // the caller's array need not outlive this call: the copies live in L
     const int64_t B = d.max_batch, dim = d.dim;
@@ -544,7 +641,11 @@ int ps_arch_create(PsArch **out, const ps_cuda_arch_desc *desc, std::string &err
     AL(a->row_token, 4 * nrow);
     AL(a->row_slot, 4 * nrow);
     const size_t ntile = nrow / PA_TM + (size_t)std::max(a->max_e, 1) + 1;
-    if (a->round) AL(a->tcx, (nrow / PT_N + (size_t)std::max(a->max_e, 1) + 1) * (size_t)((a->max_k + PT_KB - 1) / PT_KB) * PT_BLOCK);
+    if (a->round) {
+        size_t blocks = (nrow / PT_N + (size_t)std::max(a->max_e, 1) + 1) * (size_t)((a->max_k + PT_KB - 1) / PT_KB);
+        if (a->has_shift) blocks = std::max(blocks, (size_t)PT_MAX_SEG * ((size_t)B + PT_N - 1) / PT_N * (size_t)((dim + PT_KB - 1) / PT_KB) + PT_MAX_SEG * (size_t)((dim + PT_KB - 1) / PT_KB));
+        AL(a->tcx, blocks * PT_BLOCK);
+    }
     AL(a->tile_e, 4 * ntile);
     AL(a->tile_row0, 4 * ntile);
     AL(a->tile_end, 4 * ntile);
@@ -570,6 +671,12 @@ int ps_arch_create(PsArch **out, const ps_cuda_arch_desc *desc, std::string &err
     if (a->has_pass_in) AL(a->xcat, 8 * dim * B);
     if (a->max_rec) AL(a->gts, 8 * (size_t)a->max_rec * B);
     AL(a->hn, 4 * dim);
+    if (a->max_dcy) AL(a->dcy, 4 * (size_t)a->max_dcy * B);
+    if (a->has_shift) AL(a->mixb, 4 * 5 * (size_t)dim * B);
+    if (d.token_slots > 0) {
+        AL(a->tg, 4 * (size_t)std::max(d.token_dim, 1) * B);
+        AL(a->ty, 4 * (size_t)dim * B);
+    }
     if (a->vsrc_w) AL(a->vsrc, 4 * (size_t)a->vsrc_w * B);
     if (rc) return bail(rc);
     int dev = 0;
@@ -583,21 +690,18 @@ int ps_arch_create(PsArch **out, const ps_cuda_arch_desc *desc, std::string &err
         cudaFuncSetAttribute(pa_k_dec_expert_up<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024) != cudaSuccess ||
         cudaFuncSetAttribute(pa_k_dec_dense_up<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024) != cudaSuccess ||
         cudaFuncSetAttribute(pa_k_dec_dense_up<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024) != cudaSuccess ||
-        cudaFuncSetAttribute(pa_k_scan<1, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, 112 * 1024) != cudaSuccess ||
-        cudaFuncSetAttribute(pa_k_scan<1, 2>, cudaFuncAttributeMaxDynamicSharedMemorySize, 112 * 1024) != cudaSuccess ||
-        cudaFuncSetAttribute(pa_k_scan<2, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, 112 * 1024) != cudaSuccess ||
-        cudaFuncSetAttribute(pa_k_scan<2, 2>, cudaFuncAttributeMaxDynamicSharedMemorySize, 112 * 1024) != cudaSuccess ||
-        cudaFuncSetAttribute(pa_k_scan<4, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, 112 * 1024) != cudaSuccess ||
-        cudaFuncSetAttribute(pa_k_scan<4, 2>, cudaFuncAttributeMaxDynamicSharedMemorySize, 112 * 1024) != cudaSuccess ||
-        cudaFuncSetAttribute(pa_k_scan<8, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, 112 * 1024) != cudaSuccess ||
-        cudaFuncSetAttribute(pa_k_scan<8, 2>, cudaFuncAttributeMaxDynamicSharedMemorySize, 112 * 1024) != cudaSuccess ||
-        cudaFuncSetAttribute(pa_k_scan<16, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, 112 * 1024) != cudaSuccess ||
-        cudaFuncSetAttribute(pa_k_scan<16, 2>, cudaFuncAttributeMaxDynamicSharedMemorySize, 112 * 1024) != cudaSuccess ||
         cudaFuncSetAttribute(pa_k_tc_gemm<1>, cudaFuncAttributeMaxDynamicSharedMemorySize, PT_SMEM) != cudaSuccess ||
         cudaFuncSetAttribute(pa_k_tc_gemm<2>, cudaFuncAttributeMaxDynamicSharedMemorySize, PT_SMEM) != cudaSuccess) {
         cudaGetLastError();
         return bail(afail(err, PS_CUDA_ERR_CUDA, "cudaFuncSetAttribute(dynamic shared memory) failed"));
     }
+    for (int il = 1; il <= 16; il *= 2)
+        for (int nc = 1; nc <= 2; nc++)
+            for (int mode = 0; mode <= 2; mode++)
+                if (cudaFuncSetAttribute(pa_scan_kernel(il, nc, mode), cudaFuncAttributeMaxDynamicSharedMemorySize, 112 * 1024) != cudaSuccess) {
+                    cudaGetLastError();
+                    return bail(afail(err, PS_CUDA_ERR_CUDA, "cudaFuncSetAttribute(dynamic shared memory) failed"));
+                }
     if (cudaStreamCreateWithFlags(&a->side, cudaStreamNonBlocking) != cudaSuccess || cudaEventCreateWithFlags(&a->ev_fork, cudaEventDisableTiming) != cudaSuccess ||
         cudaEventCreateWithFlags(&a->ev_join, cudaEventDisableTiming) != cudaSuccess) {
         cudaGetLastError();
@@ -759,11 +863,12 @@ int ps_arch_bind(PsArch *a, const ps_cuda_arch_weights *wt, cudaStream_t stream,
     if ((rc = aalloc(a, (void **)&a->embed, 2 * dim * d.vocab_size, err)) || (rc = upload_mat(a->embed, wt->embed, dim * d.vocab_size, "embed", err))) return rc;
     if ((rc = aalloc(a, (void **)&a->head, 2 * dim * d.vocab_size, err)) || (rc = upload_mat(a->head, wt->head, dim * d.vocab_size, "head", err))) return rc;
     // a norm's weight: [dim] values, or with norm_scalar one number for all coordinates
-    auto normvec = [&](float **dst, const ps_cuda_tensor &t, const char *what) -> int {
+    auto normvec = [&](float **dst, const ps_cuda_tensor &t, const char *what, const std::vector<float> *scale = nullptr) -> int {
         int r = small_to_f32(t, d.norm_scalar ? 1 : dim, tmp, what, err);
         if (r) return r;
         if (d.norm_scalar) tmp.assign(dim, tmp[0]);
         if (d.norm_unit_offset) for (float &v : tmp) v = 1.0f + v;
+        if (scale) for (size_t c = 0; c < dim; c++) tmp[c] *= (*scale)[c];
         return upload_f32(a, dst, tmp, err);
     };
     if ((rc = normvec(&a->final_norm, wt->final_norm, "final norm"))) return rc;
@@ -772,6 +877,7 @@ int ps_arch_bind(PsArch *a, const ps_cuda_arch_weights *wt, cudaStream_t stream,
         return r ? r : upload_mat(*dst, t, n, what, err);
     };
     if (a->has_pass_in && (rc = mat(&a->pass_in, wt->pass_in, 2 * dim * dim, "pass input"))) return rc;
+    if (d.token_slots > 0 && (rc = mat(&a->tok_embed, wt->token_embed, (size_t)d.vocab_size * d.token_slots * d.token_dim, "token input table"))) return rc;
     if (d.n_pass_steps > 0 && (rc = vec(&a->pass_steps, wt->pass_steps, (size_t)d.n_pass_steps * dim, "pass steps", false))) return rc;
     a->taps.assign((size_t)d.n_layers, nullptr);
     for (int i = 0; i < d.n_layers; i++) {
@@ -805,9 +911,49 @@ int ps_arch_bind(PsArch *a, const ps_cuda_arch_weights *wt, cudaStream_t stream,
             if ((rc = upload_mat(w.wqkv, s.q, nq * dim, "q", err)) || (rc = upload_mat(w.wqkv + nq * dim, s.k, nk * dim, "k", err)) ||
                 (!l.v_is_k && (rc = upload_mat(w.wqkv + (nq + nk) * dim, s.v, nv * dim, "v", err))))
                 return rc;
-            if (l.out_gate && (rc = upload_mat(w.wqkv + (size_t)w.g_off * dim, s.g, (size_t)w.ho * dim, "output gate", err))) return rc;
+            if (l.out_gate && (rc = upload_mat(w.wqkv + (size_t)w.g_off * dim, s.g, (size_t)(l.out_gate == PS_GATE_HEAD ? l.n_heads : w.ho) * dim, "output gate", err))) return rc;
             if (l.lin_bias && (rc = vec(&w.lin, s.lin, (size_t)l.n_heads, "distance-bias slopes", false))) return rc;
-            if (l.side_kind) {
+            if (l.qk_norm == PS_QKNORM_HEAD_W && ((rc = vec(&w.q_norm, s.q_norm, (size_t)l.qk_dim, "q norm", false)) || (rc = vec(&w.k_norm, s.k_norm, (size_t)l.qk_dim, "k norm", false)))) return rc;
+            auto freqs = [&](double **dst, int dims, float factor) -> int {
+                std::vector<double> fd((size_t)dims / 2);
+                const double ms = rope_freq_host(dims, l.rope_base, factor, l.rope_original, l.rope_fast, l.rope_slow, fd.data());
+                if (dst == &w.rope_freq) w.rope_mscale = (float)ms;
+                int r = aalloc(a, (void **)dst, fd.size() * 8, err);
+                if (r) return r;
+                PA_CK(cudaMemcpy(*dst, fd.data(), fd.size() * 8, cudaMemcpyHostToDevice));
+                return 0;
+            };
+            if (l.mixer_kind == PS_MIXER_ATTENTION && l.rope_dims > 0 && (rc = freqs(&w.rope_freq, l.rope_dims, l.rope_factor))) return rc;
+            if (l.mixer_kind == PS_MIXER_ATTENTION && l.v_rope && (rc = freqs(&w.vrope_freq, l.v_dim, 0.f))) return rc;
+            if (l.mixer_kind == PS_MIXER_GLA) {
+                const size_t rk = (size_t)l.decay_rank, H = (size_t)l.n_heads;
+                if ((rc = upload_mat(w.wqkv + (nq + nk + nv) * dim, s.g, nv * dim, "g", err)) || (rc = upload_mat(w.wqkv + (nq + nk + 2 * nv) * dim, s.a1, rk * dim, "a1", err)) ||
+                    (rc = mat(&w.wa2, s.a2, nk * rk, "a2")) || (rc = vec(&w.a2b, s.a2_bias, nk, "a2 bias", false)) || (rc = small_to_f32(s.mix_norm, (size_t)l.v_dim, tmp, "mixer norm", err)))
+                    return rc;
+                std::vector<float> rep; // one weight for every head
+                for (size_t h = 0; h < H; h++) rep.insert(rep.end(), tmp.begin(), tmp.end());
+                if ((rc = upload_f32(a, &w.mix_norm, rep, err))) return rc;
+            }
+            if (l.side_kind == PS_MIXER_RWKV) {
+                const size_t W = (size_t)l.side_width, rk = (size_t)l.decay_rank;
+                size_t at = (size_t)w.z_off;
+                for (const ps_cuda_tensor *t : {&s.side_r, &s.side_k, &s.side_v, &s.side_g}) {
+                    if ((rc = upload_mat(w.wqkv + at * dim, *t, W * dim, "side r / k / v / g", err))) return rc;
+                    at += W;
+                }
+                if ((rc = upload_mat(w.wqkv + at * dim, s.side_w1, rk * dim, "side w1", err)) || (rc = mat(&w.wa2, s.side_w2, W * rk, "side w2")) || (rc = vec(&w.a2b, s.side_w0, W, "side w0", false)) ||
+                    (rc = vec(&w.bonus, s.side_u, W, "side u", false)))
+                    return rc;
+                std::vector<float> mu;
+                for (const ps_cuda_tensor *t : {&s.side_mu_r, &s.side_mu_k, &s.side_mu_v, &s.side_mu_g, &s.side_mu_w}) {
+                    if ((rc = small_to_f32(*t, dim, tmp, "side mu", err))) return rc;
+                    mu.insert(mu.end(), tmp.begin(), tmp.end());
+                }
+                if ((rc = upload_f32(a, &w.mu, mu, err)) || (rc = small_to_f32(s.side_norm, W, tmp, "side norm", err))) return rc;
+                for (float &v : tmp) v *= l.side_scale; // the side mixer's factor rides on its norm's weight
+                if ((rc = upload_f32(a, &w.mix_norm, tmp, err))) return rc;
+            }
+            if (l.side_kind == PS_MIXER_MINGRU) {
                 const size_t W = (size_t)l.side_width;
                 if ((rc = upload_mat(w.wqkv + (size_t)w.z_off * dim, s.side_z, W * dim, "side z", err)) || (rc = upload_mat(w.wqkv + ((size_t)w.z_off + W) * dim, s.side_x, W * dim, "side x", err)) ||
                     (rc = upload_mat(w.wqkv + ((size_t)w.z_off + 2 * W) * dim, s.side_g, W * dim, "side gate", err)))
@@ -852,11 +998,19 @@ int ps_arch_bind(PsArch *a, const ps_cuda_arch_weights *wt, cudaStream_t stream,
             return rc;
         }
         if (l.block_kind == PS_BLOCK_SEQUENTIAL) {
-            if (l.post_norm && (rc = normvec(&w.norm_mix_out, s.norm_mix_out, "norm of the mixer's output"))) return rc;
+            std::vector<float> sc;
+            // a layer scale rides on the output norm's weight
+            if (l.layer_scale && (rc = small_to_f32(s.scale_mix, dim, sc, "layer scale of the mixer", err))) return rc;
+            if (l.post_norm && (rc = normvec(&w.norm_mix_out, s.norm_mix_out, "norm of the mixer's output", l.layer_scale ? &sc : nullptr))) return rc;
             if (l.mlp_kind != PS_MLP_NONE) {
+                if (l.layer_scale && (rc = small_to_f32(s.scale_ff, dim, sc, "layer scale of the feed-forward", err))) return rc;
                 if (!l.raw_input && (rc = normvec(&w.norm_ff, s.norm_ff, "norm before the feed-forward"))) return rc;
-                if (l.post_norm && (rc = normvec(&w.norm_ff_out, s.norm_ff_out, "norm of the feed-forward's output"))) return rc;
+                if (l.post_norm && (rc = normvec(&w.norm_ff_out, s.norm_ff_out, "norm of the feed-forward's output", l.layer_scale ? &sc : nullptr))) return rc;
             }
+        }
+        if (l.token_slot) {
+            const size_t td = (size_t)d.token_dim;
+            if ((rc = mat(&w.wtg, s.token_gate, td * dim, "token gate")) || (rc = mat(&w.wtp, s.token_proj, td * dim, "token projection")) || (rc = vec(&w.tok_norm, s.token_norm, dim, "token norm", false))) return rc;
         }
         if (l.log_bias && ((rc = vec(&w.r1, s.r1, (size_t)l.n_heads, "distance-bias slopes", false)) || (rc = vec(&w.r2, s.r2, (size_t)l.n_heads, "distance-bias rates", false)))) return rc;
         if (l.sink == PS_SINK_LEARNED && (rc = vec(&w.sink_v, s.sink, (size_t)l.n_heads, "sink logits", false))) return rc;
@@ -883,8 +1037,10 @@ int ps_arch_bind(PsArch *a, const ps_cuda_arch_weights *wt, cudaStream_t stream,
             const size_t E = (size_t)l.n_experts, ff = (size_t)l.expert_ff;
             if (!s.gate || !s.up || !s.down) return afail(err, PS_CUDA_ERR_INVALID, "bind: layer %d has no expert tensors", i);
             const size_t sgr = (l.shared_ff > 0 && l.shared_gate) ? 1 : 0; // the shared expert's gate is one more router row
-            if ((rc = aalloc(a, (void **)&w.router, 2 * (E + sgr) * dim, err)) || (rc = upload_mat(w.router, s.router, E * dim, "router", err))) return rc;
-            if (sgr && (rc = upload_mat(w.router + E * dim, s.shared_sg, dim, "shared gate", err))) return rc;
+            const size_t Er = E + (size_t)l.route_identity;
+            if ((rc = aalloc(a, (void **)&w.router, 2 * (Er + sgr) * dim, err)) || (rc = upload_mat(w.router, s.router, Er * dim, "router", err))) return rc;
+            if (l.route_correction && (rc = vec(&w.corr, s.correction, Er, "router correction", false))) return rc;
+            if (sgr && (rc = upload_mat(w.router + Er * dim, s.shared_sg, dim, "shared gate", err))) return rc;
             if (l.shared_ff > 0) {
                 const size_t sf = (size_t)l.shared_ff;
                 if ((rc = mat(&w.wsg, s.shared_gate, sf * dim, "shared gate rows")) || (rc = mat(&w.wsu, s.shared_up, sf * dim, "shared up rows")) || (rc = mat(&w.wsd, s.shared_down, sf * dim, "shared down rows"))) return rc;
@@ -931,7 +1087,19 @@ int ps_arch_bind(PsArch *a, const ps_cuda_arch_weights *wt, cudaStream_t stream,
                     return rc;
                 continue;
             }
-            if ((rc = tile(&w.t_qkv, w.wqkv, 1, w.pw, d.dim)) || (rc = tile(&w.t_o, w.wo, 1, d.dim, w.od))) return rc;
+            if (w.seg.n > 0) { // every segment starts at a row tile of its own
+                const int nkb = (d.dim + PT_KB - 1) / PT_KB;
+                if ((rc = aalloc(a, (void **)&w.t_qkv, (size_t)w.seg.rt[w.seg.n] * nkb * PT_BLOCK, err))) return rc;
+                for (int k = 0; k < w.seg.n; k++) {
+                    const int n = w.seg.row[k + 1] - w.seg.row[k], n_rt = w.seg.rt[k + 1] - w.seg.rt[k];
+                    pa_k_tc_tile_w<<<dim3((unsigned)nkb, (unsigned)n_rt, 1), 256, 0, stream>>>(w.t_qkv + (size_t)w.seg.rt[k] * nkb * PT_BLOCK, w.wqkv + (size_t)w.seg.row[k] * d.dim, n, d.dim, n_rt, nkb);
+                    PA_CK(cudaGetLastError());
+                }
+            } else if ((rc = tile(&w.t_qkv, w.wqkv, 1, w.pw, d.dim))) {
+                return rc;
+            }
+            if ((rc = tile(&w.t_o, w.wo, 1, d.dim, w.od))) return rc;
+            if (w.wtg && ((rc = tile(&w.t_tg, w.wtg, 1, d.token_dim, d.dim)) || (rc = tile(&w.t_tp, w.wtp, 1, d.dim, d.token_dim)))) return rc;
             if (w.wuq && (rc = tile(&w.t_uq, w.wuq, 1, w.d.n_heads * (w.d.qk_dim + w.d.rot_dim), w.d.q_rank))) return rc;
             if (w.d.mlp_kind == PS_MLP_DENSE &&
                 ((w.wgate && (rc = tile(&w.t_gate, w.wgate, 1, w.d.expert_ff, d.dim))) || (rc = tile(&w.t_up, w.wup, 1, w.d.expert_ff, d.dim)) || (rc = tile(&w.t_down, w.wdown, 1, d.dim, w.d.expert_ff))))
@@ -985,13 +1153,14 @@ static int forward_t(PsArch *a, const PsArchIO &io, int bs, int pos0, int lm_hea
     const bool tc = ROUND && a->opt_tc && !single && !a->opt_simple;
     // C[m][n] = sum_k X[m][k] W[n][k] + bias[n] on the tensor cores: round + tile the activations, then the GEMM
     auto tc_dense = [&](const float *X, int ldx, int M, int K, const uint8_t *wt, int N, const float *bias, float *C, int ldc, const PaAct *act1 = nullptr, int act_from = 0,
-                        int gap = 0) -> int {
+                        int gap = 0, const PaRowMul *mul = nullptr) -> int {
         const int nkb = (K + PT_KB - 1) / PT_KB, n_ct = (M + PT_N - 1) / PT_N, n_rt = (N + PT_M - 1) / PT_M;
         pa_k_tc_prep_x<<<dim3((unsigned)nkb, (unsigned)n_ct), 256, 0, st>>>(a->tcx, X, ldx, M, K, nkb, nullptr, nullptr, nullptr, nullptr, nullptr);
         PA_LAUNCH();
         PtArgs g{};
         g.a0 = wt; g.b = a->tcx; g.nkb = nkb; g.n_rt = n_rt; g.n_ct = n_ct; g.M = M; g.N = N; g.mode = PT_MODE_DENSE; g.C = C; g.ldc = ldc; g.bias = bias; g.err = io.err_dev;
         if (act1) { g.act = *act1; g.act1 = 1; g.act_from = act_from; g.gap = gap; }
+        if (mul) g.mul = *mul;
         pa_k_tc_gemm<1><<<std::min(a->n_sm, n_ct * n_rt), PT_THREADS, PT_SMEM, st>>>(g);
         PA_LAUNCH();
         return 0;
@@ -1045,9 +1214,9 @@ static int forward_t(PsArch *a, const PsArchIO &io, int bs, int pos0, int lm_hea
         if (pend_y || add_tok || add_vec) { mv.x_out = xo; std::swap(xc, xo); }
         pend_y = pend_w = add_tok = add_vec = nullptr;
     };
-    auto dec_mv = [&](PaMv &mv, size_t smem) -> int {
+    auto dec_mv = [&](PaMv &mv, size_t smem, bool overlap = true) -> int {
         mv.ksplit = pick_ksplit(mv.N + mv.E, mv.K); mv.prefetch = a->opt_prefetch;
-        pa_launch_dep(pdl, pa_k_dec_mv<ROUND>, dim3(mv_grid(mv.N + mv.E, mv.ksplit, mv.K)), dim3(PA_DV_THREADS), smem, st, mv);
+        pa_launch_dep(pdl && overlap, pa_k_dec_mv<ROUND>, dim3(mv_grid(mv.N + mv.E, mv.ksplit, mv.K)), dim3(PA_DV_THREADS), smem, st, mv);
         PA_LAUNCH();
         return 0;
     };
@@ -1057,7 +1226,7 @@ static int forward_t(PsArch *a, const PsArchIO &io, int bs, int pos0, int lm_hea
         if (at.window > 0) blocks = std::min(blocks, cdiv(at.window, PA_DS_KEYS) + 1);
         if (at.chunk > 0) blocks = std::min(blocks, cdiv(at.chunk, PA_DS_KEYS) + 1);
         const unsigned pooled = at.pool > 0 ? cdiv(n_kv_cap / at.pool, PA_DS_KEYS) : 0; // further CTAs for the pooled blocks
-        pa_launch_dep(pdl, pa_k_dec_scores, dim3(blocks + pooled), dim3(256), pa_dec_scores_smem(at.H, at.G, at.dq), st, at, q, (const float *)io.kc[li], io.pos_dev, a->S, io.err_dev, (int)blocks,
+        pa_launch_dep(pdl, pa_k_dec_scores, dim3(blocks + pooled), dim3(256), pa_dec_scores_smem(at.H, at.G, at.dq, at.rope.dims), st, at, q, (const float *)io.kc[li], io.pos_dev, a->S, io.err_dev, (int)blocks,
                       pool_here && pooled ? io.vct[li] : (float *)nullptr);
         PA_LAUNCH();
         pa_launch_dep(pdl, pa_k_dec_pv, dim3(cdiv(at.dv, PA_DP_DIMS), at.G, pa_dec_pv_split(at.H, at.G)), dim3(256), pa_dec_pv_smem(at.H, at.G), st, at, (const float *)a->S, (const float *)io.vct[li], io.pos_dev, out,
@@ -1239,22 +1408,85 @@ static int forward_t(PsArch *a, const PsArchIO &io, int bs, int pos0, int lm_hea
         const int il = pa_scan_il(sc.dk);
         int nc = a->opt_scan_nc;
         if (nc <= 0) nc = (int64_t)cdiv(sc.dv, pa_scan_cols(sc.dk, 2)) * sc.H >= (bs > 1 ? a->n_sm * 3 / 4 : 4 * a->n_sm) ? 2 : 1;
-        const dim3 grid(cdiv(sc.dv, pa_scan_cols(sc.dk, nc)), (unsigned)sc.H), blk_s(32 * PA_SC_WARPS);
-        const size_t smem = pa_scan_smem(sc.dk, nc);
-#define PA_SCAN_CASE(IL_)                                                              \
-    case IL_:                                                                           \
-        if (nc == 2) pa_k_scan<IL_, 2><<<grid, blk_s, smem, st>>>(sc);                  \
-        else pa_k_scan<IL_, 1><<<grid, blk_s, smem, st>>>(sc);                          \
-        break;
-        switch (il) {
-            PA_SCAN_CASE(1) PA_SCAN_CASE(2) PA_SCAN_CASE(4) PA_SCAN_CASE(8)
-        default:
-            if (nc == 2) pa_k_scan<16, 2><<<grid, blk_s, smem, st>>>(sc);
-            else pa_k_scan<16, 1><<<grid, blk_s, smem, st>>>(sc);
-            break;
-        }
-#undef PA_SCAN_CASE
+        const int mode = sc.bonus ? 2 : sc.dec ? 1 : 0;
+        pa_scan_kernel(il, nc, mode)<<<dim3(cdiv(sc.dv, pa_scan_cols(sc.dk, nc)), (unsigned)sc.H), dim3(32 * PA_SC_WARPS), pa_scan_smem(sc.dk, nc, mode), st>>>(sc);
         PA_LAUNCH();
+        return 0;
+    };
+    // a recurrence with a decay per key channel between the first projection's rows and the output product: decay (low-rank, fp32), scan,
+    // head norm, weight, silu gate.  Single tokens: one launch, a cluster per head.
+    struct PaRec {
+        const float *q, *k, *v, *g, *a1;
+        int H, dk, dv;
+        PaAct act;
+        const float *bonus;
+        float o_scale, *S, *out;
+        int ldo;
+    };
+    auto recurrence = [&](const PsArchLayer &w, const PaRec &r, cudaStream_t sr, bool dep) -> int {
+        const int rank = w.d.decay_rank, n = r.H * r.dk, dkp = pa_scan_dkp(r.dk);
+        if (single) {
+            PaRecStep p{};
+            p.q = r.q; p.k = r.k; p.v = r.v; p.g = r.g; p.a1 = r.a1; p.a2 = w.wa2; p.a2b = w.a2b; p.rank = rank; p.dact = r.act; p.bonus = r.bonus; p.o_scale = r.o_scale;
+            p.S = r.S; p.norm_w = w.mix_norm; p.eps = d.norm_eps; p.out = r.out; p.pos = io.pos_dev; p.dk = r.dk; p.dv = r.dv; p.dkp = dkp;
+            while ((PA_SC_REGS << p.lg) < dkp) p.lg++;
+            const int n_cl = pa_rec_cluster(r.dv);
+            PA_CK(pa_launch_cluster(dep, n_cl, pa_k_dec_recur, dim3((unsigned)n_cl, (unsigned)r.H), dim3(256), pa_rec_step_smem(dkp, (r.dv + n_cl - 1) / n_cl, rank), sr, p));
+            PA_LAUNCH();
+            return 0;
+        }
+        pa_k_linear<false><<<dim3(cdiv(n, PA_TN), cdiv(bs, PA_TM)), blk, 0, sr>>>(r.a1, w.pw, w.wa2, w.a2b, a->dcy, n, bs, n, rank, 0, 0, 0, 0, r.act);
+        PA_LAUNCH();
+        PaScan sc{};
+        sc.q = r.q; sc.k = r.k; sc.v = r.v; sc.ldq = sc.ldk = sc.ldv = w.pw; sc.q_gs = sc.k_gs = r.dk; sc.H = sc.G = r.H; sc.dk = r.dk; sc.dv = r.dv;
+        sc.dec = a->dcy; sc.lddec = n; sc.bonus = r.bonus; sc.o_scale = r.o_scale; sc.S = r.S; sc.o = r.out; sc.ldo = r.ldo; sc.pos = io.pos_dev; sc.bs = bs;
+        int rc = scan(sc);
+        if (rc) return rc;
+        pa_k_gate_norm<<<dim3((unsigned)r.H, bs), 256, 0, sr>>>(r.out, r.ldo, r.g, w.pw, r.H * r.dv, r.H, w.mix_norm, 0, d.norm_eps, r.out, r.ldo);
+        PA_LAUNCH();
+        return 0;
+    };
+    // the time mixing beside an attention: its columns follow the heads' outputs.  A single token's runs on the side stream (a fork in the captured step).
+    auto time_mix = [&](int li) -> int {
+        const PsArchLayer &w = a->L[(size_t)li];
+        const int W = w.d.side_width, sd = W / w.d.side_heads;
+        PaRec r{};
+        r.q = a->qkv + w.z_off; r.k = r.q + W; r.v = r.k + W; r.g = r.v + W; r.a1 = r.g + W;
+        r.H = w.d.side_heads; r.dk = r.dv = sd; r.act = PaAct{0.f, 0.f, 0.f, PA_ACT_EXP_EXP}; r.bonus = w.bonus; r.o_scale = 1.0f;
+        r.S = io.kc[li] + w.state_off; r.out = a->att + w.ho; r.ldo = w.aw;
+        const bool fork = single && a->opt_fork;
+        if (fork) { PA_CK(cudaEventRecord(a->ev_fork, st)); PA_CK(cudaStreamWaitEvent(a->side, a->ev_fork, 0)); }
+        int rc = recurrence(w, r, fork ? a->side : st, pdl && !fork);
+        if (rc) return rc;
+        if (fork) PA_CK(cudaEventRecord(a->ev_join, a->side));
+        return 0;
+    };
+    // the per-layer input from the token's own row: x <- x + N(W_proj (gelu(W_gate x) * e)); its output waits for the next seam
+    auto token_input = [&](int li) -> int {
+        const PsArchLayer &w = a->L[(size_t)li];
+        const int td = d.token_dim;
+        const PaAct gelu{0.f, 0.f, 0.f, PS_ACT_GELU_TANH};
+        const PaRowMul mul{a->tok_embed + (int64_t)(w.d.token_slot - 1) * td, (int64_t)d.token_slots * td, io.tokens_dev};
+        int rc;
+        if (single) {
+            PaMv mv{};
+            seam_mv(mv, nullptr);
+            mv.W = w.wtg; mv.N = td; mv.K = dim; mv.y = a->tg; mv.act = gelu; mv.mul = mul;
+            if ((rc = dec_mv(mv, 4 * (size_t)dim))) return rc;
+            PaMv mp{};
+            mp.x = a->tg; mp.W = w.wtp; mp.N = dim; mp.K = td; mp.y = a->ty;
+            if ((rc = dec_mv(mp, 0))) return rc;
+        } else {
+            if ((rc = seam(nullptr, nullptr))) return rc;
+            if (tc) {
+                if ((rc = tc_dense(a->x, dim, bs, dim, w.t_tg, td, nullptr, a->tg, td, &gelu, 0, 0, &mul))) return rc;
+            } else {
+                pa_k_linear<ROUND><<<dim3(cdiv(td, PA_TN), cdiv(bs, PA_TM)), blk, 0, st>>>(a->x, dim, w.wtg, nullptr, a->tg, td, bs, td, dim, 0, 0, 0, 0, gelu, mul);
+                PA_LAUNCH();
+            }
+            if ((rc = linear(a->tg, td, td, w.wtp, w.t_tp, dim, a->ty, dim))) return rc;
+        }
+        pend_y = a->ty; pend_w = w.tok_norm;
         return 0;
     };
     // A sequential block from the general parts: the sublayers read the residual stream itself (raw_input) or its norm; the mixer is an
@@ -1269,7 +1501,11 @@ static int forward_t(PsArch *a, const PsArchIO &io, int bs, int pos0, int lm_hea
         const bool raw = l.raw_input != 0;
         int rc;
         // single token, attention without convolution or q / k norm: the K rows (and V rows) go from the mat-vec straight into the cache
-        const bool direct = single && l.mixer_kind == PS_MIXER_ATTENTION && l.conv_taps == 0 && l.qk_norm == PS_QKNORM_NONE;
+        const bool heads_post = l.mixer_kind == PS_MIXER_ATTENTION && (l.qk_norm == PS_QKNORM_HEAD_W || l.rope_dims > 0 || l.v_rope); // norms / rotations of the heads
+        const bool direct = single && l.mixer_kind == PS_MIXER_ATTENTION && l.conv_taps == 0 && l.qk_norm == PS_QKNORM_NONE && !heads_post;
+        const bool rwkv = l.side_kind == PS_MIXER_RWKV;
+        const PaAct tanh_act{0.f, 0.f, 0.f, PA_ACT_TANH};
+        const int w1_off = w.pw - l.decay_rank; // time mixing: the rows of the decay's first product, which leave through tanh
         if (single) {
             PaMv mv{};
             seam_mv(mv, raw ? nullptr : w.norm);
@@ -1277,13 +1513,46 @@ static int forward_t(PsArch *a, const PsArchIO &io, int bs, int pos0, int lm_hea
             if (direct) {
                 mv.qd = w.qd; mv.kd = w.kd; mv.vd = l.v_is_k ? 0 : w.vd; mv.v_is_k = l.v_is_k; mv.kc = io.kc[li]; mv.vct = io.vct[li]; mv.n_ctx = d.n_ctx; mv.pos = io.pos_dev;
             }
-            if ((rc = dec_mv(mv, 4 * (size_t)dim))) return rc;
+            if (rwkv) {
+                mv.seg_n = w.seg.n;
+                for (int k = 0; k < w.seg.n; k++) mv.seg_end[k] = w.seg.row[k + 1];
+                mv.mu = w.mu; mv.ring = io.kc[li] + w.ring_off; mv.pos = io.pos_dev; mv.act_from = w1_off; mv.act = tanh_act;
+            }
+            if ((rc = dec_mv(mv, (rwkv ? PT_MAX_SEG : 1) * 4 * (size_t)dim))) return rc;
+        } else if (rwkv) {
+            float *ring = io.kc[li] + w.ring_off;
+            if ((rc = seam(a->h, w.norm))) return rc;
+            if (tc) { // one GEMM over six operand sets
+                const int nkb = (dim + PT_KB - 1) / PT_KB, n_ct = (bs + PT_N - 1) / PT_N;
+                PtArgs g{};
+                g.seg = w.seg;
+                g.seg.set_bytes = (int64_t)n_ct * nkb * PT_BLOCK;
+                pa_k_tc_prep_shift<<<dim3((unsigned)nkb, (unsigned)n_ct, PT_MAX_SEG), 256, 0, st>>>(a->tcx, a->h, bs, dim, nkb, w.mu, ring, io.pos_dev, g.seg.set_bytes);
+                PA_LAUNCH();
+                g.a0 = w.t_qkv; g.b = a->tcx; g.nkb = nkb; g.n_rt = w.seg.rt[w.seg.n]; g.n_ct = n_ct; g.M = bs; g.N = w.pw; g.mode = PT_MODE_DENSE; g.C = a->qkv; g.ldc = w.pw; g.err = io.err_dev;
+                g.act = tanh_act; g.act1 = 1; g.act_from = w1_off;
+                pa_k_tc_gemm<1><<<std::min(a->n_sm, n_ct * g.n_rt), PT_THREADS, PT_SMEM, st>>>(g);
+                PA_LAUNCH();
+            } else {
+                pa_k_token_shift<<<dim3(cdiv(dim, 256), bs, 5), 256, 0, st>>>(a->h, dim, w.mu, ring, io.pos_dev, a->mixb, (int64_t)B * dim);
+                PA_LAUNCH();
+                for (int k = 0; k < w.seg.n; k++) {
+                    const int r0 = w.seg.row[k], n = w.seg.row[k + 1] - r0;
+                    pa_k_linear<ROUND><<<dim3(cdiv(n, PA_TN), cdiv(bs, PA_TM)), blk, 0, st>>>(k ? a->mixb + (int64_t)(k - 1) * B * dim : a->h, dim, w.wqkv + (int64_t)r0 * dim, nullptr, a->qkv + r0, w.pw, bs, n, dim, 0,
+                                                                                            0, r0 == w1_off ? 0 : 1 << 30, 0, tanh_act);
+                    PA_LAUNCH();
+                }
+            }
+            pa_k_token_keep<<<cdiv(dim, 256), 256, 0, st>>>(a->h, dim, ring, io.pos_dev, bs);
+            PA_LAUNCH();
         } else {
             if ((rc = seam(raw ? nullptr : a->h, raw ? nullptr : w.norm))) return rc;
             if ((rc = linear(raw ? a->x : a->h, dim, dim, w.wqkv, w.t_qkv, w.pw, a->qkv, w.pw))) return rc;
         }
         if (l.mixer_kind == PS_MIXER_ATTENTION) {
             float *q = a->qkv;
+            const PaRope at_rope{w.rope_freq, l.rope_dims, w.rope_mscale, 0}, at_vrope{w.vrope_freq, l.v_rope ? l.v_dim : 0, 1.0f, 0};
+            if (rwkv && (rc = time_mix(li))) return rc; // a single token's runs beside the attention, joined before the output product
             if (l.conv_taps > 0) {
                 float *tail = io.kc[li] + (int64_t)w.kd * d.n_ctx;
                 if (bs == 1) {
@@ -1301,6 +1570,12 @@ static int forward_t(PsArch *a, const PsArchIO &io, int bs, int pos0, int lm_hea
             if (l.qk_norm == PS_QKNORM_WHOLE) {
                 pa_k_qkv_whole_norm<<<bs, 256, 0, st>>>(q, w.pw, w.qd, w.kd, w.vd, w.q_norm, w.k_norm, d.norm_eps, io.kc[li], io.vct[li], d.n_ctx, io.pos_dev, w.v_off);
                 PA_LAUNCH();
+            } else if (heads_post) {
+                if (!single) { // (a single token's scores kernel does this)
+                    pa_k_qkv_post<<<bs, 256, 8 * (size_t)(l.rope_dims / 2 + (l.v_rope ? l.v_dim / 2 : 0)), st>>>(q, w.pw, H, l.n_kv_heads, l.qk_dim, l.v_dim, l.qk_norm, d.norm_eps, 0, nullptr, nullptr, 0, io.kc[li],
+                                                                                                      io.vct[li], d.n_ctx, io.pos_dev, w.q_norm, w.k_norm, 0.f, 1.f, at_rope, at_vrope);
+                    PA_LAUNCH();
+                }
             } else if (!direct) {
                 pa_k_kv_store<<<dim3(cdiv(w.kd + w.vd, 256), bs), 256, 0, st>>>(q, w.pw, w.qd, w.kd, w.vd, io.kc[li], io.vct[li], d.n_ctx, io.pos_dev, w.v_off);
                 PA_LAUNCH();
@@ -1313,17 +1588,32 @@ static int forward_t(PsArch *a, const PsArchIO &io, int bs, int pos0, int lm_hea
             at.H = H; at.G = l.n_kv_heads; at.dq = l.qk_dim; at.dv = l.v_dim; at.scale = l.score_scale; at.rel = w.rel; at.bucket = w.bucket; at.n_bucket = d.n_ctx;
             at.sink = l.sink != PS_SINK_NONE; at.sink_v = w.sink_v; at.r1 = w.r1; at.r2 = w.r2; at.window = l.window; at.chunk = l.chunk;
             at.n_ctx = d.n_ctx; at.ldS = a->ldS; at.B = B; at.pm = a->pm; at.pl = a->pl; at.ldP = a->ldP;
+            at.softcap = l.score_softcap; at.vrope = at_vrope;
+            if (heads_post && single) {
+                at.k_raw = a->qkv + w.qd; at.kc_out = io.kc[li]; at.head_norm = l.qk_norm != PS_QKNORM_NONE; at.eps = d.norm_eps; at.rope = at_rope;
+                at.qn = w.q_norm; at.kn = w.k_norm;
+                at.v_raw = a->qkv + w.v_off; at.vct_out = io.vct[li];
+            }
+            if (l.out_gate == PS_GATE_HEAD) { at.gate = a->qkv + w.g_off; at.ld_gate = w.pw; }
+            if (rwkv) at.out_scale = l.mix_scale;
             at.lin = w.lin; at.pool = l.pool; at.n_pool = w.n_pool; at.pool_off = a->pool_off; at.stat_off = a->stat_off;
             if (single) rc = attend_single(at, q, li, a->att, true);
             else rc = attend(at, q, w.pw, w.kd, li, a->att, w.aw);
             if (rc) return rc;
-            if (l.out_gate || l.side_kind) { // the heads' outputs through their gate; the side mixer's recurrence fills the columns behind them
-                const unsigned gate_ctas = cdiv(w.ho, PA_GG_THREADS), side_ctas = l.side_kind ? cdiv(l.side_width, 32) : 0;
-                pa_k_gate_gru<<<dim3(gate_ctas + side_ctas, (unsigned)std::min(bs, 64)), PA_GG_THREADS, 0, st>>>(a->att, w.aw, a->qkv, w.pw, w.ho, l.out_gate ? w.g_off : -1, l.side_kind ? l.mix_scale : 1.0f,
-                                                                                                     (int)gate_ctas, l.side_kind ? l.side_width : 0, w.z_off, w.side_b, l.side_kind ? w.side_b + l.side_width : nullptr,
+            if (rwkv && single && a->opt_fork) PA_CK(cudaStreamWaitEvent(st, a->ev_join, 0));
+            if (l.out_gate == PS_GATE_ELEMENT || l.side_kind == PS_MIXER_MINGRU) { // the heads' outputs through their gate; the side mixer's recurrence fills the columns behind them
+                const unsigned gate_ctas = cdiv(w.ho, PA_GG_THREADS), side_ctas = l.side_kind == PS_MIXER_MINGRU ? cdiv(l.side_width, 32) : 0;
+                pa_k_gate_gru<<<dim3(gate_ctas + side_ctas, (unsigned)std::min(bs, 64)), PA_GG_THREADS, 0, st>>>(a->att, w.aw, a->qkv, w.pw, w.ho, l.out_gate == PS_GATE_ELEMENT ? w.g_off : -1, l.side_kind == PS_MIXER_MINGRU ? l.mix_scale : 1.0f,
+                                                                                                     (int)gate_ctas, l.side_kind == PS_MIXER_MINGRU ? l.side_width : 0, w.z_off, w.side_b, l.side_kind ? w.side_b + l.side_width : nullptr,
                                                                                                      l.side_scale, io.kc[li] + w.state_off, io.pos_dev, bs);
                 PA_LAUNCH();
             }
+        } else if (l.mixer_kind == PS_MIXER_GLA) {
+            PaRec r{};
+            r.q = a->qkv; r.k = a->qkv + w.qd; r.v = a->qkv + 2 * w.qd; r.g = r.v + w.od; r.a1 = r.g + w.od;
+            r.H = H; r.dk = l.qk_dim; r.dv = l.v_dim; r.act = PaAct{0.f, 1.0f / l.decay_tau, 0.f, PA_ACT_ROOT_SIGMOID}; r.o_scale = 1.0f / sqrtf((float)l.qk_dim);
+            r.S = io.kc[li]; r.out = a->att; r.ldo = w.aw;
+            if ((rc = recurrence(w, r, st, pdl))) return rc;
         } else if (l.mixer_kind == PS_MIXER_RETENTION) {
             const int dq = l.qk_dim, dv = l.v_dim;
             const PaRope rope{w.rope_freq, l.rope_dims, 1.0f, 0};
@@ -1360,7 +1650,7 @@ static int forward_t(PsArch *a, const PsArchIO &io, int bs, int pos0, int lm_hea
         if (single) {
             PaMv mv{};
             mv.x = a->att; mv.W = w.wo; mv.N = dim; mv.K = w.od; mv.y = a->ao;
-            if ((rc = dec_mv(mv, 0))) return rc;
+            if ((rc = dec_mv(mv, 0, !rwkv))) return rc; // (behind a join of two streams: an ordinary launch)
         } else if ((rc = linear(a->att, w.od, w.od, w.wo, w.t_o, dim, a->ao, dim))) {
             return rc;
         }
@@ -1382,9 +1672,10 @@ static int forward_t(PsArch *a, const PsArchIO &io, int bs, int pos0, int lm_hea
         }
         // routed experts (+ shared expert)
         const int E = l.n_experts, ff = l.expert_ff, top = l.top_k, sff = l.shared_ff;
-        const PaRoute rt = pa_route_of(l);
+        PaRoute rt = pa_route_of(l);
+        rt.corr = w.corr;
         if (single) {
-            const int n_rt = E + (rt.shared_gate ? 1 : 0); // the router's rows (+ the shared gate's): logits from the unrounded input
+            const int n_rt = rt.E + (rt.shared_gate ? 1 : 0); // the router's rows (+ the shared gate's): logits from the unrounded input
             if (sff > 0) { // the shared expert's gate | up launch carries the seam and the router's rows
                 pa_launch_dep(pdl, pa_k_dec_dense_up<ROUND>, dim3(std::min(cdiv(sff + n_rt, PA_DV_ROWS / 2), up_cap)), dim3(PA_DV_THREADS), 4 * (size_t)dim, st, (const float *)xc, pend_y, pend_w, w_in,
                               xo, groups, d.norm_eps, (const bf16 *)w.wsg, (const bf16 *)w.wsu, a->y, sff, dim, act, (const bf16 *)w.router, n_rt, a->z, 0, a->res_scale);
@@ -1401,11 +1692,11 @@ static int forward_t(PsArch *a, const PsArchIO &io, int bs, int pos0, int lm_hea
                 if ((rc = dec_mv(mv, 4 * (size_t)dim))) return rc;
             }
             pa_k_dec_expert_up<ROUND><<<dim3(std::min(cdiv(ff, PA_DV_ROWS / 2), (unsigned)std::max(1, 4 * a->n_sm / top)), top), PA_DV_THREADS, 4 * (size_t)dim, st>>>(
-                xc, w_in, d.norm_eps, a->z, rt, w.wgate, w.wup, a->y, ff, dim, l.route_on_input, act, a->sel_e, a->sel_w);
+                xc, w_in, d.norm_eps, a->z, rt, w.wgate, w.wup, a->y, ff, dim, l.route_on_input, act, a->sel_e, a->sel_w, l.route_identity ? a->hn : nullptr);
             PA_LAUNCH();
             const int ksd = pick_ksplit(dim, ff);
             pa_k_dec_expert_down<ROUND><<<cdiv(dim, PA_DV_ROWS / ksd), PA_DV_THREADS, 0, st>>>(a->y, a->sel_e, a->sel_w, top, w.wdown, nullptr, nullptr, dim, ff, l.route_on_input, ksd, a->ffo,
-                                                                                               sff > 0 ? a->sh : nullptr, rt.shared_gate ? a->z + E : nullptr);
+                                                                                               sff > 0 ? a->sh : nullptr, rt.shared_gate ? a->z + rt.E : nullptr, E, a->hn);
             PA_LAUNCH();
         } else {
             if ((rc = seam(raw ? nullptr : a->h, w_in))) return rc;
@@ -1414,7 +1705,8 @@ static int forward_t(PsArch *a, const PsArchIO &io, int bs, int pos0, int lm_hea
             pa_k_router<<<bs, 256, 0, st>>>(X, w.router, dim, rt, a->sel_e, a->sel_w, a->sgate, nullptr);
             PA_LAUNCH();
             if ((rc = routed_batch(X, w))) return rc;
-            pa_k_moe_sum<<<dim3(cdiv(dim, 256), bs), 256, 0, st>>>(a->ffo, a->slot, top, sff > 0 ? a->sh : nullptr, rt.shared_gate ? a->sgate : nullptr, dim);
+            pa_k_moe_sum<<<dim3(cdiv(dim, 256), bs), 256, 0, st>>>(a->ffo, a->slot, top, sff > 0 ? a->sh : nullptr, rt.shared_gate ? a->sgate : nullptr, dim, a->sel_e, a->sel_w,
+                                                                     l.route_identity ? X : nullptr, E);
             PA_LAUNCH();
         }
         pend_y = a->ffo; pend_w = l.post_norm ? w.norm_ff_out : nullptr;
@@ -1522,7 +1814,7 @@ static int forward_t(PsArch *a, const PsArchIO &io, int bs, int pos0, int lm_hea
                 }
             } else if (single) {
                 if (l.qk_norm != PS_QKNORM_NONE) { // the scores kernel norms q and the token's key
-                    at.qn = w.q_norm; at.kn = w.k_norm; at.eps = d.norm_eps; at.qt_coef = l.q_temp_coef; at.qt_every = l.q_temp_every; at.k_raw = a->qkv + w.qd; at.kc_out = io.kc[li];
+                    at.head_norm = 1; at.qn = w.q_norm; at.kn = w.k_norm; at.eps = d.norm_eps; at.qt_coef = l.q_temp_coef; at.qt_every = l.q_temp_every; at.k_raw = a->qkv + w.qd; at.kc_out = io.kc[li];
                 }
             } else {
                 pa_k_qkv_post<<<bs, 256, 0, st>>>(a->qkv, w.ldp, H, l.n_kv_heads, l.qk_dim, l.v_dim, l.qk_norm, d.norm_eps, 0, nullptr, nullptr, 0, io.kc[li], io.vct[li], d.n_ctx, io.pos_dev, w.q_norm,
@@ -1576,6 +1868,7 @@ static int forward_t(PsArch *a, const PsArchIO &io, int bs, int pos0, int lm_hea
         if (l.block_kind == PS_BLOCK_SEQUENTIAL || w.gpar) {
             int rc = w.gpar ? par_layer(li) : w.gen2 ? gen_layer(li) : seq_layer(li);
             if (rc) return rc;
+            if (l.token_slot && (rc = token_input(li))) return rc;
             if (a->taps_on) {
                 if ((rc = seam(nullptr, nullptr))) return rc; // the tap shows the layer's whole effect
                 if (!a->taps[(size_t)li]) { rc = aalloc(a, (void **)&a->taps[(size_t)li], 4 * (size_t)dim * B, err); if (rc) return rc; }

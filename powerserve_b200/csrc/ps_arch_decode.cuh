@@ -158,6 +158,13 @@ struct PaMv {
     // rows n >= act_from (> 0) leave through the one-argument activation, `gap` entries further on
     int act_from, gap;
     PaAct act;
+    PaRowMul mul;          // rows leave through the activation `act`, times a table row (act_from is not read then)
+    // rows that read different mixtures of the normed input (seg_n > 0; with groups > 0): rows below seg_end[0] read h, rows from
+    // seg_end[s - 1] to seg_end[s] read h + (h' - h) mu[s - 1] with h' the token before's h: row (pos - 1) & 1 of the ring [2][K], zeros at
+    // position 0; CTA 0 stores h to row pos & 1.  Every CTA takes neighbouring row groups and forms only the mixtures they read.
+    int seg_n, seg_end[6];
+    const float *mu;
+    float *ring;
     int ksplit;            // warps of a CTA that share a row pair, each taking K / ksplit of the columns (1, 2, 4 or 8)
     int prefetch;          // 1: request the first row group into L2 before the dependency wait; 2: also every next group one ahead
 };
@@ -177,7 +184,11 @@ __global__ void __launch_bounds__(PA_DV_THREADS) pa_k_dec_mv(const PaMv a) {
         const int n0 = (grp * pairs + pair) * 2;
         if (a.prefetch && n0 < total) pa_prefetch2(row(n0), row(min(n0 + 1, total - 1)), k_begin, k_end, lane);
     };
-    prefetch(blockIdx.x);
+    // row groups of this CTA: every gridDim.x-th, or (mixtures) a run of neighbours
+    const int per_cta = (groups + (int)gridDim.x - 1) / (int)gridDim.x;
+    const int g_begin = a.seg_n > 0 ? blockIdx.x * per_cta : blockIdx.x, g_end = a.seg_n > 0 ? min(groups, g_begin + per_cta) : groups, g_step = a.seg_n > 0 ? 1 : gridDim.x;
+    auto segment = [&](int n) { int sg = 0; while (sg < a.seg_n - 1 && n >= a.seg_end[sg]) sg++; return sg; };
+    prefetch(g_begin);
     // launched with programmatic stream serialisation: everything above touches weights only and overlaps the kernel before
     ps_grid_dep_launch();
     ps_grid_dep_wait();
@@ -191,19 +202,39 @@ __global__ void __launch_bounds__(PA_DV_THREADS) pa_k_dec_mv(const PaMv a) {
         }
         if (a.h_out && blockIdx.x == 0)
             for (int c = threadIdx.x; c < sd; c += PA_DV_THREADS) a.h_out[c] = pa_hs[c];
+        if (a.seg_n > 0) {
+            const int p = a.pos[0], s_lo = segment(g_begin * 2 * pairs), s_hi = segment(min(g_end * 2 * pairs, total) - 1);
+            const float *prev = a.ring + (int64_t)((p - 1) & 1) * a.K;
+            float *keep = a.ring + (int64_t)(p & 1) * a.K;
+            for (int c = threadIdx.x; c < a.K; c += PA_DV_THREADS) {
+                const float h = pa_hs[c], d = (p > 0 ? prev[c] : 0.f) - h;
+                if (blockIdx.x == 0) keep[c] = h;
+                for (int sg = max(s_lo, 1); sg <= s_hi; sg++) pa_hs[sg * a.K + c] = fmaf(d, a.mu[(int64_t)(sg - 1) * a.K + c], h);
+            }
+            __syncthreads();
+        }
         xin = pa_hs;
     } else if (a.norm_w) {
         pa_norm_to_smem(pa_hs, a.x, a.norm_w, a.K, a.eps);
         xin = pa_hs;
     }
-    for (int grp = blockIdx.x; grp < groups; grp += gridDim.x) {
-        if (a.prefetch > 1 && grp + (int)gridDim.x < groups) prefetch(grp + gridDim.x); // opt-in: the next group's rows travel to L2 meanwhile
+    for (int grp = g_begin; grp < g_end; grp += g_step) {
+        if (a.prefetch > 1 && grp + g_step < g_end) prefetch(grp + g_step); // opt-in: the next group's rows travel to L2 meanwhile
         const int n0 = (grp * pairs + pair) * 2, n1 = min(n0 + 1, total - 1);
         const bool live = n0 < total;
         float s0 = 0.f, s1 = 0.f;
         if (live) {
             const bf16 *w0 = row(n0), *w1 = row(n1);
-            if (a.grp_rows > 0 && n0 / a.grp_rows == n1 / a.grp_rows) {
+            if (a.seg_n > 0) {
+                const int e0 = segment(n0), e1 = segment(n1);
+                if (e0 == e1) {
+                    pa_dot2<ROUND>(w0, w1, xin + e0 * a.K, a.K, 1.0f, lane, s0, s1, k_begin, k_end);
+                } else {
+                    float t;
+                    pa_dot2<ROUND>(w0, w0, xin + e0 * a.K, a.K, 1.0f, lane, s0, t, k_begin, k_end);
+                    pa_dot2<ROUND>(w1, w1, xin + e1 * a.K, a.K, 1.0f, lane, s1, t, k_begin, k_end);
+                }
+            } else if (a.grp_rows > 0 && n0 / a.grp_rows == n1 / a.grp_rows) {
                 pa_dot2<ROUND>(w0, w1, xin + (n0 / a.grp_rows) * a.x_gs, a.K, 1.0f, lane, s0, s1, k_begin, k_end);
             } else if (a.grp_rows > 0) { // every row reads its own head's slice of x
                 float t;
@@ -242,6 +273,8 @@ __global__ void __launch_bounds__(PA_DV_THREADS) pa_k_dec_mv(const PaMv a) {
                     } else {
                         a.vct[(int64_t)(n - a.qd - a.kd) * a.n_ctx + p] = v;
                     }
+                } else if (a.mul.table) {
+                    a.y[n] = pa_act1(v, a.act) * pa_ld(a.mul.table + (int64_t)a.mul.tok[0] * a.mul.ld + n);
                 } else if (a.act_from > 0 && n >= a.act_from) {
                     a.y[n + a.gap] = pa_act1(v, a.act);
                 } else if (a.residual) {
@@ -272,7 +305,8 @@ __global__ void __launch_bounds__(256) pa_k_dec_scores(PaAttn at, const float *_
     float *ks = sm;                        // [PA_DS_KEYS][kds]
     float *qs = ks + PA_DS_KEYS * kds;     // [H][dq]
     float *sa = qs + H * dq;               // [H][PA_DS_KEYS + 1]
-    float *Ts = sa + H * (PA_DS_KEYS + 1); // [H][H]
+    float *Ts = sa + H * (PA_DS_KEYS + 1); // [H][H], or cos / sin of the rotations
+    float2 *cs = reinterpret_cast<float2 *>(sm + (((Ts - sm) + 1) & ~1));
     const int tid = threadIdx.x;
     if (at.mix) for (int t = tid; t < H * H; t += 256) Ts[t] = at.mix[t]; // a weight: fetched before the dependency wait
     ps_grid_dep_launch();
@@ -307,6 +341,19 @@ __global__ void __launch_bounds__(256) pa_k_dec_scores(PaAttn at, const float *_
     if (at.k_raw) { // a warp per head: norm of q (times the position's temperature), and of the token's key on its way into the cache
         const int lane = tid & 31;
         const float qt = pa_q_temp(at.qt_coef, at.qt_every, pos);
+        const int rh = at.rope.dims >> 1, vh = at.vrope.dims >> 1;
+        if (rh > 0) {
+            for (int i = tid; i < rh; i += 256) cs[i] = pa_rope_cs(at.rope, pos, i);
+            __syncthreads();
+        }
+        if (own && vh > 0) // the token's value, rotated, into its V^T column
+            for (int e = tid; e < G * vh; e += 256) {
+                const int g = e / vh, m = e % vh;
+                const float va = at.v_raw[g * at.dv + m], vb = at.v_raw[g * at.dv + m + vh];
+                const float2 t = pa_rope_cs(at.vrope, pos, m);
+                at.vct_out[(int64_t)(g * at.dv + m) * at.n_ctx + pos] = va * t.x - vb * t.y;
+                at.vct_out[(int64_t)(g * at.dv + m + vh) * at.n_ctx + pos] = vb * t.x + va * t.y;
+            }
         for (int hh = tid >> 5; hh < H + (own ? G : 0); hh += 8) {
             const bool is_q = hh < H;
             const float *src = is_q ? q + hh * dq : at.k_raw + (hh - H) * dq, *w = is_q ? at.qn : at.kn;
@@ -320,11 +367,21 @@ __global__ void __launch_bounds__(256) pa_k_dec_scores(PaAttn at, const float *_
             }
 #pragma unroll
             for (int o = 16; o; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
-            const float inv = 1.0f / sqrtf(s / (float)dq + at.eps) * (is_q ? qt : 1.0f);
-            for (int c = lane; c < dq; c += 32) { // (a lane's own entries)
+            const float inv = (at.head_norm ? 1.0f / sqrtf(s / (float)dq + at.eps) : 1.0f) * (is_q ? qt : 1.0f);
+            float *kout = is_q ? nullptr : at.kc_out + (int64_t)pos * kd + (hh - H) * dq;
+            if (rh > 0) {
+                __syncwarp();
+                for (int i = lane; i < rh; i += 32) {
+                    const float va = dst[i] * inv, vb = dst[i + rh] * inv, ra = va * cs[i].x - vb * cs[i].y, rb = vb * cs[i].x + va * cs[i].y;
+                    dst[i] = ra;
+                    dst[i + rh] = rb;
+                    if (kout) { kout[i] = ra; kout[i + rh] = rb; }
+                }
+            }
+            for (int c = 2 * rh + lane; c < dq; c += 32) { // (without a rotation: a lane's own entries)
                 const float v = dst[c] * inv;
                 dst[c] = v;
-                if (!is_q) at.kc_out[(int64_t)pos * kd + (hh - H) * dq + c] = v;
+                if (kout) kout[c] = v;
             }
         }
     } else {
@@ -433,6 +490,13 @@ __global__ void __launch_bounds__(256) pa_k_dec_pv(PaAttn at, const float *__res
     for (int t = tid; t < 8 * rep; t += 256) acc[t] = 0.f;
     const int dim_l = warp % PA_DP_DIMS, part = warp / PA_DP_DIMS, n_part = 8 / PA_DP_DIMS;
     const int c0 = blockIdx.x * PA_DP_DIMS;
+    // value dim of the CTA's cc-th row (dv or more: outside); with rotated values the CTA takes two pairs (m, m + dv / 2)
+    const int vh = at.vrope.dims >> 1;
+    auto col = [&](int cc) {
+        if (vh == 0) return c0 + cc;
+        const int m = c0 / 2 + (cc & 1);
+        return m < vh ? m + (cc >= 2 ? vh : 0) : dv;
+    };
     int it = 0;
     // two stretches of keys: the tokens in sight (V^T rows of n_ctx columns), then the pooled blocks (rows of n_pool columns behind them)
     for (int seg = 0; seg < (nv > 0 ? 2 : 1); seg++) {
@@ -443,15 +507,17 @@ __global__ void __launch_bounds__(256) pa_k_dec_pv(PaAttn at, const float *__res
         __syncthreads(); // the previous chunk's buffers are free
         if (bulk) {
             if (tid == 0) {
-                const int rows = min(PA_DP_DIMS, dv - c0);
+                int rows = 0;
+                for (int cc = 0; cc < PA_DP_DIMS; cc++) rows += col(cc) < dv;
                 asm volatile("fence.proxy.async.shared::cta;" ::: "memory"); // the rows were read through the generic proxy
                 ps_mbar_expect_tx(&bar, (uint32_t)(rows * nj4 * 4));
-                for (int cc = 0; cc < rows; cc++) ps_bulk_g2s(vs + cc * chunk, vbase + (int64_t)(g * dv + c0 + cc) * ldv + j0, (uint32_t)(nj4 * 4), &bar);
+                for (int cc = 0; cc < PA_DP_DIMS; cc++)
+                    if (col(cc) < dv) ps_bulk_g2s(vs + cc * chunk, vbase + (int64_t)(g * dv + col(cc)) * ldv + j0, (uint32_t)(nj4 * 4), &bar);
             }
         } else {
             for (int t = tid; t < PA_DP_DIMS * nj4; t += 256) {
                 const int cc = t / nj4, jj = t % nj4;
-                vs[cc * chunk + jj] = (c0 + cc < dv && jj < nj) ? vbase[(int64_t)(g * dv + c0 + cc) * ldv + j0 + jj] : 0.f;
+                vs[cc * chunk + jj] = (col(cc) < dv && jj < nj) ? vbase[(int64_t)(g * dv + col(cc)) * ldv + j0 + jj] : 0.f;
             }
         }
         for (int t = tid; t < rep * nj4; t += 256) {
@@ -460,7 +526,7 @@ __global__ void __launch_bounds__(256) pa_k_dec_pv(PaAttn at, const float *__res
         }
         __syncthreads();
         if (bulk && !ps_tc_wait(&bar, it & 1)) { if (tid == 0) err[0] = 6; return; }
-        if (c0 + dim_l < dv) {
+        if (col(dim_l) < dv) {
             const float4 *v4 = reinterpret_cast<const float4 *>(vs + dim_l * chunk);
             for (int r = 0; r < rep; r++) {
                 const float4 *p4 = reinterpret_cast<const float4 *>(ps + r * chunk);
@@ -478,12 +544,21 @@ __global__ void __launch_bounds__(256) pa_k_dec_pv(PaAttn at, const float *__res
     }
     __syncthreads();
     for (int t = tid; t < PA_DP_DIMS * rep; t += 256) {
-        const int cc = t / rep, r = t % rep;
-        if (c0 + cc >= dv) continue;
-        float s = 0.f;
-        for (int pp = 0; pp < n_part; pp++) s += acc[(pp * PA_DP_DIMS + cc) * rep + r];
-        s *= inv[r];
-        att[(h0 + r) * dv + c0 + cc] = at.gate ? s * pa_sigmoid(at.gate[h0 + r]) : s;
+        const int cc = t / rep, r = t % rep, c = col(cc);
+        if (c >= dv) continue;
+        auto sum = [&](int k) {
+            float s = 0.f;
+            for (int pp = 0; pp < n_part; pp++) s += acc[(pp * PA_DP_DIMS + k) * rep + r];
+            return s * inv[r];
+        };
+        float s = sum(cc);
+        if (vh > 0) { // turned back by the query's position
+            const float2 t2 = pa_rope_cs(at.vrope, n - 1, c0 / 2 + (cc & 1));
+            const float o = sum(cc ^ 2);
+            s = cc < 2 ? s * t2.x + o * t2.y : s * t2.x - o * t2.y;
+        }
+        if (at.gate) s *= pa_sigmoid(at.gate[h0 + r]);
+        att[(h0 + r) * dv + c] = at.out_scale != 0.f ? s * at.out_scale : s;
     }
 }
 
@@ -554,14 +629,15 @@ template <bool ROUND>
 __global__ void __launch_bounds__(PA_DV_THREADS) pa_k_dec_expert_up(const float *__restrict__ x, const float *__restrict__ norm_w, float eps, const float *__restrict__ z, PaRoute rt,
                                                                     const bf16 *__restrict__ Wg, const bf16 *__restrict__ Wu, float *__restrict__ y,
                                                                     int ff, int dim, int on_input, PaAct act, int *__restrict__ sel_e,
-                                                                    float *__restrict__ sel_w) {
+                                                                    float *__restrict__ sel_w, float *__restrict__ h_out = nullptr) {
     extern __shared__ __align__(16) float pa_hs[];
     __shared__ float sc[PA_MAX_EXPERTS];
     __shared__ int se[PA_MAX_EXPERTS];
     __shared__ float sw[PA_MAX_EXPERTS];
-    if (rt.act == PS_ROUTER_TOPK_SOFTMAX) {
+    if (rt.act == PS_ROUTER_TOPK_SOFTMAX || (rt.act == PS_ROUTER_SOFTMAX && rt.groups <= 1)) {
         if (threadIdx.x < 32) {
-            pa_route_topk_warp(z, rt.E, rt.top, se, sw, threadIdx.x);
+            if (rt.act == PS_ROUTER_SOFTMAX) pa_route_softmax_warp(z, rt, se, sw, threadIdx.x);
+            else pa_route_topk_warp(z, rt.E, rt.top, se, sw, threadIdx.x);
             __syncwarp();
             if (blockIdx.x == 0 && blockIdx.y == 0)
                 for (int r = threadIdx.x; r < rt.top; r += 32) { sel_e[r] = se[r]; sel_w[r] = sw[r]; }
@@ -578,6 +654,9 @@ __global__ void __launch_bounds__(PA_DV_THREADS) pa_k_dec_expert_up(const float 
         __syncthreads();
     }
     const int r = blockIdx.y, e = se[r], lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    if (h_out && blockIdx.x == 0 && blockIdx.y == 0) // the normed input, for the choices that stand for it
+        for (int c = threadIdx.x; c < dim; c += blockDim.x) h_out[c] = pa_hs[c];
+    if (e >= rt.E - rt.identity) return;
     const float w = on_input ? sw[r] : 1.0f;
     // a warp owns one ff row at a time: its gate row and its up row are the pair; the CTAs walk the row groups with the grid's stride
     const int rows = PA_DV_ROWS / 2;
@@ -651,7 +730,7 @@ template <bool ROUND>
 __global__ void __launch_bounds__(PA_DV_THREADS) pa_k_dec_expert_down(const float *__restrict__ y, const int *__restrict__ sel_e, const float *__restrict__ sel_w, int top,
                                                                       const bf16 *__restrict__ Wd, const float *__restrict__ ao, float *__restrict__ x, int dim, int ff,
                                                                       int on_input, int ksplit, float *__restrict__ dst = nullptr, const float *__restrict__ extra = nullptr,
-                                                                      const float *__restrict__ extra_logit = nullptr) {
+                                                                      const float *__restrict__ extra_logit = nullptr, int E = 1 << 30, const float *__restrict__ h = nullptr) {
     __shared__ float part_s[8][2];
     ps_grid_dep_launch(); // the next kernel (the next layer's q|k|v rows, or the head) may start fetching its weights
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
@@ -663,10 +742,15 @@ __global__ void __launch_bounds__(PA_DV_THREADS) pa_k_dec_expert_down(const floa
     if (live) {
         for (int r = 0; r < top; r++) {
             const int e = sel_e[r];
+            if (e >= E) continue;
             pa_prefetch2(Wd + ((int64_t)e * dim + n0) * ff, Wd + ((int64_t)e * dim + n1) * ff, k_begin, k_end, lane);
         }
         for (int r = 0; r < top; r++) {
             const int e = sel_e[r];
+            if (e >= E) { // the input itself (one of the warps that share the rows adds it)
+                if (slice == 0) { t0 = fmaf(sel_w[r], h[n0], t0); t1 = fmaf(sel_w[r], h[n1], t1); }
+                continue;
+            }
             float s0, s1;
             pa_dot2<ROUND>(Wd + ((int64_t)e * dim + n0) * ff, Wd + ((int64_t)e * dim + n1) * ff, y + (int64_t)r * ff, ff, 1.0f, lane, s0, s1, k_begin, k_end);
             const float w = on_input ? 1.0f : sel_w[r];

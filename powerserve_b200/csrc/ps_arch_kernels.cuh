@@ -22,10 +22,35 @@
 //                             PS_ACT_XIELU      one argument only: alpha z^2 + z / 2 above zero, shift (exp(z) - 1 - z) + z / 2 below
 //                                               (alpha = softplus(p), shift = 1/2 + softplus(q) of the layer's two numbers)
 //                             PS_ACT_RELU2      one argument only: max(z, 0)^2
+//                             PS_ACT_RELU       max(g, 0) times u, or max(z, 0)
+// and, of one argument, what a recurrence reads: PA_ACT_TANH  tanh(z);  PA_ACT_ROOT_SIGMOID  sigmoid(z)^alpha;  PA_ACT_EXP_EXP  exp(-exp(z))
+enum { PA_ACT_TANH = 100, PA_ACT_ROOT_SIGMOID = 101, PA_ACT_EXP_EXP = 102 };
 struct PaAct {
     float limit, alpha, shift;
     int kind;
 };
+
+// the outputs of a product times a row of a bfloat16 table: row tok[m] of stride ld (table null: nothing)
+struct PaRowMul {
+    const bf16 *table;
+    int64_t ld;
+    const int32_t *tok;
+};
+
+// rotation of the first `dims` entries of a vector (pairs (i, i + dims / 2)) by the angles pos * freq[i], cos / sin times mscale.
+// The product and its reduction to [-pi, pi] are formed in double (three operations), so that the float32 argument of cosf / sinf is
+// good to 2e-7 at any position; a float32 product alone is off by pos * 6e-8.
+struct PaRope {
+    const double *freq; // [dims / 2]
+    int dims;
+    float mscale;
+    int interleaved;    // pairs (2i, 2i + 1) instead of (i, i + dims / 2)
+};
+__device__ __forceinline__ float2 pa_rope_cs(const PaRope &r, int pos, int i) {
+    const double turns = (double)pos * r.freq[i];
+    const float ang = (float)fma(-rint(turns * 0.15915494309189535), 6.283185307179586, turns);
+    return make_float2(cosf(ang) * r.mscale, sinf(ang) * r.mscale);
+}
 
 struct PaAttn {
     int H, G, dq, dv;
@@ -41,6 +66,7 @@ struct PaAttn {
     int window;             // > 0: a query sees the keys at distances 0 .. window - 1 only
     int chunk;              // > 0: a query sees the keys of its own chunk of positions only (chunks counted from position 0)
     const float *lin;       // [H] or null: score -= lin[h] * distance
+    float softcap;          // > 0: score <- softcap tanh(score / softcap)
     // pool > 0 (with a window): one mean key / value per block of `pool` positions that lies wholly before the window.  The means sit
     // behind the token rows of the cache buffers (K: row n_ctx + b; V^T: [G * dv][n_pool] behind the token part); a query's pooled
     // scores sit at pool_off + b of its score row, the single-token step's block statistics from stat_off on
@@ -55,6 +81,12 @@ struct PaAttn {
     float eps, qt_coef, qt_every;
     const float *k_raw;
     float *kc_out;
+    int head_norm;          // (with k_raw) q and k heads are normed; 0: rotated only
+    PaRope rope;            // q / k rotation after the norm (dims 0: none); the single-token scores kernel applies it with the norms
+    PaRope vrope;           // dims = dv: the cached values are rotated by their positions and every head's output is turned back by the query's
+    const float *v_raw;     // (with k_raw and vrope) the token's raw value row; the single-token scores kernel stores the rotated one to the
+    float *vct_out;         // V^T column pos
+    float out_scale;        // factor on the heads' outputs (0: 1)
     const float *gate;      // one logit per query row and head (row stride ld_gate) or null: the head's output times sigmoid(logit)
     int ld_gate;
     float *pm, *pl;         // single-token step: per head and block of keys, max and sum of exponentials of the mixed scores
@@ -76,6 +108,7 @@ __device__ __forceinline__ void pa_dot2(const bf16 *__restrict__ w0, const bf16 
 // ---------------------------------------------------------------------------------------------------------------- activations
 __device__ __forceinline__ float pa_sigmoid(float v) { return 1.0f / (1.0f + expf(-v)); }
 __device__ __forceinline__ float pa_expert_act(float g, float u, PaAct act) {
+    if (act.kind == PS_ACT_RELU) return fmaxf(g, 0.f) * u;
     if (act.kind == PS_ACT_GELU_TANH) // 0.5 g (1 + tanh(sqrt(2 / pi) (g + 0.044715 g^3))) * u
         return 0.5f * g * (1.0f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g))) * u;
     g = fminf(g, act.limit);
@@ -86,6 +119,10 @@ __device__ __forceinline__ float pa_expert_act(float g, float u, PaAct act) {
 // the one-argument forms (a feed-forward without a gate)
 __device__ __forceinline__ float pa_act1(float z, PaAct act) {
     if (act.kind == PS_ACT_RELU2) return z > 0.f ? z * z : 0.f;
+    if (act.kind == PS_ACT_RELU) return fmaxf(z, 0.f);
+    if (act.kind == PA_ACT_TANH) return tanhf(z);
+    if (act.kind == PA_ACT_ROOT_SIGMOID) return expf(-act.alpha * (fmaxf(-z, 0.f) + log1pf(expf(-fabsf(z))))); // exp(-alpha softplus(-z))
+    if (act.kind == PA_ACT_EXP_EXP) return expf(-expf(z));
     if (act.kind == PS_ACT_XIELU) return z > 0.f ? fmaf(act.alpha * z, z, 0.5f * z) : fmaf(act.shift, expm1f(z) - z, 0.5f * z);
     if (act.kind == PS_ACT_GELU_TANH) return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
     z = fminf(z, act.limit);
@@ -302,24 +339,47 @@ __device__ __forceinline__ float pa_q_temp(float coef, float every, int p) {
 }
 
 // After the q|k|v projection of a batch, one CTA per token: unit-RMS q heads (in place) and k heads (qk_norm; times the weights qn / kn
-// and, for q, the position's temperature), the value rows blended with the source layer's (v_mix), K row -> kc[pos][:], V row transposed -> vct[:][pos].
+// and, for q, the position's temperature), both rotated (rope, its angles formed once per token), the values rotated (vrope), the value rows blended with the source layer's (v_mix), K row -> kc[pos][:], V row transposed -> vct[:][pos].
 __global__ void __launch_bounds__(256) pa_k_qkv_post(float *__restrict__ qkv, int ld, int H, int G, int dq, int dv, int qk_norm, float eps, int v_mix,
                                                      const float *__restrict__ lambda, float *__restrict__ v_src, int ld_src, float *__restrict__ kc,
                                                      float *__restrict__ vct, int n_ctx, const int32_t *__restrict__ pos, const float *__restrict__ qn, const float *__restrict__ kn,
-                                                     float qt_coef, float qt_every) {
+                                                     float qt_coef, float qt_every, PaRope rope = PaRope{}, PaRope vrope = PaRope{}) {
+    extern __shared__ __align__(16) float2 pa_cs[]; // cos / sin of the rotations: rope.dims / 2 pairs, then vrope.dims / 2
     const int t = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, p = pos[t];
     float *row = qkv + (int64_t)t * ld;
     const float qt = pa_q_temp(qt_coef, qt_every, p);
-    const int qd = H * dq, kd = G * dq, vd = G * dv;
+    const int qd = H * dq, kd = G * dq, vd = G * dv, rh = rope.dims >> 1, vh = vrope.dims >> 1;
+    if (rh + vh > 0) {
+        for (int i = threadIdx.x; i < rh + vh; i += 256) pa_cs[i] = i < rh ? pa_rope_cs(rope, p, i) : pa_rope_cs(vrope, p, i - rh);
+        __syncthreads();
+    }
     for (int hh = warp; hh < H + G; hh += 8) { // q heads, then k heads
         float *v = row + hh * dq;
         const float inv = qk_norm ? pa_warp_inv_rms(v, dq, eps, lane) : 1.0f;
-        if (hh < H) {
-            if (qk_norm) for (int c = lane; c < dq; c += 32) v[c] *= inv * (qn ? qn[c] : 1.0f) * qt;
-        } else {
-            float *dst = kc + (int64_t)p * kd + (hh - H) * dq;
-            for (int c = lane; c < dq; c += 32) dst[c] = v[c] * inv * (kn ? kn[c] : 1.0f);
+        const float *w = hh < H ? qn : kn;
+        float *dst = hh < H ? v : kc + (int64_t)p * kd + (hh - H) * dq;
+        const float f = hh < H ? inv * qt : inv;
+        for (int i = lane; i < rh; i += 32) { // the rotated pairs (i, i + rh)
+            const float a = v[i] * f * (w ? w[i] : 1.0f), b = v[i + rh] * f * (w ? w[i + rh] : 1.0f);
+            const float2 cs = pa_cs[i];
+            dst[i] = a * cs.x - b * cs.y;
+            dst[i + rh] = b * cs.x + a * cs.y;
         }
+        if (hh < H) {
+            if (qk_norm) for (int c = 2 * rh + lane; c < dq; c += 32) v[c] *= f * (w ? w[c] : 1.0f);
+        } else {
+            for (int c = 2 * rh + lane; c < dq; c += 32) dst[c] = v[c] * f * (w ? w[c] : 1.0f);
+        }
+    }
+    if (vh > 0) {
+        for (int e = threadIdx.x; e < G * vh; e += 256) {
+            const int g = e / vh, m = e % vh;
+            const float a = row[qd + kd + g * dv + m], b = row[qd + kd + g * dv + m + vh];
+            const float2 cs = pa_cs[rh + m];
+            vct[(int64_t)(g * dv + m) * n_ctx + p] = a * cs.x - b * cs.y;
+            vct[(int64_t)(g * dv + m + vh) * n_ctx + p] = b * cs.x + a * cs.y;
+        }
+        return;
     }
     const float lam = v_mix == PS_VMIX_BLEND ? lambda[0] : 0.f;
     for (int c = threadIdx.x; c < vd; c += 256) {
@@ -330,22 +390,12 @@ __global__ void __launch_bounds__(256) pa_k_qkv_post(float *__restrict__ qkv, in
     }
 }
 
-// rotation of the first `dims` entries of a vector (pairs (i, i + dims / 2)) by the angles pos * freq[i], cos / sin times mscale.
-// The product and its reduction to [-pi, pi] are formed in double (three operations), so that the float32 argument of cosf / sinf is
-// good to 2e-7 at any position; a float32 product alone is off by pos * 6e-8.
-struct PaRope {
-    const double *freq; // [dims / 2]
-    int dims;
-    float mscale;
-    int interleaved;    // pairs (2i, 2i + 1) instead of (i, i + dims / 2)
-};
 __device__ __forceinline__ void pa_rope_store(const PaRope &r, const float *src, float *dst, int n, int pos, int c) {
     const int half = r.dims >> 1;
     if (c >= r.dims) { if (c < n) dst[c] = src[c]; return; }
     const int i = r.interleaved ? c >> 1 : c < half ? c : c - half;
-    const double turns = (double)pos * r.freq[i];
-    const float ang = (float)fma(-rint(turns * 0.15915494309189535), 6.283185307179586, turns);
-    const float cs = cosf(ang) * r.mscale, sn = sinf(ang) * r.mscale;
+    const float2 t = pa_rope_cs(r, pos, i);
+    const float cs = t.x, sn = t.y;
     if (r.interleaved) dst[c] = (c & 1) == 0 ? src[c] * cs - src[c + 1] * sn : src[c] * cs + src[c - 1] * sn;
     else dst[c] = c < half ? src[c] * cs - src[c + half] * sn : src[c] * cs + src[c - half] * sn;
 }
@@ -389,10 +439,11 @@ __global__ void __launch_bounds__(256) pa_k_rope_q(const float *__restrict__ q, 
 // ---------------------------------------------------------------------------------------------------------------- dense
 // C[m][n] = sum_k A[m][k] W[n][k] + bias[n].  blockIdx.z walks groups (per-head products): group z reads the columns of A from
 // z * a_gs on, the matrix z of N x K weights, and writes the columns of C from z * c_gs on.  Rows n >= act_from leave through the
-// one-argument activation, `gap` columns further on.
+// one-argument activation, `gap` columns further on; mul multiplies the outputs by a table row per token.
 template <bool ROUND>
 __global__ void __launch_bounds__(256) pa_k_linear(const float *__restrict__ A, int lda, const bf16 *__restrict__ W, const float *__restrict__ bias, float *__restrict__ C, int ldc,
-                                                   int M, int N, int K, int a_gs = 0, int c_gs = 0, int act_from = 1 << 30, int gap = 0, PaAct act = PaAct{}) {
+                                                   int M, int N, int K, int a_gs = 0, int c_gs = 0, int act_from = 1 << 30, int gap = 0, PaAct act = PaAct{},
+                                                   PaRowMul mul = PaRowMul{}) {
     PA_TILE_SMEM(1);
     const int tid = threadIdx.x, lr = tid >> 2, tx = tid & 15, ty = tid >> 4;
     const int m0 = blockIdx.y * PA_TM, n0 = blockIdx.x * PA_TN;
@@ -411,9 +462,10 @@ __global__ void __launch_bounds__(256) pa_k_linear(const float *__restrict__ A, 
         for (int j = 0; j < 4; j++) {
             const int n = n0 + tx * 4 + j;
             if (n >= N) continue;
-            const float v = acc[0][i][j] + (bias ? bias[n] : 0.f);
-            if (n < act_from) C[(int64_t)m * ldc + n] = v;
-            else C[(int64_t)m * ldc + n + gap] = pa_act1(v, act);
+            float v = acc[0][i][j] + (bias ? bias[n] : 0.f);
+            if (n >= act_from) v = pa_act1(v, act);
+            if (mul.table) v *= pa_ld(mul.table + (int64_t)mul.tok[m] * mul.ld + n);
+            C[(int64_t)m * ldc + (n < act_from ? n : n + gap)] = v;
         }
     }
 }
@@ -421,12 +473,14 @@ __global__ void __launch_bounds__(256) pa_k_linear(const float *__restrict__ A, 
 // ---------------------------------------------------------------------------------------------------------------- router
 // how a router turns its logits into chosen experts and weights
 struct PaRoute {
-    int E, top;
+    int E, top;        // router outputs; the last `identity` of them stand for the input itself, the others are experts
     int act;           // PS_ROUTER_SIGMOID: every logit through a sigmoid; PS_ROUTER_SOFTMAX: soft-max over all experts;
                        // PS_ROUTER_TOPK_SOFTMAX: the largest logits, soft-max over those alone (pa_route_topk_warp)
     int groups, keep;  // groups > 1: equal groups of neighbouring experts, a group is worth its best score, the `keep` best groups stay
     int renorm;        // the chosen scores are divided by their sum + eps
     float eps;
+    const float *corr; // [E] or null (soft-max scores without groups): added to the scores for the choice, not for the weights
+    int identity;
     int shared_gate;   // the router matrix has one more row: the logit of the shared expert's gate
 };
 // one thread: scores from the logits z, group limit, the top largest (ties: the lower expert) -> se / sw; sc is scratch of E entries,
@@ -475,6 +529,44 @@ __device__ __forceinline__ void pa_route_serial(const float *__restrict__ z, con
         for (int n = 0; n < r.top; n++) sw[n] /= sum + r.eps;
 }
 
+// one warp: soft-max over all E logits, the `top` largest scores (+ corr) choose (ties: the lower expert), weights = the scores themselves,
+// divided by their sum + eps with renorm; se / sw are in shared memory
+__device__ __forceinline__ void pa_route_softmax_warp(const float *__restrict__ z, const PaRoute &r, int *se, float *sw, int lane) {
+    float s[PA_MAX_EXPERTS / 32], v[PA_MAX_EXPERTS / 32], mx = -INFINITY, sum = 0.f;
+    unsigned taken = 0;
+#pragma unroll
+    for (int i = 0; i < PA_MAX_EXPERTS / 32; i++) { s[i] = lane + 32 * i < r.E ? z[lane + 32 * i] : -INFINITY; mx = fmaxf(mx, s[i]); }
+#pragma unroll
+    for (int o = 16; o; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+#pragma unroll
+    for (int i = 0; i < PA_MAX_EXPERTS / 32; i++) { s[i] = lane + 32 * i < r.E ? expf(s[i] - mx) : 0.f; sum += s[i]; }
+#pragma unroll
+    for (int o = 16; o; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
+    const float inv = 1.0f / sum;
+#pragma unroll
+    for (int i = 0; i < PA_MAX_EXPERTS / 32; i++) { s[i] *= inv; v[i] = s[i] + (r.corr && lane + 32 * i < r.E ? r.corr[lane + 32 * i] : 0.f); }
+    float chosen = 0.f;
+    for (int n = 0; n < r.top; n++) {
+        int be = -1;
+        float bv = 0.f, bs = 0.f;
+#pragma unroll
+        for (int i = 0; i < PA_MAX_EXPERTS / 32; i++)
+            if (lane + 32 * i < r.E && !((taken >> i) & 1) && (be < 0 || v[i] > bv)) { be = lane + 32 * i; bv = v[i]; bs = s[i]; }
+#pragma unroll
+        for (int o = 16; o; o >>= 1) {
+            const int oe = __shfl_xor_sync(0xffffffffu, be, o);
+            const float ov = __shfl_xor_sync(0xffffffffu, bv, o), os = __shfl_xor_sync(0xffffffffu, bs, o);
+            if (oe >= 0 && (be < 0 || ov > bv || (ov == bv && oe < be))) { be = oe; bv = ov; bs = os; }
+        }
+        if ((be & 31) == lane) taken |= 1u << (be >> 5);
+        chosen += bs;
+        if (lane == 0) { se[n] = be; sw[n] = bs; }
+    }
+    __syncwarp();
+    if (r.renorm)
+        for (int n = lane; n < r.top; n += 32) sw[n] /= chosen + r.eps;
+}
+
 // one warp: the `top` largest of E logits (ties: the lower expert), weights = soft-max over the chosen; se / sw are in shared memory
 __device__ __forceinline__ void pa_route_topk_warp(const float *__restrict__ z, int E, int top, int *se, float *sw, int lane) {
     float v[PA_MAX_EXPERTS / 32], z0 = 0.f, sum = 0.f;
@@ -519,9 +611,10 @@ __global__ void __launch_bounds__(256) pa_k_router(const float *__restrict__ h, 
         if (lane == 0) { zs[e] = s0 + (bias && e < r.E ? bias[e] : 0.f); zs[e1] = s1 + (bias && e1 < r.E ? bias[e1] : 0.f); }
     }
     __syncthreads();
-    if (r.act == PS_ROUTER_TOPK_SOFTMAX) {
+    if (r.act == PS_ROUTER_TOPK_SOFTMAX || (r.act == PS_ROUTER_SOFTMAX && r.groups <= 1)) {
         if (warp == 0) {
-            pa_route_topk_warp(zs, r.E, r.top, se, sw, lane);
+            if (r.act == PS_ROUTER_SOFTMAX) pa_route_softmax_warp(zs, r, se, sw, lane);
+            else pa_route_topk_warp(zs, r.E, r.top, se, sw, lane);
             __syncwarp();
             for (int n = lane; n < r.top; n += 32) { sel_e[t * r.top + n] = se[n]; sel_w[t * r.top + n] = sw[n]; }
             if (lane == 0 && r.shared_gate) sgate[t] = 1.0f / (1.0f + expf(-zs[r.E]));
@@ -542,7 +635,8 @@ __global__ void __launch_bounds__(256) pa_k_dispatch(const int *__restrict__ sel
     __shared__ int cnt[PA_MAX_EXPERTS], off[PA_MAX_EXPERTS], fill[PA_MAX_EXPERTS];
     for (int e = threadIdx.x; e < E; e += 256) { cnt[e] = 0; fill[e] = 0; }
     __syncthreads();
-    for (int i = threadIdx.x; i < n; i += 256) atomicAdd(&cnt[sel_e[i]], 1);
+    for (int i = threadIdx.x; i < n; i += 256)
+        if (sel_e[i] < E) atomicAdd(&cnt[sel_e[i]], 1); // (a choice that stands for the input itself has no expert rows)
     __syncthreads();
     if (threadIdx.x == 0) {
         int o = 0, nt = 0;
@@ -556,6 +650,7 @@ __global__ void __launch_bounds__(256) pa_k_dispatch(const int *__restrict__ sel
     __syncthreads();
     for (int i = threadIdx.x; i < n; i += 256) {
         const int e = sel_e[i];
+        if (e >= E) continue;
         const int p = off[e] + atomicAdd(&fill[e], 1);
         row_token[p] = i / top;
         row_slot[p] = i % top;
@@ -671,6 +766,7 @@ __device__ __forceinline__ float pa_score(const PaAttn &at, float dot, int h, in
     if (at.rel) s += at.rel[(int)at.bucket[min(dist, at.n_bucket - 1)] * at.H + h];
     if (at.r1) s -= at.r1[h] * logf(1.0f + at.r2[h] * (float)dist);
     if (at.lin) s -= at.lin[h] * (float)dist;
+    if (at.softcap > 0.f) s = at.softcap * tanhf(s / at.softcap);
     return s;
 }
 // pooled blocks a query at position p sees: those that end at or before p - window
@@ -798,7 +894,8 @@ __global__ void __launch_bounds__(256) pa_k_mix_softmax(PaAttn at, float *__rest
     }
 }
 
-// att[i][h * dv + c] = sum_j P[h][i][j] V^T[g * dv + c][j]
+// att[i][h * dv + c] = sum_j P[h][i][j] V^T[g * dv + c][j].  With rotated values a tile's 64 columns are 32 pairs (m, m + dv / 2), two pairs to a
+// thread, which turns them back by its query's position; then the head's gate and the factor on the heads' outputs.
 __global__ void __launch_bounds__(256) pa_k_pv(PaAttn at, const float *__restrict__ S, const float *__restrict__ vct, float *__restrict__ att, int od,
                                                const int32_t *__restrict__ pos, int bs) {
     PA_TILE_SMEM(1);
@@ -808,7 +905,15 @@ __global__ void __launch_bounds__(256) pa_k_pv(PaAttn at, const float *__restric
     const int k0 = pa_first_key(at, pos[0] + m0);    // ... and the first key its first query sees (zero before a row's own)
     float acc[1][4][4] = {};
     const float *arow = (m0 + lr < bs) ? S + ((int64_t)h * at.B + m0 + lr) * at.ldS + k0 : nullptr;
-    const float *brow = (n0 + lr < at.dv) ? vct + (int64_t)(g * at.dv + n0 + lr) * at.n_ctx + k0 : nullptr;
+    // value dim of the tile's column j (dv or more: outside)
+    const int vh = at.vrope.dims >> 1;
+    auto col = [&](int j) {
+        if (vh == 0) return n0 + j;
+        const int m = n0 / 2 + (j >> 2) * 2 + (j & 1);
+        return m < vh ? m + ((j & 2) ? vh : 0) : at.dv;
+    };
+    const int cb = col(lr);
+    const float *brow = (cb < at.dv) ? vct + (int64_t)(g * at.dv + cb) * at.n_ctx + k0 : nullptr;
     pa_tile_mm<false, float, 1>(acc, arow, 1.0f, brow, nullptr, n_keys - k0, As, Bs);
     const int nv = pa_pool_vis(at, n_keys - 1); // pooled blocks of the tile's furthest query: their weights times the mean value rows
     if (nv > 0) {
@@ -820,10 +925,23 @@ __global__ void __launch_bounds__(256) pa_k_pv(PaAttn at, const float *__restric
     for (int i = 0; i < 4; i++) {
         const int m = m0 + ty * 4 + i;
         if (m >= bs) continue;
+        float f = at.gate ? pa_sigmoid(at.gate[(int64_t)m * at.ld_gate + h]) : 1.0f;
+        if (at.out_scale != 0.f) f *= at.out_scale;
+        if (vh > 0) {
+#pragma unroll
+            for (int j = 0; j < 2; j++) {
+                const int d = n0 / 2 + tx * 2 + j;
+                if (d >= vh) continue;
+                const float2 cs = pa_rope_cs(at.vrope, pos[0] + m, d);
+                const float a = acc[0][i][j], b = acc[0][i][j + 2];
+                acc[0][i][j] = a * cs.x + b * cs.y;
+                acc[0][i][j + 2] = b * cs.x - a * cs.y;
+            }
+        }
 #pragma unroll
         for (int j = 0; j < 4; j++) {
-            const int n = n0 + tx * 4 + j;
-            if (n < at.dv) att[(int64_t)m * od + h * at.dv + n] = at.gate ? acc[0][i][j] * pa_sigmoid(at.gate[(int64_t)m * at.ld_gate + h]) : acc[0][i][j];
+            const int n = col(tx * 4 + j);
+            if (n < at.dv) att[(int64_t)m * od + h * at.dv + n] = acc[0][i][j] * f;
         }
     }
 }

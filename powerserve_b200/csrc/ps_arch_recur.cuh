@@ -11,10 +11,15 @@
 //   pa_k_conv_step       both for a single token
 //   pa_k_qkv_whole_norm  q (all heads) and k RMS-normed as one vector each with weights; K row and V^T column into the cache
 //   pa_k_rope_heads      rotate-half rotation of the first dims of every head, in place, with a scale for the heads from `h_scaled` on
+//   pa_k_token_shift     h + (h' - h) mu_s for the five inputs of a time mixing (h' the token before), and the ring that keeps the last h
 //   pa_k_scan            S_t = a_t S_(t-1) + k_t (c_t v_t)^T, o_t = S_t^T q_t (+ D v_t): retention (a fixed per head, c = 1) and the
 //                        state-space recurrence (a_t = exp(-exp(A_log) dt_t), c_t = dt_t, dt = softplus(raw + bias)); fp32 state,
 //                        16 entries of a value column per lane in registers, tokens strictly in order (the result does not
 //                        depend on how a prompt was cut)
+//                        MODE 1: a decay per key channel and token (gated linear attention); MODE 2: the same, and the current token counts
+//                        with a bonus u per channel before it joins the state (time mixing)
+//   pa_k_dec_recur       one token of the MODE 1 / 2 recurrences with everything around them: the decay's low-rank product, state, output,
+//                        the head's RMS norm over a thread-block cluster, weight and silu gate in one launch
 //   pa_k_gate_gru        after an attention: the heads' outputs times their sigmoid gate, and the minGRU beside the attention
 //                        (S_t = (1 - z) S_(t-1) + z cand per channel, rounds of 32 tokens, gates formed ahead of the dependent steps)
 //   pa_k_rglru_scan      real-gated linear recurrence of a batch: S_t = a_t S_(t-1) + sqrt(1 - a_t^2) i_t u_t with log a_t = -rate r_t
@@ -272,6 +277,23 @@ __global__ void __launch_bounds__(256) pa_k_dec_rglru(const PaRglru a) {
     }
 }
 
+// out[s][t][c] = h[t][c] + (h[t - 1][c] - h[t][c]) mu[s][c]; the row before the batch's first is row (pos - 1) & 1 of `ring` (zeros at
+// position 0).  Grid (channels / 256, tokens, sets).
+__global__ void __launch_bounds__(256) pa_k_token_shift(const float *__restrict__ h, int dim, const float *__restrict__ mu, const float *__restrict__ ring, const int32_t *__restrict__ pos,
+                                                        float *__restrict__ out, int64_t set_stride) {
+    const int c = blockIdx.x * 256 + threadIdx.x, t = blockIdx.y;
+    if (c >= dim) return;
+    const int p0 = pos[0];
+    const float v = h[(int64_t)t * dim + c];
+    const float b = t > 0 ? h[(int64_t)(t - 1) * dim + c] : p0 > 0 ? ring[(int64_t)((p0 - 1) & 1) * dim + c] : 0.f;
+    out[blockIdx.z * set_stride + (int64_t)t * dim + c] = fmaf(b - v, mu[(int64_t)blockIdx.z * dim + c], v);
+}
+// after the batch: row (last position) & 1 of the ring takes the last token's input
+__global__ void __launch_bounds__(256) pa_k_token_keep(const float *__restrict__ h, int dim, float *__restrict__ ring, const int32_t *__restrict__ pos, int bs) {
+    const int c = blockIdx.x * 256 + threadIdx.x;
+    if (c < dim) ring[(int64_t)((pos[0] + bs - 1) & 1) * dim + c] = h[(int64_t)(bs - 1) * dim + c];
+}
+
 #define PA_SC_TOK 32    // tokens staged per round (half as many for the widest states)
 #define PA_SC_WARPS 4
 #define PA_SC_REGS 16   // state entries per lane
@@ -283,6 +305,10 @@ struct PaScan {
     const float *dt;          // dt[t * lddt + h] raw step sizes: c_t = softplus(dt + dt_bias[h]), a_t = exp(-exp(a_log[h]) c_t)
     int lddt;
     const float *dt_bias, *a_log, *d_skip; // [H]; d_skip null: no skip term
+    const float *dec;         // MODE 1, 2: decays dec[t * lddec + h * dk + i]
+    int lddec;
+    const float *bonus;       // MODE 2: u [H][dk]
+    float o_scale;            // MODE 1, 2: factor on the output
     float *S;                 // [H][dv][dkp]: a value column's state entries lie together, dkp = 16 * pa_scan_il(dk)
     float *o;                 // o[t * ldo + h * dv + j]
     int ldo;
@@ -294,8 +320,8 @@ static inline int pa_scan_il(int dk) { int il = 1; while (il * PA_SC_REGS < dk) 
 static inline int pa_scan_dkp(int dk) { return PA_SC_REGS * pa_scan_il(dk); }
 static inline int pa_scan_cols(int dk, int nc) { return 32 / pa_scan_il(dk) * PA_SC_WARPS * nc; } // value columns per CTA, nc per lane
 static inline int pa_scan_tok(int dk) { return pa_scan_il(dk) <= 8 ? PA_SC_TOK : PA_SC_TOK / 2; } // tokens staged per round
-static inline size_t pa_scan_smem(int dk, int nc) {
-    return 4 * (size_t)pa_scan_tok(dk) * (2 * (2 * (size_t)pa_scan_dkp(dk) + pa_scan_cols(dk, nc) + 1) + pa_scan_cols(dk, nc) + 2);
+static inline size_t pa_scan_smem(int dk, int nc, int mode) {
+    return 4 * (size_t)pa_scan_tok(dk) * (2 * ((mode ? 3 : 2) * (size_t)pa_scan_dkp(dk) + pa_scan_cols(dk, nc) + 1) + pa_scan_cols(dk, nc) + 2);
 }
 
 __device__ __forceinline__ void pa_cp_async4(float *dst_smem, const float *src) {
@@ -307,11 +333,11 @@ __device__ __forceinline__ void pa_cp_async4(float *dst_smem, const float *src) 
 // columns from registers; the output is reduced over the IL lanes of a column by log2(IL) shuffles, always in the same order (the
 // result does not depend on NC).  The q / k / v rows (and raw step sizes) of a round of tokens arrive by asynchronous 4-byte copies
 // into one of two buffers while the round before is computed.
-template <int IL, int NC>
+template <int IL, int NC, int MODE>
 __global__ void __launch_bounds__(32 * PA_SC_WARPS) pa_k_scan(const PaScan a) {
     extern __shared__ __align__(16) float sm[];
     constexpr int CW = 32 / IL, CC = CW * PA_SC_WARPS * NC, DKP = PA_SC_REGS * IL, NT = 32 * PA_SC_WARPS, TOK = IL <= 8 ? PA_SC_TOK : PA_SC_TOK / 2;
-    constexpr int BUF = TOK * (2 * DKP + CC + 1); // floats of one input buffer: q rows, k rows, v entries, raw step sizes
+    constexpr int BUF = TOK * ((MODE ? 3 : 2) * DKP + CC + 1); // floats of one input buffer: q rows, k rows, v entries, raw step sizes (MODE 1, 2: decay rows)
     const int dk = a.dk, dv = a.dv;
     float *os = sm + 2 * BUF, *as = os + TOK * CC, *cs = as + TOK;
     const int h = blockIdx.y, g = h / (a.H / a.G), j0 = blockIdx.x * CC, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
@@ -328,7 +354,15 @@ __global__ void __launch_bounds__(32 * PA_SC_WARPS) pa_k_scan(const PaScan a) {
             S[c][4 * m] = v.x; S[c][4 * m + 1] = v.y; S[c][4 * m + 2] = v.z; S[c][4 * m + 3] = v.w;
         }
     }
-    const float rate = a.dt ? expf(a.a_log[h]) : 0.f, bias = a.dt ? a.dt_bias[h] : 0.f, fixed = a.dt ? 0.f : a.decay[h], skip = a.d_skip ? a.d_skip[h] : 0.f;
+    float u[MODE == 2 ? PA_SC_REGS : 1];
+    if (MODE == 2) {
+#pragma unroll
+        for (int e = 0; e < PA_SC_REGS; e++) { // entry (m * IL + li) * 4 + e % 4, m = e / 4
+            const int i = ((e >> 2) * IL + li) * 4 + (e & 3);
+            u[MODE == 2 ? e : 0] = i < dk ? a.bonus[(int64_t)h * dk + i] : 0.f;
+        }
+    }
+    const float rate = a.dt ? expf(a.a_log[h]) : 0.f, bias = a.dt ? a.dt_bias[h] : 0.f, fixed = (MODE || a.dt) ? 0.f : a.decay[h], skip = a.d_skip ? a.d_skip[h] : 0.f;
     for (int e = tid; e < 2 * BUF; e += NT) sm[e] = 0.f; // what the copies never write (entries beyond dk, columns beyond dv) stays zero
     __syncthreads();
     auto fetch = [&](int t0, int buf) {
@@ -339,6 +373,10 @@ __global__ void __launch_bounds__(32 * PA_SC_WARPS) pa_k_scan(const PaScan a) {
             for (int i = lane; i < dk; i += 32) {
                 pa_cp_async4(qs + tt * DKP + i, qr + i);
                 pa_cp_async4(ks + tt * DKP + i, kr + i);
+            }
+            if (MODE) {
+                const float *dr = a.dec + (int64_t)(t0 + tt) * a.lddec + h * dk;
+                for (int i = lane; i < dk; i += 32) pa_cp_async4(ds + TOK + tt * DKP + i, dr + i);
             }
             const float *vr = a.v + (int64_t)(t0 + tt) * a.ldv + h * dv + j0;
             for (int c = lane; c < CC && j0 + c < dv; c += 32) pa_cp_async4(vs + tt * CC + c, vr + c);
@@ -358,7 +396,7 @@ __global__ void __launch_bounds__(32 * PA_SC_WARPS) pa_k_scan(const PaScan a) {
             asm volatile("cp.async.wait_group 0;" ::: "memory");
         }
         __syncthreads();
-        for (int tt = tid; tt < nt; tt += NT) {
+        for (int tt = tid; MODE == 0 && tt < nt; tt += NT) {
             if (a.dt) {
                 const float d = pa_softplus(ds[tt] + bias);
                 cs[tt] = d;
@@ -368,9 +406,9 @@ __global__ void __launch_bounds__(32 * PA_SC_WARPS) pa_k_scan(const PaScan a) {
                 as[tt] = fixed;
             }
         }
-        __syncthreads();
+        if (MODE == 0) __syncthreads();
         for (int tt = 0; tt < nt; tt++) {
-            const float aa = as[tt], ct = cs[tt];
+            const float aa = MODE ? 0.f : as[tt], ct = MODE ? 1.0f : cs[tt];
             float x[NC], vv[NC], acc[NC][4];
 #pragma unroll
             for (int c = 0; c < NC; c++) {
@@ -382,6 +420,22 @@ __global__ void __launch_bounds__(32 * PA_SC_WARPS) pa_k_scan(const PaScan a) {
 #pragma unroll
             for (int m = 0; m < 4; m++) {
                 const float4 kk = k4[m * IL], qq = q4[m * IL];
+                if (MODE) {
+                    const float4 dd = (reinterpret_cast<const float4 *>(ds + TOK + tt * DKP) + li)[m * IL];
+                    const float ke[4] = {kk.x, kk.y, kk.z, kk.w}, qe[4] = {qq.x, qq.y, qq.z, qq.w}, de[4] = {dd.x, dd.y, dd.z, dd.w};
+#pragma unroll
+                    for (int e = 0; e < 4; e++) {
+                        const float uk = MODE == 2 ? u[MODE == 2 ? 4 * m + e : 0] * ke[e] : 0.f;
+#pragma unroll
+                        for (int c = 0; c < NC; c++) {
+                            float &s = S[c][4 * m + e];
+                            if (MODE == 2) acc[c][e] = fmaf(fmaf(uk, vv[c], s), qe[e], acc[c][e]); // the state before, and the bonus
+                            s = fmaf(de[e], s, ke[e] * vv[c]);
+                            if (MODE == 1) acc[c][e] = fmaf(s, qe[e], acc[c][e]);
+                        }
+                    }
+                    continue;
+                }
 #pragma unroll
                 for (int c = 0; c < NC; c++) {
                     S[c][4 * m] = fmaf(aa, S[c][4 * m], kk.x * vv[c]);         acc[c][0] = fmaf(S[c][4 * m], qq.x, acc[c][0]);
@@ -395,7 +449,7 @@ __global__ void __launch_bounds__(32 * PA_SC_WARPS) pa_k_scan(const PaScan a) {
                 float r = (acc[c][0] + acc[c][1]) + (acc[c][2] + acc[c][3]);
 #pragma unroll
                 for (int o = IL / 2; o; o >>= 1) r += __shfl_xor_sync(0xffffffffu, r, o);
-                if (li == 0) os[tt * CC + col0 + c * CW] = fmaf(skip, x[c], r);
+                if (li == 0) os[tt * CC + col0 + c * CW] = MODE ? r * a.o_scale : fmaf(skip, x[c], r);
             }
         }
         __syncthreads();
@@ -413,6 +467,117 @@ __global__ void __launch_bounds__(32 * PA_SC_WARPS) pa_k_scan(const PaScan a) {
 #pragma unroll
         for (int m = 0; m < 4; m++) Sg[m * IL] = make_float4(S[c][4 * m], S[c][4 * m + 1], S[c][4 * m + 2], S[c][4 * m + 3]);
     }
+}
+
+// One token of a recurrence with a decay per key channel, and what stands around it.  A cluster of gridDim.x CTAs takes head blockIdx.y, each
+// CTA an equal share of its value columns:
+//   decay_i = dact(W_a2[h dk + i] . a1 + b)   (fp32 inputs, never rounded; every CTA of the head forms all dk of them)
+//   bonus null:  S <- diag(decay) S + k v^T, o = S^T q o_scale;   bonus given:  o = (S + diag(u) k v^T)^T q o_scale, then the same update
+//   out = o / sqrt(mean(o^2) + eps) * norm_w * silu(g)   with the mean over the head's dv columns (partial sums through distributed shared memory)
+struct PaRecStep {
+    const float *q, *k, *v, *g, *a1;
+    const bf16 *a2;
+    const float *a2b;
+    int rank;
+    PaAct dact;
+    const float *bonus;   // [H][dk]
+    float o_scale;
+    float *S;             // [H][dv][dkp]
+    const float *norm_w;  // [H * dv]
+    float eps;
+    float *out;
+    const int32_t *pos;
+    int dk, dv, dkp, lg;  // lg: log2 of the lanes that share a value column (dkp / 16)
+};
+static inline size_t pa_rec_step_smem(int dkp, int cols, int rank) { return 4 * ((size_t)4 * dkp + 3 * (size_t)cols + rank); }
+
+__global__ void __launch_bounds__(256) pa_k_dec_recur(const PaRecStep a) {
+    extern __shared__ __align__(16) float sm[];
+    __shared__ float red[8], part_s;
+    cg::cluster_group cl = cg::this_cluster();
+    const int n_cl = gridDim.x, h = blockIdx.y, cols = (a.dv + n_cl - 1) / n_cl, j0 = blockIdx.x * cols, nc = max(0, min(cols, a.dv - j0)), dk = a.dk, dkp = a.dkp;
+    float *qs = sm, *ks = qs + dkp, *ds = ks + dkp, *us = ds + dkp, *vs = us + dkp, *gs = vs + cols, *os = gs + cols, *ls = os + cols;
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    float *Sh = a.S + ((int64_t)h * a.dv + j0) * dkp;
+    // neither a weight nor the state's address depends on the kernel before: on their way to L2 (the state is read behind the wait)
+    for (int e = tid * 32; e < nc * dkp; e += 256 * 32) asm volatile("prefetch.global.L2 [%0];" ::"l"(Sh + e));
+    for (int e = tid * 64; e < dk * a.rank; e += 256 * 64) asm volatile("prefetch.global.L2 [%0];" ::"l"(a.a2 + (int64_t)h * dk * a.rank + e));
+    ps_grid_dep_launch();
+    ps_grid_dep_wait();
+    const bool fresh = a.pos[0] == 0;
+    for (int i = tid; i < dkp; i += 256) {
+        const bool in = i < dk;
+        qs[i] = in ? a.q[h * dk + i] : 0.f;
+        ks[i] = in ? a.k[h * dk + i] : 0.f;
+        us[i] = in && a.bonus ? a.bonus[h * dk + i] : 0.f;
+    }
+    for (int j = tid; j < nc; j += 256) { vs[j] = a.v[h * a.dv + j0 + j]; gs[j] = pa_silu(a.g[h * a.dv + j0 + j]); }
+    for (int r = tid; r < a.rank; r += 256) ls[r] = a.a1[r];
+    __syncthreads();
+    for (int i = tid; i < dkp; i += 256) {
+        float d = 0.f;
+        if (i < dk) {
+            const bf16 *w = a.a2 + ((int64_t)h * dk + i) * a.rank;
+            float z = 0.f;
+            if ((a.rank & 7) == 0) {
+                for (int r = 0; r < a.rank; r += 8) {
+                    const uint4 v = __ldg(reinterpret_cast<const uint4 *>(w + r));
+                    const uint32_t u[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+                    for (int t = 0; t < 4; t++) {
+                        z = fmaf(__uint_as_float(u[t] << 16), ls[r + 2 * t], z);
+                        z = fmaf(__uint_as_float(u[t] & 0xffff0000u), ls[r + 2 * t + 1], z);
+                    }
+                }
+            } else {
+                for (int r = 0; r < a.rank; r++) z = fmaf(pa_ld(w + r), ls[r], z);
+            }
+            d = pa_act1(z + a.a2b[h * dk + i], a.dact);
+        }
+        ds[i] = d;
+    }
+    __syncthreads();
+    // 2^lg lanes share a value column, 16 state entries each (the layout of pa_k_scan); entries beyond dk are zero and stay zero
+    const int il = 1 << a.lg, li = lane & (il - 1), per_warp = 32 >> a.lg;
+    float ss = 0.f;
+    for (int jb = warp * per_warp; jb < nc; jb += 8 * per_warp) {
+        const int j = jb + (lane >> a.lg), jj = min(j, nc - 1);
+        float4 *Sg = reinterpret_cast<float4 *>(Sh + (int64_t)jj * dkp) + li;
+        const float v = vs[jj];
+        float4 s[4];
+        float acc[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+        for (int m = 0; m < 4; m++) s[m] = fresh ? make_float4(0.f, 0.f, 0.f, 0.f) : Sg[m * il];
+#pragma unroll
+        for (int m = 0; m < 4; m++) {
+            const float4 kk = (reinterpret_cast<const float4 *>(ks) + li)[m * il], qq = (reinterpret_cast<const float4 *>(qs) + li)[m * il], dd = (reinterpret_cast<const float4 *>(ds) + li)[m * il],
+                         uu = (reinterpret_cast<const float4 *>(us) + li)[m * il];
+            const float ke[4] = {kk.x, kk.y, kk.z, kk.w}, qe[4] = {qq.x, qq.y, qq.z, qq.w}, de[4] = {dd.x, dd.y, dd.z, dd.w}, ue[4] = {uu.x, uu.y, uu.z, uu.w};
+            float se[4] = {s[m].x, s[m].y, s[m].z, s[m].w};
+#pragma unroll
+            for (int e = 0; e < 4; e++) {
+                if (a.bonus) acc[e] = fmaf(fmaf(ue[e] * ke[e], v, se[e]), qe[e], acc[e]);
+                se[e] = fmaf(de[e], se[e], ke[e] * v);
+                if (!a.bonus) acc[e] = fmaf(se[e], qe[e], acc[e]);
+            }
+            s[m] = make_float4(se[0], se[1], se[2], se[3]);
+        }
+        float r = (acc[0] + acc[1]) + (acc[2] + acc[3]);
+        for (int o = il / 2; o; o >>= 1) r += __shfl_xor_sync(0xffffffffu, r, o);
+        if (j < nc) {
+#pragma unroll
+            for (int m = 0; m < 4; m++) Sg[m * il] = s[m];
+            if (li == 0) { r *= a.o_scale; os[j] = r; ss = fmaf(r, r, ss); }
+        }
+    }
+    const float mine = pa_block_sum(ss, red);
+    if (tid == 0) part_s = mine;
+    cl.sync();
+    float t = 0.f;
+    for (int c = 0; c < n_cl; c++) t += *cl.map_shared_rank(&part_s, c);
+    const float inv = 1.0f / sqrtf(t / (float)a.dv + a.eps);
+    for (int j = tid; j < nc; j += 256) a.out[h * a.dv + j0 + j] = os[j] * inv * a.norm_w[h * a.dv + j0 + j] * gs[j];
+    cl.sync(); // no CTA leaves while another reads its partial sum
 }
 
 // one CTA per (part, token); `width` entries in `parts` equal parts.  gate_first: out = N(y silu(g)) * w; else out = N(y) * silu(g) (w null: 1)
@@ -437,13 +602,18 @@ __global__ void __launch_bounds__(256) pa_k_gate_norm(const float *__restrict__ 
     }
 }
 
-// out[t][c] = sum_r slot[t][r][c] + sgate[t] * shared[t][c]   (shared null: no shared expert; sgate null: 1)
+// out[t][c] = sum_r slot[t][r][c] + sgate[t] * shared[t][c]   (shared null: no shared expert; sgate null: 1); a choice sel_e[t][r] >= E
+// stands for the input itself: sel_w[t][r] * x[t][c]
 __global__ void __launch_bounds__(256) pa_k_moe_sum(float *__restrict__ out, const float *__restrict__ slot, int top, const float *__restrict__ shared,
-                                                    const float *__restrict__ sgate, int dim) {
+                                                    const float *__restrict__ sgate, int dim, const int *__restrict__ sel_e = nullptr, const float *__restrict__ sel_w = nullptr,
+                                                    const float *__restrict__ x = nullptr, int E = 0) {
     const int t = blockIdx.y, c = blockIdx.x * 256 + threadIdx.x;
     if (c >= dim) return;
     float y = 0.f;
-    for (int r = 0; r < top; r++) y += slot[((int64_t)t * top + r) * dim + c];
+    for (int r = 0; r < top; r++) {
+        if (x && sel_e[t * top + r] >= E) y = fmaf(sel_w[t * top + r], x[(int64_t)t * dim + c], y);
+        else y += slot[((int64_t)t * top + r) * dim + c];
+    }
     if (shared) y += (sgate ? sgate[t] : 1.0f) * shared[(int64_t)t * dim + c];
     out[(int64_t)t * dim + c] = y;
 }

@@ -63,7 +63,42 @@ __global__ void __launch_bounds__(256) pa_k_tc_prep_x(uint8_t *__restrict__ dst,
     }
 }
 
+// the operand sets of a segmented product: set 0 = x, set s = x + (x' - x) mu[s - 1] with x' the row of the token before (the batch's first
+// token: row (pos - 1) & 1 of `ring`, zeros at position 0).  Grid (k blocks, column tiles, sets); set s starts s * set_bytes further on.
+__global__ void __launch_bounds__(256) pa_k_tc_prep_shift(uint8_t *__restrict__ dst, const float *__restrict__ x, int M, int K, int nkb, const float *__restrict__ mu,
+                                                          const float *__restrict__ ring, const int32_t *__restrict__ pos, int64_t set_bytes) {
+    const int kb = blockIdx.x, t = blockIdx.y, set = blockIdx.z, p0 = pos[0];
+    const float *m = set ? mu + (int64_t)(set - 1) * K : nullptr;
+    uint8_t *out = dst + set * set_bytes + ((int64_t)t * nkb + kb) * PT_BLOCK;
+    for (int c = threadIdx.x; c < 128 * 8; c += 256) {
+        const int kc = c & 7, row = c >> 3, r = t * 128 + row, k0 = kb * PT_KB + kc * 8;
+        uint16_t v[8];
+        const float *src = x + (int64_t)r * K, *prev = r > 0 ? src - K : ring + (int64_t)((p0 - 1) & 1) * K;
+        const bool first = r == 0 && p0 == 0;
+#pragma unroll
+        for (int e = 0; e < 8; e++) {
+            float val = 0.f;
+            if (r < M && k0 + e < K) {
+                val = src[k0 + e];
+                if (m) val = fmaf((first ? 0.f : prev[k0 + e]) - val, m[k0 + e], val);
+            }
+            v[e] = __bfloat16_as_ushort(__float2bfloat16_rn(val));
+        }
+        uint4 pk;
+        pk.x = v[0] | ((uint32_t)v[1] << 16); pk.y = v[2] | ((uint32_t)v[3] << 16); pk.z = v[4] | ((uint32_t)v[5] << 16); pk.w = v[6] | ((uint32_t)v[7] << 16);
+        *reinterpret_cast<uint4 *>(out + kc * 2048 + row * 16) = pk;
+    }
+}
+
 // ---------------------------------------------------------------------------------------------------- the GEMM
+// A product whose output rows read different operand sets (activations that are mixtures of the same input): row tiles rt[s] .. rt[s + 1] - 1
+// hold the rows row[s] .. row[s + 1] - 1 of the output and read set s.  n = 0: one set, all rows.
+#define PT_MAX_SEG 6
+struct PtSegs {
+    int n;
+    int rt[PT_MAX_SEG + 1], row[PT_MAX_SEG + 1];
+    int64_t set_bytes;
+};
 enum { PT_MODE_DENSE = 0, PT_MODE_EXPERT_UP = 1, PT_MODE_EXPERT_DOWN = 2 };
 
 struct PtArgs {
@@ -83,6 +118,8 @@ struct PtArgs {
     PaAct act;
     int act1;               // dense / expert up: the one-argument activation on the outputs n >= act_from (a feed-forward without a gate),
     int act_from, gap;      // which are stored `gap` columns further on
+    PaRowMul mul;           // dense: the outputs times a table row per token
+    PtSegs seg;
     int *err;
 };
 
@@ -125,6 +162,8 @@ __global__ void __launch_bounds__(PT_THREADS, 1) pa_k_tc_gemm(const PtArgs a) {
                 const uint8_t *pa0 = a.a0 + ((grp * a.n_rt + rt) * nkb) * (int64_t)PT_BLOCK;
                 const uint8_t *pa1 = NA == 2 ? a.a1 + ((grp * a.n_rt + rt) * nkb) * (int64_t)PT_BLOCK : nullptr;
                 const uint8_t *pb = a.b + ((int64_t)ct * nkb) * PT_BLOCK;
+                for (int sg = 1; sg < a.seg.n; sg++)
+                    if (rt >= a.seg.rt[sg]) pb += a.seg.set_bytes;
                 for (int kb = 0; kb < nkb; kb++, g++) {
                     const int s = g % STAGES;
                     if (g >= STAGES && !ps_tc_wait(&bar_empty[s], ((g / STAGES) - 1) & 1)) { *a.err = 1; ok = false; break; }
@@ -168,10 +207,12 @@ __global__ void __launch_bounds__(PT_THREADS, 1) pa_k_tc_gemm(const PtArgs a) {
             const int u = (int)blockIdx.x + mu * (int)gridDim.x, ct = u / a.n_rt, rt = u % a.n_rt, tb = mu & 1;
             if (!ps_tc_wait(&bar_tmem_full[tb], (mu >> 1) & 1)) { *a.err = 4; break; }
             ps_tc_fence_after();
-            const int n = rt * PT_M + 32 * warp + lane;
+            int n = rt * PT_M + 32 * warp + lane, n_end = a.N;
+            for (int sg = 0; sg < a.seg.n; sg++) // the segment's own rows
+                if (rt >= a.seg.rt[sg] && rt < a.seg.rt[sg + 1]) { n += a.seg.row[sg] - a.seg.rt[sg] * PT_M; n_end = a.seg.row[sg + 1]; break; }
             const int r0 = a.tile_row0 ? a.tile_row0[ct] : ct * PT_N, rend = a.tile_end ? a.tile_end[ct] : a.M;
             const uint32_t t_lane = tmem_base + ((uint32_t)(32 * warp) << 16) + tb * (NA * PT_N);
-            const float bias = (a.bias && n < a.N) ? a.bias[n] : 0.f;
+            const float bias = (a.bias && n < n_end) ? a.bias[n] : 0.f;
             const int n_cols = min(PT_N, rend - r0); // warp-uniform
             for (int c0 = 0; c0 < n_cols; c0 += 16) {
                 uint32_t v[16], w2[16];
@@ -187,15 +228,17 @@ __global__ void __launch_bounds__(PT_THREADS, 1) pa_k_tc_gemm(const PtArgs a) {
                                  : "r"(t_lane + PT_N + c0)
                                  : "memory");
                 ps_tc_ld_wait();
-                if (n < a.N) {
+                if (n < n_end) {
 #pragma unroll
                     for (int c = 0; c < 16; c++) {
                         const int r = r0 + c0 + c;
                         if (r >= rend) break;
                         const float acc = __uint_as_float(v[c]);
                         if (a.mode == PT_MODE_DENSE) {
-                            if (a.act1 && n >= a.act_from) a.C[(int64_t)r * a.ldc + n + a.gap] = pa_act1(acc + bias, a.act);
-                            else a.C[(int64_t)r * a.ldc + n] = acc + bias;
+                            const bool act1 = a.act1 && n >= a.act_from;
+                            float val = act1 ? pa_act1(acc + bias, a.act) : acc + bias;
+                            if (a.mul.table) val *= pa_ld(a.mul.table + (int64_t)a.mul.tok[r] * a.mul.ld + n);
+                            a.C[(int64_t)r * a.ldc + (act1 ? n + a.gap : n)] = val;
                         } else if (a.mode == PT_MODE_EXPERT_UP) {
                             a.C[(int64_t)r * a.ldc + n] = NA == 2 ? pa_expert_act(acc, __uint_as_float(w2[c]), a.act) : pa_act1(acc, a.act);
                         } else {
