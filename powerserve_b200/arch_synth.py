@@ -429,3 +429,99 @@ def momedra_weights(cfg: dict, seed: int = 0, fast: bool = False) -> Dict[str, n
             if f.get("shared"):
                 t[p + "mlp.shared.up"], t[p + "mlp.shared.down"] = mat(f["shared"]["ff"], W), mat(W, f["shared"]["ff"])
     return t
+
+
+# ------------------------------------------------------------------------------------------------------------ Tegolix
+def _tegolix_mlp(ff: int = 0, experts: int = 0, top: int = 1, identity: int = 0, shared_ff: int = 0) -> Optional[dict]:
+    """ff == 0: no feed-forward; experts == 0: dense of ff rows; else routed experts of ff rows, `identity` further router outputs that stand for the
+    input itself (+ a shared expert of shared_ff rows)"""
+    if not ff:
+        return None
+    if not experts:
+        return {"kind": "dense", "ff": ff}
+    mlp = {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": experts, "identity": identity, "top": top}}
+    if shared_ff:
+        mlp["shared"] = {"ff": shared_ff}
+    return mlp
+
+
+def tegolix_gla_layer(heads: int, dim: int, vdim: int, *, tau: float = 16.0, **mlp) -> dict:
+    return {"type": "gla", "mixer": {"heads": heads, "dim": dim, "vdim": vdim, "tau": tau}, "mlp": _tegolix_mlp(**mlp)}
+
+
+def tegolix_parallel_layer(heads: int, kv_heads: int, dim: int, vdim: int, *, window: int, rwkv: tuple, rot_dims: Optional[int] = None, rot_base: float = 10000.0,
+                           scaling: Optional[dict] = None, softcap: Optional[float] = 50.0, scale: Optional[float] = None, left_scale: float = 0.8, right_scale: float = 0.9, **mlp) -> dict:
+    """rwkv = (heads, dim) of the time mixing; scaling = {"factor", "original", "fast", "slow"} turns YaRN on"""
+    rot = {"base": rot_base, "dims": dim if rot_dims is None else rot_dims}
+    if scaling:
+        rot["scaling"] = dict(scaling)
+    left = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "mask": {"size": window}, "rot": rot, "scale": float(scale if scale is not None else dim ** -0.5)}
+    if softcap:
+        left["softcap"] = softcap
+    return {"type": "parallel", "mixer": {"left": left, "left_scale": left_scale, "right": {"heads": rwkv[0], "dim": rwkv[1]}, "right_scale": right_scale}, "mlp": _tegolix_mlp(**mlp)}
+
+
+def tegolix_config(width: int, vocab: int, layers: List[dict], *, side_dim: int, eps: float = 1e-6) -> dict:
+    return {"architecture": "Tegolix", "layers": layers, "norm": {"eps": eps}, "token_side": {"dim": side_dim}, "vocab": vocab, "width": width}
+
+
+def tegolix_weights(cfg: dict, seed: int = 0, rank: int = 6, fast: bool = False) -> Dict[str, np.ndarray]:
+    """float32 arrays of bfloat16-representable values keyed by tensor name; `rank` rows in the decays' first matrices
+    (fast = True: big matrices as random bfloat16 bit patterns)"""
+    rng = np.random.default_rng(seed)
+    W, V = cfg["width"], cfg["vocab"]
+
+    def rnd(a):
+        return (safetensors.float32_to_bf16_bits(np.asarray(a, np.float32)).astype(np.uint32) << 16).view(np.float32)
+
+    def mat(out_dim, in_dim, gain=1.0):
+        if fast:
+            e = int(np.floor(np.log2(gain / np.sqrt(in_dim)))) + 127
+            bits = rng.integers(0, 1 << 7, size=(out_dim, in_dim), dtype=np.uint16) | np.uint16(e << 7)
+            return bits | (rng.integers(0, 2, size=(out_dim, in_dim), dtype=np.uint16) << 15).astype(np.uint16)
+        return rnd(rng.standard_normal((out_dim, in_dim), dtype=np.float32) * np.float32(gain / np.sqrt(in_dim)))
+
+    def vec(n, mean=0.0, dev=0.1):
+        return rnd(mean + rng.standard_normal(n).astype(np.float32) * dev)
+
+    def unit(n):
+        return {"gate": mat(n, W, 1.5), "up": mat(n, W, 1.5), "down": mat(W, n)}
+
+    sd, nl = cfg["token_side"]["dim"], len(cfg["layers"])
+    t: Dict[str, np.ndarray] = {"embed": mat(V, W, np.sqrt(W)), "final.norm": vec(W), "head": mat(V, W), "side.embed": mat(V, nl * sd, np.sqrt(nl * sd))}
+    for i, l in enumerate(cfg["layers"]):
+        p, a, m = f"l{i}.", f"l{i}.mix.", l["mixer"]
+        t[p + "norm1"], t[p + "norm1b"], t[p + "ls1"] = vec(W), vec(W), vec(W, 0.6, 0.2)
+        t[p + "side.gate"], t[p + "side.proj"], t[p + "side.norm"] = mat(sd, W), mat(W, sd), vec(W, 0.4)
+        if l["type"] == "gla":
+            H, d, dv = m["heads"], m["dim"], m["vdim"]
+            t[a + "q"], t[a + "k"], t[a + "v"], t[a + "g"], t[a + "o"] = mat(H * d, W), mat(H * d, W), mat(H * dv, W), mat(H * dv, W), mat(W, H * dv)
+            t[a + "norm"], t[a + "a1"], t[a + "a2"], t[a + "a2.b"] = vec(dv, 1.0, 0.2), mat(rank, W), mat(H * d, rank, 1.5), vec(H * d, 0.5, 1.5)
+        else:
+            ml, mr, b = m["left"], m["right"], a + "right."
+            a += "left."
+            H, G, d, dv = ml["heads"], ml["kv_heads"], ml["dim"], ml["vdim"]
+            t[a + "q"], t[a + "k"], t[a + "v"], t[a + "g"], t[a + "o"] = mat(H * d, W), mat(G * d, W), mat(G * dv, W), mat(H, W, 2.0), mat(W, H * dv)
+            t[a + "q.norm"], t[a + "k.norm"] = vec(d, 1.4, 0.3), vec(d, 1.4, 0.3)
+            R = mr["heads"] * mr["dim"]
+            for s in "rkvg":
+                t[b + s] = mat(R, W)
+            for s in "rkvgw":
+                t[b + "mu." + s] = rnd(rng.uniform(0.1, 0.9, W))
+            t[b + "w1"], t[b + "w2"], t[b + "w0"] = mat(rank, W), mat(R, rank), rnd(rng.uniform(-6.0, 0.5, R))
+            t[b + "u"], t[b + "norm"], t[b + "o"] = vec((mr["heads"], mr["dim"]), 0.5, 0.5), vec(R, 1.0, 0.2), mat(W, R)
+        f = l.get("mlp")
+        if f is None:
+            continue
+        t[p + "norm2"], t[p + "norm2b"], t[p + "ls2"] = vec(W), vec(W), vec(W, 0.6, 0.2)
+        if f["kind"] == "dense":
+            t.update({p + "mlp." + n: x for n, x in unit(f["ff"]).items()})
+            continue
+        E = f["router"]["experts"]
+        t[p + "mlp.router"], t[p + "mlp.correction"] = mat(E + f["router"].get("identity", 0), W, 2.0), vec(E + f["router"].get("identity", 0), 0.0, 0.1)
+        for e in range(E):
+            t.update({p + f"mlp.e{e}.{n}": x for n, x in unit(f["expert"]["ff"]).items()})
+        if f.get("shared"):
+            t.update({p + "mlp.shared." + n: x for n, x in unit(f["shared"]["ff"]).items()})
+            t[p + "mlp.shared.sg"] = mat(1, W, 2.0)
+    return t
