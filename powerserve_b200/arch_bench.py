@@ -1,4 +1,4 @@
-"""bench.py --arch nufusun | vanapel | dozotar | pidenex | momedra: prefill and decode throughput of a layer-list design at layer sizes that resemble real
+"""bench.py --arch nufusun | vanapel | dozotar | pidenex | momedra | tegolix: prefill and decode throughput of a layer-list design at layer sizes that resemble real
 models (random weights), beside the closest existing model of the framework.
 
 --arch vanapel: the Vanapel design (windowed attention layers and one latent-attention layer, dense gated feed-forward) beside
@@ -18,6 +18,12 @@ ff rows against an ungated one of 3 ff / 2).
 RG-LRU with dense feed-forwards; the first two layers run twice at sizes s and m) beside Pidenex - the closest existing model: layer
 norms, layer runs, latent attention with neighbouring pairs, a gated recurrence, feed-forwards without a gate - with as many layer
 runs, equal width, head geometry, keys in sight, vocabulary and ACTIVE feed-forward rows per token.
+
+--arch tegolix: the Tegolix design (two gated-linear-attention layers, a windowed attention beside a time mixing; dense relu and routed
+feed-forwards with identity outputs and a shared expert, per-layer token inputs) beside Dozotar - the closest existing model: sequential
+blocks, matrix-state recurrences with a gated head norm, an attention in bounded sight, soft-max routing beside a shared expert - with
+retention in the gated linear attention's place, equal width, head geometry, keys in sight, layer count, vocabulary and ACTIVE
+feed-forward rows per token.
 
 --arch nufusun: prefill and decode throughput of the Nufusun design at layer sizes that resemble real models
 (random weights), beside the closest existing model of the framework - a llama stack (Q4_K) with the same width, head
@@ -417,6 +423,73 @@ def run_size_momedra(name, prompt_len, steps, warmup, seed, chunk):
     return out
 
 
+# name: (width, attention (heads, kv heads, head size, window), time mixing (heads, channels), gla (heads, dim, vdim), active ff / 2, token input, decay rank, layer types, vocab)
+TEGOLIX_SIZES = {
+    "s": (1024, (16, 4, 64, 512), (16, 64), (8, 64, 128), 1024, 128, 16, "gpgg", 32000),
+    "m": (2048, (16, 4, 128, 1024), (32, 64), (8, 128, 256), 2816, 256, 32, "gpgg", 32000),
+    "l": (4096, (32, 8, 128, 1024), (64, 64), (16, 128, 256), 7168, 256, 64, "gpg", 32000),
+}
+
+
+def _tegolix_model(name, seed, chunk, n_ctx):
+    W, (H, G, hs, win), rw, (GH, gd, gv), ff, sd, rank, kinds, V = TEGOLIX_SIZES[name]
+    layers = []
+    for i, k in enumerate(kinds):   # the first layer's feed-forward is dense (2 ff rows), the others route 2 of 8 (+ 1 identity output) of ff / 2 rows beside a shared one of ff
+        mlp = dict(ff=2 * ff) if i == 0 else dict(ff=ff // 2, experts=8, top=2, identity=1, shared_ff=ff)
+        if k == "g":
+            layers.append(arch_synth.tegolix_gla_layer(GH, gd, gv, **mlp))
+        else:
+            layers.append(arch_synth.tegolix_parallel_layer(H, G, hs, hs, window=win, rwkv=rw, rot_base=5e5, scaling={"factor": 4.0, "original": 1024, "fast": 32.0, "slow": 1.0}, **mlp))
+    cfg = arch_synth.tegolix_config(W, V, layers, side_dim=sd)
+    return cfg, _load_synth(cfg, arch_synth.tegolix_weights(cfg, seed=seed, rank=rank, fast=True), chunk, n_ctx)
+
+
+def _tegolix_comparator(name, seed, chunk, n_ctx):
+    W, (H, G, hs, win), _, (GH, gd, gv), ff, _, _, kinds, V = TEGOLIX_SIZES[name]
+    layers = []
+    for i, k in enumerate(kinds):
+        mlp = dict(ff=2 * ff) if i == 0 else dict(ff=ff // 2, experts=8, top=2, shared_ff=ff)
+        if k == "g":
+            layers.append(arch_synth.dozotar_retention_layer(GH, gd, gv, rot_base=5e5, **mlp))
+        else:
+            layers.append(arch_synth.dozotar_attention_layer(H, G, hs, hs, chunk=win, conv=4, bias_max=float(win), **mlp))
+    cfg = arch_synth.dozotar_config(W, V, layers)
+    return cfg, _load_synth(cfg, arch_synth.dozotar_weights(cfg, seed=seed, rel_rows=32, fast=True), chunk, n_ctx)
+
+
+def run_size_tegolix(name, prompt_len, steps, warmup, seed, chunk):
+    W, (H, G, hs, win), (RH, rd), (GH, gd, gv), ff, sd, rank, kinds, V = TEGOLIX_SIZES[name]
+    hbm, tflops, src = _peaks()
+    n_ctx = -(-(prompt_len + steps + warmup + 24) // 256) * 256
+    prompt = [int(v) for v in np.random.default_rng(1234).integers(0, V, prompt_len)]
+    out = {"size": name, "width": W, "attention": [H, G, hs, win], "time_mixing": [RH, rd], "gla": [GH, gd, gv], "active_ff": 2 * ff, "token_input": sd, "decay_rank": rank, "layers": kinds, "vocab": V,
+           "context": prompt_len}
+
+    def report(m, params, cache_bytes, mix_flops):
+        t_pre, t_dec, launches, e2e = _measure(m, prompt, chunk, steps, warmup)
+        m.close()
+        flops = (2 * params + mix_flops) * prompt_len / t_pre / 1e12
+        by = 2 * params + cache_bytes
+        return {"prefill_tok_s": prompt_len / t_pre, "prefill_chunk": chunk, "prefill_tflops": flops, "prefill_frac_of_bf16_peak": flops / tflops,
+                "decode_tok_s": 1 / t_dec, "decode_ms": t_dec * 1e3, "decode_launches_per_step": launches, "decode_bytes_per_token": by,
+                "decode_frac_of_hbm_peak": by / t_dec / 1e9 / hbm, "e2e_decode_tok_s": e2e}
+
+    ng, npar, nl, R = kinds.count("g"), kinds.count("p"), len(kinds), RH * rd
+    keys = min(win, prompt_len)
+    p_att = (H + 2 * G) * hs * W + H * hs * W
+    p_ff = 3 * 2 * ff * W + (nl - 1) * (10 * W + 3 * 2 * ff * W)             # one identity output in nine: counted as an expert
+    p_gla = (2 * GH * gd + 2 * GH * gv) * W + GH * gv * W
+    params = npar * (p_att + H * W + 5 * R * W + rank * (W + R)) + ng * (p_gla + rank * (W + GH * gd)) + p_ff + nl * 2 * sd * W + V * W
+    state, flops = npar * 2 * G * hs * 4 * keys + ng * 2 * GH * gd * gv * 4, npar * 2 * 2 * H * hs * keys / 2 + ng * 5 * GH * gd * gv
+    cfg, m = _tegolix_model(name, seed, chunk, n_ctx)
+    out["tegolix"] = report(m, params, state + npar * 2 * RH * rd * rd * 4, flops + npar * 7 * RH * rd * rd)
+    cfg, m = _tegolix_comparator(name, seed, chunk, n_ctx)
+    params = npar * p_att + ng * p_gla + p_ff + V * W
+    out["dozotar"] = dict(report(m, params, state, npar * 2 * 2 * H * hs * keys / 2 + ng * 4 * GH * gd * gv), layers=kinds.replace("g", "r").replace("p", "a"))
+    out["peaks"] = {"hbm_gbs": hbm, "bf16_tflops": tflops, "source": src}
+    return out
+
+
 def main(args) -> int:
     if capi.load_library().ps_cuda_device_count() == 0:
         print(json.dumps({"arch": args.arch, "unavailable": "no CUDA device: there is no CPU fallback"}))
@@ -435,6 +508,11 @@ def main(args) -> int:
     if args.arch == "momedra":
         res = [run_size_momedra(s, args.arch_prompt, max(args.steps, 8), max(args.warmup, 3), args.seed, args.arch_chunk) for s in sizes]
         print(json.dumps({"arch": "momedra", "dtype": "bf16", "data": "synthetic", "timing": "CUDA events around every call, warm-up first; weights exceed L2",
+                          "sizes": res}))
+        return 0
+    if args.arch == "tegolix":
+        res = [run_size_tegolix(s, args.arch_prompt, max(args.steps, 8), max(args.warmup, 3), args.seed, args.arch_chunk) for s in sizes]
+        print(json.dumps({"arch": "tegolix", "dtype": "bf16", "data": "synthetic", "timing": "CUDA events around every call, warm-up first; weights exceed L2",
                           "sizes": res}))
         return 0
     if args.arch == "vanapel":

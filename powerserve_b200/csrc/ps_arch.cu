@@ -77,7 +77,7 @@ struct PsArchLayer {
     float *a2b = nullptr, *bonus = nullptr, *mu = nullptr; // mu: [5][dim]
     PtSegs seg{};                         // time mixing: which operand set the first projection's rows read
     int64_t ring_off = 0;                 // the last token's input in the K buffer (two rows; floats from its start)
-    double *vrope_freq = nullptr;         // rotation of the values
+    int ang_qk = 0, ang_v = 0;            // rotated attention heads: where the angles of q / k and of the values start in the model's list of pairs
     float *corr = nullptr;                // corrections on the router's choice
     // per-layer token input
     bf16 *wtg = nullptr, *wtp = nullptr;
@@ -113,7 +113,7 @@ struct PsArch {
     float *xe = nullptr;   // the embedding output, kept for the passes of a looped model that add it back
     float *pass_steps = nullptr; // [n_pass_steps][dim]
     int pool_off = 0, stat_off = 0; // where a score row keeps its pooled scores; where the single-token step keeps their block statistics
-    float *cv = nullptr, *sh = nullptr, *ffo = nullptr, *sgate = nullptr; // convolution output; shared expert's output; summed feed-forward output; shared gate per token
+    float *cv = nullptr, *sh = nullptr, *ffo = nullptr, *sgate = nullptr, *ysh = nullptr; // convolution output; shared expert's output; summed feed-forward output; shared gate per token; its activated rows (single token)
     int max_cv = 0, max_pool = 0;
     bool has_state = false; // some layer carries state that cannot be cut back (recurrences, convolution tails)
     int max_rq = 0, max_lq = 0, max_qa = 0, max_att2 = 0, vsrc_w = 0;
@@ -149,6 +149,11 @@ struct PsArch {
     bf16 *tok_embed = nullptr;             // per-layer token input: [vocab][token_slots * token_dim]
     float *tg = nullptr, *ty = nullptr;    // its gated part [max_batch][token_dim] and its output [max_batch][dim]
     bool has_shift = false;
+    std::vector<double> ang_freq_h;        // rotated attention heads: the model's pairs (equal lists of different layers kept once)
+    std::vector<float> ang_ms_h;
+    double *ang_freq = nullptr;
+    float *ang_ms = nullptr;
+    float2 *ang = nullptr;                 // [max_batch][pairs]: cos / sin at the positions in flight
     int max_rec = 0;
 };
 
@@ -242,9 +247,7 @@ void build_bucket_table(int rows, float dmax, int n, std::vector<uint16_t> &t) {
 }
 
 // shared memory of the single-token kernels
-size_t pa_dec_scores_smem(int H, int G, int dq, int rope_dims = 0) {
-    return 4 * ((size_t)PA_DS_KEYS * (((G * dq + 3) & ~3) + 4) + (size_t)H * dq + (size_t)(PA_DS_KEYS + 1) * H + (size_t)std::max(H * H, rope_dims + 2));
-}
+size_t pa_dec_scores_smem(int H, int G, int dq) { return 4 * ((size_t)PA_DS_KEYS * (((G * dq + 3) & ~3) + 4) + (size_t)H * dq + (size_t)(PA_DS_KEYS + 1) * H + (size_t)H * H); }
 // the P.V kernel splits more than 4 query heads per kv head over blockIdx.z, 4 (or fewer) to a CTA
 int pa_dec_pv_split(int H, int G) { return (H / G + 3) / 4; }
 int pa_dec_pv_rep(int H, int G) { const int z = pa_dec_pv_split(H, G); return (H / G + z - 1) / z; }
@@ -532,7 +535,7 @@ int ps_arch_create(PsArch **out, const ps_cuda_arch_desc *desc, std::string &err
         if (l.mlp_kind == PS_MLP_DENSE && l.expert_ff <= 0) return bail(afail(err, PS_CUDA_ERR_UNSUPPORTED, "layer %d: dense feed-forward of %d rows", i, l.expert_ff));
         // the attention kernels see a latent layer as one shared key head of kv_rank + rot_dim dims whose values are the latents
         const int a_dq = latent ? l.kv_rank + l.rot_dim : l.qk_dim, a_dv = latent ? l.kv_rank : l.v_dim;
-        if ((!recur && pa_dec_scores_smem(l.n_heads, l.n_kv_heads, a_dq, l.rope_dims) > 160 * 1024) || (size_t)d.dim * 4 > 160 * 1024)
+        if ((!recur && pa_dec_scores_smem(l.n_heads, l.n_kv_heads, a_dq) > 160 * 1024) || (size_t)d.dim * 4 > 160 * 1024)
             return bail(afail(err, PS_CUDA_ERR_UNSUPPORTED, "layer %d: %d heads of size %d (or width %d) exceed the single-token kernels' shared memory", i, l.n_heads, a_dq, d.dim));
         w.qd = l.n_heads * a_dq; w.kd = l.n_kv_heads * a_dq; w.vd = l.n_kv_heads * a_dv; w.od = l.n_heads * l.v_dim;
         w.pw = latent ? l.q_rank + l.kv_rank + l.rot_dim : w.qd + w.kd + w.vd;
@@ -653,6 +656,7 @@ int ps_arch_create(PsArch **out, const ps_cuda_arch_desc *desc, std::string &err
     AL(a->z, 4 * ((size_t)std::max(a->max_e, 1) + 1));
     if (a->max_cv) AL(a->cv, 4 * (size_t)a->max_cv * B);
     AL(a->sh, 4 * dim * B);
+    AL(a->ysh, 4 * (size_t)std::max(a->max_ff, 1));
     AL(a->ffo, 4 * dim * B);
     AL(a->sgate, 4 * B);
     a->stat_off = (d.n_ctx + PA_DS_KEYS - 1) / PA_DS_KEYS;
@@ -914,17 +918,20 @@ int ps_arch_bind(PsArch *a, const ps_cuda_arch_weights *wt, cudaStream_t stream,
             if (l.out_gate && (rc = upload_mat(w.wqkv + (size_t)w.g_off * dim, s.g, (size_t)(l.out_gate == PS_GATE_HEAD ? l.n_heads : w.ho) * dim, "output gate", err))) return rc;
             if (l.lin_bias && (rc = vec(&w.lin, s.lin, (size_t)l.n_heads, "distance-bias slopes", false))) return rc;
             if (l.qk_norm == PS_QKNORM_HEAD_W && ((rc = vec(&w.q_norm, s.q_norm, (size_t)l.qk_dim, "q norm", false)) || (rc = vec(&w.k_norm, s.k_norm, (size_t)l.qk_dim, "k norm", false)))) return rc;
-            auto freqs = [&](double **dst, int dims, float factor) -> int {
+            // the place of a list of rotated pairs among the model's (an equal list that is there already serves both)
+            auto pairs = [&](int dims, float factor) -> int {
                 std::vector<double> fd((size_t)dims / 2);
-                const double ms = rope_freq_host(dims, l.rope_base, factor, l.rope_original, l.rope_fast, l.rope_slow, fd.data());
-                if (dst == &w.rope_freq) w.rope_mscale = (float)ms;
-                int r = aalloc(a, (void **)dst, fd.size() * 8, err);
-                if (r) return r;
-                PA_CK(cudaMemcpy(*dst, fd.data(), fd.size() * 8, cudaMemcpyHostToDevice));
-                return 0;
+                const float ms = (float)rope_freq_host(dims, l.rope_base, factor, l.rope_original, l.rope_fast, l.rope_slow, fd.data());
+                const size_t n = fd.size(), have = a->ang_freq_h.size();
+                for (size_t o = 0; o + n <= have; o++)
+                    if (std::equal(fd.begin(), fd.end(), a->ang_freq_h.begin() + (ptrdiff_t)o) && std::all_of(a->ang_ms_h.begin() + (ptrdiff_t)o, a->ang_ms_h.begin() + (ptrdiff_t)(o + n), [&](float v) { return v == ms; }))
+                        return (int)o;
+                a->ang_freq_h.insert(a->ang_freq_h.end(), fd.begin(), fd.end());
+                a->ang_ms_h.insert(a->ang_ms_h.end(), n, ms);
+                return (int)have;
             };
-            if (l.mixer_kind == PS_MIXER_ATTENTION && l.rope_dims > 0 && (rc = freqs(&w.rope_freq, l.rope_dims, l.rope_factor))) return rc;
-            if (l.mixer_kind == PS_MIXER_ATTENTION && l.v_rope && (rc = freqs(&w.vrope_freq, l.v_dim, 0.f))) return rc;
+            if (l.mixer_kind == PS_MIXER_ATTENTION && l.rope_dims > 0) w.ang_qk = pairs(l.rope_dims, l.rope_factor);
+            if (l.mixer_kind == PS_MIXER_ATTENTION && l.v_rope) w.ang_v = pairs(l.v_dim, 0.f);
             if (l.mixer_kind == PS_MIXER_GLA) {
                 const size_t rk = (size_t)l.decay_rank, H = (size_t)l.n_heads;
                 if ((rc = upload_mat(w.wqkv + (nq + nk + nv) * dim, s.g, nv * dim, "g", err)) || (rc = upload_mat(w.wqkv + (nq + nk + 2 * nv) * dim, s.a1, rk * dim, "a1", err)) ||
@@ -1065,6 +1072,11 @@ int ps_arch_bind(PsArch *a, const ps_cuda_arch_weights *wt, cudaStream_t stream,
                 w.act_b = (float)(0.5 + softplus((double)tmp[1]));
             }
         }
+    }
+    if (!a->ang_freq_h.empty()) {
+        const size_t n = a->ang_freq_h.size();
+        if ((rc = aalloc(a, (void **)&a->ang_freq, 8 * n, err)) || (rc = upload_f32(a, &a->ang_ms, a->ang_ms_h, err)) || (rc = aalloc(a, (void **)&a->ang, 8 * n * (size_t)d.max_batch, err))) return rc;
+        PA_CK(cudaMemcpy(a->ang_freq, a->ang_freq_h.data(), 8 * n, cudaMemcpyHostToDevice));
     }
     if (a->round) {
         // tensor-core operand blocks: every matrix once more in the layout the tcgen05 GEMM streams (ps_arch_tc.cuh)
@@ -1226,7 +1238,7 @@ static int forward_t(PsArch *a, const PsArchIO &io, int bs, int pos0, int lm_hea
         if (at.window > 0) blocks = std::min(blocks, cdiv(at.window, PA_DS_KEYS) + 1);
         if (at.chunk > 0) blocks = std::min(blocks, cdiv(at.chunk, PA_DS_KEYS) + 1);
         const unsigned pooled = at.pool > 0 ? cdiv(n_kv_cap / at.pool, PA_DS_KEYS) : 0; // further CTAs for the pooled blocks
-        pa_launch_dep(pdl, pa_k_dec_scores, dim3(blocks + pooled), dim3(256), pa_dec_scores_smem(at.H, at.G, at.dq, at.rope.dims), st, at, q, (const float *)io.kc[li], io.pos_dev, a->S, io.err_dev, (int)blocks,
+        pa_launch_dep(pdl, pa_k_dec_scores, dim3(blocks + pooled), dim3(256), pa_dec_scores_smem(at.H, at.G, at.dq), st, at, q, (const float *)io.kc[li], io.pos_dev, a->S, io.err_dev, (int)blocks,
                       pool_here && pooled ? io.vct[li] : (float *)nullptr);
         PA_LAUNCH();
         pa_launch_dep(pdl, pa_k_dec_pv, dim3(cdiv(at.dv, PA_DP_DIMS), at.G, pa_dec_pv_split(at.H, at.G)), dim3(256), pa_dec_pv_smem(at.H, at.G), st, at, (const float *)a->S, (const float *)io.vct[li], io.pos_dev, out,
@@ -1422,6 +1434,7 @@ static int forward_t(PsArch *a, const PsArchIO &io, int bs, int pos0, int lm_hea
         const float *bonus;
         float o_scale, *S, *out;
         int ldo;
+        float *ring; // time mixing: keeps the batch's last input
     };
     auto recurrence = [&](const PsArchLayer &w, const PaRec &r, cudaStream_t sr, bool dep) -> int {
         const int rank = w.d.decay_rank, n = r.H * r.dk, dkp = pa_scan_dkp(r.dk);
@@ -1435,14 +1448,15 @@ static int forward_t(PsArch *a, const PsArchIO &io, int bs, int pos0, int lm_hea
             PA_LAUNCH();
             return 0;
         }
-        pa_k_linear<false><<<dim3(cdiv(n, PA_TN), cdiv(bs, PA_TM)), blk, 0, sr>>>(r.a1, w.pw, w.wa2, w.a2b, a->dcy, n, bs, n, rank, 0, 0, 0, 0, r.act);
+        pa_k_decay<<<dim3(cdiv(n, 256), cdiv(bs, PA_DC_TOK)), 256, 4 * (size_t)rank * PA_DC_TOK, sr>>>(r.a1, w.pw, rank, w.wa2, w.a2b, n, r.act, a->dcy, bs, a->h, dim, r.ring, io.pos_dev);
         PA_LAUNCH();
         PaScan sc{};
         sc.q = r.q; sc.k = r.k; sc.v = r.v; sc.ldq = sc.ldk = sc.ldv = w.pw; sc.q_gs = sc.k_gs = r.dk; sc.H = sc.G = r.H; sc.dk = r.dk; sc.dv = r.dv;
         sc.dec = a->dcy; sc.lddec = n; sc.bonus = r.bonus; sc.o_scale = r.o_scale; sc.S = r.S; sc.o = r.out; sc.ldo = r.ldo; sc.pos = io.pos_dev; sc.bs = bs;
         int rc = scan(sc);
         if (rc) return rc;
-        pa_k_gate_norm<<<dim3((unsigned)r.H, bs), 256, 0, sr>>>(r.out, r.ldo, r.g, w.pw, r.H * r.dv, r.H, w.mix_norm, 0, d.norm_eps, r.out, r.ldo);
+        if (r.dv <= 256) pa_k_gate_norm_warp<<<dim3(cdiv(r.H, 8), bs), 256, 0, sr>>>(r.out, r.ldo, r.g, w.pw, r.dv, r.H, w.mix_norm, d.norm_eps, r.out, r.ldo);
+        else pa_k_gate_norm<<<dim3((unsigned)r.H, bs), 256, 0, sr>>>(r.out, r.ldo, r.g, w.pw, r.H * r.dv, r.H, w.mix_norm, 0, d.norm_eps, r.out, r.ldo);
         PA_LAUNCH();
         return 0;
     };
@@ -1453,7 +1467,7 @@ static int forward_t(PsArch *a, const PsArchIO &io, int bs, int pos0, int lm_hea
         PaRec r{};
         r.q = a->qkv + w.z_off; r.k = r.q + W; r.v = r.k + W; r.g = r.v + W; r.a1 = r.g + W;
         r.H = w.d.side_heads; r.dk = r.dv = sd; r.act = PaAct{0.f, 0.f, 0.f, PA_ACT_EXP_EXP}; r.bonus = w.bonus; r.o_scale = 1.0f;
-        r.S = io.kc[li] + w.state_off; r.out = a->att + w.ho; r.ldo = w.aw;
+        r.S = io.kc[li] + w.state_off; r.out = a->att + w.ho; r.ldo = w.aw; r.ring = io.kc[li] + w.ring_off;
         const bool fork = single && a->opt_fork;
         if (fork) { PA_CK(cudaEventRecord(a->ev_fork, st)); PA_CK(cudaStreamWaitEvent(a->side, a->ev_fork, 0)); }
         int rc = recurrence(w, r, fork ? a->side : st, pdl && !fork);
@@ -1527,7 +1541,7 @@ static int forward_t(PsArch *a, const PsArchIO &io, int bs, int pos0, int lm_hea
                 PtArgs g{};
                 g.seg = w.seg;
                 g.seg.set_bytes = (int64_t)n_ct * nkb * PT_BLOCK;
-                pa_k_tc_prep_shift<<<dim3((unsigned)nkb, (unsigned)n_ct, PT_MAX_SEG), 256, 0, st>>>(a->tcx, a->h, bs, dim, nkb, w.mu, ring, io.pos_dev, g.seg.set_bytes);
+                pa_k_tc_prep_shift<<<dim3((unsigned)nkb, (unsigned)n_ct, 4), 256, 0, st>>>(a->tcx, a->h, bs, dim, nkb, w.mu, ring, io.pos_dev, g.seg.set_bytes);
                 PA_LAUNCH();
                 g.a0 = w.t_qkv; g.b = a->tcx; g.nkb = nkb; g.n_rt = w.seg.rt[w.seg.n]; g.n_ct = n_ct; g.M = bs; g.N = w.pw; g.mode = PT_MODE_DENSE; g.C = a->qkv; g.ldc = w.pw; g.err = io.err_dev;
                 g.act = tanh_act; g.act1 = 1; g.act_from = w1_off;
@@ -1543,15 +1557,14 @@ static int forward_t(PsArch *a, const PsArchIO &io, int bs, int pos0, int lm_hea
                     PA_LAUNCH();
                 }
             }
-            pa_k_token_keep<<<cdiv(dim, 256), 256, 0, st>>>(a->h, dim, ring, io.pos_dev, bs);
-            PA_LAUNCH();
         } else {
             if ((rc = seam(raw ? nullptr : a->h, raw ? nullptr : w.norm))) return rc;
             if ((rc = linear(raw ? a->x : a->h, dim, dim, w.wqkv, w.t_qkv, w.pw, a->qkv, w.pw))) return rc;
         }
         if (l.mixer_kind == PS_MIXER_ATTENTION) {
             float *q = a->qkv;
-            const PaRope at_rope{w.rope_freq, l.rope_dims, w.rope_mscale, 0}, at_vrope{w.vrope_freq, l.v_rope ? l.v_dim : 0, 1.0f, 0};
+            const int n_ang = (int)a->ang_freq_h.size();
+            const PaRope at_rope{nullptr, l.rope_dims, 1.0f, 0, a->ang + w.ang_qk, n_ang}, at_vrope{nullptr, l.v_rope ? l.v_dim : 0, 1.0f, 0, a->ang + w.ang_v, n_ang};
             if (rwkv && (rc = time_mix(li))) return rc; // a single token's runs beside the attention, joined before the output product
             if (l.conv_taps > 0) {
                 float *tail = io.kc[li] + (int64_t)w.kd * d.n_ctx;
@@ -1572,7 +1585,7 @@ static int forward_t(PsArch *a, const PsArchIO &io, int bs, int pos0, int lm_hea
                 PA_LAUNCH();
             } else if (heads_post) {
                 if (!single) { // (a single token's scores kernel does this)
-                    pa_k_qkv_post<<<bs, 256, 8 * (size_t)(l.rope_dims / 2 + (l.v_rope ? l.v_dim / 2 : 0)), st>>>(q, w.pw, H, l.n_kv_heads, l.qk_dim, l.v_dim, l.qk_norm, d.norm_eps, 0, nullptr, nullptr, 0, io.kc[li],
+                    pa_k_qkv_post<<<bs, 256, 0, st>>>(q, w.pw, H, l.n_kv_heads, l.qk_dim, l.v_dim, l.qk_norm, d.norm_eps, 0, nullptr, nullptr, 0, io.kc[li],
                                                                                                       io.vct[li], d.n_ctx, io.pos_dev, w.q_norm, w.k_norm, 0.f, 1.f, at_rope, at_vrope);
                     PA_LAUNCH();
                 }
@@ -1678,25 +1691,23 @@ static int forward_t(PsArch *a, const PsArchIO &io, int bs, int pos0, int lm_hea
             const int n_rt = rt.E + (rt.shared_gate ? 1 : 0); // the router's rows (+ the shared gate's): logits from the unrounded input
             if (sff > 0) { // the shared expert's gate | up launch carries the seam and the router's rows
                 pa_launch_dep(pdl, pa_k_dec_dense_up<ROUND>, dim3(std::min(cdiv(sff + n_rt, PA_DV_ROWS / 2), up_cap)), dim3(PA_DV_THREADS), 4 * (size_t)dim, st, (const float *)xc, pend_y, pend_w, w_in,
-                              xo, groups, d.norm_eps, (const bf16 *)w.wsg, (const bf16 *)w.wsu, a->y, sff, dim, act, (const bf16 *)w.router, n_rt, a->z, 0, a->res_scale);
+                              xo, groups, d.norm_eps, (const bf16 *)w.wsg, (const bf16 *)w.wsu, a->ysh, sff, dim, act, (const bf16 *)w.router, n_rt, a->z, 0, a->res_scale);
                 PA_LAUNCH();
                 std::swap(xc, xo);
                 pend_y = pend_w = nullptr;
-                PaMv ms{};
-                ms.x = a->y; ms.W = w.wsd; ms.N = dim; ms.K = sff; ms.y = a->sh;
-                if ((rc = dec_mv(ms, 0))) return rc;
             } else {
                 PaMv mv{};
                 seam_mv(mv, w_in);
                 mv.W = nullptr; mv.N = 0; mv.K = dim; mv.Wr = w.router; mv.E = n_rt; mv.z = a->z;
                 if ((rc = dec_mv(mv, 4 * (size_t)dim))) return rc;
             }
-            pa_k_dec_expert_up<ROUND><<<dim3(std::min(cdiv(ff, PA_DV_ROWS / 2), (unsigned)std::max(1, 4 * a->n_sm / top)), top), PA_DV_THREADS, 4 * (size_t)dim, st>>>(
-                xc, w_in, d.norm_eps, a->z, rt, w.wgate, w.wup, a->y, ff, dim, l.route_on_input, act, a->sel_e, a->sel_w, l.route_identity ? a->hn : nullptr);
+            pa_launch_dep(pdl, pa_k_dec_expert_up<ROUND>, dim3(std::min(cdiv(ff, PA_DV_ROWS / 2), (unsigned)std::max(1, 4 * a->n_sm / top)), top), dim3(PA_DV_THREADS), 4 * (size_t)dim, st, (const float *)xc, w_in,
+                          d.norm_eps, (const float *)a->z, rt, (const bf16 *)w.wgate, (const bf16 *)w.wup, a->y, ff, dim, l.route_on_input, act, a->sel_e, a->sel_w, l.route_identity ? a->hn : (float *)nullptr);
             PA_LAUNCH();
             const int ksd = pick_ksplit(dim, ff);
-            pa_k_dec_expert_down<ROUND><<<cdiv(dim, PA_DV_ROWS / ksd), PA_DV_THREADS, 0, st>>>(a->y, a->sel_e, a->sel_w, top, w.wdown, nullptr, nullptr, dim, ff, l.route_on_input, ksd, a->ffo,
-                                                                                               sff > 0 ? a->sh : nullptr, rt.shared_gate ? a->z + rt.E : nullptr, E, a->hn);
+            pa_launch_dep(pdl, pa_k_dec_expert_down<ROUND>, dim3(cdiv(dim, PA_DV_ROWS / ksd)), dim3(PA_DV_THREADS), 0, st, (const float *)a->y, (const int *)a->sel_e, (const float *)a->sel_w, top,
+                          (const bf16 *)w.wdown, (const float *)nullptr, (float *)nullptr, dim, ff, l.route_on_input, ksd, a->ffo, (const float *)nullptr, rt.shared_gate ? (const float *)(a->z + rt.E) : (const float *)nullptr, E,
+                          (const float *)a->hn, sff > 0 ? (const bf16 *)w.wsd : (const bf16 *)nullptr, (const float *)a->ysh, sff);
             PA_LAUNCH();
         } else {
             if ((rc = seam(raw ? nullptr : a->h, w_in))) return rc;
@@ -1858,7 +1869,8 @@ static int forward_t(PsArch *a, const PsArchIO &io, int bs, int pos0, int lm_hea
         return 0;
     };
 
-    pa_k_embed<<<bs, 128, 0, st>>>(a->x, a->embed, io.tokens_dev, dim, d.embed_scale, a->has_pass_in ? a->xcat + dim : a->keep_embed ? a->xe : nullptr, a->has_pass_in ? 2 * dim : dim);
+    pa_k_embed<<<bs, 128, 0, st>>>(a->x, a->embed, io.tokens_dev, dim, d.embed_scale, a->has_pass_in ? a->xcat + dim : a->keep_embed ? a->xe : nullptr, a->has_pass_in ? 2 * dim : dim,
+                                   PaAngles{a->ang_freq, a->ang_ms, (int)a->ang_freq_h.size(), a->ang, io.pos_dev});
     PA_LAUNCH();
     for (int li = 0; li < d.n_layers; li++) {
         const PsArchLayer &w = a->L[(size_t)li];

@@ -22,7 +22,8 @@
 //   pa_k_dec_latent_q    latent attention with queries from the input: W_uk folded into the query, both rotations, latent and rotated key
 //                        part into the cache
 //   pa_k_dec_expert_up   norm + top-k of the router scores in the prologue, gate | up rows of the chosen experts, activation
-//   pa_k_dec_expert_down down rows of the chosen experts summed over the slots + mixer output + residual
+//   pa_k_dec_expert_down down rows of the chosen experts summed over the slots + mixer output + residual (or, for the next seam, + the
+//                        shared expert's down rows behind its gate + the input itself for identity outputs)
 #pragma once
 #include "ps_ptx.cuh"
 
@@ -305,8 +306,8 @@ __global__ void __launch_bounds__(256) pa_k_dec_scores(PaAttn at, const float *_
     float *ks = sm;                        // [PA_DS_KEYS][kds]
     float *qs = ks + PA_DS_KEYS * kds;     // [H][dq]
     float *sa = qs + H * dq;               // [H][PA_DS_KEYS + 1]
-    float *Ts = sa + H * (PA_DS_KEYS + 1); // [H][H], or cos / sin of the rotations
-    float2 *cs = reinterpret_cast<float2 *>(sm + (((Ts - sm) + 1) & ~1));
+    float *Ts = sa + H * (PA_DS_KEYS + 1); // [H][H]
+    const float2 *cs = at.rope.cs;
     const int tid = threadIdx.x;
     if (at.mix) for (int t = tid; t < H * H; t += 256) Ts[t] = at.mix[t]; // a weight: fetched before the dependency wait
     ps_grid_dep_launch();
@@ -342,15 +343,11 @@ __global__ void __launch_bounds__(256) pa_k_dec_scores(PaAttn at, const float *_
         const int lane = tid & 31;
         const float qt = pa_q_temp(at.qt_coef, at.qt_every, pos);
         const int rh = at.rope.dims >> 1, vh = at.vrope.dims >> 1;
-        if (rh > 0) {
-            for (int i = tid; i < rh; i += 256) cs[i] = pa_rope_cs(at.rope, pos, i);
-            __syncthreads();
-        }
         if (own && vh > 0) // the token's value, rotated, into its V^T column
             for (int e = tid; e < G * vh; e += 256) {
                 const int g = e / vh, m = e % vh;
                 const float va = at.v_raw[g * at.dv + m], vb = at.v_raw[g * at.dv + m + vh];
-                const float2 t = pa_rope_cs(at.vrope, pos, m);
+                const float2 t = at.vrope.cs[m];
                 at.vct_out[(int64_t)(g * at.dv + m) * at.n_ctx + pos] = va * t.x - vb * t.y;
                 at.vct_out[(int64_t)(g * at.dv + m + vh) * at.n_ctx + pos] = vb * t.x + va * t.y;
             }
@@ -372,7 +369,8 @@ __global__ void __launch_bounds__(256) pa_k_dec_scores(PaAttn at, const float *_
             if (rh > 0) {
                 __syncwarp();
                 for (int i = lane; i < rh; i += 32) {
-                    const float va = dst[i] * inv, vb = dst[i + rh] * inv, ra = va * cs[i].x - vb * cs[i].y, rb = vb * cs[i].x + va * cs[i].y;
+                    const float2 c2 = cs[i];
+                    const float va = dst[i] * inv, vb = dst[i + rh] * inv, ra = va * c2.x - vb * c2.y, rb = vb * c2.x + va * c2.y;
                     dst[i] = ra;
                     dst[i + rh] = rb;
                     if (kout) { kout[i] = ra; kout[i + rh] = rb; }
@@ -553,7 +551,7 @@ __global__ void __launch_bounds__(256) pa_k_dec_pv(PaAttn at, const float *__res
         };
         float s = sum(cc);
         if (vh > 0) { // turned back by the query's position
-            const float2 t2 = pa_rope_cs(at.vrope, n - 1, c0 / 2 + (cc & 1));
+            const float2 t2 = at.vrope.cs[c0 / 2 + (cc & 1)];
             const float o = sum(cc ^ 2);
             s = cc < 2 ? s * t2.x + o * t2.y : s * t2.x - o * t2.y;
         }
@@ -634,6 +632,8 @@ __global__ void __launch_bounds__(PA_DV_THREADS) pa_k_dec_expert_up(const float 
     __shared__ float sc[PA_MAX_EXPERTS];
     __shared__ int se[PA_MAX_EXPERTS];
     __shared__ float sw[PA_MAX_EXPERTS];
+    ps_grid_dep_launch();
+    ps_grid_dep_wait();
     if (rt.act == PS_ROUTER_TOPK_SOFTMAX || (rt.act == PS_ROUTER_SOFTMAX && rt.groups <= 1)) {
         if (threadIdx.x < 32) {
             if (rt.act == PS_ROUTER_SOFTMAX) pa_route_softmax_warp(z, rt, se, sw, threadIdx.x);
@@ -730,7 +730,8 @@ template <bool ROUND>
 __global__ void __launch_bounds__(PA_DV_THREADS) pa_k_dec_expert_down(const float *__restrict__ y, const int *__restrict__ sel_e, const float *__restrict__ sel_w, int top,
                                                                       const bf16 *__restrict__ Wd, const float *__restrict__ ao, float *__restrict__ x, int dim, int ff,
                                                                       int on_input, int ksplit, float *__restrict__ dst = nullptr, const float *__restrict__ extra = nullptr,
-                                                                      const float *__restrict__ extra_logit = nullptr, int E = 1 << 30, const float *__restrict__ h = nullptr) {
+                                                                      const float *__restrict__ extra_logit = nullptr, int E = 1 << 30, const float *__restrict__ h = nullptr,
+                                                                      const bf16 *__restrict__ Wsd = nullptr, const float *__restrict__ ysh = nullptr, int sff = 0) {
     __shared__ float part_s[8][2];
     ps_grid_dep_launch(); // the next kernel (the next layer's q|k|v rows, or the head) may start fetching its weights
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
@@ -739,6 +740,9 @@ __global__ void __launch_bounds__(PA_DV_THREADS) pa_k_dec_expert_down(const floa
     const int kc = ff / ksplit, k_begin = slice * kc, k_end = slice == ksplit - 1 ? ff : k_begin + kc;
     const bool live = n0 < dim;
     float t0 = 0.f, t1 = 0.f;
+    const int kcs = (sff / ksplit) & ~7, s_begin = slice * kcs, s_end = slice == ksplit - 1 ? sff : s_begin + kcs; // the shared expert's columns
+    if (live && Wsd) pa_prefetch2(Wsd + (int64_t)n0 * sff, Wsd + (int64_t)n1 * sff, s_begin, s_end, lane);
+    ps_grid_dep_wait();
     if (live) {
         for (int r = 0; r < top; r++) {
             const int e = sel_e[r];
@@ -756,6 +760,13 @@ __global__ void __launch_bounds__(PA_DV_THREADS) pa_k_dec_expert_down(const floa
             const float w = on_input ? 1.0f : sel_w[r];
             t0 += s0 * w;
             t1 += s1 * w;
+        }
+        if (Wsd) { // the shared expert's down rows, times its gate
+            float s0, s1;
+            pa_dot2<ROUND>(Wsd + (int64_t)n0 * sff, Wsd + (int64_t)n1 * sff, ysh, sff, 1.0f, lane, s0, s1, s_begin, s_end);
+            const float sg = extra_logit ? 1.0f / (1.0f + expf(-extra_logit[0])) : 1.0f;
+            t0 = fmaf(sg, s0, t0);
+            t1 = fmaf(sg, s1, t1);
         }
     }
     if (ksplit > 1) {

@@ -45,6 +45,16 @@ struct PaRope {
     int dims;
     float mscale;
     int interleaved;    // pairs (2i, 2i + 1) instead of (i, i + dims / 2)
+    const float2 *cs;   // rotated attention heads: cos / sin of every token in flight, formed once per forward pass (row t: cs + t * ld_cs)
+    int ld_cs;
+};
+// the angles of all rotated attention heads of a model, one list of pairs: row t of `out` receives (cos, sin) * mscale at the token's position
+struct PaAngles {
+    const double *freq;
+    const float *mscale;
+    int n;
+    float2 *out;
+    const int32_t *pos;
 };
 __device__ __forceinline__ float2 pa_rope_cs(const PaRope &r, int pos, int i) {
     const double turns = (double)pos * r.freq[i];
@@ -171,8 +181,12 @@ __device__ __forceinline__ void pa_tile_mm(float (&acc)[NB][4][4], const float *
 // ---------------------------------------------------------------------------------------------------------------- small ops
 // keep (null or [tokens] rows of stride ld_keep) receives the same rows once more: the embedding output that later passes of a looped model add back
 __global__ void __launch_bounds__(128) pa_k_embed(float *__restrict__ x, const bf16 *__restrict__ table, const int32_t *__restrict__ tokens, int dim, float scale,
-                                                  float *__restrict__ keep, int ld_keep) {
+                                                  float *__restrict__ keep, int ld_keep, PaAngles ang) {
     const int t = blockIdx.x;
+    for (int i = threadIdx.x; i < ang.n; i += blockDim.x) {
+        const PaRope r{ang.freq, 0, ang.mscale[i], 0, nullptr, 0};
+        ang.out[(int64_t)t * ang.n + i] = pa_rope_cs(r, ang.pos[t], i);
+    }
     const bf16 *row = table + (int64_t)tokens[t] * dim;
     float *out = x + (int64_t)t * dim;
     float *out2 = keep ? keep + (int64_t)t * ld_keep : nullptr;
@@ -339,20 +353,16 @@ __device__ __forceinline__ float pa_q_temp(float coef, float every, int p) {
 }
 
 // After the q|k|v projection of a batch, one CTA per token: unit-RMS q heads (in place) and k heads (qk_norm; times the weights qn / kn
-// and, for q, the position's temperature), both rotated (rope, its angles formed once per token), the values rotated (vrope), the value rows blended with the source layer's (v_mix), K row -> kc[pos][:], V row transposed -> vct[:][pos].
+// and, for q, the position's temperature), both rotated (rope), the values rotated (vrope), the value rows blended with the source layer's (v_mix), K row -> kc[pos][:], V row transposed -> vct[:][pos].
 __global__ void __launch_bounds__(256) pa_k_qkv_post(float *__restrict__ qkv, int ld, int H, int G, int dq, int dv, int qk_norm, float eps, int v_mix,
                                                      const float *__restrict__ lambda, float *__restrict__ v_src, int ld_src, float *__restrict__ kc,
                                                      float *__restrict__ vct, int n_ctx, const int32_t *__restrict__ pos, const float *__restrict__ qn, const float *__restrict__ kn,
                                                      float qt_coef, float qt_every, PaRope rope = PaRope{}, PaRope vrope = PaRope{}) {
-    extern __shared__ __align__(16) float2 pa_cs[]; // cos / sin of the rotations: rope.dims / 2 pairs, then vrope.dims / 2
     const int t = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, p = pos[t];
     float *row = qkv + (int64_t)t * ld;
     const float qt = pa_q_temp(qt_coef, qt_every, p);
     const int qd = H * dq, kd = G * dq, vd = G * dv, rh = rope.dims >> 1, vh = vrope.dims >> 1;
-    if (rh + vh > 0) {
-        for (int i = threadIdx.x; i < rh + vh; i += 256) pa_cs[i] = i < rh ? pa_rope_cs(rope, p, i) : pa_rope_cs(vrope, p, i - rh);
-        __syncthreads();
-    }
+    const float2 *rcs = rope.cs + (int64_t)t * rope.ld_cs, *vcs = vrope.cs + (int64_t)t * vrope.ld_cs;
     for (int hh = warp; hh < H + G; hh += 8) { // q heads, then k heads
         float *v = row + hh * dq;
         const float inv = qk_norm ? pa_warp_inv_rms(v, dq, eps, lane) : 1.0f;
@@ -361,7 +371,7 @@ __global__ void __launch_bounds__(256) pa_k_qkv_post(float *__restrict__ qkv, in
         const float f = hh < H ? inv * qt : inv;
         for (int i = lane; i < rh; i += 32) { // the rotated pairs (i, i + rh)
             const float a = v[i] * f * (w ? w[i] : 1.0f), b = v[i + rh] * f * (w ? w[i + rh] : 1.0f);
-            const float2 cs = pa_cs[i];
+            const float2 cs = rcs[i];
             dst[i] = a * cs.x - b * cs.y;
             dst[i + rh] = b * cs.x + a * cs.y;
         }
@@ -375,7 +385,7 @@ __global__ void __launch_bounds__(256) pa_k_qkv_post(float *__restrict__ qkv, in
         for (int e = threadIdx.x; e < G * vh; e += 256) {
             const int g = e / vh, m = e % vh;
             const float a = row[qd + kd + g * dv + m], b = row[qd + kd + g * dv + m + vh];
-            const float2 cs = pa_cs[rh + m];
+            const float2 cs = vcs[m];
             vct[(int64_t)(g * dv + m) * n_ctx + p] = a * cs.x - b * cs.y;
             vct[(int64_t)(g * dv + m + vh) * n_ctx + p] = b * cs.x + a * cs.y;
         }
@@ -932,7 +942,7 @@ __global__ void __launch_bounds__(256) pa_k_pv(PaAttn at, const float *__restric
             for (int j = 0; j < 2; j++) {
                 const int d = n0 / 2 + tx * 2 + j;
                 if (d >= vh) continue;
-                const float2 cs = pa_rope_cs(at.vrope, pos[0] + m, d);
+                const float2 cs = at.vrope.cs[(int64_t)m * at.vrope.ld_cs + d];
                 const float a = acc[0][i][j], b = acc[0][i][j + 2];
                 acc[0][i][j] = a * cs.x + b * cs.y;
                 acc[0][i][j + 2] = b * cs.x - a * cs.y;

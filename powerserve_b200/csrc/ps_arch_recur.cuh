@@ -11,7 +11,8 @@
 //   pa_k_conv_step       both for a single token
 //   pa_k_qkv_whole_norm  q (all heads) and k RMS-normed as one vector each with weights; K row and V^T column into the cache
 //   pa_k_rope_heads      rotate-half rotation of the first dims of every head, in place, with a scale for the heads from `h_scaled` on
-//   pa_k_token_shift     h + (h' - h) mu_s for the five inputs of a time mixing (h' the token before), and the ring that keeps the last h
+//   pa_k_token_shift     h + (h' - h) mu_s for the five inputs of a time mixing (h' the token before)
+//   pa_k_decay           low-rank decays per key channel and token; keeps a time mixing's last input
 //   pa_k_scan            S_t = a_t S_(t-1) + k_t (c_t v_t)^T, o_t = S_t^T q_t (+ D v_t): retention (a fixed per head, c = 1) and the
 //                        state-space recurrence (a_t = exp(-exp(A_log) dt_t), c_t = dt_t, dt = softplus(raw + bias)); fp32 state,
 //                        16 entries of a value column per lane in registers, tokens strictly in order (the result does not
@@ -25,6 +26,7 @@
 //   pa_k_rglru_scan      real-gated linear recurrence of a batch: S_t = a_t S_(t-1) + sqrt(1 - a_t^2) i_t u_t with log a_t = -rate r_t
 //                        softplus(lam), times gelu(y); rounds of 32 tokens like the minGRU; leaves the convolution's ring for the next batch
 //   pa_k_dec_rglru       convolution, both gates' block rows, recurrence and output product of a single token in one launch
+//   pa_k_gate_norm_warp  the same for parts of at most 256 entries, a warp per part
 //   pa_k_gate_norm       RMS norm in equal parts around a silu gate: (y silu(g)) normed times w, or normed y times silu(g)
 //   pa_k_moe_sum         sum of a token's expert slots (fixed order) plus the gated shared expert
 #pragma once
@@ -288,13 +290,49 @@ __global__ void __launch_bounds__(256) pa_k_token_shift(const float *__restrict_
     const float b = t > 0 ? h[(int64_t)(t - 1) * dim + c] : p0 > 0 ? ring[(int64_t)((p0 - 1) & 1) * dim + c] : 0.f;
     out[blockIdx.z * set_stride + (int64_t)t * dim + c] = fmaf(b - v, mu[(int64_t)blockIdx.z * dim + c], v);
 }
-// after the batch: row (last position) & 1 of the ring takes the last token's input
-__global__ void __launch_bounds__(256) pa_k_token_keep(const float *__restrict__ h, int dim, float *__restrict__ ring, const int32_t *__restrict__ pos, int bs) {
-    const int c = blockIdx.x * 256 + threadIdx.x;
-    if (c < dim) ring[(int64_t)((pos[0] + bs - 1) & 1) * dim + c] = h[(int64_t)(bs - 1) * dim + c];
+// The decays of a batch, dec[t][n] = act(W2[n] . a1[t] + b[n]): fp32 inputs, never rounded, one chain of FMAs in the order of the single-token
+// step's.  Grid (channels / 256, tokens / PA_DC_TOK); a thread takes one channel of PA_DC_TOK tokens.  With `ring` given (a time mixing) the
+// launch also leaves the batch's last input h in row (last position) & 1 of the ring - nothing behind the first projection reads the old row.
+#define PA_DC_TOK 8
+__global__ void __launch_bounds__(256) pa_k_decay(const float *__restrict__ a1, int lda, int rank, const bf16 *__restrict__ w2, const float *__restrict__ b, int n, PaAct act,
+                                                  float *__restrict__ dec, int bs, const float *__restrict__ h, int dim, float *__restrict__ ring, const int32_t *__restrict__ pos) {
+    extern __shared__ __align__(16) float ls[]; // [rank][PA_DC_TOK]
+    const int t0 = blockIdx.y * PA_DC_TOK, c = blockIdx.x * 256 + threadIdx.x;
+    if (ring)
+        for (int e = (blockIdx.y * gridDim.x + blockIdx.x) * 256 + threadIdx.x; e < dim; e += gridDim.x * gridDim.y * 256)
+            ring[(int64_t)((pos[0] + bs - 1) & 1) * dim + e] = h[(int64_t)(bs - 1) * dim + e];
+    for (int e = threadIdx.x; e < rank * PA_DC_TOK; e += 256) {
+        const int r = e % rank, t = e / rank;
+        ls[r * PA_DC_TOK + t] = t0 + t < bs ? a1[(int64_t)(t0 + t) * lda + r] : 0.f;
+    }
+    __syncthreads();
+    if (c >= n) return;
+    const bf16 *w = w2 + (int64_t)c * rank;
+    float z[PA_DC_TOK] = {};
+    auto add = [&](int r, float wv) {
+        const float4 u = *reinterpret_cast<const float4 *>(ls + r * PA_DC_TOK), v = *reinterpret_cast<const float4 *>(ls + r * PA_DC_TOK + 4);
+        const float x[PA_DC_TOK] = {u.x, u.y, u.z, u.w, v.x, v.y, v.z, v.w};
+#pragma unroll
+        for (int t = 0; t < PA_DC_TOK; t++) z[t] = fmaf(wv, x[t], z[t]);
+    };
+    if ((rank & 7) == 0) {
+        for (int r = 0; r < rank; r += 8) {
+            const uint4 v = __ldg(reinterpret_cast<const uint4 *>(w + r));
+            const uint32_t u[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+            for (int e = 0; e < 4; e++) { add(r + 2 * e, __uint_as_float(u[e] << 16)); add(r + 2 * e + 1, __uint_as_float(u[e] & 0xffff0000u)); }
+        }
+    } else {
+        for (int r = 0; r < rank; r++) add(r, pa_ld(w + r));
+    }
+    const float bias = b[c];
+#pragma unroll
+    for (int t = 0; t < PA_DC_TOK; t++)
+        if (t0 + t < bs) dec[(int64_t)(t0 + t) * n + c] = pa_act1(z[t] + bias, act);
 }
 
 #define PA_SC_TOK 32    // tokens staged per round (half as many for the widest states)
+#define PA_SC_FLIGHT 4  // tokens whose outputs are reduced together
 #define PA_SC_WARPS 4
 #define PA_SC_REGS 16   // state entries per lane
 struct PaScan {
@@ -407,7 +445,8 @@ __global__ void __launch_bounds__(32 * PA_SC_WARPS) pa_k_scan(const PaScan a) {
             }
         }
         if (MODE == 0) __syncthreads();
-        for (int tt = 0; tt < nt; tt++) {
+        // one token: the state, and the lane's part of the output of its columns
+        auto step = [&](int tt, float (&part)[NC]) {
             const float aa = MODE ? 0.f : as[tt], ct = MODE ? 1.0f : cs[tt];
             float x[NC], vv[NC], acc[NC][4];
 #pragma unroll
@@ -445,12 +484,36 @@ __global__ void __launch_bounds__(32 * PA_SC_WARPS) pa_k_scan(const PaScan a) {
                 }
             }
 #pragma unroll
-            for (int c = 0; c < NC; c++) {
-                float r = (acc[c][0] + acc[c][1]) + (acc[c][2] + acc[c][3]);
+            for (int c = 0; c < NC; c++) part[c] = (acc[c][0] + acc[c][1]) + (acc[c][2] + acc[c][3]);
+        };
+        // ... reduced over the column's lanes in the same order for every token
+        auto finish = [&](int tt, float (&part)[NC]) {
 #pragma unroll
-                for (int o = IL / 2; o; o >>= 1) r += __shfl_xor_sync(0xffffffffu, r, o);
-                if (li == 0) os[tt * CC + col0 + c * CW] = MODE ? r * a.o_scale : fmaf(skip, x[c], r);
-            }
+            for (int c = 0; c < NC; c++)
+                if (li == 0) os[tt * CC + col0 + c * CW] = MODE ? part[c] * a.o_scale : fmaf(skip, vs[tt * CC + col0 + c * CW], part[c]);
+        };
+        int tt = 0;
+        for (; tt + PA_SC_FLIGHT <= nt; tt += PA_SC_FLIGHT) { // several tokens in flight: nothing is stored between their loads
+            float part[PA_SC_FLIGHT][NC];
+#pragma unroll
+            for (int f = 0; f < PA_SC_FLIGHT; f++) step(tt + f, part[f]);
+#pragma unroll
+            for (int o = IL / 2; o; o >>= 1)
+#pragma unroll
+                for (int f = 0; f < PA_SC_FLIGHT; f++)
+#pragma unroll
+                    for (int c = 0; c < NC; c++) part[f][c] += __shfl_xor_sync(0xffffffffu, part[f][c], o);
+#pragma unroll
+            for (int f = 0; f < PA_SC_FLIGHT; f++) finish(tt + f, part[f]);
+        }
+        for (; tt < nt; tt++) {
+            float part[NC];
+            step(tt, part);
+#pragma unroll
+            for (int o = IL / 2; o; o >>= 1)
+#pragma unroll
+                for (int c = 0; c < NC; c++) part[c] += __shfl_xor_sync(0xffffffffu, part[c], o);
+            finish(tt, part);
         }
         __syncthreads();
         for (int tt = warp; tt < nt; tt += PA_SC_WARPS) {
@@ -599,6 +662,30 @@ __global__ void __launch_bounds__(256) pa_k_gate_norm(const float *__restrict__ 
             const float gsl = pa_silu(gr[c0 + c]), wv = w ? w[c0 + c] : 1.0f;
             orow[c0 + c] = gate_first ? yr[c0 + c] * gsl * inv * wv : yr[c0 + c] * inv * wv * gsl;
         }
+    }
+}
+
+// norm first (out = N(y) w silu(g)), parts of at most 256 entries: a warp per part, eight parts per CTA.  Grid (parts / 8, tokens)
+__global__ void __launch_bounds__(256) pa_k_gate_norm_warp(const float *__restrict__ y, int ldy, const float *__restrict__ gate, int ldg, int ps, int parts, const float *__restrict__ w, float eps,
+                                                           float *__restrict__ out, int ldo) {
+    const int t = blockIdx.y, part = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+    if (part >= parts) return;
+    const float *yr = y + (int64_t)t * ldy + part * ps, *gr = gate + (int64_t)t * ldg + part * ps;
+    float v[8], g[8], s = 0.f;
+#pragma unroll
+    for (int i = 0; i < 8; i++) {
+        const int c = lane + 32 * i;
+        v[i] = c < ps ? yr[c] : 0.f;
+        g[i] = c < ps ? gr[c] : 0.f;
+        s = fmaf(v[i], v[i], s);
+    }
+#pragma unroll
+    for (int o = 16; o; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
+    const float inv = 1.0f / sqrtf(s / (float)ps + eps);
+#pragma unroll
+    for (int i = 0; i < 8; i++) {
+        const int c = lane + 32 * i;
+        if (c < ps) out[(int64_t)t * ldo + part * ps + c] = v[i] * inv * (w ? w[part * ps + c] : 1.0f) * pa_silu(g[i]);
     }
 }
 

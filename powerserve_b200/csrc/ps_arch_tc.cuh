@@ -17,6 +17,7 @@
 #define PT_KB 64
 #define PT_BLOCK (128 * PT_KB * 2) // bytes of one operand block (either side)
 #define PT_THREADS 192
+#define PT_MAX_SEG 6 // operand sets of one product
 #define PT_SMEM (192 * 1024 + 1024)
 
 // ---------------------------------------------------------------------------------------------------- operand builders
@@ -64,36 +65,35 @@ __global__ void __launch_bounds__(256) pa_k_tc_prep_x(uint8_t *__restrict__ dst,
 }
 
 // the operand sets of a segmented product: set 0 = x, set s = x + (x' - x) mu[s - 1] with x' the row of the token before (the batch's first
-// token: row (pos - 1) & 1 of `ring`, zeros at position 0).  Grid (k blocks, column tiles, sets); set s starts s * set_bytes further on.
+// token: row (pos - 1) & 1 of `ring`, zeros at position 0).  Grid (k blocks, column tiles, 4): a CTA takes 32 rows, a thread eight entries of all sets; set s starts s * set_bytes further on.
 __global__ void __launch_bounds__(256) pa_k_tc_prep_shift(uint8_t *__restrict__ dst, const float *__restrict__ x, int M, int K, int nkb, const float *__restrict__ mu,
                                                           const float *__restrict__ ring, const int32_t *__restrict__ pos, int64_t set_bytes) {
-    const int kb = blockIdx.x, t = blockIdx.y, set = blockIdx.z, p0 = pos[0];
-    const float *m = set ? mu + (int64_t)(set - 1) * K : nullptr;
-    uint8_t *out = dst + set * set_bytes + ((int64_t)t * nkb + kb) * PT_BLOCK;
-    for (int c = threadIdx.x; c < 128 * 8; c += 256) {
-        const int kc = c & 7, row = c >> 3, r = t * 128 + row, k0 = kb * PT_KB + kc * 8;
-        uint16_t v[8];
-        const float *src = x + (int64_t)r * K, *prev = r > 0 ? src - K : ring + (int64_t)((p0 - 1) & 1) * K;
-        const bool first = r == 0 && p0 == 0;
+    const int kb = blockIdx.x, t = blockIdx.y, p0 = pos[0];
+    const int kc = threadIdx.x & 7, row = blockIdx.z * 32 + (threadIdx.x >> 3), r = t * 128 + row, k0 = kb * PT_KB + kc * 8;
+    uint8_t *out = dst + ((int64_t)t * nkb + kb) * PT_BLOCK + kc * 2048 + row * 16;
+    const float *src = x + (int64_t)r * K, *prev = r > 0 ? src - K : ring + (int64_t)((p0 - 1) & 1) * K;
+    const bool first = r == 0 && p0 == 0;
+    float h[8], d[8];
 #pragma unroll
-        for (int e = 0; e < 8; e++) {
-            float val = 0.f;
-            if (r < M && k0 + e < K) {
-                val = src[k0 + e];
-                if (m) val = fmaf((first ? 0.f : prev[k0 + e]) - val, m[k0 + e], val);
-            }
-            v[e] = __bfloat16_as_ushort(__float2bfloat16_rn(val));
-        }
+    for (int e = 0; e < 8; e++) {
+        const bool in = r < M && k0 + e < K;
+        h[e] = in ? src[k0 + e] : 0.f;
+        d[e] = in ? (first ? 0.f : prev[k0 + e]) - h[e] : 0.f;
+    }
+#pragma unroll
+    for (int set = 0; set < PT_MAX_SEG; set++) {
+        uint16_t v[8];
+#pragma unroll
+        for (int e = 0; e < 8; e++) v[e] = __bfloat16_as_ushort(__float2bfloat16_rn(set && k0 + e < K ? fmaf(d[e], mu[(int64_t)(set - 1) * K + k0 + e], h[e]) : h[e]));
         uint4 pk;
         pk.x = v[0] | ((uint32_t)v[1] << 16); pk.y = v[2] | ((uint32_t)v[3] << 16); pk.z = v[4] | ((uint32_t)v[5] << 16); pk.w = v[6] | ((uint32_t)v[7] << 16);
-        *reinterpret_cast<uint4 *>(out + kc * 2048 + row * 16) = pk;
+        *reinterpret_cast<uint4 *>(out + set * set_bytes) = pk;
     }
 }
 
 // ---------------------------------------------------------------------------------------------------- the GEMM
 // A product whose output rows read different operand sets (activations that are mixtures of the same input): row tiles rt[s] .. rt[s + 1] - 1
 // hold the rows row[s] .. row[s + 1] - 1 of the output and read set s.  n = 0: one set, all rows.
-#define PT_MAX_SEG 6
 struct PtSegs {
     int n;
     int rt[PT_MAX_SEG + 1], row[PT_MAX_SEG + 1];
@@ -227,6 +227,11 @@ __global__ void __launch_bounds__(PT_THREADS, 1) pa_k_tc_gemm(const PtArgs a) {
                                    "=r"(w2[10]), "=r"(w2[11]), "=r"(w2[12]), "=r"(w2[13]), "=r"(w2[14]), "=r"(w2[15])
                                  : "r"(t_lane + PT_N + c0)
                                  : "memory");
+                float mulv[16]; // the table rows' entries: sixteen independent loads beside the tensor-memory loads
+                if (NA == 1 && a.mul.table) {
+#pragma unroll
+                    for (int c = 0; c < 16; c++) mulv[c] = pa_ld(a.mul.table + (int64_t)a.mul.tok[min(r0 + c0 + c, rend - 1)] * a.mul.ld + min(n, n_end - 1));
+                }
                 ps_tc_ld_wait();
                 if (n < n_end) {
 #pragma unroll
@@ -237,7 +242,7 @@ __global__ void __launch_bounds__(PT_THREADS, 1) pa_k_tc_gemm(const PtArgs a) {
                         if (a.mode == PT_MODE_DENSE) {
                             const bool act1 = a.act1 && n >= a.act_from;
                             float val = act1 ? pa_act1(acc + bias, a.act) : acc + bias;
-                            if (a.mul.table) val *= pa_ld(a.mul.table + (int64_t)a.mul.tok[r] * a.mul.ld + n);
+                            if (NA == 1 && a.mul.table) val *= mulv[c];
                             a.C[(int64_t)r * a.ldc + (act1 ? n + a.gap : n)] = val;
                         } else if (a.mode == PT_MODE_EXPERT_UP) {
                             a.C[(int64_t)r * a.ldc + n] = NA == 2 ? pa_expert_act(acc, __uint_as_float(w2[c]), a.act) : pa_act1(acc, a.act);
