@@ -131,7 +131,7 @@ struct PsArch {
     cudaStream_t side = nullptr;
     cudaEvent_t ev_fork = nullptr, ev_join = nullptr;
     int opt_fork = 1;
-    int opt_mv_cap = 0; // > 0: resident mat-vec CTAs per SM (0: two beside overlapping launches, four for long streams or without overlap)
+    int opt_mv_cap = 0; // > 0: resident mat-vec CTAs per SM (0: four)
     int opt_prefetch = 1; // 1: a mat-vec CTA requests its first row group into L2 before the dependency wait; 2: every next group too
     int opt_pdl = 1;    // single-token kernels on the main stream are launched with programmatic stream serialisation
     int opt_scan_nc = 0; // value columns per lane of the recurrence scan (0: chosen by the grid's size)
@@ -485,7 +485,7 @@ int ps_arch_create(PsArch **out, const ps_cuda_arch_desc *desc, std::string &err
         if ((l.route_identity || l.route_correction) && (!w.gen2 || l.mlp_kind != PS_MLP_ROUTED || l.route_identity < 0 || l.router_act != PS_ROUTER_SOFTMAX || l.route_groups > 1 || l.route_on_input))
             return bail(afail(err, PS_CUDA_ERR_UNSUPPORTED, "layer %d: identity experts (%d) and corrected choices need a soft-max router without groups in a sequential block", i, l.route_identity));
         if ((l.layer_scale && (!l.post_norm || l.block_kind != PS_BLOCK_SEQUENTIAL)) || l.token_slot < 0 || l.token_slot > d.token_slots ||
-            (l.token_slot > 0 && (d.token_dim <= 0 || l.block_kind != PS_BLOCK_SEQUENTIAL || d.norm_kind != PS_NORM_RMS || d.norm_groups > 1 || l.pass_in)))
+            (l.token_slot > 0 && (d.token_dim <= 0 || d.token_dim > 4096 || l.block_kind != PS_BLOCK_SEQUENTIAL || d.norm_kind != PS_NORM_RMS || d.norm_groups > 1 || l.pass_in)))
             return bail(afail(err, PS_CUDA_ERR_UNSUPPORTED, "layer %d: layer scales need output norms in a sequential block; a token input (part %d of %d) a sequential block with plain RMS norms", i, l.token_slot, d.token_slots));
 
         if (l.v_is_k && l.v_dim != l.qk_dim) return bail(afail(err, PS_CUDA_ERR_UNSUPPORTED, "layer %d: values from keys of size %d cannot have size %d", i, l.qk_dim, l.v_dim));
@@ -694,6 +694,10 @@ int ps_arch_create(PsArch **out, const ps_cuda_arch_desc *desc, std::string &err
         cudaFuncSetAttribute(pa_k_dec_expert_up<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024) != cudaSuccess ||
         cudaFuncSetAttribute(pa_k_dec_dense_up<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024) != cudaSuccess ||
         cudaFuncSetAttribute(pa_k_dec_dense_up<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024) != cudaSuccess ||
+        cudaFuncSetAttribute(pa_k_dec_token_input<true>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1) != cudaSuccess ||
+        cudaFuncSetAttribute(pa_k_dec_token_input<false>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1) != cudaSuccess ||
+        cudaFuncSetAttribute(pa_k_dec_token_input<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 176 * 1024) != cudaSuccess ||
+        cudaFuncSetAttribute(pa_k_dec_token_input<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, 176 * 1024) != cudaSuccess ||
         cudaFuncSetAttribute(pa_k_tc_gemm<1>, cudaFuncAttributeMaxDynamicSharedMemorySize, PT_SMEM) != cudaSuccess ||
         cudaFuncSetAttribute(pa_k_tc_gemm<2>, cudaFuncAttributeMaxDynamicSharedMemorySize, PT_SMEM) != cudaSuccess) {
         cudaGetLastError();
@@ -1155,14 +1159,21 @@ static int forward_t(PsArch *a, const PsArchIO &io, int bs, int pos0, int lm_hea
         return ks;
     };
     // the mat-vec CTAs walk the row groups with the grid's stride: at most four resident CTAs per SM, one wave
-    // (two per SM when the launches overlap: the next kernel's CTAs need room beside them to fetch their weights early)
     const bool pdl = a->opt_pdl != 0;
-    auto mv_grid = [&](int rows, int ks, int K) {
-        // a long stream (>= 48 MB) gains more from four resident CTAs per SM than from the next kernel's early start
-        const int cap = a->opt_mv_cap > 0 ? a->opt_mv_cap : (!pdl || (int64_t)rows * K * 2 >= ((int64_t)48 << 20)) ? 4 : 2;
+    auto mv_grid = [&](int rows, int ks) {
+        const int cap = a->opt_mv_cap > 0 ? a->opt_mv_cap : 4; // as many as stay resident
         return std::min(cdiv(rows, PA_DV_ROWS / ks), (unsigned)(cap * a->n_sm));
     };
     const bool tc = ROUND && a->opt_tc && !single && !a->opt_simple;
+    // a dense product with few units: cut its token tiles until the grid fills the GPU.  Every cut reads the weights once more and shortens the
+    // epilogue, so it pays for short sums and tiny grids (measured)
+    auto cut_tiles = [&](PtArgs &g) {
+        const int units = g.n_rt * g.n_ct, most = g.nkb <= 16 || units <= 8 ? 8 : g.nkb <= 40 && (g.a1 || units <= 16) ? 2 : 1;
+        g.n_sub = 1;
+        while (g.n_sub < most && cdiv(g.M, PT_N / (2 * g.n_sub)) * (unsigned)g.n_rt <= (unsigned)a->n_sm) g.n_sub *= 2;
+        g.n_ct = (int)cdiv(g.M, PT_N / g.n_sub);
+        return std::min(a->n_sm, g.n_ct * g.n_rt);
+    };
     // C[m][n] = sum_k X[m][k] W[n][k] + bias[n] on the tensor cores: round + tile the activations, then the GEMM
     auto tc_dense = [&](const float *X, int ldx, int M, int K, const uint8_t *wt, int N, const float *bias, float *C, int ldc, const PaAct *act1 = nullptr, int act_from = 0,
                         int gap = 0, const PaRowMul *mul = nullptr) -> int {
@@ -1173,7 +1184,8 @@ static int forward_t(PsArch *a, const PsArchIO &io, int bs, int pos0, int lm_hea
         g.a0 = wt; g.b = a->tcx; g.nkb = nkb; g.n_rt = n_rt; g.n_ct = n_ct; g.M = M; g.N = N; g.mode = PT_MODE_DENSE; g.C = C; g.ldc = ldc; g.bias = bias; g.err = io.err_dev;
         if (act1) { g.act = *act1; g.act1 = 1; g.act_from = act_from; g.gap = gap; }
         if (mul) g.mul = *mul;
-        pa_k_tc_gemm<1><<<std::min(a->n_sm, n_ct * n_rt), PT_THREADS, PT_SMEM, st>>>(g);
+        const int ctas = cut_tiles(g);
+        pa_k_tc_gemm<1><<<ctas, PT_THREADS, PT_SMEM, st>>>(g);
         PA_LAUNCH();
         return 0;
     };
@@ -1228,7 +1240,7 @@ static int forward_t(PsArch *a, const PsArchIO &io, int bs, int pos0, int lm_hea
     };
     auto dec_mv = [&](PaMv &mv, size_t smem, bool overlap = true) -> int {
         mv.ksplit = pick_ksplit(mv.N + mv.E, mv.K); mv.prefetch = a->opt_prefetch;
-        pa_launch_dep(pdl && overlap, pa_k_dec_mv<ROUND>, dim3(mv_grid(mv.N + mv.E, mv.ksplit, mv.K)), dim3(PA_DV_THREADS), smem, st, mv);
+        pa_launch_dep(pdl && overlap, pa_k_dec_mv<ROUND>, dim3(mv_grid(mv.N + mv.E, mv.ksplit)), dim3(PA_DV_THREADS), smem, st, mv);
         PA_LAUNCH();
         return 0;
     };
@@ -1310,7 +1322,8 @@ static int forward_t(PsArch *a, const PsArchIO &io, int bs, int pos0, int lm_hea
             PtArgs g{};
             g.a0 = tg; g.a1 = tu; g.b = a->tcx; g.nkb = nkb; g.n_rt = (ff + PT_M - 1) / PT_M; g.n_ct = n_ct; g.M = bs; g.N = ff; g.mode = PT_MODE_EXPERT_UP;
             g.C = a->y; g.ldc = ff; g.act = act; g.err = io.err_dev;
-            pa_k_tc_gemm<2><<<std::min(a->n_sm, n_ct * g.n_rt), PT_THREADS, PT_SMEM, st>>>(g);
+            const int ctas = cut_tiles(g);
+            pa_k_tc_gemm<2><<<ctas, PT_THREADS, PT_SMEM, st>>>(g);
         } else {
             pa_k_dense_up<ROUND><<<dim3(cdiv(ff, PA_TN), cdiv(bs, PA_TM)), blk, 0, st>>>(X, dim, wg, wu, a->y, bs, ff, dim, act);
         }
@@ -1483,13 +1496,10 @@ static int forward_t(PsArch *a, const PsArchIO &io, int bs, int pos0, int lm_hea
         const PaRowMul mul{a->tok_embed + (int64_t)(w.d.token_slot - 1) * td, (int64_t)d.token_slots * td, io.tokens_dev};
         int rc;
         if (single) {
-            PaMv mv{};
-            seam_mv(mv, nullptr);
-            mv.W = w.wtg; mv.N = td; mv.K = dim; mv.y = a->tg; mv.act = gelu; mv.mul = mul;
-            if ((rc = dec_mv(mv, 4 * (size_t)dim))) return rc;
-            PaMv mp{};
-            mp.x = a->tg; mp.W = w.wtp; mp.N = dim; mp.K = td; mp.y = a->ty;
-            if ((rc = dec_mv(mp, 0))) return rc;
+            PaTokIn p{xc, pend_y, pend_w, xo, d.norm_eps, a->res_scale, w.wtg, w.wtp, dim, td, mul, a->ty};
+            PA_CK(pa_launch_cluster(pdl, PA_TI_CLUSTER, pa_k_dec_token_input<ROUND>, dim3(PA_TI_CLUSTER), dim3(PA_TI_THREADS), 4 * (size_t)(((dim + 3) & ~3) + td), st, p));
+            PA_LAUNCH();
+            std::swap(xc, xo);
         } else {
             if ((rc = seam(nullptr, nullptr))) return rc;
             if (tc) {
@@ -1545,7 +1555,8 @@ static int forward_t(PsArch *a, const PsArchIO &io, int bs, int pos0, int lm_hea
                 PA_LAUNCH();
                 g.a0 = w.t_qkv; g.b = a->tcx; g.nkb = nkb; g.n_rt = w.seg.rt[w.seg.n]; g.n_ct = n_ct; g.M = bs; g.N = w.pw; g.mode = PT_MODE_DENSE; g.C = a->qkv; g.ldc = w.pw; g.err = io.err_dev;
                 g.act = tanh_act; g.act1 = 1; g.act_from = w1_off;
-                pa_k_tc_gemm<1><<<std::min(a->n_sm, n_ct * g.n_rt), PT_THREADS, PT_SMEM, st>>>(g);
+                const int ctas = cut_tiles(g);
+                pa_k_tc_gemm<1><<<ctas, PT_THREADS, PT_SMEM, st>>>(g);
                 PA_LAUNCH();
             } else {
                 pa_k_token_shift<<<dim3(cdiv(dim, 256), bs, 5), 256, 0, st>>>(a->h, dim, w.mu, ring, io.pos_dev, a->mixb, (int64_t)B * dim);
@@ -1902,7 +1913,7 @@ static int forward_t(PsArch *a, const PsArchIO &io, int bs, int pos0, int lm_hea
             mv.qd = w.qd; mv.kd = w.kd; mv.vd = w.vd; mv.kc = io.kc[li]; mv.vct = io.vct[li]; mv.n_ctx = d.n_ctx; mv.pos = io.pos_dev;
             if (routed) { mv.Wr = w.router; mv.E = l.n_experts; mv.z = a->z; }
             mv.ksplit = pick_ksplit(nqkv + mv.E, dim); mv.prefetch = a->opt_prefetch;
-            pa_launch_dep(pdl, pa_k_dec_mv<ROUND>, dim3(mv_grid(nqkv + mv.E, mv.ksplit, dim)), dim3(PA_DV_THREADS), 4 * (size_t)dim, st, mv);
+            pa_launch_dep(pdl, pa_k_dec_mv<ROUND>, dim3(mv_grid(nqkv + mv.E, mv.ksplit)), dim3(PA_DV_THREADS), 4 * (size_t)dim, st, mv);
             if (routed) {
                 // gate | up of the chosen experts: reads x and the router logits only, so it runs on the side stream while the main
                 // stream goes through scores, P.V and the output projection (a fork in the captured graph); joined before `down`
@@ -1947,7 +1958,7 @@ static int forward_t(PsArch *a, const PsArchIO &io, int bs, int pos0, int lm_hea
             mv.x = a->att; mv.W = w.wo; mv.bias = w.bo; mv.N = dim; mv.K = w.od; mv.y = a->ao;
             if (!routed) mv.residual = a->x; // no feed-forward: the layer ends here
             mv.ksplit = pick_ksplit(dim, w.od); mv.prefetch = a->opt_prefetch;
-            pa_launch_dep(pdl, pa_k_dec_mv<ROUND>, dim3(mv_grid(dim, mv.ksplit, w.od)), dim3(PA_DV_THREADS), 0, st, mv);
+            pa_launch_dep(pdl, pa_k_dec_mv<ROUND>, dim3(mv_grid(dim, mv.ksplit)), dim3(PA_DV_THREADS), 0, st, mv);
         } else if (tc) {
             int rc = tc_dense(a->att, w.od, bs, w.od, w.t_o, dim, w.bo, a->ao, dim);
             if (rc) return rc;
@@ -1998,7 +2009,7 @@ static int forward_t(PsArch *a, const PsArchIO &io, int bs, int pos0, int lm_hea
             mv.x = a->x; mv.norm_w = a->final_norm; mv.eps = d.norm_eps; mv.W = a->head; mv.N = d.vocab_size; mv.K = dim; mv.y = a->logits;
             if (a->has_seq) seam_mv(mv, a->final_norm);
             mv.ksplit = pick_ksplit(d.vocab_size, dim); mv.prefetch = a->opt_prefetch;
-            pa_launch_dep(pdl, pa_k_dec_mv<ROUND>, dim3(mv_grid(d.vocab_size, mv.ksplit, dim)), dim3(PA_DV_THREADS), 4 * (size_t)dim, st, mv);
+            pa_launch_dep(pdl, pa_k_dec_mv<ROUND>, dim3(mv_grid(d.vocab_size, mv.ksplit)), dim3(PA_DV_THREADS), 4 * (size_t)dim, st, mv);
         } else if (tc) {
             int rc = tc_dense(a->h, dim, bs, dim, a->t_head, d.vocab_size, nullptr, a->logits, d.vocab_size);
             if (rc) return rc;

@@ -21,6 +21,7 @@
 //                        logits as further rows), activation; without a gate a warp's pair is two neighbouring up rows
 //   pa_k_dec_latent_q    latent attention with queries from the input: W_uk folded into the query, both rotations, latent and rotated key
 //                        part into the cache
+//   pa_k_dec_token_input per-layer token input: seam, gate rows, the token's table row and the projection in one cluster
 //   pa_k_dec_expert_up   norm + top-k of the router scores in the prologue, gate | up rows of the chosen experts, activation
 //   pa_k_dec_expert_down down rows of the chosen experts summed over the slots + mixer output + residual (or, for the next seam, + the
 //                        shared expert's down rows behind its gate + the input itself for identity outputs)
@@ -96,19 +97,111 @@ __device__ __forceinline__ void pa_norm_to_smem(float *hs, const float *__restri
     __syncthreads();
 }
 
-// block-wide seam between two blocks (256 threads): hs = G(x + y_scale P(y) + add_tok + add_vec; w_in) with P(y) = G(y; w_out) (w_out
+struct PaNoHook { __device__ __forceinline__ void operator()() const {} };
+// the seam below for one part whose vectors fit into registers (dim a multiple of 4, at most 16 NT): every load of a phase is in flight at
+// once, the sums come out of registers.  `between` runs behind the first loads.
+template <int NT, typename F>
+__device__ __forceinline__ void pa_seam_regs(float *hs, const float *__restrict__ x, const float *__restrict__ y, const float *__restrict__ w_out, const float *__restrict__ w_in,
+                                             float *__restrict__ x_out, int dim, float eps, int center, const float *__restrict__ add_tok, const float *__restrict__ add_vec, float y_scale, float *red,
+                                             const F &between) {
+    constexpr int V = 4;
+    const int n4 = dim >> 2, tid = threadIdx.x;
+    auto ld = [&](const float *p, int c) { return p && c < n4 ? reinterpret_cast<const float4 *>(p)[c] : make_float4(0.f, 0.f, 0.f, 0.f); };
+    auto stats = [&](const float4 (&v)[V], float &mu) { // 1 / sqrt(mean((v - mu)^2) + eps)
+        mu = 0.f;
+        if (center) {
+            float m = 0.f;
+#pragma unroll
+            for (int i = 0; i < V; i++) m += (v[i].x + v[i].y) + (v[i].z + v[i].w);
+            mu = pa_block_sum(m, red) / (float)dim;
+        }
+        float s = 0.f;
+#pragma unroll
+        for (int i = 0; i < V; i++) {
+            if (tid + i * NT >= n4) continue;
+            const float a = v[i].x - mu, b = v[i].y - mu, c = v[i].z - mu, d = v[i].w - mu;
+            s = fmaf(a, a, s); s = fmaf(b, b, s); s = fmaf(c, c, s); s = fmaf(d, d, s);
+        }
+        return 1.0f / sqrtf(pa_block_sum(s, red) / (float)dim + eps);
+    };
+    float4 v[V];
+    {
+        float4 t[V];
+#pragma unroll
+        for (int i = 0; i < V; i++) { t[i] = ld(y, tid + i * NT); v[i] = ld(x, tid + i * NT); }
+        between();
+        if (y && w_out) {
+            float4 w[V];
+#pragma unroll
+            for (int i = 0; i < V; i++) w[i] = ld(w_out, tid + i * NT);
+            float mu;
+            const float f = stats(t, mu) * y_scale;
+#pragma unroll
+            for (int i = 0; i < V; i++) {
+                v[i].x = fmaf((t[i].x - mu) * f, w[i].x, v[i].x); v[i].y = fmaf((t[i].y - mu) * f, w[i].y, v[i].y);
+                v[i].z = fmaf((t[i].z - mu) * f, w[i].z, v[i].z); v[i].w = fmaf((t[i].w - mu) * f, w[i].w, v[i].w);
+            }
+        } else if (y) {
+#pragma unroll
+            for (int i = 0; i < V; i++) { v[i].x = fmaf(y_scale, t[i].x, v[i].x); v[i].y = fmaf(y_scale, t[i].y, v[i].y); v[i].z = fmaf(y_scale, t[i].z, v[i].z); v[i].w = fmaf(y_scale, t[i].w, v[i].w); }
+        }
+    }
+    if (add_tok || add_vec) {
+#pragma unroll
+        for (int i = 0; i < V; i++) {
+            const float4 p = ld(add_tok, tid + i * NT), q = ld(add_vec, tid + i * NT);
+            v[i].x += p.x + q.x; v[i].y += p.y + q.y; v[i].z += p.z + q.z; v[i].w += p.w + q.w;
+        }
+    }
+    if (x_out && blockIdx.x == 0 && blockIdx.y == 0) {
+#pragma unroll
+        for (int i = 0; i < V; i++)
+            if (tid + i * NT < n4) reinterpret_cast<float4 *>(x_out)[tid + i * NT] = v[i];
+    }
+    if (w_in) {
+        float4 w[V];
+#pragma unroll
+        for (int i = 0; i < V; i++) w[i] = ld(w_in, tid + i * NT);
+        float mu;
+        const float f = stats(v, mu);
+#pragma unroll
+        for (int i = 0; i < V; i++) { v[i].x = (v[i].x - mu) * f * w[i].x; v[i].y = (v[i].y - mu) * f * w[i].y; v[i].z = (v[i].z - mu) * f * w[i].z; v[i].w = (v[i].w - mu) * f * w[i].w; }
+    }
+#pragma unroll
+    for (int i = 0; i < V; i++)
+        if (tid + i * NT < n4) reinterpret_cast<float4 *>(hs)[tid + i * NT] = v[i];
+    __syncthreads();
+}
+
+// norm weights on their way to L2 before the dependency wait (a few CTAs ask for all)
+__device__ __forceinline__ void pa_prefetch_norms(const float *a, const float *b, int dim) {
+    if (blockIdx.x >= 2 || blockIdx.y) return;
+    for (int c = threadIdx.x * 32; c < dim; c += blockDim.x * 32) {
+        if (a) asm volatile("prefetch.global.L2 [%0];" ::"l"(a + c));
+        if (b) asm volatile("prefetch.global.L2 [%0];" ::"l"(b + c));
+    }
+}
+
+// block-wide seam between two blocks (NT threads): hs = G(x + y_scale P(y) + add_tok + add_vec; w_in) with P(y) = G(y; w_out) (w_out
 // null: y itself; y / add_tok / add_vec null: nothing joins), G over `groups` equal parts, the part's mean taken off first when
 // `center`.  CTA 0 also stores the updated residual to x_out - a buffer other than x, which the other CTAs are still reading.
+template <int NT = 256, typename F = PaNoHook>
 __device__ __forceinline__ void pa_seam_to_smem(float *hs, const float *__restrict__ x, const float *__restrict__ y, const float *__restrict__ w_out,
                                                 const float *__restrict__ w_in, float *__restrict__ x_out, int dim, int groups, float eps, int center = 0,
-                                                const float *__restrict__ add_tok = nullptr, const float *__restrict__ add_vec = nullptr, float y_scale = 1.0f) {
-    __shared__ float red[8];
+                                                const float *__restrict__ add_tok = nullptr, const float *__restrict__ add_vec = nullptr, float y_scale = 1.0f,
+                                                const F &between = F{}) {
+    __shared__ float red[NT / 32];
+    if (groups == 1 && (dim & 3) == 0 && dim <= 16 * NT) {
+        pa_seam_regs<NT>(hs, x, y, w_out, w_in, x_out, dim, eps, center, add_tok, add_vec, y_scale, red, between);
+        return;
+    }
+    between();
     const int gs = dim / groups;
     for (int g = 0; g < groups; g++) {
         const int c0 = g * gs;
         float inv = 1.0f, mu = 0.f;
-        if (y && w_out) inv = pa_block_stats(y + c0, gs, center, eps, red, mu);
-        for (int c = threadIdx.x; c < gs; c += 256) {
+        if (y && w_out) inv = pa_block_stats<NT>(y + c0, gs, center, eps, red, mu);
+        for (int c = threadIdx.x; c < gs; c += NT) {
             float v = x[c0 + c];
             if (y) v += y_scale * (w_out ? (y[c0 + c] - mu) * inv * w_out[c0 + c] : y[c0 + c]);
             if (add_tok || add_vec) v += (add_tok ? add_tok[c0 + c] : 0.f) + (add_vec ? add_vec[c0 + c] : 0.f);
@@ -117,8 +210,8 @@ __device__ __forceinline__ void pa_seam_to_smem(float *hs, const float *__restri
         }
         if (w_in) {
             float mu2;
-            const float inv2 = pa_block_stats(hs + c0, gs, center, eps, red, mu2); // (a thread's own entries)
-            for (int c = threadIdx.x; c < gs; c += 256) hs[c0 + c] = (hs[c0 + c] - mu2) * inv2 * w_in[c0 + c];
+            const float inv2 = pa_block_stats<NT>(hs + c0, gs, center, eps, red, mu2); // (a thread's own entries)
+            for (int c = threadIdx.x; c < gs; c += NT) hs[c0 + c] = (hs[c0 + c] - mu2) * inv2 * w_in[c0 + c];
         }
     }
     __syncthreads();
@@ -159,7 +252,6 @@ struct PaMv {
     // rows n >= act_from (> 0) leave through the one-argument activation, `gap` entries further on
     int act_from, gap;
     PaAct act;
-    PaRowMul mul;          // rows leave through the activation `act`, times a table row (act_from is not read then)
     // rows that read different mixtures of the normed input (seg_n > 0; with groups > 0): rows below seg_end[0] read h, rows from
     // seg_end[s - 1] to seg_end[s] read h + (h' - h) mu[s - 1] with h' the token before's h: row (pos - 1) & 1 of the ring [2][K], zeros at
     // position 0; CTA 0 stores h to row pos & 1.  Every CTA takes neighbouring row groups and forms only the mixtures they read.
@@ -171,7 +263,7 @@ struct PaMv {
 };
 
 template <bool ROUND>
-__global__ void __launch_bounds__(PA_DV_THREADS) pa_k_dec_mv(const PaMv a) {
+__global__ void __launch_bounds__(PA_DV_THREADS, 4) pa_k_dec_mv(const PaMv a) {
     extern __shared__ __align__(16) float pa_hs[];
     __shared__ float part_s[8][2];
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
@@ -190,6 +282,7 @@ __global__ void __launch_bounds__(PA_DV_THREADS) pa_k_dec_mv(const PaMv a) {
     const int g_begin = a.seg_n > 0 ? blockIdx.x * per_cta : blockIdx.x, g_end = a.seg_n > 0 ? min(groups, g_begin + per_cta) : groups, g_step = a.seg_n > 0 ? 1 : gridDim.x;
     auto segment = [&](int n) { int sg = 0; while (sg < a.seg_n - 1 && n >= a.seg_end[sg]) sg++; return sg; };
     prefetch(g_begin);
+    pa_prefetch_norms(a.seam_w, a.norm_w, a.groups > 0 ? (a.cat ? a.seam_dim : a.K) : 0);
     // launched with programmatic stream serialisation: everything above touches weights only and overlaps the kernel before
     ps_grid_dep_launch();
     ps_grid_dep_wait();
@@ -274,8 +367,6 @@ __global__ void __launch_bounds__(PA_DV_THREADS) pa_k_dec_mv(const PaMv a) {
                     } else {
                         a.vct[(int64_t)(n - a.qd - a.kd) * a.n_ctx + p] = v;
                     }
-                } else if (a.mul.table) {
-                    a.y[n] = pa_act1(v, a.act) * pa_ld(a.mul.table + (int64_t)a.mul.tok[0] * a.mul.ld + n);
                 } else if (a.act_from > 0 && n >= a.act_from) {
                     a.y[n + a.gap] = pa_act1(v, a.act);
                 } else if (a.residual) {
@@ -288,6 +379,105 @@ __global__ void __launch_bounds__(PA_DV_THREADS) pa_k_dec_mv(const PaMv a) {
             }
         }
         if (ks > 1) __syncthreads(); // part_s is written again by the next group
+    }
+}
+
+// ---------------------------------------------------------------------------------------------------- per-layer token input
+// eight rows at once (neighbours of stride K; K and the address multiples of eight): s[i] = w_i . f(x), reduced over the warp
+template <bool ROUND> __device__ __forceinline__ void pa_dot8(const bf16 *__restrict__ w, const float *x, int K, int lane, float (&s)[8]) {
+#pragma unroll
+    for (int i = 0; i < 8; i++) s[i] = 0.f;
+    for (int k = lane * 8; k < K; k += 256) {
+        uint4 v[8];
+#pragma unroll
+        for (int i = 0; i < 8; i++) v[i] = __ldg(reinterpret_cast<const uint4 *>(w + (int64_t)i * K + k));
+        const float4 x0 = *reinterpret_cast<const float4 *>(x + k), x1 = *reinterpret_cast<const float4 *>(x + k + 4);
+        const float xv[8] = {pa_rnd<ROUND>(x0.x), pa_rnd<ROUND>(x0.y), pa_rnd<ROUND>(x0.z), pa_rnd<ROUND>(x0.w), pa_rnd<ROUND>(x1.x), pa_rnd<ROUND>(x1.y), pa_rnd<ROUND>(x1.z), pa_rnd<ROUND>(x1.w)};
+#pragma unroll
+        for (int i = 0; i < 8; i++) {
+            const uint32_t u[4] = {v[i].x, v[i].y, v[i].z, v[i].w};
+#pragma unroll
+            for (int t = 0; t < 4; t++) {
+                s[i] = fmaf(__uint_as_float(u[t] << 16), xv[2 * t], s[i]);
+                s[i] = fmaf(__uint_as_float(u[t] & 0xffff0000u), xv[2 * t + 1], s[i]);
+            }
+        }
+    }
+#pragma unroll
+    for (int o = 16; o; o >>= 1)
+#pragma unroll
+        for (int i = 0; i < 8; i++) s[i] += __shfl_xor_sync(0xffffffffu, s[i], o);
+}
+
+// x <- x + seam; y = W_proj (gelu(W_gate x) * e) in one launch of one cluster: each CTA forms its share of the gated vector and hands it to
+// every other through distributed shared memory, then takes its share of the projection's rows.  y waits for the next seam.
+#define PA_TI_THREADS 512
+#define PA_TI_CLUSTER 16 // (beyond the portable size: asked for by attribute)
+struct PaTokIn {
+    const float *x, *seam_y, *seam_w;
+    float *x_out;
+    float eps, y_scale;
+    const bf16 *Wg, *Wp; // [td][dim], [dim][td]
+    int dim, td;
+    PaRowMul e;
+    float *y;
+};
+template <bool ROUND>
+__global__ void __launch_bounds__(PA_TI_THREADS) pa_k_dec_token_input(const PaTokIn a) {
+    extern __shared__ __align__(16) float pa_hs[]; // [dim] the stream, [td] the gated vector
+    cg::cluster_group cl = cg::this_cluster();
+    const int n_cl = gridDim.x, me = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, dim = a.dim, td = a.td;
+    float *gs = pa_hs + ((dim + 3) & ~3);
+    const int per_g = (td + n_cl - 1) / n_cl, g0 = min(me * per_g, td), g1 = min(g0 + per_g, td);
+    const int per_p = ((dim + n_cl - 1) / n_cl + 7) & ~7, p0 = min(me * per_p, dim), p1 = min(p0 + per_p, dim);
+    for (int64_t e = threadIdx.x * 64; e < (int64_t)(g1 - g0) * dim; e += PA_TI_THREADS * 64) asm volatile("prefetch.global.L2 [%0];" ::"l"(a.Wg + (int64_t)g0 * dim + e));
+    for (int64_t e = threadIdx.x * 64; e < (int64_t)(p1 - p0) * td; e += PA_TI_THREADS * 64) asm volatile("prefetch.global.L2 [%0];" ::"l"(a.Wp + (int64_t)p0 * td + e));
+    pa_prefetch_norms(a.seam_w, nullptr, dim);
+    ps_grid_dep_launch();
+    ps_grid_dep_wait();
+    cl.barrier_arrive(); // this CTA runs: its shared memory may be written
+    const bf16 *erow = a.e.table + (int64_t)a.e.tok[0] * a.e.ld;
+    if (warp == PA_TI_THREADS / 32 - 1)
+        for (int n = g0 + lane * 32; n < g1; n += 32 * 32) asm volatile("prefetch.global.L2 [%0];" ::"l"(erow + n));
+    pa_seam_to_smem<PA_TI_THREADS>(pa_hs, a.x, a.seam_y, a.seam_w, nullptr, a.x_out, dim, 1, a.eps, 0, nullptr, nullptr, a.y_scale);
+    cl.barrier_wait();
+    const PaAct gelu{0.f, 0.f, 0.f, PS_ACT_GELU_TANH};
+    for (int n = g0 + 2 * warp; n < g1; n += 2 * (PA_TI_THREADS / 32)) {
+        const int n1 = min(n + 1, g1 - 1);
+        float s0, s1;
+        const float e0 = pa_ld(erow + n), e1 = pa_ld(erow + n1);
+        pa_dot2<ROUND>(a.Wg + (int64_t)n * dim, a.Wg + (int64_t)n1 * dim, pa_hs, dim, 1.0f, lane, s0, s1);
+        if (lane < n_cl) { // a lane per CTA
+            float *dst = cl.map_shared_rank(gs, lane);
+            dst[n] = pa_act1(s0, gelu) * e0;
+            dst[n1] = pa_act1(n1 == n ? s0 : s1, gelu) * e1;
+        }
+    }
+    cl.sync();
+    if ((td & 7) == 0) {
+        for (int n = p0 + 8 * warp; n < p1; n += 8 * (PA_TI_THREADS / 32)) {
+            if (n + 8 <= p1) {
+                float s[8];
+                pa_dot8<ROUND>(a.Wp + (int64_t)n * td, gs, td, lane, s);
+#pragma unroll
+                for (int i = 0; i < 8; i++)
+                    if (lane == i) a.y[n + i] = s[i];
+            } else {
+                for (int m = n; m < p1; m++) {
+                    float s0, s1;
+                    pa_dot2<ROUND>(a.Wp + (int64_t)m * td, a.Wp + (int64_t)m * td, gs, td, 1.0f, lane, s0, s1);
+                    if (lane == 0) a.y[m] = s0;
+                }
+            }
+        }
+    } else {
+        for (int n = p0 + 2 * warp; n < p1; n += 2 * (PA_TI_THREADS / 32)) {
+            const int n1 = min(n + 1, p1 - 1);
+            float s0, s1;
+            pa_dot2<ROUND>(a.Wp + (int64_t)n * td, a.Wp + (int64_t)n1 * td, gs, td, 1.0f, lane, s0, s1);
+            if (lane == 0) a.y[n] = s0;
+            if (lane == 1 && n1 != n) a.y[n1] = s1;
+        }
     }
 }
 
@@ -463,6 +653,24 @@ __global__ void __launch_bounds__(256) pa_k_dec_pv(PaAttn at, const float *__res
         ps_fence_barrier_init();
         asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
     }
+    const int c0 = blockIdx.x * PA_DP_DIMS;
+    // value dim of the CTA's cc-th row (dv or more: outside); with rotated values the CTA takes two pairs (m, m + dv / 2)
+    const int vh = at.vrope.dims >> 1;
+    auto col = [&](int cc) {
+        if (vh == 0) return c0 + cc;
+        const int m = c0 / 2 + (cc & 1);
+        return m < vh ? m + (cc >= 2 ? vh : 0) : dv;
+    };
+    // a chunk's V^T rows: 1-D bulk copies, issued by one thread (the first chunk's travel while the statistics are merged)
+    auto copy_rows = [&](const float *vbase, int ldv, int j0, int nj4) {
+        int rows = 0;
+        for (int cc = 0; cc < PA_DP_DIMS; cc++) rows += col(cc) < dv;
+        asm volatile("fence.proxy.async.shared::cta;" ::: "memory"); // the rows were read through the generic proxy
+        ps_mbar_expect_tx(&bar, (uint32_t)(rows * nj4 * 4));
+        for (int cc = 0; cc < PA_DP_DIMS; cc++)
+            if (col(cc) < dv) ps_bulk_g2s(vs + cc * chunk, vbase + (int64_t)(g * dv + col(cc)) * ldv + j0, (uint32_t)(nj4 * 4), &bar);
+    };
+    if (bulk && tid == 0) copy_rows(vct, at.n_ctx, lo & ~3, (min(chunk, n - (lo & ~3)) + 3) & ~3);
     // soft-max statistics of every head of the group from the scores kernel's per-block pairs: a warp per head
     const int nb = (n + PA_DS_KEYS - 1) / PA_DS_KEYS;
     const int nv = pa_pool_vis(at, n - 1), nvb = (nv + PA_DS_KEYS - 1) / PA_DS_KEYS; // pooled blocks in sight, and their statistics
@@ -487,14 +695,6 @@ __global__ void __launch_bounds__(256) pa_k_dec_pv(PaAttn at, const float *__res
     }
     for (int t = tid; t < 8 * rep; t += 256) acc[t] = 0.f;
     const int dim_l = warp % PA_DP_DIMS, part = warp / PA_DP_DIMS, n_part = 8 / PA_DP_DIMS;
-    const int c0 = blockIdx.x * PA_DP_DIMS;
-    // value dim of the CTA's cc-th row (dv or more: outside); with rotated values the CTA takes two pairs (m, m + dv / 2)
-    const int vh = at.vrope.dims >> 1;
-    auto col = [&](int cc) {
-        if (vh == 0) return c0 + cc;
-        const int m = c0 / 2 + (cc & 1);
-        return m < vh ? m + (cc >= 2 ? vh : 0) : dv;
-    };
     int it = 0;
     // two stretches of keys: the tokens in sight (V^T rows of n_ctx columns), then the pooled blocks (rows of n_pool columns behind them)
     for (int seg = 0; seg < (nv > 0 ? 2 : 1); seg++) {
@@ -504,23 +704,26 @@ __global__ void __launch_bounds__(256) pa_k_dec_pv(PaAttn at, const float *__res
         const int nj = min(chunk, s_n - j0), nj4 = (nj + 3) & ~3;
         __syncthreads(); // the previous chunk's buffers are free
         if (bulk) {
-            if (tid == 0) {
-                int rows = 0;
-                for (int cc = 0; cc < PA_DP_DIMS; cc++) rows += col(cc) < dv;
-                asm volatile("fence.proxy.async.shared::cta;" ::: "memory"); // the rows were read through the generic proxy
-                ps_mbar_expect_tx(&bar, (uint32_t)(rows * nj4 * 4));
-                for (int cc = 0; cc < PA_DP_DIMS; cc++)
-                    if (col(cc) < dv) ps_bulk_g2s(vs + cc * chunk, vbase + (int64_t)(g * dv + col(cc)) * ldv + j0, (uint32_t)(nj4 * 4), &bar);
-            }
+            if (tid == 0 && it > 0) copy_rows(vbase, ldv, j0, nj4);
         } else {
             for (int t = tid; t < PA_DP_DIMS * nj4; t += 256) {
                 const int cc = t / nj4, jj = t % nj4;
                 vs[cc * chunk + jj] = (col(cc) < dv && jj < nj) ? vbase[(int64_t)(g * dv + col(cc)) * ldv + j0 + jj] : 0.f;
             }
         }
-        for (int t = tid; t < rep * nj4; t += 256) {
-            const int r = t / nj4, jj = t % nj4;
-            ps[r * chunk + jj] = (jj < nj && j0 + jj >= s_lo) ? expf(b[(int64_t)(h0 + r) * at.ldS + s_off + j0 + jj] - ms[r]) : 0.f;
+        for (int r = 0; r < rep; r++) {
+            const float *br = b + (int64_t)(h0 + r) * at.ldS + s_off + j0;
+            const float m = ms[r];
+            for (int jb = tid; jb < nj4; jb += 4 * 256) { // four scores in flight per thread
+                float v[4];
+#pragma unroll
+                for (int u = 0; u < 4; u++) v[u] = br[min(jb + 256 * u, nj - 1)];
+#pragma unroll
+                for (int u = 0; u < 4; u++) {
+                    const int jj = jb + 256 * u;
+                    if (jj < nj4) ps[r * chunk + jj] = (jj < nj && j0 + jj >= s_lo) ? expf(v[u] - m) : 0.f;
+                }
+            }
         }
         __syncthreads();
         if (bulk && !ps_tc_wait(&bar, it & 1)) { if (tid == 0) err[0] = 6; return; }
@@ -632,27 +835,26 @@ __global__ void __launch_bounds__(PA_DV_THREADS) pa_k_dec_expert_up(const float 
     __shared__ float sc[PA_MAX_EXPERTS];
     __shared__ int se[PA_MAX_EXPERTS];
     __shared__ float sw[PA_MAX_EXPERTS];
+    pa_prefetch_norms(norm_w, nullptr, norm_w ? dim : 0);
     ps_grid_dep_launch();
     ps_grid_dep_wait();
-    if (rt.act == PS_ROUTER_TOPK_SOFTMAX || (rt.act == PS_ROUTER_SOFTMAX && rt.groups <= 1)) {
-        if (threadIdx.x < 32) {
-            if (rt.act == PS_ROUTER_SOFTMAX) pa_route_softmax_warp(z, rt, se, sw, threadIdx.x);
-            else pa_route_topk_warp(z, rt.E, rt.top, se, sw, threadIdx.x);
-            __syncwarp();
+    auto route = [&]() { // (the prologue's barriers publish se / sw)
+        if (rt.act == PS_ROUTER_TOPK_SOFTMAX || (rt.act == PS_ROUTER_SOFTMAX && rt.groups <= 1)) {
+            if (threadIdx.x < 32) {
+                if (rt.act == PS_ROUTER_SOFTMAX) pa_route_softmax_warp(z, rt, se, sw, threadIdx.x);
+                else pa_route_topk_warp(z, rt.E, rt.top, se, sw, threadIdx.x);
+                __syncwarp();
+                if (blockIdx.x == 0 && blockIdx.y == 0)
+                    for (int r = threadIdx.x; r < rt.top; r += 32) { sel_e[r] = se[r]; sel_w[r] = sw[r]; }
+            }
+        } else if (threadIdx.x == 0) {
+            pa_route_serial(z, rt, sc, se, sw);
             if (blockIdx.x == 0 && blockIdx.y == 0)
-                for (int r = threadIdx.x; r < rt.top; r += 32) { sel_e[r] = se[r]; sel_w[r] = sw[r]; }
+                for (int r = 0; r < rt.top; r++) { sel_e[r] = se[r]; sel_w[r] = sw[r]; }
         }
-    } else if (threadIdx.x == 0) {
-        pa_route_serial(z, rt, sc, se, sw);
-        if (blockIdx.x == 0 && blockIdx.y == 0)
-            for (int r = 0; r < rt.top; r++) { sel_e[r] = se[r]; sel_w[r] = sw[r]; }
-    }
-    if (norm_w) {
-        pa_norm_to_smem(pa_hs, x, norm_w, dim, eps); // (its barriers also publish se / sw)
-    } else { // the experts read the residual stream itself
-        for (int c = threadIdx.x; c < dim; c += blockDim.x) pa_hs[c] = x[c];
-        __syncthreads();
-    }
+    };
+    // the input, normed (norm_w null: as it is, the experts read the residual stream itself)
+    pa_seam_to_smem(pa_hs, x, nullptr, nullptr, norm_w, nullptr, dim, 1, eps, 0, nullptr, nullptr, 1.0f, route);
     const int r = blockIdx.y, e = se[r], lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     if (h_out && blockIdx.x == 0 && blockIdx.y == 0) // the normed input, for the choices that stand for it
         for (int c = threadIdx.x; c < dim; c += blockDim.x) h_out[c] = pa_hs[c];
@@ -691,6 +893,7 @@ __global__ void __launch_bounds__(PA_DV_THREADS) pa_k_dec_dense_up(const float *
     if (!Wg) { // no gate: a warp's pair is two neighbouring up rows, y[n] = act(up[n] . h)
         const int n = (blockIdx.x * rows + warp) * 2;
         if (n < ff) pa_prefetch2(Wu + (int64_t)n * dim, Wu + (int64_t)min(n + 1, ff - 1) * dim, 0, dim, lane);
+        pa_prefetch_norms(seam_w, norm_w, dim);
         ps_grid_dep_launch();
         ps_grid_dep_wait();
         pa_seam_to_smem(pa_hs, x, seam_y, seam_w, norm_w, x_out, dim, groups, eps, center, nullptr, nullptr, y_scale);
@@ -706,6 +909,7 @@ __global__ void __launch_bounds__(PA_DV_THREADS) pa_k_dec_dense_up(const float *
     {
         const int n = blockIdx.x * rows + warp;
         if (n < ff) pa_prefetch2(Wg + (int64_t)n * dim, Wu + (int64_t)n * dim, 0, dim, lane);
+        pa_prefetch_norms(seam_w, norm_w, dim);
     }
     ps_grid_dep_launch();
     ps_grid_dep_wait();

@@ -276,7 +276,7 @@ __global__ void __launch_bounds__(256) pa_k_combine(float *__restrict__ x, const
 }
 
 // ---------------------------------------------------------------------------------------------------------------- sequential blocks
-// block-wide sum over 256 threads, broadcast to all (two barriers)
+// block-wide sum (red: one entry per warp), broadcast to all (two barriers)
 __device__ __forceinline__ float pa_block_sum(float s, float *red) {
 #pragma unroll
     for (int o = 16; o; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
@@ -288,17 +288,17 @@ __device__ __forceinline__ float pa_block_sum(float s, float *red) {
     return t;
 }
 
-// block-wide statistics of v[0 .. n) (each thread its own strided entries): mu = mean when `center`, else 0;
+// block-wide (NT threads) statistics of v[0 .. n) (each thread its own strided entries): mu = mean when `center`, else 0;
 // returns 1 / sqrt(mean((v - mu)^2) + eps)
-__device__ __forceinline__ float pa_block_stats(const float *v, int n, int center, float eps, float *red, float &mu) {
+template <int NT = 256> __device__ __forceinline__ float pa_block_stats(const float *v, int n, int center, float eps, float *red, float &mu) {
     mu = 0.f;
     if (center) {
         float m = 0.f;
-        for (int c = threadIdx.x; c < n; c += 256) m += v[c];
+        for (int c = threadIdx.x; c < n; c += NT) m += v[c];
         mu = pa_block_sum(m, red) / (float)n;
     }
     float s = 0.f;
-    for (int c = threadIdx.x; c < n; c += 256) { const float d = v[c] - mu; s = fmaf(d, d, s); }
+    for (int c = threadIdx.x; c < n; c += NT) { const float d = v[c] - mu; s = fmaf(d, d, s); }
     return 1.0f / sqrtf(pa_block_sum(s, red) / (float)n + eps);
 }
 
@@ -539,28 +539,32 @@ __device__ __forceinline__ void pa_route_serial(const float *__restrict__ z, con
         for (int n = 0; n < r.top; n++) sw[n] /= sum + r.eps;
 }
 
-// one warp: soft-max over all E logits, the `top` largest scores (+ corr) choose (ties: the lower expert), weights = the scores themselves,
+// NS * 32 >= E.  One warp: soft-max over all E logits, the `top` largest scores (+ corr) choose (ties: the lower expert), weights = the scores themselves,
 // divided by their sum + eps with renorm; se / sw are in shared memory
-__device__ __forceinline__ void pa_route_softmax_warp(const float *__restrict__ z, const PaRoute &r, int *se, float *sw, int lane) {
-    float s[PA_MAX_EXPERTS / 32], v[PA_MAX_EXPERTS / 32], mx = -INFINITY, sum = 0.f;
+template <int NS> __device__ __forceinline__ void pa_route_softmax_warp_n(const float *__restrict__ z, const PaRoute &r, int *se, float *sw, int lane) {
+    float s[NS], v[NS], mx = -INFINITY, sum = 0.f;
     unsigned taken = 0;
 #pragma unroll
-    for (int i = 0; i < PA_MAX_EXPERTS / 32; i++) { s[i] = lane + 32 * i < r.E ? z[lane + 32 * i] : -INFINITY; mx = fmaxf(mx, s[i]); }
+    for (int i = 0; i < NS; i++) {
+        s[i] = lane + 32 * i < r.E ? z[lane + 32 * i] : -INFINITY;
+        v[i] = r.corr && lane + 32 * i < r.E ? r.corr[lane + 32 * i] : 0.f;
+        mx = fmaxf(mx, s[i]);
+    }
 #pragma unroll
     for (int o = 16; o; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
 #pragma unroll
-    for (int i = 0; i < PA_MAX_EXPERTS / 32; i++) { s[i] = lane + 32 * i < r.E ? expf(s[i] - mx) : 0.f; sum += s[i]; }
+    for (int i = 0; i < NS; i++) { s[i] = lane + 32 * i < r.E ? expf(s[i] - mx) : 0.f; sum += s[i]; }
 #pragma unroll
     for (int o = 16; o; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
     const float inv = 1.0f / sum;
 #pragma unroll
-    for (int i = 0; i < PA_MAX_EXPERTS / 32; i++) { s[i] *= inv; v[i] = s[i] + (r.corr && lane + 32 * i < r.E ? r.corr[lane + 32 * i] : 0.f); }
+    for (int i = 0; i < NS; i++) { s[i] *= inv; v[i] += s[i]; }
     float chosen = 0.f;
     for (int n = 0; n < r.top; n++) {
         int be = -1;
         float bv = 0.f, bs = 0.f;
 #pragma unroll
-        for (int i = 0; i < PA_MAX_EXPERTS / 32; i++)
+        for (int i = 0; i < NS; i++)
             if (lane + 32 * i < r.E && !((taken >> i) & 1) && (be < 0 || v[i] > bv)) { be = lane + 32 * i; bv = v[i]; bs = s[i]; }
 #pragma unroll
         for (int o = 16; o; o >>= 1) {
@@ -575,6 +579,10 @@ __device__ __forceinline__ void pa_route_softmax_warp(const float *__restrict__ 
     __syncwarp();
     if (r.renorm)
         for (int n = lane; n < r.top; n += 32) sw[n] /= chosen + r.eps;
+}
+__device__ __forceinline__ void pa_route_softmax_warp(const float *__restrict__ z, const PaRoute &r, int *se, float *sw, int lane) {
+    if (r.E <= 32) pa_route_softmax_warp_n<1>(z, r, se, sw, lane);
+    else pa_route_softmax_warp_n<PA_MAX_EXPERTS / 32>(z, r, se, sw, lane);
 }
 
 // one warp: the `top` largest of E logits (ties: the lower expert), weights = soft-max over the chosen; se / sw are in shared memory

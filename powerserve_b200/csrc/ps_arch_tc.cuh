@@ -1,7 +1,7 @@
 // ps_arch_tc.cuh - tcgen05 GEMM for the layer-list executor's bfloat16 products: C[token][n] = sum_k X[token][k] W[n][k].
 //
 // The WEIGHT rows are the MMA's M side (128 output features per unit), the tokens its N side (128 per unit), so one
-// accumulator column is one token and an epilogue warp's 32 tensor-memory lanes are 32 consecutive output features: the
+// accumulator column is one token (a grid with few units cuts the token tiles into parts of 64, 32 or 16) and an epilogue warp's 32 tensor-memory lanes are 32 consecutive output features: the
 // stores of a column are coalesced.  Both operands reach shared memory as ready-made canonical K-major no-swizzle blocks
 // ([k-chunk of 8][row][8 elements], 16 KB per 128 rows x 64 k) through ONE 1-D bulk copy each:
 //   * weights are re-tiled once at bind time (pa_k_tc_tile_w), per expert for the routed feed-forward;
@@ -105,6 +105,7 @@ struct PtArgs {
     const uint8_t *a0, *a1; // weight blocks [group][row tiles][k blocks]; a1 = the second matrix of a fused pair (gate | up)
     const uint8_t *b;       // activation blocks [column tiles][k blocks]
     int nkb, n_rt, n_ct;    // n_ct: column tiles (an upper bound when n_ct_dev is given)
+    int n_sub;              // dense: a column tile is cut into n_sub equal parts (0: one), n_ct counts the parts - more, narrower units for a grid that would not fill the GPU
     const int *n_ct_dev;
     const int *tile_e, *tile_row0, *tile_end; // routed: group, first row and end row of every column tile
     int M, N;               // dense: token rows; N: output features
@@ -134,6 +135,7 @@ __global__ void __launch_bounds__(PT_THREADS, 1) pa_k_tc_gemm(const PtArgs a) {
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int nkb = a.nkb, n_ct = a.n_ct_dev ? min(*a.n_ct_dev, a.n_ct) : a.n_ct;
     const int n_units = n_ct * a.n_rt;
+    const int n_sub = max(a.n_sub, 1), tn = PT_N / n_sub; // tokens of a unit
     const int my_units = (n_units > (int)blockIdx.x) ? (n_units - 1 - (int)blockIdx.x) / (int)gridDim.x + 1 : 0;
 
     if (tid == 0) {
@@ -161,24 +163,26 @@ __global__ void __launch_bounds__(PT_THREADS, 1) pa_k_tc_gemm(const PtArgs a) {
                 const int64_t grp = a.tile_e ? a.tile_e[ct] : 0;
                 const uint8_t *pa0 = a.a0 + ((grp * a.n_rt + rt) * nkb) * (int64_t)PT_BLOCK;
                 const uint8_t *pa1 = NA == 2 ? a.a1 + ((grp * a.n_rt + rt) * nkb) * (int64_t)PT_BLOCK : nullptr;
-                const uint8_t *pb = a.b + ((int64_t)ct * nkb) * PT_BLOCK;
+                const uint8_t *pb = a.b + ((int64_t)(ct / n_sub) * nkb) * PT_BLOCK + (ct % n_sub) * tn * 16;
                 for (int sg = 1; sg < a.seg.n; sg++)
                     if (rt >= a.seg.rt[sg]) pb += a.seg.set_bytes;
                 for (int kb = 0; kb < nkb; kb++, g++) {
                     const int s = g % STAGES;
                     if (g >= STAGES && !ps_tc_wait(&bar_empty[s], ((g / STAGES) - 1) & 1)) { *a.err = 1; ok = false; break; }
                     uint8_t *st = smem + (size_t)s * STAGE_BYTES;
-                    ps_mbar_expect_tx(&bar_full[s], STAGE_BYTES);
+                    ps_mbar_expect_tx(&bar_full[s], NA * PT_BLOCK + PT_BLOCK / n_sub);
                     ps_bulk_g2s(st, pa0 + (int64_t)kb * PT_BLOCK, PT_BLOCK, &bar_full[s]);
                     if (NA == 2) ps_bulk_g2s(st + PT_BLOCK, pa1 + (int64_t)kb * PT_BLOCK, PT_BLOCK, &bar_full[s]);
-                    ps_bulk_g2s(st + NA * PT_BLOCK, pb + (int64_t)kb * PT_BLOCK, PT_BLOCK, &bar_full[s]);
+                    if (n_sub == 1) ps_bulk_g2s(st + NA * PT_BLOCK, pb + (int64_t)kb * PT_BLOCK, PT_BLOCK, &bar_full[s]);
+                    else // the part's tokens of every k-chunk, at the places they have in the whole tile
+                        for (int c = 0; c < 8; c++) ps_bulk_g2s(st + NA * PT_BLOCK + c * 2048, pb + (int64_t)kb * PT_BLOCK + c * 2048, (uint32_t)(tn * 16), &bar_full[s]);
                 }
             }
         }
     } else if (warp == 5) {
         // ===== MMA issuer: kind::f16 with bfloat16 operands (a_format = b_format = 1), fp32 accumulators, K-major both
         if (lane == 0) {
-            const uint32_t idesc = (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(PT_N >> 3) << 17) | ((uint32_t)(PT_M >> 4) << 24);
+            const uint32_t idesc = (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(tn >> 3) << 17) | ((uint32_t)(PT_M >> 4) << 24);
             int g = 0;
             bool ok = true;
             for (int mu = 0; mu < my_units && ok; mu++) {
@@ -210,10 +214,10 @@ __global__ void __launch_bounds__(PT_THREADS, 1) pa_k_tc_gemm(const PtArgs a) {
             int n = rt * PT_M + 32 * warp + lane, n_end = a.N;
             for (int sg = 0; sg < a.seg.n; sg++) // the segment's own rows
                 if (rt >= a.seg.rt[sg] && rt < a.seg.rt[sg + 1]) { n += a.seg.row[sg] - a.seg.rt[sg] * PT_M; n_end = a.seg.row[sg + 1]; break; }
-            const int r0 = a.tile_row0 ? a.tile_row0[ct] : ct * PT_N, rend = a.tile_end ? a.tile_end[ct] : a.M;
+            const int r0 = a.tile_row0 ? a.tile_row0[ct] : ct * tn, rend = a.tile_end ? a.tile_end[ct] : a.M;
             const uint32_t t_lane = tmem_base + ((uint32_t)(32 * warp) << 16) + tb * (NA * PT_N);
             const float bias = (a.bias && n < n_end) ? a.bias[n] : 0.f;
-            const int n_cols = min(PT_N, rend - r0); // warp-uniform
+            const int n_cols = min(tn, rend - r0); // warp-uniform
             for (int c0 = 0; c0 < n_cols; c0 += 16) {
                 uint32_t v[16], w2[16];
                 asm volatile("tcgen05.ld.sync.aligned.32x32b.x16.b32 {%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15}, [%16];"
