@@ -366,10 +366,14 @@ __device__ __forceinline__ void pa_cp_async4(float *dst_smem, const float *src) 
     asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"((uint32_t)__cvta_generic_to_shared(dst_smem)), "l"(src) : "memory");
 }
 
+__device__ __forceinline__ void pa_cp_async16(float *dst_smem, const float *src) {
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((uint32_t)__cvta_generic_to_shared(dst_smem)), "l"(src) : "memory");
+}
+
 // grid (dv / columns per CTA, H).  A lane owns entries i = (m * IL + li) * 4 + e (m, e < 4) of NC columns: k and q come out of shared
 // memory as float4 (lanes of a column read neighbouring float4s, lanes of different columns the same ones) and serve the lane's NC
 // columns from registers; the output is reduced over the IL lanes of a column by log2(IL) shuffles, always in the same order (the
-// result does not depend on NC).  The q / k / v rows (and raw step sizes) of a round of tokens arrive by asynchronous 4-byte copies
+// result does not depend on NC).  The q / k / v rows (and raw step sizes) of a round of tokens arrive by asynchronous copies (16 bytes where rows and sizes allow)
 // into one of two buffers while the round before is computed.
 template <int IL, int NC, int MODE>
 __global__ void __launch_bounds__(32 * PA_SC_WARPS) pa_k_scan(const PaScan a) {
@@ -403,11 +407,23 @@ __global__ void __launch_bounds__(32 * PA_SC_WARPS) pa_k_scan(const PaScan a) {
     const float rate = a.dt ? expf(a.a_log[h]) : 0.f, bias = a.dt ? a.dt_bias[h] : 0.f, fixed = (MODE || a.dt) ? 0.f : a.decay[h], skip = a.d_skip ? a.d_skip[h] : 0.f;
     for (int e = tid; e < 2 * BUF; e += NT) sm[e] = 0.f; // what the copies never write (entries beyond dk, columns beyond dv) stays zero
     __syncthreads();
+    auto al = [](const float *p, int ld, int n) { return ((reinterpret_cast<uintptr_t>(p) & 15) | ((ld | n) & 3)) == 0; };
+    const bool wide = al(a.q, a.ldq, a.q_gs | dk) && al(a.k, a.ldk, a.k_gs) && al(a.v, a.ldv, dv) && (!MODE || al(a.dec, a.lddec, dk));
     auto fetch = [&](int t0, int buf) {
         float *qs = sm + buf * BUF, *ks = qs + TOK * DKP, *vs = ks + TOK * DKP, *ds = vs + TOK * CC;
         const int nt = min(TOK, a.bs - t0);
         for (int tt = warp; tt < nt; tt += PA_SC_WARPS) {
             const float *qr = a.q + (int64_t)(t0 + tt) * a.ldq + g * a.q_gs, *kr = a.k + (int64_t)(t0 + tt) * a.ldk + g * a.k_gs;
+            if (wide) {
+                for (int i = lane * 4; i < dk; i += 128) {
+                    pa_cp_async16(qs + tt * DKP + i, qr + i);
+                    pa_cp_async16(ks + tt * DKP + i, kr + i);
+                    if (MODE) pa_cp_async16(ds + TOK + tt * DKP + i, a.dec + (int64_t)(t0 + tt) * a.lddec + h * dk + i);
+                }
+                const float *vr = a.v + (int64_t)(t0 + tt) * a.ldv + h * dv + j0;
+                for (int c = lane * 4; c < CC && j0 + c < dv; c += 128) pa_cp_async16(vs + tt * CC + c, vr + c);
+                continue;
+            }
             for (int i = lane; i < dk; i += 32) {
                 pa_cp_async4(qs + tt * DKP + i, qr + i);
                 pa_cp_async4(ks + tt * DKP + i, kr + i);
