@@ -145,7 +145,7 @@ struct PsArch {
     float *gts = nullptr;                  // rg-lru: gate logits of a batch
     float *hn = nullptr;                   // single-token step: the normed input, for the experts
     float *dcy = nullptr, *mixb = nullptr; // decays of a batch [max_batch][H * dk]; the five mixtures a time mixing reads [5][max_batch][dim]
-    int max_dcy = 0, max_seg_rt = 0;
+    int max_dcy = 0;
     bf16 *tok_embed = nullptr;             // per-layer token input: [vocab][token_slots * token_dim]
     float *tg = nullptr, *ty = nullptr;    // its gated part [max_batch][token_dim] and its output [max_batch][dim]
     bool has_shift = false;

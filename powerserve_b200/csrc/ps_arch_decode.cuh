@@ -10,9 +10,10 @@
 //                          its group norm, the sum is group-normed for this product; CTA 0 stores the sum to the second residual buffer),
 //                          per-head products (a row reads its head's slice of the input);
 //                          general parallel blocks: one range of rows leaves through the feed-forward's activation; a pass projection
-//                          appends the embedding output to the seam's sum
+//                          appends the embedding output to the seam's sum;
+//                          time mixing: ranges of rows read different mixtures of the normed input with the token before's
 //   pa_k_dec_scores      scores of all heads for 16 keys per CTA (thread per key and head out of shared memory), distance bias (table,
-//                        logarithmic or linear), head mixing, norms of q and of the token's own key per head, per-block soft-max statistics; with a window the grid starts at the first
+//                        logarithmic or linear), head mixing, norms and rotation of q and of the token's own key per head, rotation of its value, per-block soft-max statistics; with a window the grid starts at the first
 //                        key in sight; pooled windows: further CTAs take 16 block means each, and the last CTA forms the mean of the
 //                        block that the token completes
 //   pa_k_dec_pv          soft-max statistics (+ sink logit) per head, weights staged once per CTA, P.V along contiguous V^T rows; many

@@ -6,7 +6,8 @@
 // residual add, what a new pass of a looped model adds, norm of the sum), unit-RMS q / k (with weights and a query temperature, or the value blend) on the way into the cache,
 // the latent attention's norms and rotations (half-split or neighbouring pairs).  Pooled windows: pa_k_pool_blocks forms the mean key /
 // value of every block of positions that a batch completes; the scores / soft-max / P.V kernels take the blocks as further keys behind
-// the tokens.  pa_k_dense_up1 is the first half of a feed-forward without a gate.
+// the tokens.  Rotated heads: pa_k_embed forms the angles of a forward pass, pa_k_qkv_post rotates q / k / values, pa_k_pv turns the heads'
+// outputs back.  pa_k_dense_up1 is the first half of a feed-forward without a gate.
 // The single-token kernels (bs == 1) live in ps_arch_decode.cuh.
 #pragma once
 
