@@ -131,7 +131,7 @@ struct PsArch {
     cudaStream_t side = nullptr;
     cudaEvent_t ev_fork = nullptr, ev_join = nullptr;
     int opt_fork = 1;
-    int opt_mv_cap = 0; // > 0: resident mat-vec CTAs per SM (0: four)
+    int opt_mv_cap = 0; // > 0: resident mat-vec CTAs per SM (0: four, or two beside the experts of a parallel block)
     int opt_prefetch = 1; // 1: a mat-vec CTA requests its first row group into L2 before the dependency wait; 2: every next group too
     int opt_pdl = 1;    // single-token kernels on the main stream are launched with programmatic stream serialisation
     int opt_scan_nc = 0; // value columns per lane of the recurrence scan (0: chosen by the grid's size)
@@ -1160,8 +1160,9 @@ static int forward_t(PsArch *a, const PsArchIO &io, int bs, int pos0, int lm_hea
     };
     // the mat-vec CTAs walk the row groups with the grid's stride: at most four resident CTAs per SM, one wave
     const bool pdl = a->opt_pdl != 0;
-    auto mv_grid = [&](int rows, int ks) {
-        const int cap = a->opt_mv_cap > 0 ? a->opt_mv_cap : 4; // as many as stay resident
+    auto mv_grid = [&](int rows, int ks, int K) {
+        // as many as stay resident; two where the experts of a parallel block run beside the attention and the stream is short (< 48 MB)
+        const int cap = a->opt_mv_cap > 0 ? a->opt_mv_cap : a->has_par && pdl && (int64_t)rows * K * 2 < ((int64_t)48 << 20) ? 2 : 4;
         return std::min(cdiv(rows, PA_DV_ROWS / ks), (unsigned)(cap * a->n_sm));
     };
     const bool tc = ROUND && a->opt_tc && !single && !a->opt_simple;
@@ -1240,7 +1241,7 @@ static int forward_t(PsArch *a, const PsArchIO &io, int bs, int pos0, int lm_hea
     };
     auto dec_mv = [&](PaMv &mv, size_t smem, bool overlap = true) -> int {
         mv.ksplit = pick_ksplit(mv.N + mv.E, mv.K); mv.prefetch = a->opt_prefetch;
-        pa_launch_dep(pdl && overlap, pa_k_dec_mv<ROUND>, dim3(mv_grid(mv.N + mv.E, mv.ksplit)), dim3(PA_DV_THREADS), smem, st, mv);
+        pa_launch_dep(pdl && overlap, pa_k_dec_mv<ROUND>, dim3(mv_grid(mv.N + mv.E, mv.ksplit, mv.K)), dim3(PA_DV_THREADS), smem, st, mv);
         PA_LAUNCH();
         return 0;
     };
@@ -1913,7 +1914,7 @@ static int forward_t(PsArch *a, const PsArchIO &io, int bs, int pos0, int lm_hea
             mv.qd = w.qd; mv.kd = w.kd; mv.vd = w.vd; mv.kc = io.kc[li]; mv.vct = io.vct[li]; mv.n_ctx = d.n_ctx; mv.pos = io.pos_dev;
             if (routed) { mv.Wr = w.router; mv.E = l.n_experts; mv.z = a->z; }
             mv.ksplit = pick_ksplit(nqkv + mv.E, dim); mv.prefetch = a->opt_prefetch;
-            pa_launch_dep(pdl, pa_k_dec_mv<ROUND>, dim3(mv_grid(nqkv + mv.E, mv.ksplit)), dim3(PA_DV_THREADS), 4 * (size_t)dim, st, mv);
+            pa_launch_dep(pdl, pa_k_dec_mv<ROUND>, dim3(mv_grid(nqkv + mv.E, mv.ksplit, dim)), dim3(PA_DV_THREADS), 4 * (size_t)dim, st, mv);
             if (routed) {
                 // gate | up of the chosen experts: reads x and the router logits only, so it runs on the side stream while the main
                 // stream goes through scores, P.V and the output projection (a fork in the captured graph); joined before `down`
@@ -1958,7 +1959,7 @@ static int forward_t(PsArch *a, const PsArchIO &io, int bs, int pos0, int lm_hea
             mv.x = a->att; mv.W = w.wo; mv.bias = w.bo; mv.N = dim; mv.K = w.od; mv.y = a->ao;
             if (!routed) mv.residual = a->x; // no feed-forward: the layer ends here
             mv.ksplit = pick_ksplit(dim, w.od); mv.prefetch = a->opt_prefetch;
-            pa_launch_dep(pdl, pa_k_dec_mv<ROUND>, dim3(mv_grid(dim, mv.ksplit)), dim3(PA_DV_THREADS), 0, st, mv);
+            pa_launch_dep(pdl, pa_k_dec_mv<ROUND>, dim3(mv_grid(dim, mv.ksplit, w.od)), dim3(PA_DV_THREADS), 0, st, mv);
         } else if (tc) {
             int rc = tc_dense(a->att, w.od, bs, w.od, w.t_o, dim, w.bo, a->ao, dim);
             if (rc) return rc;
@@ -2009,7 +2010,7 @@ static int forward_t(PsArch *a, const PsArchIO &io, int bs, int pos0, int lm_hea
             mv.x = a->x; mv.norm_w = a->final_norm; mv.eps = d.norm_eps; mv.W = a->head; mv.N = d.vocab_size; mv.K = dim; mv.y = a->logits;
             if (a->has_seq) seam_mv(mv, a->final_norm);
             mv.ksplit = pick_ksplit(d.vocab_size, dim); mv.prefetch = a->opt_prefetch;
-            pa_launch_dep(pdl, pa_k_dec_mv<ROUND>, dim3(mv_grid(d.vocab_size, mv.ksplit)), dim3(PA_DV_THREADS), 4 * (size_t)dim, st, mv);
+            pa_launch_dep(pdl, pa_k_dec_mv<ROUND>, dim3(mv_grid(d.vocab_size, mv.ksplit, dim)), dim3(PA_DV_THREADS), 4 * (size_t)dim, st, mv);
         } else if (tc) {
             int rc = tc_dense(a->h, dim, bs, dim, a->t_head, d.vocab_size, nullptr, a->logits, d.vocab_size);
             if (rc) return rc;
